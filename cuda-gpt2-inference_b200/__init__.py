@@ -21,6 +21,7 @@ from dataclasses import dataclass
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "lib", "libb200gpt2.so")
+DECODER_LIB_PATH = os.path.join(_HERE, "lib", "libb200decoder.so")  # the layered decoders alone (build.py --target decoder)
 
 B200_OK = 0
 (B200_ERR_NULL, B200_ERR_SHAPE, B200_ERR_ALIGN, B200_ERR_CUDA, B200_ERR_DEVICE, B200_ERR_TIMEOUT,
@@ -29,7 +30,7 @@ B200_TF32, B200_TF32X3, B200_BF16, B200_BF16X3 = 0, 1, 2, 3
 ACT_NONE, ACT_GELU = 0, 1
 
 EXPORTS = (
-    "b200_ctx_create", "b200_ctx_destroy", "b200_ctx_set_stream", "b200_ctx_sync_check",
+    "b200_ctx_create", "b200_ctx_destroy", "b200_ctx_set_stream", "b200_ctx_own_stream", "b200_ctx_sync_check",
     "b200_ctx_launch_count", "b200_ctx_reset_launch_count", "b200_status_string",
     "b200_ctx_last_error", "b200_ctx_wait_timeout_probe", "b200_ctx_peer_wait_probe",
     "b200_matmul_forward", "b200_matmul_forward_bf16", "b200_convert_bf16", "b200_matmul_forward_bf16x3", "b200_split_bf16",
@@ -47,6 +48,9 @@ EXPORTS = (
     "b200_gpt2_set_profile", "b200_gpt2_read_profile",
     "b200_gpt2_forward_static", "b200_gpt2_static_prepare",
     "b200_gpt2_enable_kv_cache", "b200_gpt2_prefill", "b200_gpt2_decode_step", "b200_gpt2_decode_step_host", "b200_gpt2_generate_greedy", "b200_gpt2_generate", "b200_sample_rows",
+    "b200_decoder_create", "b200_decoder_destroy", "b200_decoder_vocab", "b200_decoder_load_safetensors", "b200_decoder_set_tensor",
+    "b200_decoder_finish_load", "b200_decoder_set_graph", "b200_decoder_open", "b200_decoder_close", "b200_decoder_length",
+    "b200_decoder_step", "b200_decoder_prefill_device", "b200_decoder_decode_device", "b200_decoder_generate",
     "b200_gpt2_create_tp", "b200_gpt2_set_allreduce", "b200_gpt2_set_tp_overlap", "b200_gpt2_param_offsets_tp", "b200_gpt2_shard_params_host",
 )
 
@@ -84,13 +88,43 @@ class B200Error(RuntimeError):
     pass
 
 
+class _Absent:
+    """Stands for a function that the loaded library does not have (the decoder-only build lacks GPT-2's)."""
+
+
+class _Symbols:
+    def __init__(self, cdll):
+        self.cdll = cdll
+
+    def __getattr__(self, name):
+        try:
+            return getattr(self.cdll, name)
+        except AttributeError:
+            return _Absent()
+
+
+def build_library(target: str = "gpt2") -> str:
+    """Compiles what is missing of lib/ (see build.py) and makes lib() load that library."""
+    global LIB_PATH
+    import importlib.util
+    spec = importlib.util.spec_from_file_location("cuda_gpt2_inference_b200_build", os.path.join(_HERE, "build.py"))
+    b = importlib.util.module_from_spec(spec)
+    spec.loader.exec_module(b)
+    if target == "decoder" and b.fresh("gpt2"):
+        target = "gpt2"  # the whole library is there already
+    path = b.build(target=target)
+    if _lib is None:
+        LIB_PATH = path
+    return path
+
+
 def lib() -> C.CDLL:
     """Loads libb200gpt2.so; raises if it has not been built (no fallback exists)."""
     global _lib
     if _lib is None:
         if not os.path.exists(LIB_PATH):
             raise B200Error(f"{LIB_PATH} is missing: build it with `python {os.path.join(_HERE, 'build.py')}`")
-        l = C.CDLL(LIB_PATH)
+        l = _Symbols(C.CDLL(LIB_PATH))
         vp, i, sz = C.c_void_p, C.c_int, C.c_size_t
         l.b200_ctx_create.argtypes = [C.POINTER(vp), i, vp]
         l.b200_ctx_destroy.argtypes = [vp]
@@ -176,7 +210,23 @@ def lib() -> C.CDLL:
         l.b200_gpt2_param_offsets_tp.argtypes = [vp, i, i, C.POINTER(sz)]
         l.b200_gpt2_param_offsets_tp.restype = sz
         l.b200_gpt2_shard_params_host.argtypes = [vp, i, i, vp, vp]
-        _lib = l
+        l.b200_ctx_own_stream.argtypes = [vp]
+        ip = C.POINTER(i)
+        l.b200_decoder_create.argtypes = [C.POINTER(vp), vp, C.c_char_p, i, i, i, i]
+        l.b200_decoder_destroy.argtypes = [vp]
+        l.b200_decoder_vocab.argtypes = [vp]
+        l.b200_decoder_load_safetensors.argtypes = [vp, C.c_char_p]
+        l.b200_decoder_set_tensor.argtypes = [vp, C.c_char_p, vp, i, C.POINTER(C.c_long), i]
+        l.b200_decoder_finish_load.argtypes = [vp]
+        l.b200_decoder_set_graph.argtypes = [vp, i]
+        l.b200_decoder_open.argtypes = [vp, ip]
+        l.b200_decoder_close.argtypes = [vp, i]
+        l.b200_decoder_length.argtypes = [vp, i]
+        l.b200_decoder_step.argtypes = [vp, i, vp, vp, vp, i, vp, vp]
+        l.b200_decoder_prefill_device.argtypes = [vp, i, vp, vp, vp, i, vp]
+        l.b200_decoder_decode_device.argtypes = [vp, i, vp]
+        l.b200_decoder_generate.argtypes = [vp, i, vp, vp, i, C.c_float, i, C.c_float, C.c_uint, vp]
+        _lib = l.cdll
     return _lib
 
 
@@ -194,7 +244,8 @@ def _ptr(t):
 class Context:
     """One context per GPU / host thread: owns the stream binding and the device status word."""
 
-    def __init__(self, device: int = 0, stream=None):
+    def __init__(self, device: int = 0, stream=None, own_stream: bool = False):
+        """stream: a torch stream or a raw handle (None: the default stream); own_stream: one the context makes itself."""
         self._h = C.c_void_p()
         self.device = device
         handle = None
@@ -203,6 +254,8 @@ class Context:
         st = lib().b200_ctx_create(C.byref(self._h), device, handle)
         if st != B200_OK:
             raise B200Error(f"b200_ctx_create: {lib().b200_status_string(st).decode()}")
+        if own_stream:
+            self.check(lib().b200_ctx_own_stream(self._h), "own_stream")
 
     def check(self, st: int, what: str):
         if st != B200_OK:
@@ -441,6 +494,17 @@ class GPT2:
         ctx.check(lib().b200_gpt2_create_tp(C.byref(self._h), ctx._h, C.byref(cc), max_B, max_T, tp_size, tp_rank),
                   "gpt2_create")
 
+    @classmethod
+    def from_folder(cls, ctx: Context, folder: str, max_B: int = 1, max_T: int | None = None):
+        """config.json with the fields of GPT2Config and model.bin, the raw fp32 parameters in param_offsets order."""
+        import json
+        with open(os.path.join(folder, "config.json")) as f:
+            j = json.load(f)
+        cfg = GPT2Config(**{k: j[k] for k in GPT2Config.__dataclass_fields__ if k in j})
+        m = cls(ctx, cfg, max_B, max_T or cfg.max_seq_len)
+        m.load_params_file(os.path.join(folder, "model.bin"), int(j.get("header_bytes", 0)))
+        return m
+
     @property
     def logits_width(self) -> int:
         Vp = self.cfg.padded_vocab_size
@@ -661,6 +725,130 @@ class GPT2:
         if self._h:
             lib().b200_gpt2_destroy(self._h)
             self._h = C.c_void_p()
+
+
+class Decoder:
+    """A layered decoder (config.json with a list of layers; driver/decoder.cu): weights, slots of
+    per-sequence cache and state, steps of any number of tokens, and generation.
+
+    dtype "bfloat16": bf16 weights and matrix products, fp32 residual, norms, scores and recurrences;
+    "float32": everything in fp32.  max_rows tokens run at a time (default: max_seq, at most 8192)."""
+    ARITHMETIC = {"bfloat16": 0, "float32": 1}
+    ARCHITECTURES = ("Vunolorn",)
+
+    def __init__(self, ctx: Context, config, dtype: str = "bfloat16", max_slots: int = 16, max_seq: int = 4096, max_rows: int | None = None):
+        import json
+        self.ctx, self.config = ctx, json.loads(config) if isinstance(config, str) else config
+        self.max_slots, self.max_seq = max_slots, max_seq
+        self.max_rows = max_rows or min(max_seq, 8192)
+        self._h = C.c_void_p()
+        ctx.check(lib().b200_decoder_create(C.byref(self._h), ctx._h, json.dumps(self.config).encode(), self.ARITHMETIC[dtype],
+                                            max_slots, max_seq, self.max_rows), "decoder_create")
+        self.vocab = int(lib().b200_decoder_vocab(self._h))
+
+    @classmethod
+    def from_folder(cls, ctx: Context, folder: str, **kw):
+        with open(os.path.join(folder, "config.json")) as f:
+            m = cls(ctx, f.read(), **kw)
+        m.load_safetensors(os.path.join(folder, "model.safetensors"))
+        return m
+
+    def load_safetensors(self, path: str):
+        self.ctx.check(lib().b200_decoder_load_safetensors(self._h, os.fsencode(path)), "load_safetensors")
+
+    def load_tensors(self, tensors):
+        """{name: numpy array}: float32, or uint16 holding bf16 bits."""
+        import numpy as np
+        for name, a in tensors.items():
+            a = np.ascontiguousarray(a)
+            if a.dtype not in (np.float32, np.uint16):
+                raise B200Error(f"{name}: float32 or bf16 bits as uint16, not {a.dtype}")
+            shape = (C.c_long * a.ndim)(*a.shape)
+            self.ctx.check(lib().b200_decoder_set_tensor(self._h, name.encode(), _ptr(a), int(a.dtype == np.float32), shape, a.ndim), "set_tensor")
+        self.ctx.check(lib().b200_decoder_finish_load(self._h), "finish_load")
+
+    def set_graph(self, on: bool):
+        self.ctx.check(lib().b200_decoder_set_graph(self._h, int(on)), "set_graph")
+
+    def open(self) -> int:
+        slot = C.c_int()
+        self.ctx.check(lib().b200_decoder_open(self._h, C.byref(slot)), "open")
+        return slot.value
+
+    def close_slot(self, slot: int):
+        self.ctx.check(lib().b200_decoder_close(self._h, slot), "close")
+
+    def length(self, slot: int) -> int:
+        return int(lib().b200_decoder_length(self._h, slot))
+
+    @staticmethod
+    def _pack(entries):
+        import numpy as np
+        slots = np.array([s for s, _ in entries], dtype=np.int32)
+        parts = [np.asarray(t, dtype=np.int32).reshape(-1) for _, t in entries]
+        return slots, np.array([p.size for p in parts], dtype=np.int32), np.ascontiguousarray(np.concatenate(parts))
+
+    def step(self, entries, want=None):
+        """entries: [(slot, next token ids)]; want: places among all of the step's tokens (default: the
+        last token of every entry).  Returns the logits there, [len(want), vocab] float32."""
+        import numpy as np
+        slots, counts, tokens = self._pack(entries)
+        want = np.cumsum(counts, dtype=np.int32) - 1 if want is None else np.asarray(want, dtype=np.int32).reshape(-1)
+        want = np.ascontiguousarray(want, dtype=np.int32)
+        out = np.empty((want.size, self.vocab), dtype=np.float32)
+        self.ctx.check(lib().b200_decoder_step(self._h, len(entries), _ptr(slots), _ptr(counts), _ptr(tokens), want.size, _ptr(want), _ptr(out)),
+                       "decoder_step")
+        return out
+
+    def prefill_device(self, entries, want=None):
+        """step() without waiting and without results on the host (for measurements)."""
+        import numpy as np
+        slots, counts, tokens = self._pack(entries)
+        want = np.cumsum(counts, dtype=np.int32) - 1 if want is None else np.asarray(want, dtype=np.int32)
+        want = np.ascontiguousarray(want, dtype=np.int32)
+        self.ctx.check(lib().b200_decoder_prefill_device(self._h, len(entries), _ptr(slots), _ptr(counts), _ptr(tokens), want.size, _ptr(want)),
+                       "decoder_prefill_device")
+
+    def decode_device(self, slots):
+        """One token for each slot, ids as the last step left them on the device (for measurements)."""
+        import numpy as np
+        s = np.asarray(slots, dtype=np.int32)
+        self.ctx.check(lib().b200_decoder_decode_device(self._h, s.size, _ptr(s)), "decoder_decode_device")
+
+    def generate(self, prompts, n_new: int, temperature: float = 0.0, top_k: int = 0, top_p: float = 0.0, seed: int = 0):
+        """Continuations [len(prompts), n_new] of prompts of unequal lengths (temperature 0: greedy)."""
+        import numpy as np
+        parts = [np.ascontiguousarray(np.asarray(p, dtype=np.int32).reshape(-1)) for p in prompts]
+        ptrs = (C.c_void_p * len(parts))(*[p.ctypes.data for p in parts])
+        lens = np.array([p.size for p in parts], dtype=np.int32)
+        out = np.empty((len(parts), n_new), dtype=np.int32)
+        self.ctx.check(lib().b200_decoder_generate(self._h, len(parts), ptrs, _ptr(lens), n_new, float(temperature), int(top_k), float(top_p),
+                                                   int(seed) & 0xFFFFFFFF, _ptr(out)), "decoder_generate")
+        return out
+
+    def close(self):
+        if self._h:
+            lib().b200_decoder_destroy(self._h)
+            self._h = C.c_void_p()
+
+
+def architecture(folder: str) -> str:
+    """The architecture that a model folder's config.json names."""
+    import json
+    with open(os.path.join(folder, "config.json")) as f:
+        return json.load(f).get("architecture", "")
+
+
+# Model registry: architecture -> (class, what build.py has to have built for it)
+MODELS = {"GPT2": (GPT2, "gpt2"), **{a: (Decoder, "decoder") for a in Decoder.ARCHITECTURES}}
+
+
+def model_class(folder: str):
+    """(class, build target) of the model in a folder, chosen by its config.json."""
+    name = architecture(folder)
+    if name not in MODELS:
+        raise B200Error(f"unknown architecture {name!r} (known: {', '.join(MODELS)})")
+    return MODELS[name]
 
 
 def gpt2_static_prepare(ctx: Context) -> int:

@@ -36,6 +36,7 @@ struct b200_ctx {
     int device = 0;
     int num_sms = 148;
     cudaStream_t stream = nullptr;
+    cudaStream_t own_stream = nullptr;  // b200_ctx_own_stream
     int* d_status = nullptr;  // device word: first device-side error code of any kernel
     int* h_status = nullptr;  // pinned host copy of that word, filled by b200_ctx_sync_check
     // CTA-pair GEMM with K slices: one flag word per (slice, tile, CTA, epilogue warp); all zero between launches

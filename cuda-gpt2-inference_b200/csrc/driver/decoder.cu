@@ -1,0 +1,1180 @@
+// Layered decoders: models whose configuration lists their layers, each with a mixer of some kind and a
+// feed-forward, served from per-sequence slots that hold whatever the mixers remember (key/value cache, recurrent
+// state, convolution history).
+//
+//   configuration  ModelSpec, read from config.json; a Design (registry below) fixes what all models of an
+//                  architecture share
+//   weights        safetensors or single tensors -> concatenated, padded matrices on the device
+//   slots          opened and closed by the caller or the generation loop; a slot carries one sequence's
+//                  length and needs no clearing (a sequence at position 0 starts from zero state)
+//   step           any number of tokens of any open sequences: the general path (prompts, portions), or, with one
+//                  token for each of at most 16 sequences in 16-bit arithmetic, the fused decode path, replayed
+//                  as a CUDA graph
+//   generate       the scheduler: admits requests to slots, runs their prompts in portions, then decodes all
+//                  active sequences together
+#include <cmath>
+#include <cstdio>
+#include <cstdlib>
+#include <cstring>
+#include <deque>
+#include <map>
+#include <new>
+#include <stdexcept>
+#include <string>
+#include <vector>
+#include "../api/ctx.h"
+#include "../kernels/decoder_kernels.h"
+#include "json.h"
+#include "weights.h"
+
+using namespace b200;
+
+namespace {
+
+// ------------------------------------------------------------------ configuration
+// What the models of one architecture have in common and config.json does not say.
+struct Design {
+    const char* name;
+    int mlp_act;        // of a dense feed-forward
+    bool qk_norm;       // attention: per-head RMS norm of queries and keys, with weights
+    bool value_norm;    // attention: values divided by their root mean square
+};
+const Design kDesigns[] = {
+    {"Vunolorn", ACT_GELU_ERF, true, true},
+};
+
+enum MixerKind { MIX_MAMBA1, MIX_DELTA, MIX_PARALLEL };
+
+struct AttentionSpec { int heads, kv_heads, dim, vdim, rot_dims; double rot_base; float scale; };
+struct LayerSpec {
+    MixerKind kind;
+    int conv = 0, dt_rank = 0, inner = 0, state = 0;           // mamba1 (and conv of delta)
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0;            // delta
+    AttentionSpec att{};                                       // parallel, left
+    int gru_width = 0;                                         // parallel, right
+    float left_scale = 1.f, right_scale = 1.f;
+    int ff = 0;                                                // 0: no feed-forward
+};
+struct ModelSpec {
+    const Design* design = nullptr;
+    int vocab = 0, width = 0;
+    float embed_scale = 1.f, eps = 1e-5f;
+    std::vector<LayerSpec> layers;
+};
+
+void positive(int v, const char* what) { if (v < 1) throw std::runtime_error(std::string("config: '") + what + "' must be positive"); }
+void head_groups(int heads, int kv_heads) {
+    positive(heads, "heads");
+    positive(kv_heads, "kv_heads");
+    if (heads % kv_heads) throw std::runtime_error("config: 'heads' must be a multiple of 'kv_heads'");
+}
+
+AttentionSpec parse_attention(const Json& m) {
+    AttentionSpec a{};
+    a.heads = m.integer("heads"); a.kv_heads = m.integer("kv_heads");
+    head_groups(a.heads, a.kv_heads);
+    a.dim = m.integer("dim"); a.vdim = m.integer("vdim");
+    positive(a.dim, "dim"); positive(a.vdim, "vdim");
+    if (a.dim > 256 || a.vdim > 256) throw std::runtime_error("config: attention heads of more than 256 dimensions");
+    a.scale = (float)m.number("scale");
+    if (!(a.scale > 0.f)) throw std::runtime_error("config: attention 'scale' must be positive");
+    const Json& r = m.at("rot");
+    a.rot_dims = r.integer("dims");
+    a.rot_base = r.number("base");
+    if (a.rot_dims < 0 || a.rot_dims % 2 || a.rot_dims > a.dim) throw std::runtime_error("config: rot.dims must be even and at most dim");
+    return a;
+}
+
+// mixer registry: config name -> reader of its sizes
+struct MixerType {
+    const char* name;
+    void (*parse)(const Json&, LayerSpec&);
+};
+const MixerType kMixers[] = {
+    {"mamba1", [](const Json& m, LayerSpec& l) {
+         l.kind = MIX_MAMBA1;
+         l.conv = m.integer("conv"); l.dt_rank = m.integer("dt_rank"); l.inner = m.integer("inner"); l.state = m.integer("state");
+         positive(l.conv, "conv"); positive(l.dt_rank, "dt_rank"); positive(l.inner, "inner"); positive(l.state, "state");
+         if (!selective_state_pad(l.state)) throw std::runtime_error("config: mamba1 'state' beyond 256");
+     }},
+    {"delta", [](const Json& m, LayerSpec& l) {
+         l.kind = MIX_DELTA;
+         l.conv = m.integer("conv"); l.heads = m.integer("heads"); l.kv_heads = m.integer("kv_heads");
+         l.dim = m.integer("dim"); l.vdim = m.integer("vdim");
+         positive(l.conv, "conv"); head_groups(l.heads, l.kv_heads); positive(l.dim, "dim"); positive(l.vdim, "vdim");
+         if (!delta_state_pad(l.dim)) throw std::runtime_error("config: delta 'dim' beyond 256");
+         if (l.vdim > 2048) throw std::runtime_error("config: delta 'vdim' beyond 2048");
+     }},
+    {"parallel", [](const Json& m, LayerSpec& l) {
+         l.kind = MIX_PARALLEL;
+         l.att = parse_attention(m.at("left"));
+         l.gru_width = m.at("right").integer("width");
+         positive(l.gru_width, "width");
+         l.left_scale = (float)m.number("left_scale");
+         l.right_scale = (float)m.number("right_scale");
+     }},
+};
+
+ModelSpec parse_config(const char* text) {
+    const Json j = Json::parse(text, text + strlen(text));
+    ModelSpec s;
+    const std::string& arch = j.string("architecture");
+    for (const Design& d : kDesigns)
+        if (arch == d.name) s.design = &d;
+    if (!s.design) throw std::runtime_error("config: unknown architecture '" + arch + "'");
+    s.vocab = j.integer("vocab"); s.width = j.integer("width");
+    positive(s.vocab, "vocab"); positive(s.width, "width");
+    s.embed_scale = (float)j.at("embedding").number("scale");
+    s.eps = (float)j.at("norm").number("eps");
+    const Json& layers = j.at("layers");
+    if (layers.kind != Json::ARR || layers.arr.empty()) throw std::runtime_error("config: 'layers' must be a list");
+    for (const Json& lj : layers.arr) {
+        LayerSpec l;
+        const std::string& type = lj.string("type");
+        const MixerType* mt = nullptr;
+        for (const MixerType& t : kMixers)
+            if (type == t.name) mt = &t;
+        if (!mt) throw std::runtime_error("config: unknown mixer '" + type + "'");
+        mt->parse(lj.at("mixer"), l);
+        const Json& mlp = lj.at("mlp");
+        if (!mlp.is_null()) {
+            if (mlp.string("kind") != "dense") throw std::runtime_error("config: unknown feed-forward '" + mlp.string("kind") + "'");
+            l.ff = mlp.integer("ff");
+            positive(l.ff, "ff");
+        }
+        s.layers.push_back(l);
+    }
+    return s;
+}
+
+// ------------------------------------------------------------------ the model on the device
+// A matrix [N, K] in the model's element type; N and K are padded with zeros.
+struct Matrix { void* w = nullptr; int N = 0, K = 0; float* bias = nullptr; };
+
+struct Mlp { Matrix up, down; };
+struct Layer {
+    const LayerSpec* spec = nullptr;
+    float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
+    Matrix in, o;            // the mixer's joint input projection and its output projection
+    Mlp mlp;
+    // mamba1: in = [x: np | z: np]; xp = [dt: rank_p | B: sp | C: sp]
+    Matrix xp, dt;
+    float *conv_w = nullptr, *conv_b = nullptr, *A2 = nullptr, *dt_b = nullptr, *D = nullptr;
+    int np = 0, sp = 0, rank_p = 0;
+    // delta: in = [q: G*Dl | k: G*Dl | v: H*Dvl | gate: H*Dvl | a: H | b: H]
+    float *negA = nullptr, *dt_bias = nullptr, *head_norm = nullptr;
+    int Dl = 0, Dvl = 0, k_col = 0, v_col = 0, gate_col = 0, a_col = 0, b_col = 0;
+    // parallel: in = [q | k | v | z | x | g], o over [attention: att_p | minGRU]
+    CachedAttention att{};
+    int z_col = 0, x_col = 0, g_col = 0, att_p = 0;
+    // what the slots hold
+    float *hist = nullptr, *S = nullptr;
+};
+
+struct Slot { bool open = false; int len = 0, bank = 0; };
+
+int round4(int n) { return (n + 3) & ~3; }
+
+}  // namespace
+
+struct b200_decoder {
+    b200_ctx* ctx = nullptr;
+    ModelSpec spec;
+    bool f32 = false;
+    int max_slots = 0, max_seq = 0, max_rows = 0, Tp = 0;
+    int C = 0, Cp = 0, Vp = 0;
+    bool ready = false;
+    bool use_graph = true;
+    TensorStore* store = nullptr;
+    std::vector<void*> owned;             // every device allocation
+    std::vector<Layer> layers;
+    void* embed = nullptr;
+    float* final_norm = nullptr;
+    Matrix head;
+    std::map<std::pair<int, double>, float2*> rot_tables;
+    std::vector<Slot> slots;
+    // activations of the general path
+    float *x = nullptr, *proj = nullptr, *y = nullptr, *aux = nullptr, *wide = nullptr;
+    void *h = nullptr, *conv = nullptr, *mix = nullptr, *q = nullptr, *low = nullptr;
+    float* logits = nullptr;
+    int logits_rows = 0;
+    // ... and of the decode path (fp32, 16 rows)
+    float *dx[2] = {nullptr, nullptr}, *dproj = nullptr, *dmix = nullptr, *dy = nullptr, *dconv = nullptr, *daux = nullptr, *dlogits = nullptr;
+    void* dh = nullptr;
+    float* partial = nullptr;
+    unsigned int* counters = nullptr;
+    // step descriptors: a ring of pinned buffers, one device buffer per path
+    static constexpr int kRing = 8;
+    int* pinned[kRing] = {};
+    cudaEvent_t ring_ev[kRing] = {};
+    int ring = 0;
+    size_t desc_ints = 0;
+    int* desc = nullptr;
+    SeqDesc* dseqs = nullptr;   // decode path: [16] descriptors, then 16 token ids
+    int* dtokens = nullptr;
+    std::map<int, cudaGraphExec_t> graphs;    // decode path, by B
+    std::map<int, uint64_t> graph_launches;
+    int* gen_log = nullptr;
+    size_t gen_log_ints = 0;
+};
+
+namespace {
+
+size_t elem(const b200_decoder* m) { return m->f32 ? 4 : 2; }
+
+void* device_zeros(b200_decoder* m, size_t bytes) {
+    void* p = nullptr;
+    if (bytes == 0) bytes = 16;
+    cudaError_t e = cudaMalloc(&p, bytes);
+    if (e != cudaSuccess) throw std::runtime_error(std::string("cudaMalloc: ") + cudaGetErrorString(e));
+    m->owned.push_back(p);
+    e = cudaMemset(p, 0, bytes);
+    if (e != cudaSuccess) throw std::runtime_error(std::string("cudaMemset: ") + cudaGetErrorString(e));
+    return p;
+}
+void* upload(b200_decoder* m, const void* src, size_t bytes) {
+    void* p = device_zeros(m, bytes);
+    const cudaError_t e = cudaMemcpy(p, src, bytes, cudaMemcpyHostToDevice);
+    if (e != cudaSuccess) throw std::runtime_error(std::string("cudaMemcpy: ") + cudaGetErrorString(e));
+    return p;
+}
+
+// ------------------------------------------------------------------ weights
+// Assembles a padded matrix from blocks of tensors, then uploads it in the model's element type.
+class MatrixBuilder {
+   public:
+    MatrixBuilder(b200_decoder* m, int N, int K) : m_(m), N_(N), K_(K) {
+        if (m->f32) f_.assign((size_t)N * K, 0.f);
+        else h_.assign((size_t)N * K, 0);
+    }
+    // rows `rows` of t (columns [0, cols)) to (row0, col0), times scale
+    void put(const HostTensor& t, int src_row0, int rows, int cols, int row0, int col0) {
+        for (int r = 0; r < rows; ++r) {
+            const size_t s = (size_t)(src_row0 + r) * cols, d = (size_t)(row0 + r) * K_ + col0;
+            if (m_->f32) for (int c = 0; c < cols; ++c) f_[d + c] = t.value(s + c);
+            else if (t.f32) for (int c = 0; c < cols; ++c) h_[d + c] = bf16_bits(t.value(s + c));
+            else memcpy(&h_[d], t.data + 2 * s, (size_t)cols * 2);
+        }
+    }
+    Matrix build() {
+        Matrix x;
+        x.N = N_; x.K = K_;
+        x.w = m_->f32 ? upload(m_, f_.data(), f_.size() * 4) : upload(m_, h_.data(), h_.size() * 2);
+        return x;
+    }
+
+   private:
+    b200_decoder* m_;
+    int N_, K_;
+    std::vector<float> f_;
+    std::vector<uint16_t> h_;
+};
+
+float* vector_f32(b200_decoder* m, const HostTensor& t, size_t padded) {
+    std::vector<float> v(padded, 0.f);
+    for (size_t i = 0; i < t.count(); ++i) v[i] = t.value(i);
+    return static_cast<float*>(upload(m, v.data(), padded * 4));
+}
+
+float2* rotation_table(b200_decoder* m, int dims, double base) {
+    const auto key = std::make_pair(dims, base);
+    auto it = m->rot_tables.find(key);
+    if (it != m->rot_tables.end()) return it->second;
+    const int half = dims / 2;
+    std::vector<float2> t((size_t)m->Tp * half);
+    for (int i = 0; i < half; ++i) {
+        const double f = pow(base, -2.0 * i / dims);
+        for (int p = 0; p < m->Tp; ++p) t[(size_t)p * half + i] = make_float2((float)cos(p * f), (float)sin(p * f));
+    }
+    return m->rot_tables[key] = static_cast<float2*>(upload(m, t.data(), t.size() * sizeof(float2)));
+}
+
+// convolution weights [channels, taps] -> [taps][np], channel c of the tensor to channel dst(c)
+void put_taps(std::vector<float>& w, int np, const HostTensor& t, int channels, int taps, int head, int head_l, int base) {
+    for (int c = 0; c < channels; ++c) {
+        const int d = base + c / head * head_l + c % head;
+        for (int j = 0; j < taps; ++j) w[(size_t)j * np + d] = t.value((size_t)c * taps + j);
+    }
+}
+
+void load_mamba1(b200_decoder* m, Layer& L, const std::string& p) {
+    const LayerSpec& s = *L.spec;
+    const TensorStore& w = *m->store;
+    const int C = m->C, n = s.inner;
+    L.np = pad_dim(n); L.sp = selective_state_pad(s.state); L.rank_p = pad_dim(s.dt_rank);
+    {
+        const HostTensor& t = w.get(p + ".in", {2L * n, C});
+        MatrixBuilder b(m, 2 * L.np, m->Cp);
+        b.put(t, 0, n, C, 0, 0);
+        b.put(t, n, n, C, L.np, 0);
+        L.in = b.build();
+    }
+    {
+        const HostTensor& t = w.get(p + ".x", {(long)s.dt_rank + 2L * s.state, n});
+        MatrixBuilder b(m, pad_dim(L.rank_p + 2 * L.sp), L.np);
+        b.put(t, 0, s.dt_rank, n, 0, 0);
+        b.put(t, s.dt_rank, s.state, n, L.rank_p, 0);
+        b.put(t, s.dt_rank + s.state, s.state, n, L.rank_p + L.sp, 0);
+        L.xp = b.build();
+    }
+    {
+        MatrixBuilder b(m, L.np, L.rank_p);
+        b.put(w.get(p + ".dt", {n, s.dt_rank}), 0, n, s.dt_rank, 0, 0);
+        L.dt = b.build();
+    }
+    {
+        MatrixBuilder b(m, m->Cp, L.np);
+        b.put(w.get(p + ".o", {C, n}), 0, C, n, 0, 0);
+        L.o = b.build();
+    }
+    std::vector<float> taps((size_t)s.conv * L.np, 0.f);
+    put_taps(taps, L.np, w.get(p + ".conv", {n, s.conv}), n, s.conv, n, n, 0);
+    L.conv_w = static_cast<float*>(upload(m, taps.data(), taps.size() * 4));
+    L.conv_b = vector_f32(m, w.get(p + ".conv.b", {n}), L.np);
+    L.dt_b = vector_f32(m, w.get(p + ".dt.b", {n}), L.np);
+    L.D = vector_f32(m, w.get(p + ".D", {n}), L.np);
+    const HostTensor& a = w.get(p + ".A_log", {n, s.state});
+    std::vector<float> A2((size_t)n * L.sp, 0.f);  // exponents for base 2
+    for (int c = 0; c < n; ++c)
+        for (int k = 0; k < s.state; ++k) A2[(size_t)c * L.sp + k] = (float)(-exp((double)a.value((size_t)c * s.state + k)) * 1.4426950408889634);
+    L.A2 = static_cast<float*>(upload(m, A2.data(), A2.size() * 4));
+    L.hist = static_cast<float*>(device_zeros(m, (size_t)2 * m->max_slots * (s.conv - 1) * L.np * 4));
+    L.S = static_cast<float*>(device_zeros(m, (size_t)m->max_slots * n * L.sp * 4));
+}
+
+void load_delta(b200_decoder* m, Layer& L, const std::string& p) {
+    const LayerSpec& s = *L.spec;
+    const TensorStore& w = *m->store;
+    const int C = m->C, H = s.heads, G = s.kv_heads, D = s.dim, Dv = s.vdim;
+    L.Dl = round4(D); L.Dvl = round4(Dv);
+    L.k_col = G * L.Dl; L.v_col = 2 * G * L.Dl;
+    L.np = L.v_col + H * L.Dvl;  // the convolved columns
+    L.gate_col = L.np; L.a_col = L.gate_col + H * L.Dvl; L.b_col = L.a_col + H;
+    MatrixBuilder b(m, pad_dim(L.b_col + H), m->Cp);
+    std::vector<float> taps((size_t)s.conv * L.np, 0.f);
+    const struct { const char* n; int heads, dim, dim_l, col; } parts[] = {{".q", G, D, L.Dl, 0}, {".k", G, D, L.Dl, L.k_col}, {".v", H, Dv, L.Dvl, L.v_col}};
+    for (const auto& a : parts) {
+        const HostTensor& t = w.get(p + a.n, {(long)a.heads * a.dim, C});
+        for (int h = 0; h < a.heads; ++h) b.put(t, h * a.dim, a.dim, C, a.col + h * a.dim_l, 0);
+        put_taps(taps, L.np, w.get(p + a.n + ".conv", {(long)a.heads * a.dim, s.conv}), a.heads * a.dim, s.conv, a.dim, a.dim_l, a.col);
+    }
+    const HostTensor& g = w.get(p + ".g", {(long)H * Dv, C});
+    for (int h = 0; h < H; ++h) b.put(g, h * Dv, Dv, C, L.gate_col + h * L.Dvl, 0);
+    b.put(w.get(p + ".a", {H, C}), 0, H, C, L.a_col, 0);
+    b.put(w.get(p + ".b", {H, C}), 0, H, C, L.b_col, 0);
+    L.in = b.build();
+    MatrixBuilder o(m, m->Cp, pad_dim(H * Dv));
+    o.put(w.get(p + ".o", {C, (long)H * Dv}), 0, C, H * Dv, 0, 0);
+    L.o = o.build();
+    L.conv_w = static_cast<float*>(upload(m, taps.data(), taps.size() * 4));
+    const HostTensor& a = w.get(p + ".A_log", {H});
+    std::vector<float> negA(H);
+    for (int h = 0; h < H; ++h) negA[h] = (float)-exp((double)a.value(h));
+    L.negA = static_cast<float*>(upload(m, negA.data(), negA.size() * 4));
+    L.dt_bias = vector_f32(m, w.get(p + ".dt_bias", {H}), H);
+    L.head_norm = vector_f32(m, w.get(p + ".norm", {Dv}), Dv);
+    L.hist = static_cast<float*>(device_zeros(m, (size_t)2 * m->max_slots * (s.conv - 1) * L.np * 4));
+    L.S = static_cast<float*>(device_zeros(m, (size_t)m->max_slots * H * Dv * delta_state_pad(D) * 4));
+}
+
+void load_parallel(b200_decoder* m, Layer& L, const std::string& p) {
+    const LayerSpec& s = *L.spec;
+    const AttentionSpec& a = s.att;
+    const TensorStore& w = *m->store;
+    const int C = m->C, W = s.gru_width;
+    const std::string l = p + ".left", r = p + ".right";
+    CachedAttention& c = L.att;
+    c.H = a.heads; c.G = a.kv_heads; c.D = a.dim; c.Dv = a.vdim;
+    c.Dp = attention_pad(a.dim); c.Dvp = attention_pad(a.vdim); c.Tp = m->Tp;
+    c.q_col = 0; c.k_col = a.heads * a.dim; c.v_col = c.k_col + a.kv_heads * a.dim;
+    L.z_col = (c.v_col + a.kv_heads * a.vdim + 7) & ~7;
+    L.x_col = L.z_col + ((W + 7) & ~7);
+    L.g_col = L.x_col + ((W + 7) & ~7);
+    const int N = pad_dim(L.g_col + W);
+    MatrixBuilder b(m, N, m->Cp);
+    b.put(w.get(l + ".q", {(long)a.heads * a.dim, C}), 0, a.heads * a.dim, C, c.q_col, 0);
+    b.put(w.get(l + ".k", {(long)a.kv_heads * a.dim, C}), 0, a.kv_heads * a.dim, C, c.k_col, 0);
+    b.put(w.get(l + ".v", {(long)a.kv_heads * a.vdim, C}), 0, a.kv_heads * a.vdim, C, c.v_col, 0);
+    b.put(w.get(r + ".z", {W, C}), 0, W, C, L.z_col, 0);
+    b.put(w.get(r + ".x", {W, C}), 0, W, C, L.x_col, 0);
+    b.put(w.get(r + ".g", {W, C}), 0, W, C, L.g_col, 0);
+    L.in = b.build();
+    std::vector<float> bias(N, 0.f);
+    const HostTensor &zb = w.get(r + ".z.b", {W}), &xb = w.get(r + ".x.b", {W});
+    for (int i = 0; i < W; ++i) { bias[L.z_col + i] = zb.value(i); bias[L.x_col + i] = xb.value(i); }
+    L.in.bias = static_cast<float*>(upload(m, bias.data(), bias.size() * 4));
+    // one output projection over both mixers; their scales are applied to its input
+    L.att_p = (a.heads * a.vdim + 7) & ~7;
+    MatrixBuilder o(m, m->Cp, pad_dim(L.att_p + W));
+    o.put(w.get(l + ".o", {C, (long)a.heads * a.vdim}), 0, C, a.heads * a.vdim, 0, 0);
+    o.put(w.get(r + ".o", {C, W}), 0, C, W, 0, L.att_p);
+    L.o = o.build();
+    c.rot_dims = a.rot_dims;
+    c.rot = a.rot_dims > 0 ? rotation_table(m, a.rot_dims, a.rot_base) : nullptr;
+    if (m->spec.design->qk_norm) {
+        c.q_norm = vector_f32(m, w.get(l + ".q.norm", {a.dim}), a.dim);
+        c.k_norm = vector_f32(m, w.get(l + ".k.norm", {a.dim}), a.dim);
+    }
+    c.v_norm = m->spec.design->value_norm;
+    c.scale = a.scale; c.eps = m->spec.eps; c.out_scale = s.left_scale;
+    c.K = device_zeros(m, (size_t)m->max_slots * c.G * c.Tp * c.Dp * elem(m));
+    c.V = device_zeros(m, (size_t)m->max_slots * c.G * c.Tp * c.Dvp * elem(m));
+    L.S = static_cast<float*>(device_zeros(m, (size_t)m->max_slots * W * 4));
+}
+
+void load_all(b200_decoder* m) {
+    const TensorStore& w = *m->store;
+    const int C = m->C, V = m->spec.vocab;
+    {
+        MatrixBuilder b(m, V, m->Cp);
+        b.put(w.get("embed", {V, C}), 0, V, C, 0, 0);
+        m->embed = b.build().w;
+    }
+    m->layers.assign(m->spec.layers.size(), Layer());
+    for (size_t i = 0; i < m->layers.size(); ++i) {
+        Layer& L = m->layers[i];
+        L.spec = &m->spec.layers[i];
+        const std::string p = "l" + std::to_string(i);
+        L.norm1 = vector_f32(m, w.get(p + ".norm1", {C}), m->Cp);
+        L.norm1b = vector_f32(m, w.get(p + ".norm1b", {C}), m->Cp);
+        if (L.spec->kind == MIX_MAMBA1) load_mamba1(m, L, p + ".mix");
+        else if (L.spec->kind == MIX_DELTA) load_delta(m, L, p + ".mix");
+        else load_parallel(m, L, p + ".mix");
+        if (L.spec->ff > 0) {
+            const int F = L.spec->ff, Fp = pad_dim(F);
+            L.norm2 = vector_f32(m, w.get(p + ".norm2", {C}), m->Cp);
+            L.norm2b = vector_f32(m, w.get(p + ".norm2b", {C}), m->Cp);
+            MatrixBuilder up(m, Fp, m->Cp), down(m, m->Cp, Fp);
+            up.put(w.get(p + ".mlp.up", {F, C}), 0, F, C, 0, 0);
+            down.put(w.get(p + ".mlp.down", {C, F}), 0, C, F, 0, 0);
+            L.mlp.up = up.build();
+            L.mlp.down = down.build();
+        }
+    }
+    m->final_norm = vector_f32(m, w.get("final.norm", {C}), m->Cp);
+    MatrixBuilder b(m, m->Vp, m->Cp);
+    b.put(w.get("head", {V, C}), 0, V, C, 0, 0);
+    m->head = b.build();
+}
+
+// activations, sized from the loaded layers
+void allocate(b200_decoder* m) {
+    size_t proj = 0, mix = 0, conv = 0, aux = 0, wide = 0, q = 0, low = 0, partial = 0, counters = 16;
+    auto up = [](size_t& a, size_t b) { if (b > a) a = b; };
+    for (const Layer& L : m->layers) {
+        up(proj, L.in.N);
+        up(mix, L.o.K);
+        if (L.spec->ff) up(mix, L.mlp.up.N);
+        if (L.spec->kind == MIX_MAMBA1) { up(conv, L.np); up(aux, L.xp.N); up(wide, L.np); up(low, L.rank_p); }
+        else if (L.spec->kind == MIX_DELTA) { up(conv, 2 * L.np); up(wide, L.spec->heads * L.Dvl); }  // (fp32 in either arithmetic)
+        else {
+            up(q, (size_t)L.att.H * L.att.Dp);
+            up(partial, attention_decode_partial_floats(L.att, 16));
+            up(counters, (size_t)16 * L.att.H);
+        }
+    }
+    const size_t M = m->max_rows, e = elem(m);
+    m->x = static_cast<float*>(device_zeros(m, M * m->Cp * 4));
+    m->h = device_zeros(m, M * m->Cp * e);
+    m->y = static_cast<float*>(device_zeros(m, M * m->Cp * 4));
+    m->proj = static_cast<float*>(device_zeros(m, M * proj * 4));
+    m->mix = device_zeros(m, M * mix * e);
+    m->conv = device_zeros(m, M * conv * (m->f32 ? 4 : 2));
+    m->aux = static_cast<float*>(device_zeros(m, M * aux * 4));
+    m->wide = static_cast<float*>(device_zeros(m, M * wide * 4));
+    m->low = device_zeros(m, M * low * e);
+    m->q = device_zeros(m, M * q * e);
+    if (!m->f32) {
+        for (float*& p : m->dx) p = static_cast<float*>(device_zeros(m, (size_t)16 * m->Cp * 4));
+        m->dy = static_cast<float*>(device_zeros(m, (size_t)16 * m->Cp * 4));
+        m->dh = device_zeros(m, (size_t)16 * m->Cp * 4);
+        m->dproj = static_cast<float*>(device_zeros(m, (size_t)16 * proj * 4));
+        m->dmix = static_cast<float*>(device_zeros(m, (size_t)16 * mix * 4));
+        m->dconv = static_cast<float*>(device_zeros(m, (size_t)16 * conv * 4));
+        m->daux = static_cast<float*>(device_zeros(m, (size_t)16 * aux * 4));
+        m->dlogits = static_cast<float*>(device_zeros(m, (size_t)16 * m->Vp * 4));
+        m->partial = static_cast<float*>(device_zeros(m, partial * 4));
+        m->counters = static_cast<unsigned int*>(device_zeros(m, counters * 4));
+    }
+    // descriptors: sequences, tokens, the sequence of every row, wanted rows, query-tile pairs
+    m->desc_ints = (size_t)m->max_slots * 8 + 3 * M + 2 * (M / 256 + m->max_slots + 1) + 64;
+    if (m->desc_ints < 16 * 9) m->desc_ints = 16 * 9;
+    m->desc = static_cast<int*>(device_zeros(m, m->desc_ints * 4));
+    m->dseqs = static_cast<SeqDesc*>(device_zeros(m, 16 * (sizeof(SeqDesc) + 4)));
+    m->dtokens = reinterpret_cast<int*>(m->dseqs + 16);
+    for (int i = 0; i < b200_decoder::kRing; ++i) {
+        if (cudaHostAlloc(&m->pinned[i], m->desc_ints * 4, cudaHostAllocDefault) != cudaSuccess ||
+            cudaEventCreateWithFlags(&m->ring_ev[i], cudaEventDisableTiming) != cudaSuccess)
+            throw std::runtime_error("pinned descriptor buffers");
+    }
+}
+
+int finish_load(b200_decoder* m) {
+    b200_device_guard guard(m->ctx);
+    try {
+        load_all(m);
+        allocate(m);
+    } catch (const std::exception& e) {
+        m->ctx->last_error = e.what();
+        return B200_ERR_STATE;
+    }
+    delete m->store;
+    m->store = nullptr;
+    const cudaError_t e = cudaDeviceSynchronize();  // the fills above ran on the default stream
+    if (e != cudaSuccess) return b200_fail_cuda(m->ctx, e, "loading weights");
+    m->ready = true;
+    return B200_OK;
+}
+
+#define TRY(call) do { const int st__ = (call); if (st__ != B200_OK) return st__; } while (0)
+
+// ------------------------------------------------------------------ general path
+// out = act(in W^T + bias); out is fp32, or with elem_out the model's element type
+int product(b200_decoder* m, void* out, const void* in, const Matrix& w, int M, int act = ACT_NONE, bool elem_out = false) {
+    b200_ctx* ctx = m->ctx;
+    if (m->f32) {
+        if (M <= 16 && act == ACT_NONE && (size_t)(M <= 8 ? 8 : 16) * w.K * 4 <= (size_t)160 * 1024)
+            return launch_skinny_gemm(ctx, static_cast<float*>(out), static_cast<const float*>(in), static_cast<const float*>(w.w), w.bias, M, w.K, w.N, 0);
+        return launch_gemm_fp32(ctx, static_cast<float*>(out), static_cast<const float*>(in), static_cast<const float*>(w.w), w.bias, M, w.K, w.N, act);
+    }
+    const int flags = act == ACT_GELU_ERF ? GEMM_GELU_ERF : (act == ACT_GELU_TANH ? GEMM_GELU : 0);
+    return launch_gemm_bf16(ctx, elem_out ? nullptr : static_cast<float*>(out), elem_out ? static_cast<uint16_t*>(out) : nullptr,
+                            static_cast<const uint16_t*>(in), static_cast<const uint16_t*>(w.w), w.bias, M, w.K, w.N, flags);
+}
+
+struct StepView {
+    const SeqDesc* seqs; const int* tokens; const int* row_seq; const int* want; const int2* pairs;
+    int E, M, max_n, n_want, num_pairs;
+};
+
+int mixer_mamba1(b200_decoder* m, const Layer& L, const StepView& v) {
+    b200_ctx* ctx = m->ctx;
+    const LayerSpec& s = *L.spec;
+    TRY(product(m, m->proj, m->h, L.in, v.M));
+    ShortConvArgs c{};
+    c.x = m->proj; c.ldx = L.in.N; c.out = m->conv; c.ld_out = L.np; c.w = L.conv_w; c.bias = L.conv_b; c.hist = L.hist; c.seqs = v.seqs;
+    c.np = L.np; c.taps = s.conv; c.max_slots = m->max_slots;
+    TRY(launch_short_conv(ctx, c, v.E, v.max_n, m->f32));
+    TRY(product(m, m->aux, m->conv, L.xp, v.M));
+    TRY(launch_slice(ctx, m->low, L.rank_p, m->aux, L.xp.N, s.dt_rank, v.M, m->f32));
+    TRY(product(m, m->wide, m->low, L.dt, v.M));
+    SelectiveScanArgs a{};
+    a.x = m->conv; a.ldx = L.np; a.dt = m->wide; a.lddt = L.np; a.bc = m->aux; a.ldbc = L.xp.N; a.b_col = L.rank_p; a.c_col = L.rank_p + L.sp;
+    a.z = m->proj + L.np; a.ldz = L.in.N; a.A2 = L.A2; a.dt_b = L.dt_b; a.D = L.D; a.S = L.S; a.out = m->mix; a.ldo = L.o.K; a.seqs = v.seqs;
+    a.inner = s.inner; a.state_pad = L.sp;
+    return launch_selective_scan(ctx, a, v.E, v.max_n, m->f32, m->f32);
+}
+
+DeltaArgs delta_args(const b200_decoder* m, const Layer& L, const SeqDesc* seqs, const float* proj) {
+    const LayerSpec& s = *L.spec;
+    DeltaArgs a{};
+    a.ld = L.np; a.k_col = L.k_col; a.v_col = L.v_col;
+    a.gates = proj; a.ldg = L.in.N; a.a_col = L.a_col; a.b_col = L.b_col;
+    a.negA = L.negA; a.dt_bias = L.dt_bias; a.S = L.S; a.seqs = seqs;
+    a.H = s.heads; a.G = s.kv_heads; a.D = s.dim; a.Dl = L.Dl; a.Dv = s.vdim; a.Dvl = L.Dvl;
+    a.conv_w = L.conv_w; a.hist = L.hist; a.taps = s.conv; a.np = L.np; a.max_slots = m->max_slots;
+    a.norm_w = L.head_norm; a.gate_col = L.gate_col; a.eps = m->spec.eps;
+    return a;
+}
+
+int mixer_delta(b200_decoder* m, const Layer& L, const StepView& v) {
+    b200_ctx* ctx = m->ctx;
+    const LayerSpec& s = *L.spec;
+    TRY(product(m, m->proj, m->h, L.in, v.M));
+    ShortConvArgs c{};
+    c.x = m->proj; c.ldx = L.in.N; c.out = m->conv; c.ld_out = L.np; c.w = L.conv_w; c.hist = L.hist; c.seqs = v.seqs;
+    c.np = L.np; c.taps = s.conv; c.max_slots = m->max_slots;
+    TRY(launch_short_conv(ctx, c, v.E, v.max_n, true));
+    DeltaArgs a = delta_args(m, L, v.seqs, m->proj);
+    a.qkv = static_cast<const float*>(m->conv);
+    a.out = m->wide; a.ldo = s.heads * L.Dvl;
+    TRY(launch_delta_scan(ctx, a, v.E));
+    return launch_gated_head_norm(ctx, m->mix, L.o.K, m->wide, a.ldo, m->proj + L.gate_col, L.in.N, L.head_norm, v.M, s.heads, s.vdim, L.Dvl,
+                                  m->spec.eps, m->f32);
+}
+
+MinGruArgs gru_args(const b200_decoder* m, const Layer& L, const SeqDesc* seqs, const float* proj, void* out, size_t out_elem) {
+    MinGruArgs g{};
+    g.zx = proj; g.ld = L.in.N; g.z_col = L.z_col; g.x_col = L.x_col; g.g_col = L.g_col; g.S = L.S;
+    g.out = static_cast<char*>(out) + (size_t)L.att_p * out_elem; g.ldo = L.o.K; g.seqs = seqs; g.width = L.spec->gru_width; g.out_scale = L.spec->right_scale;
+    (void)m;
+    return g;
+}
+
+int mixer_parallel(b200_decoder* m, const Layer& L, const StepView& v) {
+    b200_ctx* ctx = m->ctx;
+    TRY(product(m, m->proj, m->h, L.in, v.M));
+    TRY(launch_attention_prep(ctx, L.att, m->proj, L.in.N, m->q, v.seqs, v.row_seq, v.M, m->f32));
+    if (!m->f32 && attention_cached_has_mma(L.att))
+        TRY(launch_attention_cached_mma(ctx, L.att, m->q, m->mix, L.o.K, v.seqs, v.pairs, v.num_pairs, v.M, m->max_slots));
+    else
+        TRY(launch_attention_cached_simt(ctx, L.att, m->q, m->mix, L.o.K, v.seqs, v.E, v.max_n, m->f32));
+    return launch_min_gru(ctx, gru_args(m, L, v.seqs, m->proj, m->mix, elem(m)), v.E, m->f32);
+}
+
+// rows of the step -> logits of the wanted rows in m->logits
+int enqueue_general(b200_decoder* m, const StepView& v) {
+    b200_ctx* ctx = m->ctx;
+    ResidualNormArgs n{};
+    n.C = m->C; n.Cp = m->Cp; n.eps = m->spec.eps; n.vocab = m->spec.vocab;
+    n.x_out = m->x; n.h = m->h; n.M = v.M;
+    n.tok = v.tokens; n.embed = m->embed; n.embed_scale = m->spec.embed_scale;
+    n.w = m->layers[0].norm1;
+    TRY(launch_residual_rms(ctx, n, m->f32));
+    n.tok = nullptr;
+    n.x = m->x;
+    n.y = m->y;
+    for (size_t i = 0; i < m->layers.size(); ++i) {
+        const Layer& L = m->layers[i];
+        if (L.spec->kind == MIX_MAMBA1) TRY(mixer_mamba1(m, L, v));
+        else if (L.spec->kind == MIX_DELTA) TRY(mixer_delta(m, L, v));
+        else TRY(mixer_parallel(m, L, v));
+        TRY(product(m, m->y, m->mix, L.o, v.M));
+        const bool last = i + 1 == m->layers.size();
+        n.wb = L.norm1b;
+        if (L.spec->ff > 0) {
+            n.w = L.norm2;
+            TRY(launch_residual_rms(ctx, n, m->f32));
+            TRY(product(m, m->mix, m->h, L.mlp.up, v.M, m->spec.design->mlp_act, true));
+            TRY(product(m, m->y, m->mix, L.mlp.down, v.M));
+            n.wb = L.norm2b;
+        }
+        if (!last) {
+            n.w = m->layers[i + 1].norm1;
+            TRY(launch_residual_rms(ctx, n, m->f32));
+        }
+    }
+    if (v.n_want == 0) return B200_OK;
+    n.w = m->final_norm;  // only the wanted rows go on
+    n.rows = v.want;
+    n.M = v.n_want;
+    n.x_out = nullptr;
+    TRY(launch_residual_rms(ctx, n, m->f32));
+    return product(m, m->logits, m->h, m->head, v.n_want);
+}
+
+// ------------------------------------------------------------------ decode path
+// One token for each of B <= 16 sequences: descriptors and tokens come from dseqs / dtokens, the logits go to
+// dlogits.  Every norm runs in the prologue of the product that follows it; the residual stream alternates
+// between two buffers because the product's other CTAs still read the old one.
+int enqueue_decode(b200_decoder* m, int B) {
+    b200_ctx* ctx = m->ctx;
+    float *xa = m->dx[0], *xb = m->dx[1];
+    const float *pending = nullptr, *pending_w = nullptr;  // branch output and the norm behind it, not yet in the residual
+    bool first = true;
+    const bool fused = decode_gemm_fits(m->Cp, B);
+    auto residual = [&](float* out, int ldo, const Matrix& w, const float* norm, int act) {
+        DecodeGemmArgs a{};
+        a.out = out; a.ldo = ldo; a.W = static_cast<const uint16_t*>(w.w); a.bias = w.bias; a.B = B; a.N = w.N; a.K = w.K; a.act = act;
+        a.status = ctx->d_status;
+        int st;
+        if (fused) {
+            a.x = xa; a.y = pending; a.wb = pending_w; a.w = norm; a.x_out = xb; a.C = m->C; a.eps = m->spec.eps; a.vocab = m->spec.vocab;
+            if (first) { a.tok = m->dtokens; a.embed = static_cast<const uint16_t*>(m->embed); a.embed_scale = m->spec.embed_scale; }
+            st = launch_decode_gemm(ctx, a, DPRO_RESIDUAL);
+        } else {
+            // rows too long for the prologue: a kernel of its own, with fp32 rows between them
+            ResidualNormArgs n{};
+            n.C = m->C; n.Cp = m->Cp; n.eps = m->spec.eps; n.vocab = m->spec.vocab; n.M = B;
+            n.x = xa; n.y = pending; n.wb = pending_w; n.w = norm; n.x_out = xb; n.h = m->dh;
+            st = B200_OK;
+            if (first) {  // the embedding's rows are bf16: into the residual first
+                ResidualNormArgs e = n;
+                e.x = nullptr; e.y = nullptr; e.w = nullptr; e.tok = m->dtokens; e.embed = m->embed; e.embed_scale = m->spec.embed_scale; e.x_out = xa;
+                st = launch_residual_rms(ctx, e, false);
+            }
+            if (st == B200_OK) st = launch_residual_rms(ctx, n, true);
+            a.x = static_cast<const float*>(m->dh); a.ldx = m->Cp;
+            if (st == B200_OK) st = launch_decode_gemm(ctx, a, DPRO_PLAIN);
+        }
+        first = false;
+        std::swap(xa, xb);
+        return st;
+    };
+    auto plain = [&](float* out, const float* in, int ldx, const Matrix& w) {
+        DecodeGemmArgs a{};
+        a.out = out; a.ldo = w.N; a.W = static_cast<const uint16_t*>(w.w); a.bias = w.bias; a.B = B; a.N = w.N; a.K = w.K;
+        a.x = in; a.ldx = ldx; a.status = ctx->d_status;
+        return launch_decode_gemm(ctx, a, DPRO_PLAIN);
+    };
+    for (const Layer& L : m->layers) {
+        const LayerSpec& s = *L.spec;
+        TRY(residual(m->dproj, L.in.N, L.in, L.norm1, ACT_NONE));
+        if (s.kind == MIX_MAMBA1) {
+            DecodeGemmArgs a{};
+            a.out = m->daux; a.ldo = L.xp.N; a.W = static_cast<const uint16_t*>(L.xp.w); a.B = B; a.N = L.xp.N; a.K = L.np;
+            a.seqs = m->dseqs; a.conv_w = L.conv_w; a.conv_b = L.conv_b; a.hist = L.hist; a.taps = s.conv; a.max_slots = m->max_slots;
+            a.status = ctx->d_status;
+            if (decode_gemm_fits(L.np, B)) {
+                a.x = m->dproj; a.ldx = L.in.N; a.conv_out = m->dconv;
+                TRY(launch_decode_gemm(ctx, a, DPRO_CONV));
+            } else {
+                ShortConvArgs c{};
+                c.x = m->dproj; c.ldx = L.in.N; c.out = m->dconv; c.ld_out = L.np; c.w = L.conv_w; c.bias = L.conv_b; c.hist = L.hist; c.seqs = m->dseqs;
+                c.np = L.np; c.taps = s.conv; c.max_slots = m->max_slots;
+                TRY(launch_short_conv(ctx, c, B, 1, true));
+                a.x = m->dconv; a.ldx = L.np;
+                TRY(launch_decode_gemm(ctx, a, DPRO_PLAIN));
+            }
+            SelectiveScanArgs c{};
+            c.x = m->dconv; c.ldx = L.np; c.bc = m->daux; c.ldbc = L.xp.N; c.b_col = L.rank_p; c.c_col = L.rank_p + L.sp;
+            c.z = m->dproj + L.np; c.ldz = L.in.N; c.A2 = L.A2; c.dt_b = L.dt_b; c.D = L.D; c.S = L.S; c.out = m->dmix; c.ldo = L.o.K; c.seqs = m->dseqs;
+            c.inner = s.inner; c.state_pad = L.sp;
+            c.Wdt = static_cast<const uint16_t*>(L.dt.w); c.rank = s.dt_rank; c.ld_wdt = L.rank_p;
+            TRY(launch_selective_scan(ctx, c, B, 1, true, true));
+        } else if (s.kind == MIX_DELTA) {
+            DeltaArgs a = delta_args(m, L, m->dseqs, m->dproj);
+            a.qkv = m->dproj; a.ld = L.in.N;
+            a.out = m->dmix; a.ldo = L.o.K;
+            TRY(launch_delta_step(ctx, a, B));
+        } else {
+            TRY(launch_attention_cached_decode(ctx, L.att, m->dproj, L.in.N, m->dmix, L.o.K, m->dseqs, B, m->partial, m->counters,
+                                               gru_args(m, L, m->dseqs, m->dproj, m->dmix, 4)));
+        }
+        TRY(plain(m->dy, m->dmix, L.o.K, L.o));
+        pending = m->dy;
+        pending_w = L.norm1b;
+        if (s.ff > 0) {
+            TRY(residual(m->dmix, L.mlp.up.N, L.mlp.up, L.norm2, m->spec.design->mlp_act));
+            TRY(plain(m->dy, m->dmix, L.mlp.up.N, L.mlp.down));
+            pending_w = L.norm2b;
+        }
+    }
+    return residual(m->dlogits, m->Vp, m->head, m->final_norm, ACT_NONE);
+}
+
+// ------------------------------------------------------------------ steps
+// the next pinned descriptor buffer, free to be written
+int ring_buffer(b200_decoder* m, int** out) {
+    m->ring = (m->ring + 1) % b200_decoder::kRing;
+    B200_CUDA(m->ctx, cudaEventSynchronize(m->ring_ev[m->ring]));
+    *out = m->pinned[m->ring];
+    return B200_OK;
+}
+
+struct Entry { int slot; const int* tokens; int n; };
+
+SeqDesc describe(b200_decoder* m, int slot, int row0, int n) {
+    Slot& s = m->slots[slot];
+    SeqDesc d{};
+    d.row0 = row0; d.n = n; d.slot = slot; d.pos0 = s.len; d.bank = s.bank;
+    s.len += n;
+    s.bank ^= 1;
+    return d;
+}
+
+// decode path: tokens == nullptr keeps the ids that are in dtokens already
+int decode_step(b200_decoder* m, const std::vector<int>& slots, const int* tokens) {
+    b200_ctx* ctx = m->ctx;
+    const int B = (int)slots.size();
+    int* host;
+    TRY(ring_buffer(m, &host));
+    SeqDesc* sd = reinterpret_cast<SeqDesc*>(host);
+    for (int b = 0; b < B; ++b) sd[b] = describe(m, slots[b], b, 1);
+    B200_CUDA(ctx, cudaMemcpyAsync(m->dseqs, sd, B * sizeof(SeqDesc), cudaMemcpyHostToDevice, ctx->stream));
+    if (tokens) {
+        int* t = host + 16 * 8;
+        for (int b = 0; b < B; ++b) t[b] = tokens[b];
+        B200_CUDA(ctx, cudaMemcpyAsync(m->dtokens, t, B * 4, cudaMemcpyHostToDevice, ctx->stream));
+    }
+    B200_CUDA(ctx, cudaEventRecord(m->ring_ev[m->ring], ctx->stream));
+    if (!m->use_graph || ctx->stream == nullptr) return enqueue_decode(m, B);
+    auto it = m->graphs.find(B);
+    if (it == m->graphs.end()) {
+        // The first step of a batch size runs eagerly (kernel attributes are set outside of capture) and is
+        // captured behind that, for the following ones.
+        TRY(enqueue_decode(m, B));
+        B200_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+        const uint64_t before = ctx->launches;
+        cudaGraph_t graph = nullptr;
+        B200_CUDA(ctx, cudaStreamBeginCapture(ctx->stream, cudaStreamCaptureModeThreadLocal));
+        const int st = enqueue_decode(m, B);
+        const cudaError_t e = cudaStreamEndCapture(ctx->stream, &graph);
+        m->graph_launches[B] = ctx->launches - before;
+        ctx->launches = before;
+        if (st != B200_OK) { if (graph) cudaGraphDestroy(graph); return st; }
+        if (e != cudaSuccess) return b200_fail_cuda(ctx, e, "cudaStreamEndCapture");
+        cudaGraphExec_t exec = nullptr;
+        const cudaError_t ie = cudaGraphInstantiate(&exec, graph, 0);
+        cudaGraphDestroy(graph);
+        if (ie != cudaSuccess) return b200_fail_cuda(ctx, ie, "cudaGraphInstantiate");
+        m->graphs.emplace(B, exec);
+        return B200_OK;
+    }
+    B200_CUDA(ctx, cudaGraphLaunch(it->second, ctx->stream));
+    ctx->launches += m->graph_launches[B];
+    return B200_OK;
+}
+
+int general_step(b200_decoder* m, const std::vector<Entry>& entries, const std::vector<int>& want) {
+    b200_ctx* ctx = m->ctx;
+    int M = 0, max_n = 0;
+    for (const Entry& e : entries) { M += e.n; if (e.n > max_n) max_n = e.n; }
+    const int E = (int)entries.size(), nw = (int)want.size();
+    if (nw > m->logits_rows) {
+        B200_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+        if (m->logits) cudaFree(m->logits);
+        m->logits = nullptr;
+        m->logits_rows = 0;
+        B200_CUDA(ctx, cudaMalloc(&m->logits, (size_t)nw * m->Vp * 4));
+        m->logits_rows = nw;
+    }
+    int* host;
+    TRY(ring_buffer(m, &host));
+    SeqDesc* sd = reinterpret_cast<SeqDesc*>(host);
+    int* tok = host + 8 * E;
+    int* row_seq = tok + M;
+    int* w = row_seq + M;
+    int* pr = w + nw;
+    if ((pr - host) & 1) ++pr;  // int2
+    struct Pair { int seq, pair, keys; };
+    std::vector<Pair> pairs;
+    int row = 0;
+    for (int i = 0; i < E; ++i) {
+        const Entry& e = entries[i];
+        sd[i] = describe(m, e.slot, row, e.n);
+        for (int t = 0; t < e.n; ++t) { tok[row + t] = e.tokens[t]; row_seq[row + t] = i; }
+        for (int p = 0; p * 256 < e.n; ++p) pairs.push_back({i, p, sd[i].pos0 + (e.n < (p + 1) * 256 ? e.n : (p + 1) * 256)});
+        row += e.n;
+    }
+    for (int i = 0; i < nw; ++i) w[i] = want[i];
+    // most keys first (stable, so the list is the same for the same step)
+    for (size_t i = 1; i < pairs.size(); ++i)
+        for (size_t j = i; j > 0 && pairs[j - 1].keys < pairs[j].keys; --j) std::swap(pairs[j - 1], pairs[j]);
+    for (size_t i = 0; i < pairs.size(); ++i) { pr[2 * i] = pairs[i].seq; pr[2 * i + 1] = pairs[i].pair; }
+    const size_t used = (pr - host) + 2 * pairs.size();
+    if (used > m->desc_ints) return B200_ERR_LIMIT;
+    B200_CUDA(ctx, cudaMemcpyAsync(m->desc, host, used * 4, cudaMemcpyHostToDevice, ctx->stream));
+    B200_CUDA(ctx, cudaEventRecord(m->ring_ev[m->ring], ctx->stream));
+    StepView v;
+    v.seqs = reinterpret_cast<const SeqDesc*>(m->desc);
+    v.tokens = m->desc + (tok - host);
+    v.row_seq = m->desc + (row_seq - host);
+    v.want = m->desc + (w - host);
+    v.pairs = reinterpret_cast<const int2*>(m->desc + (pr - host));
+    v.E = E; v.M = M; v.max_n = max_n; v.n_want = nw; v.num_pairs = (int)pairs.size();
+    return enqueue_general(m, v);
+}
+
+}  // namespace
+
+extern "C" {
+
+int b200_decoder_create(b200_decoder** out, b200_ctx* ctx, const char* config_json, int arithmetic, int max_slots, int max_seq, int max_rows) {
+    if (!out || !ctx || !config_json) return B200_ERR_NULL;
+    *out = nullptr;
+    if (arithmetic != B200_DECODER_BF16 && arithmetic != B200_DECODER_FP32) return B200_ERR_SHAPE;
+    if (max_slots < 1 || max_seq < 1 || max_rows < 1) return B200_ERR_SHAPE;
+    b200_decoder* m = new (std::nothrow) b200_decoder();
+    if (!m) return B200_ERR_CUDA;
+    try {
+        m->spec = parse_config(config_json);
+    } catch (const std::exception& e) {
+        ctx->last_error = e.what();
+        delete m;
+        return B200_ERR_SHAPE;
+    }
+    m->ctx = ctx;
+    m->f32 = arithmetic == B200_DECODER_FP32;
+    m->max_slots = max_slots; m->max_seq = max_seq; m->max_rows = max_rows;
+    m->Tp = (max_seq + 127) / 128 * 128;
+    m->C = m->spec.width; m->Cp = pad_dim(m->C); m->Vp = pad_dim(m->spec.vocab);
+    m->slots.assign(max_slots, Slot());
+    m->store = new TensorStore();
+    *out = m;
+    return B200_OK;
+}
+
+int b200_decoder_destroy(b200_decoder* m) {
+    if (!m) return B200_ERR_NULL;
+    b200_device_guard guard(m->ctx);
+    cudaStreamSynchronize(m->ctx->stream);
+    for (auto& g : m->graphs) cudaGraphExecDestroy(g.second);
+    for (void* p : m->owned) cudaFree(p);
+    if (m->logits) cudaFree(m->logits);
+    if (m->gen_log) cudaFree(m->gen_log);
+    for (int i = 0; i < b200_decoder::kRing; ++i) {
+        if (m->pinned[i]) cudaFreeHost(m->pinned[i]);
+        if (m->ring_ev[i]) cudaEventDestroy(m->ring_ev[i]);
+    }
+    m->ctx->tmap_cache.clear();  // the addresses may come back with other shapes
+    delete m->store;
+    delete m;
+    return B200_OK;
+}
+
+int b200_decoder_vocab(const b200_decoder* m) { return m ? m->spec.vocab : 0; }
+
+int b200_decoder_set_tensor(b200_decoder* m, const char* name, const void* data, int is_f32, const long* shape, int ndim) {
+    if (!m || !name || !data || !shape) return B200_ERR_NULL;
+    if (m->ready) return B200_ERR_STATE;
+    m->store->set(name, data, is_f32 != 0, std::vector<long>(shape, shape + ndim));
+    return B200_OK;
+}
+
+int b200_decoder_finish_load(b200_decoder* m) {
+    if (!m) return B200_ERR_NULL;
+    if (m->ready) return B200_ERR_STATE;
+    return finish_load(m);
+}
+
+int b200_decoder_load_safetensors(b200_decoder* m, const char* path) {
+    if (!m || !path) return B200_ERR_NULL;
+    if (m->ready) return B200_ERR_STATE;
+    try {
+        m->store->open_safetensors(path);
+    } catch (const std::exception& e) {
+        m->ctx->last_error = e.what();
+        return B200_ERR_STATE;
+    }
+    return finish_load(m);
+}
+
+int b200_decoder_set_graph(b200_decoder* m, int use_graph) {
+    if (!m) return B200_ERR_NULL;
+    m->use_graph = use_graph != 0;
+    return B200_OK;
+}
+
+int b200_decoder_open(b200_decoder* m, int* slot) {
+    if (!m || !slot) return B200_ERR_NULL;
+    for (int i = 0; i < m->max_slots; ++i)
+        if (!m->slots[i].open) {
+            m->slots[i] = Slot();
+            m->slots[i].open = true;
+            *slot = i;
+            return B200_OK;
+        }
+    m->ctx->last_error = "no free slot";
+    return B200_ERR_LIMIT;
+}
+
+int b200_decoder_close(b200_decoder* m, int slot) {
+    if (!m) return B200_ERR_NULL;
+    if (slot < 0 || slot >= m->max_slots || !m->slots[slot].open) return B200_ERR_STATE;
+    m->slots[slot].open = false;
+    return B200_OK;
+}
+
+int b200_decoder_length(const b200_decoder* m, int slot) {
+    return (m && slot >= 0 && slot < m->max_slots && m->slots[slot].open) ? m->slots[slot].len : -1;
+}
+
+int b200_decoder_step(b200_decoder* m, int n_entries, const int* slots, const int* counts, const int* tokens, int n_want, const int* want_rows,
+                      float* logits_host) {
+    if (!m || !slots || !counts || !tokens) return B200_ERR_NULL;
+    if (n_want < 0 || (n_want > 0 && !want_rows)) return B200_ERR_NULL;
+    if (!m->ready) return B200_ERR_STATE;
+    b200_ctx* ctx = m->ctx;
+    if (n_entries < 1 || n_entries > m->max_slots) return B200_ERR_SHAPE;
+    long total = 0;
+    bool single = true;
+    std::vector<char> seen(m->max_slots, 0);
+    for (int i = 0; i < n_entries; ++i) {
+        const int s = slots[i];
+        if (s < 0 || s >= m->max_slots || !m->slots[s].open || seen[s]) { ctx->last_error = "step: slot not open, or named twice"; return B200_ERR_STATE; }
+        seen[s] = 1;
+        if (counts[i] < 1) { ctx->last_error = "step: an entry without tokens"; return B200_ERR_SHAPE; }
+        if ((long)m->slots[s].len + counts[i] > m->max_seq) { ctx->last_error = "step: sequence beyond max_seq"; return B200_ERR_LIMIT; }
+        total += counts[i];
+        single = single && counts[i] == 1;
+    }
+    for (long i = 0; i < total; ++i)
+        if (tokens[i] < 0 || tokens[i] >= m->spec.vocab) { ctx->last_error = "step: token id outside the vocabulary"; return B200_ERR_SHAPE; }
+    for (int i = 0; i < n_want; ++i)
+        if (want_rows[i] < 0 || want_rows[i] >= total) { ctx->last_error = "step: wanted row outside the step"; return B200_ERR_SHAPE; }
+    b200_device_guard guard(ctx);
+    const size_t V = m->spec.vocab;
+    if (single && !m->f32 && n_entries <= 16) {
+        TRY(decode_step(m, std::vector<int>(slots, slots + n_entries), tokens));
+        if (logits_host)
+            for (int i = 0; i < n_want; ++i)
+                B200_CUDA(ctx, cudaMemcpyAsync(logits_host + i * V, m->dlogits + (size_t)want_rows[i] * m->Vp, V * 4, cudaMemcpyDeviceToHost, ctx->stream));
+        return b200_ctx_sync_check(ctx);
+    }
+    // more rows than the activation buffers hold: in portions, each with its share of the wanted rows
+    std::vector<int> done(n_entries, 0), row0(n_entries, 0);
+    for (int i = 1; i < n_entries; ++i) row0[i] = row0[i - 1] + counts[i - 1];
+    int first = 0;
+    while (first < n_entries) {
+        std::vector<Entry> part;
+        std::vector<int> rows_of;  // the step's row of every row of this portion
+        int room = m->max_rows;
+        for (int i = first; i < n_entries && room > 0; ++i) {
+            const int left = counts[i] - done[i], n = left < room ? left : room;
+            if (n == 0) continue;
+            part.push_back({slots[i], tokens + row0[i] + done[i], n});
+            for (int t = 0; t < n; ++t) rows_of.push_back(row0[i] + done[i] + t);
+            done[i] += n;
+            room -= n;
+        }
+        while (first < n_entries && done[first] == counts[first]) ++first;
+        std::vector<int> want, dst;
+        std::map<int, int> at;
+        if (n_want > 0) for (size_t r = 0; r < rows_of.size(); ++r) at[rows_of[r]] = (int)r;
+        for (int i = 0; i < n_want; ++i) {
+            auto it = at.find(want_rows[i]);
+            if (it != at.end()) { want.push_back(it->second); dst.push_back(i); }
+        }
+        // the logits' product takes as many rows as the activation buffers hold
+        std::vector<int> head(want.begin(), want.size() > (size_t)m->max_rows ? want.begin() + m->max_rows : want.end());
+        if (head.size() < want.size()) { ctx->last_error = "step: more wanted rows than max_rows"; return B200_ERR_LIMIT; }
+        TRY(general_step(m, part, want));
+        if (logits_host)
+            for (size_t i = 0; i < dst.size(); ++i)
+                B200_CUDA(ctx, cudaMemcpyAsync(logits_host + dst[i] * V, m->logits + i * m->Vp, V * 4, cudaMemcpyDeviceToHost, ctx->stream));
+    }
+    return b200_ctx_sync_check(ctx);
+}
+
+int b200_decoder_decode_device(b200_decoder* m, int n, const int* slots) {
+    if (!m || !slots) return B200_ERR_NULL;
+    if (!m->ready || m->f32) return B200_ERR_STATE;
+    if (n < 1 || n > 16 || n > m->max_slots) return B200_ERR_SHAPE;
+    for (int i = 0; i < n; ++i) {
+        if (slots[i] < 0 || slots[i] >= m->max_slots || !m->slots[slots[i]].open) return B200_ERR_STATE;
+        if (m->slots[slots[i]].len + 1 > m->max_seq) return B200_ERR_LIMIT;
+    }
+    b200_device_guard guard(m->ctx);
+    return decode_step(m, std::vector<int>(slots, slots + n), nullptr);
+}
+
+int b200_decoder_prefill_device(b200_decoder* m, int n_entries, const int* slots, const int* counts, const int* tokens, int n_want, const int* want_rows) {
+    if (!m || !slots || !counts || !tokens || (n_want > 0 && !want_rows)) return B200_ERR_NULL;
+    if (!m->ready) return B200_ERR_STATE;
+    long total = 0;
+    std::vector<Entry> e;
+    for (int i = 0; i < n_entries; ++i) {
+        if (slots[i] < 0 || slots[i] >= m->max_slots || !m->slots[slots[i]].open || counts[i] < 1) return B200_ERR_STATE;
+        if (m->slots[slots[i]].len + counts[i] > m->max_seq) return B200_ERR_LIMIT;
+        e.push_back({slots[i], tokens + total, counts[i]});
+        total += counts[i];
+    }
+    if (n_entries < 1 || n_entries > m->max_slots || total > m->max_rows || n_want > m->max_rows) return B200_ERR_LIMIT;
+    for (int i = 0; i < n_want; ++i)
+        if (want_rows[i] < 0 || want_rows[i] >= total) return B200_ERR_SHAPE;
+    b200_device_guard guard(m->ctx);
+    return general_step(m, e, std::vector<int>(want_rows, want_rows + n_want));
+}
+
+// Requests of unequal lengths, greedy (temperature <= 0) or sampled.  As many requests as there are slots (at most
+// 16) are active; a request that has its n_new tokens makes room for the next one.
+int b200_decoder_generate(b200_decoder* m, int n_req, const int* const* prompts, const int* lens, int n_new, float temperature, int top_k, float top_p,
+                          unsigned int seed, int* out_host) {
+    if (!m || !prompts || !lens || !out_host) return B200_ERR_NULL;
+    if (!m->ready) return B200_ERR_STATE;
+    if (n_req < 1 || n_new < 1 || top_k < 0) return B200_ERR_SHAPE;
+    b200_ctx* ctx = m->ctx;
+    for (int r = 0; r < n_req; ++r) {
+        if (lens[r] < 1) return B200_ERR_SHAPE;
+        if ((long)lens[r] + n_new - 1 > m->max_seq) { ctx->last_error = "generate: prompt and continuation beyond max_seq"; return B200_ERR_LIMIT; }
+        for (int t = 0; t < lens[r]; ++t)
+            if (prompts[r][t] < 0 || prompts[r][t] >= m->spec.vocab) { ctx->last_error = "generate: token id outside the vocabulary"; return B200_ERR_SHAPE; }
+    }
+    b200_device_guard guard(ctx);
+    // sampled ids: [request][n_new] on the device; the current id of every active sequence in dtokens
+    const size_t log_ints = (size_t)n_req * n_new;
+    if (log_ints > m->gen_log_ints) {
+        B200_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+        if (m->gen_log) cudaFree(m->gen_log);
+        m->gen_log = nullptr;
+        m->gen_log_ints = 0;
+        B200_CUDA(ctx, cudaMalloc(&m->gen_log, log_ints * 4));
+        m->gen_log_ints = log_ints;
+    }
+    struct Active { int req, slot, produced; };
+    std::vector<Active> act;
+    std::vector<int> opened;  // slots to give back if a step fails
+    const int V = m->spec.vocab;
+    // the token that will stand at position p of request r uses noise stream p * 4096 + r, whatever else is in the batch
+    auto draw = [&](int row, const Active& a, const float* logits) {
+        return launch_sample_rows(ctx, m->dtokens + row, logits, 1, V, m->Vp, temperature, seed, (unsigned)(lens[a.req] + a.produced) * 4096u + (unsigned)a.req,
+                                  top_k, top_p);
+    };
+    auto record = [&](int row, Active& a) -> int {
+        B200_CUDA(ctx, cudaMemcpyAsync(m->gen_log + (size_t)a.req * n_new + a.produced, m->dtokens + row, 4, cudaMemcpyDeviceToDevice, ctx->stream));
+        a.produced++;
+        return B200_OK;
+    };
+    auto retire = [&]() -> int {
+        for (size_t i = 0; i < act.size();) {
+            if (act[i].produced < n_new) { ++i; continue; }
+            b200_decoder_close(m, act[i].slot);
+            const size_t last = act.size() - 1;
+            if (i != last) {
+                B200_CUDA(ctx, cudaMemcpyAsync(m->dtokens + i, m->dtokens + last, 4, cudaMemcpyDeviceToDevice, ctx->stream));
+                act[i] = act[last];
+            }
+            act.pop_back();
+        }
+        return B200_OK;
+    };
+    auto run = [&]() -> int {
+        int next = 0;
+        while (next < n_req || !act.empty()) {
+            // admit: the prompts of the new requests, together as far as they fit into a step, longer ones in portions
+            std::vector<Active> fresh;
+            while (next < n_req && act.size() + fresh.size() < 16) {
+                int slot;
+                if (b200_decoder_open(m, &slot) != B200_OK) break;
+                opened.push_back(slot);
+                fresh.push_back({next++, slot, 0});
+            }
+            if (fresh.empty() && act.empty()) { ctx->last_error = "generate: no free slot"; return B200_ERR_LIMIT; }
+            size_t f = 0;
+            int fed = 0;  // tokens of request fresh[f] that have been run
+            while (f < fresh.size()) {
+                std::vector<Entry> part;
+                std::vector<int> want;
+                std::vector<size_t> ends;
+                int room = m->max_rows, row = 0;
+                while (f < fresh.size() && room > 0) {
+                    const int left = lens[fresh[f].req] - fed, n = left < room ? left : room;
+                    part.push_back({fresh[f].slot, prompts[fresh[f].req] + fed, n});
+                    row += n;
+                    room -= n;
+                    if (n < left) { fed += n; break; }
+                    want.push_back(row - 1);
+                    ends.push_back(f++);
+                    fed = 0;
+                }
+                TRY(general_step(m, part, want));
+                for (size_t i = 0; i < ends.size(); ++i) {
+                    act.push_back(fresh[ends[i]]);
+                    const int r = (int)act.size() - 1;
+                    TRY(draw(r, act[r], m->logits + i * m->Vp));
+                    TRY(record(r, act[r]));
+                }
+            }
+            TRY(retire());
+            if (act.empty()) continue;
+            const float* logits = m->dlogits;
+            std::vector<int> slots;
+            for (const Active& a : act) slots.push_back(a.slot);
+            if (!m->f32) {
+                TRY(decode_step(m, slots, nullptr));
+            } else {  // the general path wants the ids on the host
+                std::vector<int> ids(act.size());
+                B200_CUDA(ctx, cudaMemcpyAsync(ids.data(), m->dtokens, ids.size() * 4, cudaMemcpyDeviceToHost, ctx->stream));
+                B200_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+                std::vector<Entry> part;
+                std::vector<int> want;
+                for (size_t i = 0; i < act.size(); ++i) { part.push_back({act[i].slot, &ids[i], 1}); want.push_back((int)i); }
+                TRY(general_step(m, part, want));
+                logits = m->logits;
+            }
+            if (temperature <= 0.f) TRY(launch_sample_rows(ctx, m->dtokens, logits, (int)act.size(), V, m->Vp, 0.f, seed, 0u, 0, 0.f));
+            else for (size_t i = 0; i < act.size(); ++i) TRY(draw((int)i, act[i], logits + i * m->Vp));
+            for (size_t i = 0; i < act.size(); ++i) TRY(record((int)i, act[i]));
+            TRY(retire());
+        }
+        return B200_OK;
+    };
+    const int st = run();
+    for (int s : opened) if (st != B200_OK && m->slots[s].open) b200_decoder_close(m, s);
+    if (st != B200_OK) return st;
+    B200_CUDA(ctx, cudaMemcpyAsync(out_host, m->gen_log, log_ints * 4, cudaMemcpyDeviceToHost, ctx->stream));
+    return b200_ctx_sync_check(ctx);
+}
+
+}  // extern "C"

@@ -1,0 +1,170 @@
+// Launchers of the kernels behind driver/decoder.cu (layered decoders with per-sequence state).
+// As in kernels.h they validate nothing, enqueue on ctx->stream and bump ctx->launches once per
+// kernel launch.
+//
+// A step's tokens are rows: the rows of one sequence are consecutive and described by a SeqDesc.
+// Activations come in one of two element types: 16-bit (bf16 GEMM operands) or fp32 (the 32-bit
+// arithmetic); `f32` selects the type of the buffers declared void*.  Every leading dimension is
+// padded (pad_dim) and the padding holds zeros, so rows can be read in 16-byte pieces.
+#pragma once
+#include "kernels.h"
+
+namespace b200 {
+
+struct SeqDesc {
+    int row0;  // first row of the step
+    int n;     // tokens in this step
+    int slot;  // where the sequence's cache and state live
+    int pos0;  // position of its first token in this step
+    int bank;  // short-convolution history to read (0 / 1); the other bank is written
+    int pad[3];
+};
+
+// leading dimension of a matrix operand with n columns: whole 16-byte pieces, at least one 64-element K block
+inline int pad_dim(int n) { return n < 64 ? 64 : (n + 7) & ~7; }
+
+// ---- row-wise (rmsnorm.cu)
+// Residual stream of M rows:  r = embed[tok] * scale (tok != null), or x, or x + rms(y) * wb (y != null);
+// x_out = r (if not null);  h = rms(r) * w as f32 / bf16 (if w).  rows != null: row i of the output
+// is made from row rows[i] of the inputs.  C columns of Cp.
+struct ResidualNormArgs {
+    const float* x; const float* y; const float* wb; const float* w;
+    float* x_out; void* h;
+    const int* tok; const void* embed; float embed_scale; int vocab;
+    const int* rows;
+    int M, C, Cp; float eps;
+};
+int launch_residual_rms(b200_ctx* ctx, const ResidualNormArgs& a, bool f32);
+// out[r, h*Dv + d] = o / rms(o over the head) * w[d] * silu(gate);  o, gate [M] rows with heads Dvl apart
+int launch_gated_head_norm(b200_ctx* ctx, void* out, int ld_out, const float* o, int ld_o, const float* gate, int ld_gate,
+                           const float* w, int M, int H, int Dv, int Dvl, float eps, bool f32);
+// dst[r, 0..n) = src[r, col0 ..]  (fp32 -> bf16 or fp32), columns n..ld_dst zero
+int launch_slice(b200_ctx* ctx, void* dst, int ld_dst, const float* src, int ld_src, int n, int M, bool f32);
+
+// ---- matrix products
+enum : int { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_GELU_ERF = 2 };
+// out[M,N] = act(inp[M,K] W[N,K]^T + bias) on the fp32 FMA pipe (no reduced precision anywhere); K, N multiples of 4
+int launch_gemm_fp32(b200_ctx* ctx, float* out, const float* inp, const float* W, const float* bias, int M, int K, int N, int act);
+
+// Decode product (gemm_decode.cu): B <= 16 rows against bf16 weights.  Prologues that form the input:
+//   DPRO_PLAIN     x [B, K] fp32
+//   DPRO_RESIDUAL  r = embed[tok] * scale, or x, or x + rms(y) * wb; input = rms(r) * w; r is stored to
+//                  x_out by one CTA (a buffer other than x)
+//   DPRO_CONV      short causal convolution + bias + silu of column block [0, K) of x (leading dimension ldx)
+//                  with the history bank; the convolved row goes to conv_out, the new history to the other bank
+enum : int { DPRO_PLAIN = 0, DPRO_RESIDUAL = 1, DPRO_CONV = 2 };
+struct DecodeGemmArgs {
+    float* out; int ldo;
+    const uint16_t* W;   // [N, K]
+    const float* bias;
+    int B, N, K, act;
+    const float* x; int ldx;
+    // DPRO_RESIDUAL
+    const float* y; const float* wb; const float* w; float* x_out;
+    const int* tok; const uint16_t* embed; float embed_scale; int vocab;
+    int C; float eps;
+    // DPRO_CONV
+    const SeqDesc* seqs; const float* conv_w; const float* conv_b; float* hist; int taps; int max_slots; float* conv_out;
+    int* status;
+};
+int launch_decode_gemm(b200_ctx* ctx, const DecodeGemmArgs& a, int prologue);
+bool decode_gemm_fits(int K, int B);  // whether DPRO_RESIDUAL / DPRO_CONV can hold B rows of K on chip
+
+// ---- recurrences (recurrent.cu)
+// y = silu(causal depthwise convolution of columns [0, n) of x + bias); weights [taps][np]; history
+// [2 banks][max_slots][taps - 1][np] fp32
+struct ShortConvArgs {
+    const float* x; int ldx;
+    void* out; int ld_out;
+    const float* w; const float* bias;
+    float* hist;
+    const SeqDesc* seqs;
+    int np, taps, max_slots;  // np: channels rounded up to a multiple of 4 (weights zero beyond)
+};
+int launch_short_conv(b200_ctx* ctx, const ShortConvArgs& a, int E, int max_n, bool f32);
+
+// Selective scan with a diagonal state per channel:
+//   dt = softplus(dt_raw + dt_b);  S[c,:] = 2^(dt A2[c,:]) S[c,:] + dt x B;  y = (S C + D x) * silu(z)
+// With Wdt (decode, one token per sequence) dt_raw is formed here: dt_raw[c] = Wdt[c,:] . bc[0..rank).
+struct SelectiveScanArgs {
+    const void* x; int ldx;           // convolved input: bf16 (f32: fp32)
+    const float* dt; int lddt;        // dt_raw, null with Wdt
+    const float* bc; int ldbc;        // per token: [dt: ..| B: at b_col | C: at c_col]
+    int b_col, c_col;
+    const float* z; int ldz;
+    const float* A2;                  // [inner][state_pad]: -exp(A_log) * log2(e), zero beyond the state
+    const float* dt_b; const float* D;
+    float* S;                         // [slots][inner][state_pad]
+    void* out; int ldo;
+    const SeqDesc* seqs;
+    int inner, state_pad;
+    const uint16_t* Wdt; int rank, ld_wdt;
+};
+int selective_state_pad(int state);   // 0: unsupported
+int launch_selective_scan(b200_ctx* ctx, const SelectiveScanArgs& a, int E, int max_n, bool x_f32, bool out_f32);
+
+// Gated delta rule; q, k, v are the convolved projections of a row, head g's q at g*Dl, k at k_col + g*Dl,
+// head h's v at v_col + h*Dvl.  q and k are made unit vectors here (q also times D^-1/2), and
+//   g = exp(-exp(A_log) softplus(a + dt_bias)), beta = sigmoid(b)
+// State [slots][H][Dv][Dpad] fp32.  o goes to out [M, H*Dvl] fp32.
+struct DeltaArgs {
+    const float* qkv; int ld; int k_col, v_col;
+    const float* gates; int ldg; int a_col, b_col;  // columns of the projection holding a and b per head
+    const float* negA;      // [H] -exp(A_log)
+    const float* dt_bias;   // [H]
+    float* S;
+    float* out; int ldo;
+    const SeqDesc* seqs;
+    int H, G, D, Dl, Dv, Dvl;
+    // one-token form: convolution, output norm and gate included; qkv is the raw projection
+    const float* conv_w; float* hist; int taps, np, max_slots;
+    const float* norm_w; int gate_col; float eps;
+};
+int delta_state_pad(int D);  // 0: unsupported
+int launch_delta_scan(b200_ctx* ctx, const DeltaArgs& a, int E);
+int launch_delta_step(b200_ctx* ctx, const DeltaArgs& a, int E);  // one token per sequence, fused
+
+// minGRU: z = sigmoid(zx[z_col ..]), u = zx[x_col ..], candidate = u + 1/2 (u >= 0) or sigmoid(u);
+// S = (1 - z) S + z candidate;  out = S * silu(zx[g_col ..]) * out_scale
+struct MinGruArgs {
+    const float* zx; int ld; int z_col, x_col, g_col;
+    float* S;  // [slots][width]
+    void* out; int ldo;
+    const SeqDesc* seqs;
+    int width; float out_scale;
+};
+int launch_min_gru(b200_ctx* ctx, const MinGruArgs& a, int E, bool f32);
+
+// ---- attention over a per-slot key/value cache (attention_cached.cu)
+// Cache layout: K [slots][G][Tp][Dp], V [slots][G][Tp][Dvp], fp16 or fp32; Tp a multiple of 128.
+struct CachedAttention {
+    int H, G, D, Dv, Dp, Dvp, Tp;
+    int q_col, k_col, v_col;     // columns of the projection; heads D / Dv apart
+    int rot_dims;                // 0: no rotation
+    const float2* rot;           // [Tp][rot_dims / 2] (cos, sin)
+    const float* q_norm;         // weights of the per-head RMS norms of q and k (null: none)
+    const float* k_norm;
+    int v_norm;                  // values are divided by their root mean square
+    float scale, eps;
+    void* K; void* V;
+    float out_scale;
+};
+inline int attention_pad(int d) { return d <= 64 ? 64 : (d + 63) & ~63; }
+// norms and rotation of a step's q (-> q_out [M][H * Dp]) and k, v (-> cache)
+int launch_attention_prep(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, void* q_out, const SeqDesc* seqs,
+                          const int* row_seq, int M, bool f32);
+// causal attention of a step's rows over positions 0 .. their own; out[row, h*Dv + d] (bf16 or fp32)
+// pairs: (sequence, pair of query tiles) work list of the tensor-core kernel, most keys first
+bool attention_cached_has_mma(const CachedAttention& c);
+int launch_attention_cached_mma(b200_ctx* ctx, const CachedAttention& c, const void* q, void* out, int ldo, const SeqDesc* seqs,
+                                const int2* pairs, int num_pairs, int M, int max_slots);
+int launch_attention_cached_simt(b200_ctx* ctx, const CachedAttention& c, const void* q, void* out, int ldo, const SeqDesc* seqs,
+                                 int E, int max_n, bool f32);
+// One token per sequence: norms, rotation, cache append and attention in one kernel (fp16 cache, fp32
+// out [B][ldo]); with gru.S also a minGRU step in further CTAs of the launch.
+constexpr int kDecodeAttMaxSplits = 16;
+int launch_attention_cached_decode(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, float* out, int ldo,
+                                   const SeqDesc* seqs, int B, float* partial, unsigned int* counters, const MinGruArgs& gru);
+size_t attention_decode_partial_floats(const CachedAttention& c, int B);
+
+}  // namespace b200

@@ -4,6 +4,7 @@
 #include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include "kernels.h"
+#include "decoder_math.cuh"
 #include "../prim/sm100.cuh"
 
 namespace b200 {
@@ -103,7 +104,7 @@ __device__ __forceinline__ float gemm_bias_chunk(const float* bias, int N, int c
 __device__ __forceinline__ void gemm_drain_accumulator_bf16(const GemmArgs& args, const float* bias, const CUtensorMap* tmap_out, uint32_t tmem_acc,
                                                             int q, int lane, int row0, int col0, uint8_t* stage2, float bias_first,
                                                             int c_begin, int c_end, int nbuf) {
-    const bool do_gelu = (args.flags & GEMM_GELU) != 0;
+    const bool do_gelu = (args.flags & GEMM_GELU) != 0, do_erf = (args.flags & GEMM_GELU_ERF) != 0;
     const bool planes = args.out_planes != 0;
     if (lane == 0) tma_store_wait_read();  // the stores of the previous tile have left the staging buffers
     __syncwarp();
@@ -149,6 +150,9 @@ __device__ __forceinline__ void gemm_drain_accumulator_bf16(const GemmArgs& args
                 if (do_gelu) {
 #pragma unroll
                     for (int i = 0; i < 8; ++i) v[i] = gelu_tanh(v[i]);
+                } else if (do_erf) {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) v[i] = gelu_erf(v[i]);
                 }
                 uint32_t pk[4];
                 if (args.out_planes == 2) {

@@ -436,7 +436,8 @@ int launch_gemm_bf16(b200_ctx* ctx, float* out, uint16_t* out_h, const uint16_t*
                      const float* bias, int M, int K, int N, int flags,
                      unsigned long long* argmax_keys, int argmax_cols, int store_period) {
     if (K % 8 || N % 8) { ctx->last_error = "bf16 GEMM: K and N must be multiples of 8"; return B200_ERR_SHAPE; }
-    return launch_gemm_any(ctx, out, out_h, inp, weight, bias, nullptr, M, K, N, flags & (GEMM_GELU | GEMM_ROUND_OUT_TF32 | GEMM_ACCUM_OUT), B200_TF32, argmax_keys, argmax_cols, true, store_period, nullptr);
+    if ((flags & GEMM_GELU_ERF) && !out_h) { ctx->last_error = "GEMM_GELU_ERF: 16-bit output only"; return B200_ERR_STATE; }
+    return launch_gemm_any(ctx, out, out_h, inp, weight, bias, nullptr, M, K, N, flags & (GEMM_GELU | GEMM_GELU_ERF | GEMM_ROUND_OUT_TF32 | GEMM_ACCUM_OUT), B200_TF32, argmax_keys, argmax_cols, true, store_period, nullptr);
 }
 
 // e4m3 operands: always on CTA pairs (the kernel clips ragged edges itself)

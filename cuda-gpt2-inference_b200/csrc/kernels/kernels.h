@@ -55,7 +55,8 @@ int preload_attention_kernel(b200_ctx* ctx);
 // GEMM_ACCUM_OUT: out += result instead of out = result (fp32 output without a residual operand: the
 // tiles leave as TMA reductions).  With out = the residual stream this is the residual add.
 // GEMM_PLANES_FP16: a split output (launch_gemm_bf16x3 with out_planes) is written as two fp16 planes instead of bf16
-enum : int { GEMM_GELU = 1, GEMM_ROUND_OUT_TF32 = 2, GEMM_ACCUM_OUT = 4, GEMM_PLANES_FP16 = 8 };
+// GEMM_GELU_ERF: the exact gelu instead of the tanh form (16-bit outputs only)
+enum : int { GEMM_GELU = 1, GEMM_ROUND_OUT_TF32 = 2, GEMM_ACCUM_OUT = 4, GEMM_PLANES_FP16 = 8, GEMM_GELU_ERF = 16 };
 struct GemmRowStats;
 int launch_gemm_tf32(b200_ctx* ctx, float* out, const float* inp, const float* weight,
                      const float* bias, const float* residual, int M, int K, int N, int flags,

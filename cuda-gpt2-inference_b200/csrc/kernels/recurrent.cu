@@ -1,0 +1,664 @@
+// Layers that carry a state from token to token: the short causal convolution in front of them, the
+// selective scan (diagonal state per channel), the gated delta rule (matrix state per head) and the minGRU.
+//
+// All of them treat a step's rows as sequences (SeqDesc): a sequence that starts (pos0 = 0) begins with
+// a zero state whatever its slot holds, any other continues from the slot, so a prompt may be cut anywhere
+// and a slot needs no clearing.  State and everything that enters a recurrence is fp32.
+#include <cuda_bf16.h>
+#include "decoder_kernels.h"
+#include "decoder_math.cuh"
+#include "../prim/sm100.cuh"
+
+namespace b200 {
+namespace {
+
+// ------------------------------------------------------------------ short convolution
+// A thread computes 4 neighbouring channels of kConvTok consecutive tokens; TAPS > 0 keeps the window in registers.
+constexpr int kConvTok = 16;
+
+template <int TAPS, bool F32>
+__global__ void __launch_bounds__(128)
+short_conv_kernel(const ShortConvArgs a) {
+    griddep_wait();
+    griddep_launch_dependents();
+    const SeqDesc sd = a.seqs[blockIdx.z];
+    const int t0 = blockIdx.y * kConvTok;
+    const int c4 = blockIdx.x * blockDim.x + threadIdx.x;
+    if (t0 >= sd.n || c4 * 4 >= a.np) return;
+    const int taps = TAPS > 0 ? TAPS : a.taps, hrows = taps - 1;
+    const float* hr = a.hist + ((size_t)sd.bank * a.max_slots + sd.slot) * hrows * a.np;
+    float* hw = a.hist + ((size_t)(sd.bank ^ 1) * a.max_slots + sd.slot) * hrows * a.np;
+    const float* xin = a.x + (size_t)sd.row0 * a.ldx;
+    auto input = [&](int i) {  // the input of token i of this step (negative: from the history)
+        if (i >= 0) return load4(xin + (size_t)i * a.ldx, c4);
+        if (sd.pos0 + i < 0) return make_float4(0.f, 0.f, 0.f, 0.f);
+        return load4(hr + (size_t)(hrows + i) * a.np, c4);
+    };
+    const float4 bias = a.bias ? __ldg(reinterpret_cast<const float4*>(a.bias) + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const int t1 = min(sd.n, t0 + kConvTok);
+    auto emit = [&](int t, float4 s) {
+        store4<F32>(a.out, (size_t)(sd.row0 + t) * (a.ld_out >> 2) + c4, make_float4(silu(s.x), silu(s.y), silu(s.z), silu(s.w)));
+    };
+    if (TAPS > 0) {
+        constexpr int W = TAPS > 0 ? TAPS : 1;
+        float4 w[W], win[W];
+#pragma unroll
+        for (int j = 0; j < W; ++j) w[j] = __ldg(reinterpret_cast<const float4*>(a.w + (size_t)j * a.np) + c4);
+#pragma unroll
+        for (int j = 0; j + 1 < W; ++j) win[j] = input(t0 - (W - 1) + j);
+        for (int tb = t0; tb < t1; tb += 4) {
+            float4 nx[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) nx[u] = tb + u < t1 ? input(tb + u) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                win[W - 1] = nx[u];
+                float4 s = bias;
+#pragma unroll
+                for (int j = 0; j < W; ++j) {
+                    s.x = fmaf(win[j].x, w[j].x, s.x); s.y = fmaf(win[j].y, w[j].y, s.y);
+                    s.z = fmaf(win[j].z, w[j].z, s.z); s.w = fmaf(win[j].w, w[j].w, s.w);
+                }
+                if (tb + u < t1) emit(tb + u, s);
+#pragma unroll
+                for (int j = 0; j + 1 < W; ++j) win[j] = win[j + 1];
+            }
+        }
+    } else {
+        for (int t = t0; t < t1; ++t) {
+            float4 s = bias;
+            for (int j = 0; j < taps; ++j) {
+                const float4 x = input(t - hrows + j), w = __ldg(reinterpret_cast<const float4*>(a.w + (size_t)j * a.np) + c4);
+                s.x = fmaf(x.x, w.x, s.x); s.y = fmaf(x.y, w.y, s.y); s.z = fmaf(x.z, w.z, s.z); s.w = fmaf(x.w, w.w, s.w);
+            }
+            emit(t, s);
+        }
+    }
+    if (t1 == sd.n)  // the last taps - 1 inputs are the history of the next step
+        for (int e = 0; e < hrows; ++e) *(reinterpret_cast<float4*>(hw + (size_t)e * a.np) + c4) = input(sd.n - hrows + e);
+}
+
+// ------------------------------------------------------------------ selective scan
+// A CTA walks one sequence for 32 channels; four (or eight) lanes share a channel and keep NS of its states
+// each in registers.  Tiles of 32 tokens are staged in shared memory two deep (cp.async): dt_raw, x and z
+// of the channels, B and C of the tokens; softplus is applied to a staged tile once, y leaves through the
+// dt tile so that the gate and the store are coalesced.
+constexpr int kScanCh = 32, kScanTok = 32;
+
+template <int NS, int LPC, bool XF32, bool OF32, bool STEP>
+__global__ void __launch_bounds__(kScanCh * LPC)
+selective_scan_kernel(const SelectiveScanArgs a) {
+    constexpr int THREADS = kScanCh * LPC, SP = NS * LPC;
+    constexpr int TOK = STEP ? 1 : kScanTok;
+    constexpr int XB = XF32 ? 4 : 2;
+    struct Tile {
+        float dt[TOK][kScanCh];
+        float z[TOK][kScanCh];
+        float bc[2][TOK][SP];
+        uint8_t x[TOK * kScanCh * XB];
+    };
+    extern __shared__ __align__(16) uint8_t raw[];
+    Tile* tiles = reinterpret_cast<Tile*>(raw);
+    const int tid = threadIdx.x;
+    const int c0 = blockIdx.x * kScanCh, ch = tid / LPC, sub = tid % LPC, c = c0 + ch;
+    const bool live = c < a.inner;
+    const int cc = live ? c : a.inner - 1;
+    float A2[NS];
+#pragma unroll
+    for (int i = 0; i < NS; ++i) A2[i] = __ldg(a.A2 + (size_t)cc * SP + sub * NS + i);
+    const float Dc_ch = __ldg(a.D + min(c0 + (tid & (kScanCh - 1)), a.inner - 1));  // of the channel this thread stores
+    const float dtb_ch = __ldg(a.dt_b + min(c0 + (tid & (kScanCh - 1)), a.inner - 1));
+    griddep_wait();
+    griddep_launch_dependents();
+    const SeqDesc sd = a.seqs[blockIdx.y];
+    float* Sg = a.S + ((size_t)sd.slot * a.inner + cc) * SP + sub * NS;
+    float S[NS];
+#pragma unroll
+    for (int i = 0; i < NS; ++i) S[i] = (sd.pos0 > 0) ? Sg[i] : 0.f;
+
+    // channels beyond the end are read as the padding's zeros as far as the rows reach, else not at all
+    auto stage = [&](int t0, Tile& T) {
+        const int nt = min(TOK, sd.n - t0);
+        for (int i = tid; i < nt * (kScanCh / 4); i += THREADS) {
+            const int t = i >> 3, q = (i & 7) * 4;
+            const size_t r = (size_t)(sd.row0 + t0 + t);
+            if (c0 + q < a.inner) {
+                if (!STEP) cp_async16(&T.dt[t][q], a.dt + r * a.lddt + c0 + q);
+                cp_async16(&T.z[t][q], a.z + r * a.ldz + c0 + q);
+                if (XF32) cp_async16(T.x + (t * kScanCh + q) * XB, static_cast<const float*>(a.x) + r * a.ldx + c0 + q);
+                else cp_async8(T.x + (t * kScanCh + q) * XB, static_cast<const uint16_t*>(a.x) + r * a.ldx + c0 + q);
+            }
+        }
+        for (int i = tid; i < nt * (SP / 4) * 2; i += THREADS) {
+            const int which = i / (nt * (SP / 4)), k = i - which * nt * (SP / 4);
+            const int t = k / (SP / 4), q = (k - t * (SP / 4)) * 4;
+            cp_async16(&T.bc[which][t][q], a.bc + (size_t)(sd.row0 + t0 + t) * a.ldbc + (which ? a.c_col : a.b_col) + q);
+        }
+        cp_async_commit();
+    };
+    auto xval = [&](const Tile& T, int t, int k) {
+        return XF32 ? reinterpret_cast<const float*>(T.x)[t * kScanCh + k] : bf16_to_f(reinterpret_cast<const uint16_t*>(T.x)[t * kScanCh + k]);
+    };
+    stage(0, tiles[0]);
+    for (int t0 = 0, it = 0; t0 < sd.n; t0 += TOK, ++it) {
+        Tile& T = tiles[STEP ? 0 : (it & 1)];
+        const int nt = min(TOK, sd.n - t0);
+        if (!STEP && t0 + TOK < sd.n) { stage(t0 + TOK, tiles[(it + 1) & 1]); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+        if (STEP) {
+            // dt_raw of the CTA's channels: the low-rank projection, LPC lanes per channel
+            float s = 0.f;
+            const float* lr = a.bc + (size_t)sd.row0 * a.ldbc;
+            const uint16_t* wr = a.Wdt + (size_t)cc * a.ld_wdt;
+            for (int r = sub * 2; r < a.rank; r += LPC * 2) {  // columns beyond the rank are zero in Wdt
+                const uint32_t wp = __ldg(reinterpret_cast<const uint32_t*>(wr + r));
+                s = fmaf(__uint_as_float(wp << 16), lr[r], s);
+                s = fmaf(__uint_as_float(wp & 0xffff0000u), lr[r + 1], s);
+            }
+#pragma unroll
+            for (int m = 1; m < LPC; m <<= 1) s += __shfl_xor_sync(0xffffffffu, s, m);
+            if (sub == 0) T.dt[0][ch] = s;
+            __syncthreads();
+        }
+        for (int i = tid; i < nt * kScanCh; i += THREADS) {  // THREADS is a multiple of kScanCh: always the same channel
+            float& d = (&T.dt[0][0])[i];
+            d = softplusf_(d + dtb_ch);
+        }
+        __syncthreads();
+        // y of four tokens at a time: their lane sums are formed together
+        for (int tb = 0; tb < nt; tb += 4) {
+            float y[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                y[u] = 0.f;
+                if (STEP && u > 0) continue;
+                const int t = min(tb + u, TOK - 1);
+                if (tb + u < nt) {
+                    const float dt = T.dt[t][ch], dx = dt * xval(T, t, ch);
+#pragma unroll
+                    for (int i = 0; i < NS; ++i) {
+                        S[i] = fmaf(ex2(dt * A2[i]), S[i], dx * T.bc[0][t][sub * NS + i]);
+                        y[u] = fmaf(S[i], T.bc[1][t][sub * NS + i], y[u]);
+                    }
+                }
+            }
+            reduce_scatter<4, LPC>(y, tid);
+            const int t = tb + scatter_first<4, LPC>(tid);
+            __syncwarp();  // the lanes of the channel have read dt of these tokens
+            if (t < nt && scatter_owner<4, LPC>(tid)) T.dt[t][ch] = y[0];
+        }
+        __syncthreads();
+        for (int i = tid; i < nt * kScanCh; i += THREADS) {
+            const int t = i / kScanCh, k = i & (kScanCh - 1);
+            if (c0 + k < a.inner) {
+                const float v = (T.dt[t][k] + Dc_ch * xval(T, t, k)) * silu(T.z[t][k]);
+                store1<OF32>(a.out, (size_t)(sd.row0 + t0 + t) * a.ldo + c0 + k, v);
+            }
+        }
+        __syncthreads();  // the tile may be staged again
+    }
+    if (live) {
+#pragma unroll
+        for (int i = 0; i < NS; ++i) Sg[i] = S[i];
+    }
+}
+
+// ------------------------------------------------------------------ gated delta rule
+// The columns of a head's state S [D, Dv] do not touch one another: with S the state before the token,
+//   u = beta (v - g S^T k),   o = g S^T q + (k.q) u,   S <- g S + k u^T
+// - both products read the old state, so one reduction serves them.  L = D / 16 lanes share a group of four
+// columns and keep 16 rows of each in registers (as pairs: one instruction does two multiply-adds); lane l
+// owns rows 4 (l + L i) .. + 3, so the lanes read consecutive 16-byte pieces of k and q.
+constexpr int kDeltaTok = 16, kDeltaRows = 16, kDeltaCols = 4;
+constexpr int kDeltaThreads = 128;
+
+template <int L>
+struct DeltaCore {
+    static constexpr int D = 16 * L;
+    uint64_t S[kDeltaCols][kDeltaRows / 2];
+    __device__ __forceinline__ void zero() {
+#pragma unroll
+        for (int c = 0; c < kDeltaCols; ++c)
+#pragma unroll
+            for (int i = 0; i < kDeltaRows / 2; ++i) S[c][i] = 0ull;
+    }
+    // column j of this group at base + j * D; columns from ncol on are left alone
+    __device__ __forceinline__ void load(const float* base, int l, int ncol) {
+#pragma unroll
+        for (int c = 0; c < kDeltaCols; ++c)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                ulonglong2 v = make_ulonglong2(0ull, 0ull);
+                if (c < ncol) v = *reinterpret_cast<const ulonglong2*>(base + (size_t)c * D + 4 * (l + L * i));
+                S[c][2 * i] = v.x;
+                S[c][2 * i + 1] = v.y;
+            }
+    }
+    __device__ __forceinline__ void store(float* base, int l, int ncol) const {
+#pragma unroll
+        for (int c = 0; c < kDeltaCols; ++c)
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                if (c < ncol) *reinterpret_cast<ulonglong2*>(base + (size_t)c * D + 4 * (l + L * i)) = make_ulonglong2(S[c][2 * i], S[c][2 * i + 1]);
+    }
+    // One token.  q, k: D floats in shared memory; v: the group's four values, there too; lane: lane in the warp.
+    // Returns o of column ocol(lane) (valid where owns_o(lane)); with fewer than eight lanes a lane holds
+    // several columns: o[0 .. kHeld).
+    static constexpr int kHeld = L >= 8 ? 1 : 8 / L;         // totals a lane holds after the reduction
+    static constexpr int kOut = kHeld > 4 ? 4 : kHeld;
+    // of the eight totals, 0-3 are S^T k and 4-7 are S^T q of the four columns; lane bit 0 separates the two
+    static __device__ __forceinline__ int ocol(int lane) { return scatter_first<8, L>(lane) & 3; }
+    static __device__ __forceinline__ bool owns_o(int lane) { return (lane & 1) && scatter_owner<8, L>(lane); }
+    __device__ __forceinline__ void token(const float* q, const float* k, const float* v, float g, float beta, float kq, int lane,
+                                          float (&o)[kOut]) {
+        const int l = lane & (L - 1);
+        uint64_t kr[8], acc[8];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const ulonglong2 kv = *reinterpret_cast<const ulonglong2*>(k + 4 * (l + L * i));
+            kr[2 * i] = kv.x;
+            kr[2 * i + 1] = kv.y;
+        }
+#pragma unroll
+        for (int c = 0; c < 8; ++c) acc[c] = 0ull;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const ulonglong2 qv = *reinterpret_cast<const ulonglong2*>(q + 4 * (l + L * i));
+#pragma unroll
+            for (int c = 0; c < kDeltaCols; ++c) {
+                acc[c] = fma2(kr[2 * i], S[c][2 * i], acc[c]);
+                acc[4 + c] = fma2(qv.x, S[c][2 * i], acc[4 + c]);
+                acc[c] = fma2(kr[2 * i + 1], S[c][2 * i + 1], acc[c]);
+                acc[4 + c] = fma2(qv.y, S[c][2 * i + 1], acc[4 + c]);
+            }
+        }
+        float t[8];
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+            float x, y;
+            unpack2(acc[c], x, y);
+            t[c] = x + y;
+        }
+        reduce_scatter<8, L>(t, lane);
+        const int first = scatter_first<8, L>(lane);  // t[j] is total number first + j
+        // u on the lanes that hold S^T k (first < 4), handed to the whole group
+        float um[kOut];
+#pragma unroll
+        for (int j = 0; j < kOut; ++j) um[j] = beta * (v[(first + j) & 3] - g * t[j]);
+        const int base = lane & ~(L - 1);
+        float u[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            // the lane whose totals include number c: halving by bits 0, 1, 2 in turn
+            int src = 0;
+            if (L >= 4 && (c & 2)) src |= 2;
+            if (L >= 8 && (c & 1)) src |= 4;
+            u[c] = __shfl_sync(0xffffffffu, um[kHeld >= 4 ? c : (kHeld == 2 ? (c & 1) : 0)], base + src);
+        }
+#pragma unroll
+        for (int j = 0; j < kOut; ++j) {
+            const int col = (first + j) & 3;
+            const float uc = (kHeld >= 4) ? u[j & 3] : (col & 2 ? (col & 1 ? u[3] : u[2]) : (col & 1 ? u[1] : u[0]));
+            o[j] = fmaf(g, t[j], kq * uc);
+        }
+        const uint64_t gg = pack2(g, g);
+#pragma unroll
+        for (int c = 0; c < kDeltaCols; ++c) {
+            const uint64_t uu = pack2(u[c], u[c]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) S[c][i] = fma2(kr[i], uu, mul2(gg, S[c][i]));
+        }
+    }
+};
+
+// Prefill: a CTA walks one (sequence, head) for cols = blockDim.x / L * 4 columns of Dv, in tiles of 16 tokens
+// staged two deep; q and k of a staged tile are made unit vectors in place, one warp per token.
+template <int L>
+__global__ void __launch_bounds__(kDeltaThreads)
+delta_scan_kernel(const DeltaArgs a) {
+    constexpr int D = 16 * L;
+    extern __shared__ __align__(16) float sm[];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nwarps = blockDim.x >> 5;
+    const int cols = blockDim.x / L * kDeltaCols;
+    const int tile_f = kDeltaTok * (2 * D + cols);
+    float* coef = sm + 2 * tile_f;  // [2][16][4]: g, beta, k.q
+    const int h = blockIdx.x, c0 = blockIdx.y * cols;
+    const int kvh = h / (a.H / a.G);
+    const float negA = __ldg(a.negA + h), dtb = __ldg(a.dt_bias + h);
+    const float qscale = rsqrtf((float)a.D);
+    // rows of k and q beyond the head's dimension stay zero in both tiles
+    for (int i = tid; i < 2 * tile_f; i += blockDim.x) sm[i] = 0.f;
+    griddep_wait();
+    griddep_launch_dependents();
+    const SeqDesc sd = a.seqs[blockIdx.z];
+    const int grp = tid / L, l = tid & (L - 1);
+    const int gc = c0 + grp * kDeltaCols;         // first column of this group
+    const int ncol = min(kDeltaCols, a.Dv - gc);  // may be <= 0
+    DeltaCore<L> core;
+    float* Sg = a.S + (((size_t)sd.slot * a.H + h) * a.Dv + (gc < a.Dv ? gc : 0)) * D;
+    if (sd.pos0 > 0) core.load(Sg, l, ncol);
+    else core.zero();
+    __syncthreads();
+
+    const int d4 = a.Dl >> 2, v4 = min(cols, a.Dvl - c0) >> 2;
+    auto stage = [&](int t0, int buf) {
+        float* q = sm + buf * tile_f;
+        const int nt = min(kDeltaTok, sd.n - t0);
+        const int per = 2 * d4 + v4;
+        for (int i = tid; i < nt * per; i += blockDim.x) {
+            const int t = i / per, j = i - t * per;
+            const float* row = a.qkv + (size_t)(sd.row0 + t0 + t) * a.ld;
+            if (j < d4) cp_async16(q + t * D + j * 4, row + kvh * a.Dl + j * 4);
+            else if (j < 2 * d4) cp_async16(q + (kDeltaTok + t) * D + (j - d4) * 4, row + a.k_col + kvh * a.Dl + (j - d4) * 4);
+            else cp_async16(q + 2 * kDeltaTok * D + t * cols + (j - 2 * d4) * 4, row + a.v_col + h * a.Dvl + c0 + (j - 2 * d4) * 4);
+        }
+        cp_async_commit();
+        if (tid < nt) {
+            const float* gr = a.gates + (size_t)(sd.row0 + t0 + tid) * a.ldg;
+            coef[(buf * kDeltaTok + tid) * 4] = expf(negA * softplusf_(gr[a.a_col + h] + dtb));
+            coef[(buf * kDeltaTok + tid) * 4 + 1] = sigmoidf_(gr[a.b_col + h]);
+        }
+    };
+    stage(0, 0);
+    for (int t0 = 0, it = 0; t0 < sd.n; t0 += kDeltaTok, ++it) {
+        const int buf = it & 1, nt = min(kDeltaTok, sd.n - t0);
+        if (t0 + kDeltaTok < sd.n) { stage(t0 + kDeltaTok, buf ^ 1); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+        float* q = sm + buf * tile_f;
+        float* k = q + kDeltaTok * D;
+        const float* v = k + kDeltaTok * D;
+        for (int t = warp; t < nt; t += nwarps) {
+            float sq = 0.f, sk = 0.f, dot = 0.f;
+            for (int d = lane; d < D; d += 32) {
+                const float qv = q[t * D + d], kv = k[t * D + d];
+                sq = fmaf(qv, qv, sq);
+                sk = fmaf(kv, kv, sk);
+                dot = fmaf(qv, kv, dot);
+            }
+            sq = warp_sum(sq); sk = warp_sum(sk); dot = warp_sum(dot);
+            const float rq = qscale / sqrtf(sq + 1e-6f), rk = 1.0f / sqrtf(sk + 1e-6f);
+            for (int d = lane; d < D; d += 32) { q[t * D + d] *= rq; k[t * D + d] *= rk; }
+            if (lane == 0) coef[(buf * kDeltaTok + t) * 4 + 2] = dot * rq * rk;
+        }
+        __syncthreads();
+        const int oc = DeltaCore<L>::ocol(lane);
+        const bool ow = DeltaCore<L>::owns_o(lane);
+        for (int t = 0; t < nt; ++t) {
+            const float4 cf = *reinterpret_cast<const float4*>(coef + (buf * kDeltaTok + t) * 4);
+            float o[DeltaCore<L>::kOut];
+            core.token(q + t * D, k + t * D, v + t * cols + grp * kDeltaCols, cf.x, cf.y, cf.z, lane, o);
+            if (ow) {
+                float* orow = a.out + (size_t)(sd.row0 + t0 + t) * a.ldo + h * a.Dvl + gc;
+#pragma unroll
+                for (int j = 0; j < DeltaCore<L>::kOut; ++j)
+                    if (oc + j < ncol) orow[oc + j] = o[j];
+            }
+        }
+        __syncthreads();
+    }
+    core.store(Sg, l, ncol);
+}
+
+// Decode: one CTA per (head, sequence) takes its token through convolution, unit norms, the rule, the
+// output norm and the gate.
+constexpr int kDeltaStepThreads = 256;
+template <int L>
+__global__ void __launch_bounds__(kDeltaStepThreads)
+delta_step_kernel(const DeltaArgs a) {
+    constexpr int D = 16 * L;
+    extern __shared__ __align__(16) float sm[];  // q [D], k [D], v and o [Dvl + 4 each]
+    __shared__ float red[8];
+    float* q = sm;
+    float* k = q + D;
+    float* v = k + D;
+    const int vpad = (a.Dvl + kDeltaStepThreads / L * kDeltaCols - 1) & ~3;
+    float* o = v + vpad;
+    const int tid = threadIdx.x, lane = tid & 31;
+    const int h = blockIdx.x, per = a.H / a.G, kvh = h / per;
+    const float negA = __ldg(a.negA + h), dtb = __ldg(a.dt_bias + h);
+    for (int i = tid; i < 2 * D + 2 * vpad; i += kDeltaStepThreads) sm[i] = 0.f;
+    griddep_wait();
+    griddep_launch_dependents();
+    const SeqDesc sd = a.seqs[blockIdx.y];
+    const float* row = a.qkv + (size_t)sd.row0 * a.ld;
+    __syncthreads();
+    const int hrows = a.taps - 1;
+    const float* hr = a.hist + ((size_t)sd.bank * a.max_slots + sd.slot) * hrows * a.np;
+    float* hw = a.hist + ((size_t)(sd.bank ^ 1) * a.max_slots + sd.slot) * hrows * a.np;
+    for (int i = tid; i < 2 * a.Dl + a.Dvl; i += kDeltaStepThreads) {
+        int ch;
+        float* dst;
+        bool keep;  // this CTA writes the history of the channel (q and k are shared by the heads of a group)
+        if (i < a.Dl) { ch = kvh * a.Dl + i; dst = q + i; keep = h % per == 0; }
+        else if (i < 2 * a.Dl) { ch = a.k_col + kvh * a.Dl + i - a.Dl; dst = k + i - a.Dl; keep = h % per == 0; }
+        else { ch = a.v_col + h * a.Dvl + i - 2 * a.Dl; dst = v + i - 2 * a.Dl; keep = true; }
+        float s = 0.f;
+        for (int j = 0; j < a.taps; ++j) {
+            const int back = hrows - j;
+            float x = 0.f;
+            if (back == 0) x = row[ch];
+            else if (back <= sd.pos0) x = hr[(size_t)j * a.np + ch];
+            if (keep && j > 0) hw[(size_t)(j - 1) * a.np + ch] = x;
+            s = fmaf(x, __ldg(a.conv_w + (size_t)j * a.np + ch), s);
+        }
+        *dst = silu(s);
+    }
+    __syncthreads();
+    float sq = 0.f, sk = 0.f, dot = 0.f;  // every warp for itself
+    for (int d = lane; d < D; d += 32) { sq = fmaf(q[d], q[d], sq); sk = fmaf(k[d], k[d], sk); dot = fmaf(q[d], k[d], dot); }
+    sq = warp_sum(sq); sk = warp_sum(sk); dot = warp_sum(dot);
+    const float rq = rsqrtf((float)a.D) / sqrtf(sq + 1e-6f), rk = 1.0f / sqrtf(sk + 1e-6f);
+    const float g = expf(negA * softplusf_(row[a.a_col + h] + dtb)), beta = sigmoidf_(row[a.b_col + h]);
+    __syncthreads();
+    for (int d = tid; d < D; d += kDeltaStepThreads) { q[d] *= rq; k[d] *= rk; }
+    __syncthreads();
+    const int grp = tid / L, l = tid & (L - 1);
+    const int oc = DeltaCore<L>::ocol(lane);
+    const bool ow = DeltaCore<L>::owns_o(lane);
+    for (int c0 = 0; c0 < a.Dv; c0 += kDeltaStepThreads / L * kDeltaCols) {
+        const int gc = c0 + grp * kDeltaCols, ncol = min(kDeltaCols, a.Dv - gc);
+        DeltaCore<L> core;
+        float* Sg = a.S + (((size_t)sd.slot * a.H + h) * a.Dv + (gc < a.Dv ? gc : 0)) * D;
+        if (sd.pos0 > 0) core.load(Sg, l, ncol);
+        else core.zero();
+        float ov[DeltaCore<L>::kOut];
+        core.token(q, k, v + gc, g, beta, dot * rq * rk, lane, ov);
+        if (ow) {
+#pragma unroll
+            for (int j = 0; j < DeltaCore<L>::kOut; ++j)
+                if (oc + j < ncol) o[gc + oc + j] = ov[j];
+        }
+        core.store(Sg, l, ncol);
+    }
+    __syncthreads();
+    float s = 0.f;
+    for (int d = tid; d < a.Dv; d += kDeltaStepThreads) s += o[d] * o[d];
+    const float r = 1.0f / sqrtf(block_sum(s, red) / (float)a.Dv + a.eps);
+    for (int d = tid; d < a.Dv; d += kDeltaStepThreads)
+        a.out[(size_t)sd.row0 * a.ldo + h * a.Dv + d] = o[d] * r * __ldg(a.norm_w + d) * silu(row[a.gate_col + h * a.Dvl + d]);
+}
+
+// ------------------------------------------------------------------ minGRU
+// A CTA walks one sequence for 32 channels, 128 tokens at a time: each of 16 warps takes 8 consecutive
+// tokens (lane = channel), first as the affine map S -> A S + b that they amount to, and once the maps
+// of the warps before it are known - through shared memory - as the states themselves.
+constexpr int kGruWarps = 16, kGruTok = 8;
+template <bool F32>
+__global__ void __launch_bounds__(kGruWarps * 32)
+min_gru_kernel(const MinGruArgs a) {
+    __shared__ float mapA[2][kGruWarps][32], mapB[2][kGruWarps][32];
+    griddep_wait();
+    griddep_launch_dependents();
+    const SeqDesc sd = a.seqs[blockIdx.y];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int c = blockIdx.x * 32 + lane;
+    const bool live = c < a.width;
+    float* Sg = a.S + (size_t)sd.slot * a.width + c;
+    float S = (live && sd.pos0 > 0) ? *Sg : 0.f;  // state before the block of tokens (the same in every warp)
+    const float* base = a.zx + (size_t)sd.row0 * a.ld + c;
+    for (int t0 = 0, it = 0; t0 < sd.n; t0 += kGruWarps * kGruTok, ++it) {
+        float (&mA)[kGruWarps][32] = mapA[it & 1];
+        float (&mB)[kGruWarps][32] = mapB[it & 1];
+        const int tw = t0 + warp * kGruTok;
+        float zi[kGruTok], ui[kGruTok], gi[kGruTok];
+#pragma unroll
+        for (int i = 0; i < kGruTok; ++i) {
+            zi[i] = ui[i] = gi[i] = 0.f;
+            if (live && tw + i < sd.n) {
+                const float* r = base + (size_t)(tw + i) * a.ld;
+                zi[i] = r[a.z_col];
+                ui[i] = r[a.x_col];
+                gi[i] = r[a.g_col];
+            }
+        }
+        float A = 1.f, b = 0.f;
+#pragma unroll
+        for (int i = 0; i < kGruTok; ++i) {
+            const float z = tw + i < sd.n ? sigmoidf_(zi[i]) : 0.f;
+            const float cand = ui[i] >= 0.f ? ui[i] + 0.5f : sigmoidf_(ui[i]);
+            zi[i] = 1.f - z;
+            ui[i] = z * cand;
+            A *= zi[i];
+            b = fmaf(zi[i], b, ui[i]);
+        }
+        mA[warp][lane] = A;
+        mB[warp][lane] = b;
+        __syncthreads();  // (two sets of maps: the next block's writes do not meet this block's reads)
+        float s = S;
+#pragma unroll
+        for (int w = 0; w < kGruWarps; ++w) {
+            if (w == warp) s = S;
+            S = fmaf(mA[w][lane], S, mB[w][lane]);
+        }
+#pragma unroll
+        for (int i = 0; i < kGruTok; ++i) {
+            s = fmaf(zi[i], s, ui[i]);
+            if (live && tw + i < sd.n) store1<F32>(a.out, (size_t)(sd.row0 + tw + i) * a.ldo + c, s * silu(gi[i]) * a.out_scale);
+        }
+    }
+    if (live && warp == 0) *Sg = S;
+}
+
+template <int NS, int LPC, bool XF32, bool OF32, bool STEP>
+int launch_scan_one(b200_ctx* ctx, const SelectiveScanArgs& a, int E) {
+    constexpr int TOK = STEP ? 1 : kScanTok;
+    constexpr size_t tile = (size_t)TOK * kScanCh * 8 + (size_t)2 * TOK * NS * LPC * 4 + (size_t)TOK * kScanCh * (XF32 ? 4 : 2);
+    constexpr size_t smem = ((tile + 15) & ~(size_t)15) * (STEP ? 1 : 2);
+    static_assert(smem <= 227 * 1024, "tiles in shared memory");
+    static bool attr_set[64] = {};
+    if (!attr_set[ctx->device & 63]) {
+        B200_CUDA(ctx, cudaFuncSetAttribute(selective_scan_kernel<NS, LPC, XF32, OF32, STEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        attr_set[ctx->device & 63] = true;
+    }
+    cudaError_t le = launch_pdl(ctx, selective_scan_kernel<NS, LPC, XF32, OF32, STEP>, dim3((a.inner + kScanCh - 1) / kScanCh, E), dim3(kScanCh * LPC), smem, a);
+    ctx->launches++;
+    B200_CUDA(ctx, le);
+    return B200_OK;
+}
+
+template <int NS, int LPC>
+int launch_scan_types(b200_ctx* ctx, const SelectiveScanArgs& a, int E, bool x_f32, bool out_f32) {
+    if (a.Wdt) return launch_scan_one<NS, LPC, true, true, true>(ctx, a, E);
+    if (x_f32 && out_f32) return launch_scan_one<NS, LPC, true, true, false>(ctx, a, E);
+    if (!x_f32 && !out_f32) return launch_scan_one<NS, LPC, false, false, false>(ctx, a, E);
+    return B200_ERR_SHAPE;
+}
+
+template <int L>
+int launch_delta_one(b200_ctx* ctx, const DeltaArgs& a, int E, bool step) {
+    constexpr int D = 16 * L;
+    cudaError_t le;
+    if (step) {
+        const int vpad = (a.Dvl + kDeltaStepThreads / L * kDeltaCols - 1) & ~3;
+        const size_t smem = (size_t)(2 * D + 2 * vpad) * 4;
+        if (smem > 48 * 1024) return B200_ERR_LIMIT;
+        le = launch_pdl(ctx, delta_step_kernel<L>, dim3(a.H, E), dim3(kDeltaStepThreads), smem, a);
+    } else {
+        int groups = (a.Dv + kDeltaCols - 1) / kDeltaCols;
+        int threads = (groups * L + 31) & ~31;
+        if (threads > kDeltaThreads) threads = kDeltaThreads;
+        // a short grid: narrower column blocks put more SMs to work
+        while (threads > 32 && (long)a.H * E * ((groups * L + threads - 1) / threads) < 2L * ctx->num_sms) threads >>= 1;
+        threads = (threads + 31) & ~31;
+        const int cols = threads / L * kDeltaCols;
+        const size_t smem = (size_t)(2 * kDeltaTok * (2 * D + cols) + 2 * kDeltaTok * 4) * 4;
+        static bool attr_set[64] = {};
+        if (!attr_set[ctx->device & 63]) {
+            B200_CUDA(ctx, cudaFuncSetAttribute(delta_scan_kernel<L>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+            attr_set[ctx->device & 63] = true;
+        }
+        if (smem > 200 * 1024) return B200_ERR_LIMIT;
+        le = launch_pdl(ctx, delta_scan_kernel<L>, dim3(a.H, (a.Dv + cols - 1) / cols, E), dim3(threads), smem, a);
+    }
+    ctx->launches++;
+    B200_CUDA(ctx, le);
+    return B200_OK;
+}
+
+int launch_delta(b200_ctx* ctx, const DeltaArgs& a, int E, bool step) {
+    switch (delta_state_pad(a.D)) {
+        case 32: return launch_delta_one<2>(ctx, a, E, step);
+        case 64: return launch_delta_one<4>(ctx, a, E, step);
+        case 128: return launch_delta_one<8>(ctx, a, E, step);
+        case 256: return launch_delta_one<16>(ctx, a, E, step);
+        default: return B200_ERR_LIMIT;
+    }
+}
+
+}  // namespace
+
+int launch_short_conv(b200_ctx* ctx, const ShortConvArgs& a, int E, int max_n, bool f32) {
+    const dim3 grid((a.np / 4 + 127) / 128, (max_n + kConvTok - 1) / kConvTok, E), block(128);
+    cudaError_t le;
+    switch (a.taps) {
+        case 2: le = f32 ? launch_pdl(ctx, short_conv_kernel<2, true>, grid, block, 0, a) : launch_pdl(ctx, short_conv_kernel<2, false>, grid, block, 0, a); break;
+        case 3: le = f32 ? launch_pdl(ctx, short_conv_kernel<3, true>, grid, block, 0, a) : launch_pdl(ctx, short_conv_kernel<3, false>, grid, block, 0, a); break;
+        case 4: le = f32 ? launch_pdl(ctx, short_conv_kernel<4, true>, grid, block, 0, a) : launch_pdl(ctx, short_conv_kernel<4, false>, grid, block, 0, a); break;
+        default: le = f32 ? launch_pdl(ctx, short_conv_kernel<0, true>, grid, block, 0, a) : launch_pdl(ctx, short_conv_kernel<0, false>, grid, block, 0, a); break;
+    }
+    ctx->launches++;
+    B200_CUDA(ctx, le);
+    return B200_OK;
+}
+
+int selective_state_pad(int state) {
+    for (int p = 4; p <= 256; p <<= 1)
+        if (state <= p) return p;
+    return 0;
+}
+
+int launch_selective_scan(b200_ctx* ctx, const SelectiveScanArgs& a, int E, int max_n, bool x_f32, bool out_f32) {
+    (void)max_n;
+    switch (a.state_pad) {
+        case 4: return launch_scan_types<1, 4>(ctx, a, E, x_f32, out_f32);
+        case 8: return launch_scan_types<2, 4>(ctx, a, E, x_f32, out_f32);
+        case 16: return launch_scan_types<4, 4>(ctx, a, E, x_f32, out_f32);
+        case 32: return launch_scan_types<8, 4>(ctx, a, E, x_f32, out_f32);
+        case 64: return launch_scan_types<16, 4>(ctx, a, E, x_f32, out_f32);
+        case 128: return launch_scan_types<16, 8>(ctx, a, E, x_f32, out_f32);
+        case 256: return launch_scan_types<32, 8>(ctx, a, E, x_f32, out_f32);
+        default: return B200_ERR_LIMIT;
+    }
+}
+
+int delta_state_pad(int D) {
+    for (int p = 32; p <= 256; p <<= 1)
+        if (D <= p) return p;
+    return 0;
+}
+
+int launch_delta_scan(b200_ctx* ctx, const DeltaArgs& a, int E) { return launch_delta(ctx, a, E, false); }
+int launch_delta_step(b200_ctx* ctx, const DeltaArgs& a, int E) { return launch_delta(ctx, a, E, true); }
+
+int launch_min_gru(b200_ctx* ctx, const MinGruArgs& a, int E, bool f32) {
+    const dim3 grid((a.width + 31) / 32, E);
+    cudaError_t le = f32 ? launch_pdl(ctx, min_gru_kernel<true>, grid, dim3(kGruWarps * 32), 0, a)
+                         : launch_pdl(ctx, min_gru_kernel<false>, grid, dim3(kGruWarps * 32), 0, a);
+    ctx->launches++;
+    B200_CUDA(ctx, le);
+    return B200_OK;
+}
+
+}  // namespace b200

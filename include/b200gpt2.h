@@ -67,6 +67,8 @@ typedef struct b200_ctx b200_ctx;
  * void* (NULL = legacy default stream, the reference's behaviour). */
 int b200_ctx_create(b200_ctx** out, int device, void* stream);
 int b200_ctx_destroy(b200_ctx* ctx);
+/* A non-blocking stream of the context's own, destroyed with it (for hosts without one to bind). */
+int b200_ctx_own_stream(b200_ctx* ctx);
 int b200_ctx_set_stream(b200_ctx* ctx, void* stream);
 /* Synchronises the stream, then returns B200_ERR_TIMEOUT / B200_ERR_CUDA if a kernel
  * recorded a device-side wait that ran out or CUDA reports an error; clears the word. */
@@ -439,6 +441,56 @@ int b200_gpt2_read_profile(b200_gpt2* model, double* ms, long* launches);
 /* Device pointer of an intermediate activation of the last forward, for tests:
  * name in {"encoded","ln_out","qkv","atty","branch","fch","residual","argmax"}; NULL if unknown. */
 void* b200_gpt2_activation(b200_gpt2* model, const char* name);
+
+/* ---------------------------------------------------------------- layered decoders */
+/* Decoder-only models whose configuration lists their layers (config.json; "architecture" selects the
+ * design, e.g. "Vunolorn"), each with a mixer - selective scan, gated delta rule, or softmax attention
+ * beside a minGRU - and a feed-forward.  Sequences live in slots, which hold a sequence's key/value cache,
+ * recurrent state and convolution history; a step runs any number of new tokens of any open slots.
+ *
+ * arithmetic: B200_DECODER_BF16 - bf16 weights and matrix-product operands, fp16 key/value cache, fp32
+ * accumulation, residual stream, norms, attention scores and recurrences; B200_DECODER_FP32 - everything
+ * in fp32 on the FMA pipe. */
+enum { B200_DECODER_BF16 = 0, B200_DECODER_FP32 = 1 };
+typedef struct b200_decoder b200_decoder;
+
+/* max_slots sequences of up to max_seq tokens each; max_rows tokens run at a time (a longer step is cut
+ * into portions).  B200_ERR_SHAPE with the reason in b200_ctx_last_error if the configuration is not valid. */
+int b200_decoder_create(b200_decoder** out, b200_ctx* ctx, const char* config_json, int arithmetic, int max_slots,
+                        int max_seq, int max_rows);
+int b200_decoder_destroy(b200_decoder* model);
+int b200_decoder_vocab(const b200_decoder* model);
+/* Weights: a safetensors file, or tensors one by one (host memory, bf16 or fp32; copied) and finish_load.
+ * Names and shapes are checked against the configuration. */
+int b200_decoder_load_safetensors(b200_decoder* model, const char* path);
+int b200_decoder_set_tensor(b200_decoder* model, const char* name, const void* data, int is_f32, const long* shape, int ndim);
+int b200_decoder_finish_load(b200_decoder* model);
+/* decode steps replayed as CUDA graphs (default 1; needs a stream other than the default one) */
+int b200_decoder_set_graph(b200_decoder* model, int use_graph);
+
+/* slots */
+int b200_decoder_open(b200_decoder* model, int* slot);
+int b200_decoder_close(b200_decoder* model, int slot);
+int b200_decoder_length(const b200_decoder* model, int slot);  /* tokens run so far; -1 if not open */
+
+/* One step: counts[i] >= 1 next tokens of slot slots[i] (host ids, entry after entry).  want_rows: places
+ * among the step's tokens, counted over all entries, whose logits go to logits_host [n_want, vocab] in
+ * that order.  Synchronous. */
+int b200_decoder_step(b200_decoder* model, int n_entries, const int* slots, const int* counts, const int* tokens,
+                      int n_want, const int* want_rows, float* logits_host);
+/* The same without waiting and without results on the host (one portion: at most max_rows tokens), and
+ * a decode step of one token each for n <= 16 slots that takes the ids left on the device by the last one:
+ * for measurements. */
+int b200_decoder_prefill_device(b200_decoder* model, int n_entries, const int* slots, const int* counts, const int* tokens,
+                                int n_want, const int* want_rows);
+int b200_decoder_decode_device(b200_decoder* model, int n, const int* slots);
+
+/* Continuations of n_req prompts of lens[r] tokens each: out_host [n_req, n_new].  Sampling as in
+ * b200_gpt2_generate (temperature <= 0: greedy).  Requests are admitted to free slots (at most 16 active),
+ * prompts run in portions, active requests decode together; a finished one makes room for the next.  A
+ * request's draws do not depend on what else is active.  Synchronous. */
+int b200_decoder_generate(b200_decoder* model, int n_req, const int* const* prompts, const int* lens, int n_new,
+                          float temperature, int top_k, float top_p, unsigned int seed, int* out_host);
 
 /* ---------------------------------------------------------------- no-allocation forward */
 /* No counterpart in the reference (which has no driver at all).
