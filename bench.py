@@ -1122,6 +1122,9 @@ def main():
                     choices=["all", "matmul", "matmul_bf16", "matmul_bf16x3", "matmul_fp8", "attention", "attention_fp16", "layernorm",
                              "fused_residual_layernorm", "rowwise"],
                     help="per-kernel sweep at 8192 rows instead of the forward benchmark")
+    ap.add_argument("--layered", nargs="?", const="all", default=None,
+                    help="instead of the forward benchmark: prefill and decode of the layered decoders beside GPT-2 of equal width "
+                         "and depth (sizes 768, 1600, with commas between them; default all)")
     ap.add_argument("--case", type=int, default=None, help="with --op: run only this case of the family")
     ap.add_argument("--modes", default="tf32", choices=["tf32", "both"], help="with --op matmul: also time 3xTF32")
     ap.add_argument("--flush-l2", action="store_true", help="with --op: cold L2 before every launch")
@@ -1133,6 +1136,10 @@ def main():
         return run_reference(args)
     if args.op:
         return run_kernel_sweep(args)
+    if args.layered:
+        import bench_layered
+        import __graft_entry__ as ge
+        return bench_layered.run(args, ge.load_package, _peaks(), ClockSampler(0))
     return run_ours(args)
 
 

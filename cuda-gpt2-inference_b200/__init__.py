@@ -49,8 +49,9 @@ EXPORTS = (
     "b200_gpt2_forward_static", "b200_gpt2_static_prepare",
     "b200_gpt2_enable_kv_cache", "b200_gpt2_prefill", "b200_gpt2_decode_step", "b200_gpt2_decode_step_host", "b200_gpt2_generate_greedy", "b200_gpt2_generate", "b200_sample_rows",
     "b200_decoder_create", "b200_decoder_destroy", "b200_decoder_vocab", "b200_decoder_load_safetensors", "b200_decoder_set_tensor",
-    "b200_decoder_finish_load", "b200_decoder_set_graph", "b200_decoder_open", "b200_decoder_close", "b200_decoder_length",
+    "b200_decoder_check_config", "b200_decoder_finish_load", "b200_decoder_set_graph", "b200_decoder_open", "b200_decoder_close", "b200_decoder_length",
     "b200_decoder_step", "b200_decoder_prefill_device", "b200_decoder_decode_device", "b200_decoder_generate",
+    "b200_decoder_set_profile", "b200_decoder_read_profile",
     "b200_gpt2_create_tp", "b200_gpt2_set_allreduce", "b200_gpt2_set_tp_overlap", "b200_gpt2_param_offsets_tp", "b200_gpt2_shard_params_host",
 )
 
@@ -214,6 +215,7 @@ def lib() -> C.CDLL:
         ip = C.POINTER(i)
         l.b200_decoder_create.argtypes = [C.POINTER(vp), vp, C.c_char_p, i, i, i, i]
         l.b200_decoder_destroy.argtypes = [vp]
+        l.b200_decoder_check_config.argtypes = [C.c_char_p, C.c_char_p, i]
         l.b200_decoder_vocab.argtypes = [vp]
         l.b200_decoder_load_safetensors.argtypes = [vp, C.c_char_p]
         l.b200_decoder_set_tensor.argtypes = [vp, C.c_char_p, vp, i, C.POINTER(C.c_long), i]
@@ -225,6 +227,8 @@ def lib() -> C.CDLL:
         l.b200_decoder_step.argtypes = [vp, i, vp, vp, vp, i, vp, vp]
         l.b200_decoder_prefill_device.argtypes = [vp, i, vp, vp, vp, i, vp]
         l.b200_decoder_decode_device.argtypes = [vp, i, vp]
+        l.b200_decoder_set_profile.argtypes = [vp, i]
+        l.b200_decoder_read_profile.argtypes = [vp, i, vp, vp, vp, ip]
         l.b200_decoder_generate.argtypes = [vp, i, vp, vp, i, C.c_float, i, C.c_float, C.c_uint, vp]
         _lib = l.cdll
     return _lib
@@ -746,6 +750,14 @@ class Decoder:
                                             max_slots, max_seq, self.max_rows), "decoder_create")
         self.vocab = int(lib().b200_decoder_vocab(self._h))
 
+    @staticmethod
+    def check_config(config) -> str:
+        """What is wrong with a configuration ("" if nothing); needs no device."""
+        import json
+        msg = C.create_string_buffer(512)
+        st = lib().b200_decoder_check_config(json.dumps(config).encode(), msg, 512)
+        return "" if st == B200_OK else msg.value.decode()
+
     @classmethod
     def from_folder(cls, ctx: Context, folder: str, **kw):
         with open(os.path.join(folder, "config.json")) as f:
@@ -814,6 +826,16 @@ class Decoder:
         import numpy as np
         s = np.asarray(slots, dtype=np.int32)
         self.ctx.check(lib().b200_decoder_decode_device(self._h, s.size, _ptr(s)), "decoder_decode_device")
+
+    def set_profile(self, on: bool):
+        self.ctx.check(lib().b200_decoder_set_profile(self._h, int(on)), "set_profile")
+
+    def read_profile(self) -> dict[str, tuple[float, int]]:
+        """{operator: (milliseconds, launches)} of the general steps since the previous read-out; synchronises."""
+        cap = 64
+        names, ms, n, count = (C.c_char_p * cap)(), (C.c_double * cap)(), (C.c_long * cap)(), C.c_int()
+        self.ctx.check(lib().b200_decoder_read_profile(self._h, cap, names, ms, n, C.byref(count)), "read_profile")
+        return {names[k].decode(): (float(ms[k]), int(n[k])) for k in range(count.value)}
 
     def generate(self, prompts, n_new: int, temperature: float = 0.0, top_k: int = 0, top_p: float = 0.0, seed: int = 0):
         """Continuations [len(prompts), n_new] of prompts of unequal lengths (temperature 0: greedy)."""

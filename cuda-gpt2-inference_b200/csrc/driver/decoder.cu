@@ -216,6 +216,10 @@ struct b200_decoder {
     std::map<int, uint64_t> graph_launches;
     int* gen_log = nullptr;
     size_t gen_log_ints = 0;
+    // per-operator timing (b200_decoder_set_profile): one event pair per launch
+    bool profile = false;
+    std::vector<cudaEvent_t> ev_pool;
+    std::vector<const char*> ev_name;
 };
 
 namespace {
@@ -528,6 +532,25 @@ int finish_load(b200_decoder* m) {
 
 #define TRY(call) do { const int st__ = (call); if (st__ != B200_OK) return st__; } while (0)
 
+int prof_mark(b200_decoder* m, const char* name) {
+    const size_t used = 2 * m->ev_name.size() - (name ? 0 : 1);  // a start, or the stop of the last start
+    while (m->ev_pool.size() <= used) {
+        cudaEvent_t e;
+        B200_CUDA(m->ctx, cudaEventCreate(&e));
+        m->ev_pool.push_back(e);
+    }
+    B200_CUDA(m->ctx, cudaEventRecord(m->ev_pool[used], m->ctx->stream));
+    if (name) m->ev_name.push_back(name);
+    return B200_OK;
+}
+// an operator of a step, timed under its name when profiling is on
+#define OP(name, call)                            \
+    do {                                          \
+        if (m->profile) TRY(prof_mark(m, name));  \
+        TRY(call);                                \
+        if (m->profile) TRY(prof_mark(m, nullptr)); \
+    } while (0)
+
 // ------------------------------------------------------------------ general path
 // out = act(in W^T + bias); out is fp32, or with elem_out the model's element type
 int product(b200_decoder* m, void* out, const void* in, const Matrix& w, int M, int act = ACT_NONE, bool elem_out = false) {
@@ -550,19 +573,20 @@ struct StepView {
 int mixer_mamba1(b200_decoder* m, const Layer& L, const StepView& v) {
     b200_ctx* ctx = m->ctx;
     const LayerSpec& s = *L.spec;
-    TRY(product(m, m->proj, m->h, L.in, v.M));
+    OP("gemm mamba1 in", product(m, m->proj, m->h, L.in, v.M));
     ShortConvArgs c{};
     c.x = m->proj; c.ldx = L.in.N; c.out = m->conv; c.ld_out = L.np; c.w = L.conv_w; c.bias = L.conv_b; c.hist = L.hist; c.seqs = v.seqs;
     c.np = L.np; c.taps = s.conv; c.max_slots = m->max_slots;
-    TRY(launch_short_conv(ctx, c, v.E, v.max_n, m->f32));
-    TRY(product(m, m->aux, m->conv, L.xp, v.M));
-    TRY(launch_slice(ctx, m->low, L.rank_p, m->aux, L.xp.N, s.dt_rank, v.M, m->f32));
-    TRY(product(m, m->wide, m->low, L.dt, v.M));
+    OP("conv mamba1", launch_short_conv(ctx, c, v.E, v.max_n, m->f32));
+    OP("gemm mamba1 x", product(m, m->aux, m->conv, L.xp, v.M));
+    OP("slice", launch_slice(ctx, m->low, L.rank_p, m->aux, L.xp.N, s.dt_rank, v.M, m->f32));
+    OP("gemm mamba1 dt", product(m, m->wide, m->low, L.dt, v.M));
     SelectiveScanArgs a{};
     a.x = m->conv; a.ldx = L.np; a.dt = m->wide; a.lddt = L.np; a.bc = m->aux; a.ldbc = L.xp.N; a.b_col = L.rank_p; a.c_col = L.rank_p + L.sp;
     a.z = m->proj + L.np; a.ldz = L.in.N; a.A2 = L.A2; a.dt_b = L.dt_b; a.D = L.D; a.S = L.S; a.out = m->mix; a.ldo = L.o.K; a.seqs = v.seqs;
     a.inner = s.inner; a.state_pad = L.sp;
-    return launch_selective_scan(ctx, a, v.E, v.max_n, m->f32, m->f32);
+    OP("selective scan", launch_selective_scan(ctx, a, v.E, v.max_n, m->f32, m->f32));
+    return B200_OK;
 }
 
 DeltaArgs delta_args(const b200_decoder* m, const Layer& L, const SeqDesc* seqs, const float* proj) {
@@ -580,17 +604,18 @@ DeltaArgs delta_args(const b200_decoder* m, const Layer& L, const SeqDesc* seqs,
 int mixer_delta(b200_decoder* m, const Layer& L, const StepView& v) {
     b200_ctx* ctx = m->ctx;
     const LayerSpec& s = *L.spec;
-    TRY(product(m, m->proj, m->h, L.in, v.M));
+    OP("gemm delta in", product(m, m->proj, m->h, L.in, v.M));
     ShortConvArgs c{};
     c.x = m->proj; c.ldx = L.in.N; c.out = m->conv; c.ld_out = L.np; c.w = L.conv_w; c.hist = L.hist; c.seqs = v.seqs;
     c.np = L.np; c.taps = s.conv; c.max_slots = m->max_slots;
-    TRY(launch_short_conv(ctx, c, v.E, v.max_n, true));
+    OP("conv delta", launch_short_conv(ctx, c, v.E, v.max_n, true));
     DeltaArgs a = delta_args(m, L, v.seqs, m->proj);
     a.qkv = static_cast<const float*>(m->conv);
     a.out = m->wide; a.ldo = s.heads * L.Dvl;
-    TRY(launch_delta_scan(ctx, a, v.E));
-    return launch_gated_head_norm(ctx, m->mix, L.o.K, m->wide, a.ldo, m->proj + L.gate_col, L.in.N, L.head_norm, v.M, s.heads, s.vdim, L.Dvl,
-                                  m->spec.eps, m->f32);
+    OP("delta scan", launch_delta_scan(ctx, a, v.E));
+    OP("head norm", launch_gated_head_norm(ctx, m->mix, L.o.K, m->wide, a.ldo, m->proj + L.gate_col, L.in.N, L.head_norm, v.M, s.heads, s.vdim, L.Dvl,
+                                           m->spec.eps, m->f32));
+    return B200_OK;
 }
 
 MinGruArgs gru_args(const b200_decoder* m, const Layer& L, const SeqDesc* seqs, const float* proj, void* out, size_t out_elem) {
@@ -603,13 +628,14 @@ MinGruArgs gru_args(const b200_decoder* m, const Layer& L, const SeqDesc* seqs, 
 
 int mixer_parallel(b200_decoder* m, const Layer& L, const StepView& v) {
     b200_ctx* ctx = m->ctx;
-    TRY(product(m, m->proj, m->h, L.in, v.M));
-    TRY(launch_attention_prep(ctx, L.att, m->proj, L.in.N, m->q, v.seqs, v.row_seq, v.M, m->f32));
+    OP("gemm parallel in", product(m, m->proj, m->h, L.in, v.M));
+    OP("attention prep", launch_attention_prep(ctx, L.att, m->proj, L.in.N, m->q, v.seqs, v.row_seq, v.M, m->f32));
     if (!m->f32 && attention_cached_has_mma(L.att))
-        TRY(launch_attention_cached_mma(ctx, L.att, m->q, m->mix, L.o.K, v.seqs, v.pairs, v.num_pairs, v.M, m->max_slots));
+        OP("attention", launch_attention_cached_mma(ctx, L.att, m->q, m->mix, L.o.K, v.seqs, v.pairs, v.num_pairs, v.M, m->max_slots));
     else
-        TRY(launch_attention_cached_simt(ctx, L.att, m->q, m->mix, L.o.K, v.seqs, v.E, v.max_n, m->f32));
-    return launch_min_gru(ctx, gru_args(m, L, v.seqs, m->proj, m->mix, elem(m)), v.E, m->f32);
+        OP("attention", launch_attention_cached_simt(ctx, L.att, m->q, m->mix, L.o.K, v.seqs, v.E, v.max_n, m->f32));
+    OP("min gru", launch_min_gru(ctx, gru_args(m, L, v.seqs, m->proj, m->mix, elem(m)), v.E, m->f32));
+    return B200_OK;
 }
 
 // rows of the step -> logits of the wanted rows in m->logits
@@ -620,7 +646,7 @@ int enqueue_general(b200_decoder* m, const StepView& v) {
     n.x_out = m->x; n.h = m->h; n.M = v.M;
     n.tok = v.tokens; n.embed = m->embed; n.embed_scale = m->spec.embed_scale;
     n.w = m->layers[0].norm1;
-    TRY(launch_residual_rms(ctx, n, m->f32));
+    OP("embed norm", launch_residual_rms(ctx, n, m->f32));
     n.tok = nullptr;
     n.x = m->x;
     n.y = m->y;
@@ -629,19 +655,19 @@ int enqueue_general(b200_decoder* m, const StepView& v) {
         if (L.spec->kind == MIX_MAMBA1) TRY(mixer_mamba1(m, L, v));
         else if (L.spec->kind == MIX_DELTA) TRY(mixer_delta(m, L, v));
         else TRY(mixer_parallel(m, L, v));
-        TRY(product(m, m->y, m->mix, L.o, v.M));
+        OP(L.spec->kind == MIX_MAMBA1 ? "gemm mamba1 o" : (L.spec->kind == MIX_DELTA ? "gemm delta o" : "gemm parallel o"), product(m, m->y, m->mix, L.o, v.M));
         const bool last = i + 1 == m->layers.size();
         n.wb = L.norm1b;
         if (L.spec->ff > 0) {
             n.w = L.norm2;
-            TRY(launch_residual_rms(ctx, n, m->f32));
-            TRY(product(m, m->mix, m->h, L.mlp.up, v.M, m->spec.design->mlp_act, true));
-            TRY(product(m, m->y, m->mix, L.mlp.down, v.M));
+            OP("residual norms", launch_residual_rms(ctx, n, m->f32));
+            OP("gemm mlp up", product(m, m->mix, m->h, L.mlp.up, v.M, m->spec.design->mlp_act, true));
+            OP("gemm mlp down", product(m, m->y, m->mix, L.mlp.down, v.M));
             n.wb = L.norm2b;
         }
         if (!last) {
             n.w = m->layers[i + 1].norm1;
-            TRY(launch_residual_rms(ctx, n, m->f32));
+            OP("residual norms", launch_residual_rms(ctx, n, m->f32));
         }
     }
     if (v.n_want == 0) return B200_OK;
@@ -649,8 +675,9 @@ int enqueue_general(b200_decoder* m, const StepView& v) {
     n.rows = v.want;
     n.M = v.n_want;
     n.x_out = nullptr;
-    TRY(launch_residual_rms(ctx, n, m->f32));
-    return product(m, m->logits, m->h, m->head, v.n_want);
+    OP("final norm", launch_residual_rms(ctx, n, m->f32));
+    OP("gemm head", product(m, m->logits, m->h, m->head, v.n_want));
+    return B200_OK;
 }
 
 // ------------------------------------------------------------------ decode path
@@ -890,6 +917,7 @@ int b200_decoder_destroy(b200_decoder* m) {
     b200_device_guard guard(m->ctx);
     cudaStreamSynchronize(m->ctx->stream);
     for (auto& g : m->graphs) cudaGraphExecDestroy(g.second);
+    for (cudaEvent_t e : m->ev_pool) cudaEventDestroy(e);
     for (void* p : m->owned) cudaFree(p);
     if (m->logits) cudaFree(m->logits);
     if (m->gen_log) cudaFree(m->gen_log);
@@ -900,6 +928,18 @@ int b200_decoder_destroy(b200_decoder* m) {
     m->ctx->tmap_cache.clear();  // the addresses may come back with other shapes
     delete m->store;
     delete m;
+    return B200_OK;
+}
+
+int b200_decoder_check_config(const char* config_json, char* message, int message_bytes) {
+    if (!config_json) return B200_ERR_NULL;
+    if (message && message_bytes > 0) message[0] = 0;
+    try {
+        parse_config(config_json);
+    } catch (const std::exception& e) {
+        if (message && message_bytes > 0) snprintf(message, message_bytes, "%s", e.what());
+        return B200_ERR_SHAPE;
+    }
     return B200_OK;
 }
 
@@ -1175,6 +1215,36 @@ int b200_decoder_generate(b200_decoder* m, int n_req, const int* const* prompts,
     if (st != B200_OK) return st;
     B200_CUDA(ctx, cudaMemcpyAsync(out_host, m->gen_log, log_ints * 4, cudaMemcpyDeviceToHost, ctx->stream));
     return b200_ctx_sync_check(ctx);
+}
+
+int b200_decoder_set_profile(b200_decoder* m, int enabled) {
+    if (!m) return B200_ERR_NULL;
+    m->profile = enabled != 0;
+    return B200_OK;
+}
+
+int b200_decoder_read_profile(b200_decoder* m, int cap, const char** names, double* ms, long* launches, int* count) {
+    if (!m || !names || !ms || !launches || !count) return B200_ERR_NULL;
+    b200_ctx* ctx = m->ctx;
+    B200_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    *count = 0;
+    for (size_t i = 0; i < m->ev_name.size(); ++i) {
+        float t = 0.f;
+        B200_CUDA(ctx, cudaEventElapsedTime(&t, m->ev_pool[2 * i], m->ev_pool[2 * i + 1]));
+        int k = 0;
+        while (k < *count && strcmp(names[k], m->ev_name[i])) ++k;
+        if (k == *count) {
+            if (k == cap) continue;
+            names[k] = m->ev_name[i];
+            ms[k] = 0.0;
+            launches[k] = 0;
+            ++*count;
+        }
+        ms[k] += t;
+        launches[k]++;
+    }
+    m->ev_name.clear();
+    return B200_OK;
 }
 
 }  // extern "C"

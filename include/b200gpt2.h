@@ -459,6 +459,8 @@ typedef struct b200_decoder b200_decoder;
 int b200_decoder_create(b200_decoder** out, b200_ctx* ctx, const char* config_json, int arithmetic, int max_slots,
                         int max_seq, int max_rows);
 int b200_decoder_destroy(b200_decoder* model);
+/* Reads a configuration without a device: B200_OK, or B200_ERR_SHAPE with the reason in message (may be NULL). */
+int b200_decoder_check_config(const char* config_json, char* message, int message_bytes);
 int b200_decoder_vocab(const b200_decoder* model);
 /* Weights: a safetensors file, or tensors one by one (host memory, bf16 or fp32; copied) and finish_load.
  * Names and shapes are checked against the configuration. */
@@ -484,6 +486,11 @@ int b200_decoder_step(b200_decoder* model, int n_entries, const int* slots, cons
 int b200_decoder_prefill_device(b200_decoder* model, int n_entries, const int* slots, const int* counts, const int* tokens,
                                 int n_want, const int* want_rows);
 int b200_decoder_decode_device(b200_decoder* model, int n, const int* slots);
+
+/* Event-timed general steps: names, summed milliseconds and launches of every operator since the last read-out
+ * (at most cap; the names are static strings).  read_profile synchronises. */
+int b200_decoder_set_profile(b200_decoder* model, int enabled);
+int b200_decoder_read_profile(b200_decoder* model, int cap, const char** names, double* ms, long* launches, int* count);
 
 /* Continuations of n_req prompts of lens[r] tokens each: out_host [n_req, n_new].  Sampling as in
  * b200_gpt2_generate (temperature <= 0: greedy).  Requests are admitted to free slots (at most 16 active),
