@@ -470,7 +470,7 @@ void allocate(b200_decoder* m) {
         up(mix, L.o.K);
         if (L.spec->ff) up(mix, L.mlp.up.N);
         if (L.spec->kind == MIX_MAMBA1) { up(conv, L.np); up(aux, L.xp.N); up(wide, L.np); up(low, L.rank_p); }
-        else if (L.spec->kind == MIX_DELTA) { up(conv, 2 * L.np); up(wide, L.spec->heads * L.Dvl); }  // (fp32 in either arithmetic)
+        else if (L.spec->kind == MIX_DELTA) { up(conv, 2 * L.np); up(wide, L.spec->heads * L.Dvl); up(aux, 4 * L.spec->heads); }  // (fp32 in either arithmetic)
         else {
             up(q, (size_t)L.att.H * L.att.Dp);
             up(partial, attention_decode_partial_floats(L.att, 16));
@@ -608,9 +608,13 @@ int mixer_delta(b200_decoder* m, const Layer& L, const StepView& v) {
     ShortConvArgs c{};
     c.x = m->proj; c.ldx = L.in.N; c.out = m->conv; c.ld_out = L.np; c.w = L.conv_w; c.hist = L.hist; c.seqs = v.seqs;
     c.np = L.np; c.taps = s.conv; c.max_slots = m->max_slots;
-    OP("conv delta", launch_short_conv(ctx, c, v.E, v.max_n, true));
+    c.ch0 = L.v_col;
+    OP("conv delta v", launch_short_conv(ctx, c, v.E, v.max_n, true));
     DeltaArgs a = delta_args(m, L, v.seqs, m->proj);
     a.qkv = static_cast<const float*>(m->conv);
+    a.raw = m->proj; a.ld_raw = L.in.N;
+    a.coef = reinterpret_cast<float4*>(m->aux);
+    OP("delta prep", launch_delta_prep(ctx, a, v.E, v.max_n));
     a.out = m->wide; a.ldo = s.heads * L.Dvl;
     OP("delta scan", launch_delta_scan(ctx, a, v.E));
     OP("head norm", launch_gated_head_norm(ctx, m->mix, L.o.K, m->wide, a.ldo, m->proj + L.gate_col, L.in.N, L.head_norm, v.M, s.heads, s.vdim, L.Dvl,

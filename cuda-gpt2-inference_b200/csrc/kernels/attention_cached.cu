@@ -57,39 +57,111 @@ __device__ __forceinline__ void head_vector(float* buf, const float* src, int n,
 }
 
 // ------------------------------------------------------------------ prep
-// one warp per (row, vector): H queries, G keys, G values
-template <typename T>
+// One warp per row walks its vectors (H queries, G keys, G values), four requested at a time.  V > 0: a lane holds V consecutive elements of a vector (head sizes up to 32 V, multiples of V; the
+// rotation's partner is another lane's); V = 0: any size, through shared memory.
+template <typename T, int V>
+__device__ __forceinline__ void store_vec(T* dst, const float (&v)[V > 0 ? V : 1]);
+template <> __device__ __forceinline__ void store_vec<float, 2>(float* dst, const float (&v)[2]) { *reinterpret_cast<float2*>(dst) = make_float2(v[0], v[1]); }
+template <> __device__ __forceinline__ void store_vec<float, 4>(float* dst, const float (&v)[4]) { *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]); }
+template <> __device__ __forceinline__ void store_vec<__half, 2>(__half* dst, const float (&v)[2]) { *reinterpret_cast<__half2*>(dst) = __halves2half2(to_half(v[0]), to_half(v[1])); }
+template <> __device__ __forceinline__ void store_vec<__half, 4>(__half* dst, const float (&v)[4]) {
+    const __half2 a = __halves2half2(to_half(v[0]), to_half(v[1])), b = __halves2half2(to_half(v[2]), to_half(v[3]));
+    *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+template <int V>
+__device__ __forceinline__ void load_vec(float (&v)[V], const float* p) {
+    if (V == 2) { const float2 x = *reinterpret_cast<const float2*>(p); v[0] = x.x; v[1] = x.y; }
+    else { const float4 x = *reinterpret_cast<const float4*>(p); v[0] = x.x; v[1] = x.y; v[2 % V] = x.z; v[3 % V] = x.w; }
+}
+
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
 attention_prep_kernel(const CachedAttention c, const float* __restrict__ proj, int ld, T* __restrict__ q_out,
                       const SeqDesc* __restrict__ seqs, const int* __restrict__ row_seq, int M) {
-    __shared__ float bufs[8][kMaxHead];
+    __shared__ float bufs[V > 0 ? 1 : 8][V > 0 ? 1 : kMaxHead];
     griddep_wait();
     griddep_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int per_row = c.H + 2 * c.G;
-    const size_t u = (size_t)blockIdx.x * 8 + warp;
-    if (u >= (size_t)M * per_row) return;
-    const int row = (int)(u / per_row), j = (int)(u % per_row);
-    const SeqDesc sd = seqs[row_seq[row]];
-    const int pos = sd.pos0 + row - sd.row0;
+    const int row = blockIdx.x * 8 + warp;
+    if (row >= M) return;
+    const int seq = row_seq[row];
+    const int row0 = seqs[seq].row0, slot = seqs[seq].slot, pos = seqs[seq].pos0 + row - row0;
     const float* src = proj + (size_t)row * ld;
-    float* buf = bufs[warp];
-    T* dst;
-    int n_pad;
-    if (j < c.H + c.G) {
-        const bool is_q = j < c.H;
-        head_vector(buf, is_q ? src + c.q_col + j * c.D : src + c.k_col + (j - c.H) * c.D, c.D, c.Dp, (is_q ? c.q_norm : c.k_norm) != nullptr,
-                    is_q ? c.q_norm : c.k_norm, c.eps, c.rot_dims, c.rot + (size_t)pos * (c.rot_dims >> 1), lane);
-        n_pad = c.Dp;
-        dst = is_q ? q_out + ((size_t)row * c.H + j) * c.Dp
-                   : static_cast<T*>(c.K) + (((size_t)sd.slot * c.G + j - c.H) * c.Tp + pos) * c.Dp;
+    const float2* rot = c.rot + (size_t)pos * (c.rot_dims >> 1);
+    const int nvec = c.H + 2 * c.G;
+    auto where = [&](int j, int& n, int& n_pad, int& col) -> T* {
+        if (j < c.H) { n = c.D; n_pad = c.Dp; col = c.q_col + j * c.D; return q_out + ((size_t)row * c.H + j) * c.Dp; }
+        if (j < c.H + c.G) {
+            n = c.D; n_pad = c.Dp; col = c.k_col + (j - c.H) * c.D;
+            return static_cast<T*>(c.K) + (((size_t)slot * c.G + j - c.H) * c.Tp + pos) * c.Dp;
+        }
+        n = c.Dv; n_pad = c.Dvp; col = c.v_col + (j - c.H - c.G) * c.Dv;
+        return static_cast<T*>(c.V) + (((size_t)slot * c.G + j - c.H - c.G) * c.Tp + pos) * c.Dvp;
+    };
+    if constexpr (V == 0) {
+        float* buf = bufs[V > 0 ? 0 : warp];
+        for (int j = 0; j < nvec; ++j) {
+            int n, n_pad, col;
+            T* dst = where(j, n, n_pad, col);
+            const bool is_v = j >= c.H + c.G;
+            const float* w = is_v ? nullptr : (j < c.H ? c.q_norm : c.k_norm);
+            head_vector(buf, src + col, n, n_pad, is_v ? c.v_norm != 0 : w != nullptr, w, c.eps, is_v ? 0 : c.rot_dims, rot, lane);
+            for (int d = lane; d < n_pad; d += 32) dst[d] = to_cache<T>(buf[d]);
+            __syncwarp();
+        }
+        return;
     } else {
-        const int g = j - c.H - c.G;
-        head_vector(buf, src + c.v_col + g * c.Dv, c.Dv, c.Dvp, c.v_norm != 0, nullptr, c.eps, 0, nullptr, lane);
-        n_pad = c.Dvp;
-        dst = static_cast<T*>(c.V) + (((size_t)sd.slot * c.G + g) * c.Tp + pos) * c.Dvp;
+        constexpr int VV = V > 0 ? V : 1;
+        const int e0 = lane * VV, half = c.rot_dims >> 1, hl = half / VV;  // hl: lanes per half of the rotation
+        float cs[VV], sn[VV], wq[VV], wk[VV];
+        const int side = e0 < half ? 0 : (e0 < c.rot_dims ? 1 : 2);
+#pragma unroll
+        for (int i = 0; i < VV; ++i) {
+            cs[i] = 1.f;
+            sn[i] = 0.f;
+            if (side < 2) { const float2 r = rot[e0 + i - side * half]; cs[i] = r.x; sn[i] = side ? r.y : -r.y; }
+            wq[i] = (c.q_norm && e0 + i < c.D) ? __ldg(c.q_norm + e0 + i) : 1.f;
+            wk[i] = (c.k_norm && e0 + i < c.D) ? __ldg(c.k_norm + e0 + i) : 1.f;
+        }
+        const int partner = side == 0 ? lane + hl : (side == 1 ? lane - hl : lane);
+        constexpr int U = 4;  // vectors requested at a time
+        for (int j0 = 0; j0 < nvec; j0 += U) {
+            float v[U][VV];
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                int n = 0, n_pad, col;
+#pragma unroll
+                for (int i = 0; i < VV; ++i) v[u][i] = 0.f;
+                if (j0 + u < nvec) where(j0 + u, n, n_pad, col);
+                if (e0 < n) load_vec<VV>(v[u], src + col + e0);
+            }
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int j = j0 + u;
+                if (j < nvec) {
+                    int n, n_pad, col;
+                    T* dst = where(j, n, n_pad, col);
+                    const bool is_q = j < c.H, is_v = j >= c.H + c.G;
+                    if (is_v ? c.v_norm != 0 : (is_q ? c.q_norm : c.k_norm) != nullptr) {
+                        float s = 0.f;
+#pragma unroll
+                        for (int i = 0; i < VV; ++i) s = fmaf(v[u][i], v[u][i], s);
+                        const float r = 1.0f / sqrtf(warp_sum(s) / (float)n + c.eps);
+#pragma unroll
+                        for (int i = 0; i < VV; ++i) v[u][i] *= is_v ? r : r * (is_q ? wq[i] : wk[i]);
+                    }
+                    if (!is_v && c.rot_dims > 0) {
+#pragma unroll
+                        for (int i = 0; i < VV; ++i) {
+                            const float other = __shfl_sync(0xffffffffu, v[u][i], partner);
+                            v[u][i] = fmaf(other, sn[i], v[u][i] * cs[i]);
+                        }
+                    }
+                    if (e0 < n_pad) store_vec<T, V>(dst + e0, v[u]);  // (elements beyond the head are zero)
+                }
+            }
+        }
     }
-    for (int d = lane; d < n_pad; d += 32) dst[d] = to_cache<T>(buf[d]);
 }
 
 // ------------------------------------------------------------------ fp32 FMA attention
@@ -895,14 +967,28 @@ int launch_decode_lk(b200_ctx* ctx, const CachedAttention& c, const float* proj,
 
 }  // namespace
 
-int launch_attention_prep(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, void* q_out, const SeqDesc* seqs,
-                          const int* row_seq, int M, bool f32) {
-    const unsigned grid = (unsigned)(((size_t)M * (c.H + 2 * c.G) + 7) / 8);
-    cudaError_t le = f32 ? launch_pdl(ctx, attention_prep_kernel<float>, dim3(grid), dim3(256), 0, c, proj, ld, static_cast<float*>(q_out), seqs, row_seq, M)
-                         : launch_pdl(ctx, attention_prep_kernel<__half>, dim3(grid), dim3(256), 0, c, proj, ld, static_cast<__half*>(q_out), seqs, row_seq, M);
+namespace {
+template <typename T>
+int launch_prep(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, void* q_out, const SeqDesc* seqs, const int* row_seq, int M) {
+    const dim3 grid((M + 7) / 8), block(256);
+    // V consecutive elements per lane: everything in multiples of V, the padded heads within a warp's reach
+    auto fits = [&](int v) {
+        return c.Dp <= 32 * v && c.Dvp <= 32 * v && c.D % v == 0 && c.Dv % v == 0 && (c.rot_dims / 2) % v == 0 && c.q_col % v == 0 && c.k_col % v == 0 &&
+               c.v_col % v == 0 && ld % v == 0;
+    };
+    cudaError_t le;
+    if (fits(2)) le = launch_pdl(ctx, attention_prep_kernel<T, 2>, grid, block, 0, c, proj, ld, static_cast<T*>(q_out), seqs, row_seq, M);
+    else if (fits(4)) le = launch_pdl(ctx, attention_prep_kernel<T, 4>, grid, block, 0, c, proj, ld, static_cast<T*>(q_out), seqs, row_seq, M);
+    else le = launch_pdl(ctx, attention_prep_kernel<T, 0>, grid, block, 0, c, proj, ld, static_cast<T*>(q_out), seqs, row_seq, M);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
+}
+}  // namespace
+
+int launch_attention_prep(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, void* q_out, const SeqDesc* seqs,
+                          const int* row_seq, int M, bool f32) {
+    return f32 ? launch_prep<float>(ctx, c, proj, ld, q_out, seqs, row_seq, M) : launch_prep<__half>(ctx, c, proj, ld, q_out, seqs, row_seq, M);
 }
 
 bool attention_cached_has_mma(const CachedAttention& c) { return c.Dp <= 128 && c.Dvp <= 128; }

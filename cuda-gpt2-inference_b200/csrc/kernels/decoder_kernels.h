@@ -80,6 +80,7 @@ struct ShortConvArgs {
     float* hist;
     const SeqDesc* seqs;
     int np, taps, max_slots;  // np: channels rounded up to a multiple of 4 (weights zero beyond)
+    int ch0;                  // first channel (a multiple of 4): the ones before are left alone
 };
 int launch_short_conv(b200_ctx* ctx, const ShortConvArgs& a, int E, int max_n, bool f32);
 
@@ -103,12 +104,17 @@ struct SelectiveScanArgs {
 int selective_state_pad(int state);   // 0: unsupported
 int launch_selective_scan(b200_ctx* ctx, const SelectiveScanArgs& a, int E, int max_n, bool x_f32, bool out_f32);
 
-// Gated delta rule; q, k, v are the convolved projections of a row, head g's q at g*Dl, k at k_col + g*Dl,
-// head h's v at v_col + h*Dvl.  q and k are made unit vectors here (q also times D^-1/2), and
-//   g = exp(-exp(A_log) softplus(a + dt_bias)), beta = sigmoid(b)
-// State [slots][H][Dv][Dpad] fp32.  o goes to out [M, H*Dvl] fp32.
+// Gated delta rule.  In a row head g's q lies at g*Dl, its k at k_col + g*Dl, head h's v at v_col + h*Dvl.
+//   decay = exp(-exp(A_log) softplus(a + dt_bias)), beta = sigmoid(b)
+// State [slots][H][Dv][Dpad] fp32.
+//   prep   convolution + silu of raw's q and k columns -> unit vectors (q also times D^-1/2) in qkv, and coef
+//          (the v columns are a plain short convolution)
+//   scan   qkv, coef -> o in out [M, H*Dvl] fp32
+//   step   one token per sequence, everything from the raw projection (qkv, ld) to the normalised, gated output
 struct DeltaArgs {
     const float* qkv; int ld; int k_col, v_col;
+    const float* raw; int ld_raw;
+    float4* coef;           // [M][H] {decay, beta, k.q, -}
     const float* gates; int ldg; int a_col, b_col;  // columns of the projection holding a and b per head
     const float* negA;      // [H] -exp(A_log)
     const float* dt_bias;   // [H]
@@ -116,13 +122,13 @@ struct DeltaArgs {
     float* out; int ldo;
     const SeqDesc* seqs;
     int H, G, D, Dl, Dv, Dvl;
-    // one-token form: convolution, output norm and gate included; qkv is the raw projection
     const float* conv_w; float* hist; int taps, np, max_slots;
     const float* norm_w; int gate_col; float eps;
 };
 int delta_state_pad(int D);  // 0: unsupported
+int launch_delta_prep(b200_ctx* ctx, const DeltaArgs& a, int E, int max_n);
 int launch_delta_scan(b200_ctx* ctx, const DeltaArgs& a, int E);
-int launch_delta_step(b200_ctx* ctx, const DeltaArgs& a, int E);  // one token per sequence, fused
+int launch_delta_step(b200_ctx* ctx, const DeltaArgs& a, int E);
 
 // minGRU: z = sigmoid(zx[z_col ..]), u = zx[x_col ..], candidate = u + 1/2 (u >= 0) or sigmoid(u);
 // S = (1 - z) S + z candidate;  out = S * silu(zx[g_col ..]) * out_scale

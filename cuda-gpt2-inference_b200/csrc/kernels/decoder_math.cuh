@@ -6,14 +6,26 @@
 
 namespace b200 {
 
-__device__ __forceinline__ float sigmoidf_(float z) {
-    const float e = expf(-fabsf(z));
-    const float r = 1.0f / (1.0f + e);
-    return z >= 0.f ? r : e * r;
-}
+// 1 / (1 + e^-z): one exponential and one reciprocal on the special-function unit, relative error of a few 2^-22
+// (an overflowing exponential gives 0)
+__device__ __forceinline__ float sigmoidf_(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float silu(float z) { return z * sigmoidf_(z); }
-__device__ __forceinline__ float softplusf_(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// log(1 + e^z) = max(z, 0) + log(1 + e), e = e^-|z|; where 1 + e would drop e's digits, from the series of log
+__device__ __forceinline__ float softplusf_(float z) {
+    const float e = __expf(-fabsf(z));
+    const float series = e * fmaf(e, fmaf(e, fmaf(e, fmaf(e, 0.2f, -0.25f), 1.0f / 3.0f), -0.5f), 1.0f);
+    return fmaxf(z, 0.f) + (e < 0.03f ? series : __logf(1.0f + e));
+}
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
+// The same for a 16-bit result: erf by the rational approximation 7.1.26 of Abramowitz and Stegun, Handbook of
+// Mathematical Functions (absolute error below 1.5e-7, here and there a few rounding errors more)
+__device__ __forceinline__ float gelu_erf_h(float z) {
+    const float x = fabsf(z) * 0.70710678118654752f;
+    const float t = __fdividef(1.0f, fmaf(0.3275911f, x, 1.0f));
+    const float p = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+    const float erfc = p * __expf(-x * x);  // of |z| / sqrt(2)
+    return z >= 0.f ? z - 0.5f * z * erfc : 0.5f * z * erfc;
+}
 // 2^x on the special-function unit
 __device__ __forceinline__ float ex2(float x) {
     float y;
@@ -71,6 +83,26 @@ __device__ __forceinline__ void cp_async8(void* smem_dst, const void* src) {
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// which lane of a group holds total number `idx` after reduce_scatter<CNT, L>, and where in its v
+template <int CNT, int L>
+__device__ constexpr int scatter_lane(int idx) {
+    int lane = 0, cnt = CNT;
+    for (int m = 1; m < L && cnt > 1; m <<= 1) {
+        cnt >>= 1;
+        if (idx >= cnt) { lane |= m; idx -= cnt; }
+    }
+    return lane;
+}
+template <int CNT, int L>
+__device__ constexpr int scatter_slot(int idx) {
+    int cnt = CNT;
+    for (int m = 1; m < L && cnt > 1; m <<= 1) {
+        cnt >>= 1;
+        if (idx >= cnt) idx -= cnt;
+    }
+    return idx;
+}
 
 // CNT values per lane, summed over the L lanes of an aligned group and spread over them: on return the
 // lane holds max(1, CNT / L) of the totals in v[0 ..).  Lane bit b (mask 2^b < L) decides between the

@@ -152,7 +152,7 @@ __device__ __forceinline__ void gemm_drain_accumulator_bf16(const GemmArgs& args
                     for (int i = 0; i < 8; ++i) v[i] = gelu_tanh(v[i]);
                 } else if (do_erf) {
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) v[i] = gelu_erf(v[i]);
+                    for (int i = 0; i < 8; ++i) v[i] = gelu_erf_h(v[i]);
                 }
                 uint32_t pk[4];
                 if (args.out_planes == 2) {

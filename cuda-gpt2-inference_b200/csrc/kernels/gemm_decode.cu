@@ -49,16 +49,23 @@ __device__ __forceinline__ void split8(float4 a, float4 b, uint4& hi, uint4& lo)
 
 // Input rows in shared memory: row b at b * stride, groups of eight columns as 16 bytes of hi and 16 of lo.
 // stride = 4 * columns + 16, so that the lanes of a quarter warp (two rows, four groups) touch all banks once.
+//
+// Narrow outputs: K is cut into slices computed by the CTAs of a cluster (blockIdx.x / cluster size = first tile),
+// whose partial sums the first of them reads out of the others' shared memory, in rank order.
 template <int NT, int PRO>  // NT: blocks of eight input rows
 __global__ void __launch_bounds__(kThreads)
-decode_gemm_kernel(const DecodeGemmArgs a) {
+decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice) {
     extern __shared__ __align__(16) uint8_t xs[];
     __shared__ float red[NT][kWarps][16][9];
+    __shared__ float part[NT * 128];
     __shared__ float red1[kWarps];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
-    const int K = a.K, K8 = K >> 3, N = a.N, B = a.B;
+    const int K = a.K, N = a.N, B = a.B;
     const int tiles = (N + 15) >> 4;
-    const int chunk = PRO == DPRO_PLAIN ? min(K, kPlainChunk) : K;  // staged columns
+    const int rank = slices > 1 ? (int)cluster_ctarank() : 0;
+    const int tile0 = blockIdx.x / slices, tile_step = gridDim.x / slices;
+    const int kb = min(K, rank * kslice), ke = min(K, kb + kslice);  // this CTA's columns (may be none)
+    const int chunk = PRO == DPRO_PLAIN ? min(kslice, kPlainChunk) : kslice;  // staged columns
     const int stride = chunk * 4 + 16;
     const uint16_t* __restrict__ W = a.W;
     // this warp's pieces of a chunk: 32 columns each, number warp, warp + 8, ...
@@ -76,15 +83,17 @@ decode_gemm_kernel(const DecodeGemmArgs a) {
         }
     };
     // the weights do not depend on the previous kernel: their first pieces are on the way while it finishes
-    request(blockIdx.x, 0, min(K, chunk), warp);
+    request(tile0, kb, min(ke, kb + chunk), warp);
     griddep_wait();
     griddep_launch_dependents();
 
-    if (PRO == DPRO_RESIDUAL) {
-        // 256 / NR threads per row, NR = rows handled at a time
+    if (PRO == DPRO_RESIDUAL) {  // (never sliced: the norms want whole rows)
+        // 256 / NR threads per row, NR = rows handled at a time; x and y arrive by asynchronous copies, all at once
         const int NR = B > 4 ? 8 : (B > 2 ? 4 : B);
         const int tpr = kThreads / NR, rsub = tid / tpr, t = tid - rsub * tpr;
+        const int K4 = K >> 2, K8 = K >> 3;
         const float inv_c = 1.0f / (float)a.C;
+        float* ys = reinterpret_cast<float*>(xs + (size_t)NT * 8 * stride) + (size_t)rsub * K;
         auto row_sum = [&](float v) {  // over the threads of a row (32 or more of them)
             v = warp_sum(v);
             if (tpr == 32) return v;
@@ -102,29 +111,39 @@ decode_gemm_kernel(const DecodeGemmArgs a) {
         for (int b0 = 0; b0 < used; b0 += NR) {
             const int b = b0 + rsub;
             const bool live = b < B;
-            const float* y = a.y ? a.y + (size_t)(live ? b : 0) * K : nullptr;
             uint8_t* xrow = xs + (size_t)b * stride;
+            int tok = 0;
+            if (live) {
+                if (a.tok) {
+                    tok = a.tok[b];
+                    if (tok < 0 || tok >= a.vocab) { if (t == 0 && blockIdx.x == 0) atomicCAS(a.status, 0, 201); tok = 0; }
+                } else {
+                    for (int i = t; i < K4; i += tpr) cp_async16(xrow + i * 16, a.x + (size_t)b * K + i * 4);
+                }
+                if (a.y) for (int i = t; i < K4; i += tpr) cp_async16(ys + i * 4, a.y + (size_t)b * K + i * 4);
+            }
+            cp_async_commit();
+            cp_async_wait<0>();  // a thread reads back only what it has copied itself
             float rstd_y = 0.f;
-            if (y) {
+            if (a.y) {
                 float s = 0.f;
-                for (int i = t; i < 2 * K8; i += tpr) s += sq4(load4(y, i));
+                if (live) {
+#pragma unroll 4
+                    for (int i = t; i < K4; i += tpr) s += sq4(load4(ys, i));
+                }
                 rstd_y = 1.0f / sqrtf(row_sum(s) * inv_c + a.eps);
             }
-            int tok = 0;
-            if (a.tok && live) {
-                tok = a.tok[b];
-                if (tok < 0 || tok >= a.vocab) { if (t == 0 && blockIdx.x == 0) atomicCAS(a.status, 0, 201); tok = 0; }
-            }
             float s = 0.f;
-            for (int i = t; i < 2 * K8; i += tpr) {  // float4 number i of the row
+#pragma unroll 4
+            for (int i = t; i < K4; i += tpr) {  // float4 number i of the row
                 float4 r = make_float4(0.f, 0.f, 0.f, 0.f);
                 if (live) {
                     if (a.tok) {
                         r = load4(a.embed + (size_t)tok * K, i);
                         r.x *= a.embed_scale; r.y *= a.embed_scale; r.z *= a.embed_scale; r.w *= a.embed_scale;
-                    } else r = load4(a.x + (size_t)b * K, i);
-                    if (y) {
-                        const float4 yv = load4(y, i), wv = __ldg(reinterpret_cast<const float4*>(a.wb) + i);
+                    } else r = *reinterpret_cast<const float4*>(xrow + i * 16);
+                    if (a.y) {
+                        const float4 yv = load4(ys, i), wv = __ldg(reinterpret_cast<const float4*>(a.wb) + i);
                         r.x += yv.x * rstd_y * wv.x; r.y += yv.y * rstd_y * wv.y; r.z += yv.z * rstd_y * wv.z; r.w += yv.w * rstd_y * wv.w;
                     }
                     if (blockIdx.x == 0) *(reinterpret_cast<float4*>(a.x_out + (size_t)b * K) + i) = r;
@@ -134,6 +153,7 @@ decode_gemm_kernel(const DecodeGemmArgs a) {
             }
             const float rstd = 1.0f / sqrtf(row_sum(s) * inv_c + a.eps);
             __syncthreads();  // a group of eight columns may have been formed by two threads
+#pragma unroll 2
             for (int i = t; i < K8; i += tpr) {
                 float4* p = reinterpret_cast<float4*>(xrow + i * 32);
                 float4 v0 = p[0], v1 = p[1];
@@ -147,9 +167,10 @@ decode_gemm_kernel(const DecodeGemmArgs a) {
             }
         }
     } else if (PRO == DPRO_CONV) {
-        const int hist_rows = a.taps - 1;
-        for (int i = tid; i < NT * 8 * K8; i += kThreads) {
-            const int b = i / K8, k = (i - b * K8) * 8;
+        const int hist_rows = a.taps - 1, n8 = (ke - kb) >> 3;
+        const bool writer = tile0 == 0;  // the CTAs of the first tile store what they form of their columns
+        for (int i = tid; i < NT * 8 * n8; i += kThreads) {
+            const int b = i / n8, k = kb + (i - b * n8) * 8;
             float4 v[2] = {make_float4(0.f, 0.f, 0.f, 0.f), make_float4(0.f, 0.f, 0.f, 0.f)};
             if (b < B) {
                 const SeqDesc sd = a.seqs[b];
@@ -159,65 +180,77 @@ decode_gemm_kernel(const DecodeGemmArgs a) {
                 for (int q = 0; q < 2; ++q) {
                     const int k4 = (k >> 2) + q;
                     float4 acc = __ldg(reinterpret_cast<const float4*>(a.conv_b) + k4);
+#pragma unroll 4
                     for (int j = 0; j < a.taps; ++j) {
                         const int back = a.taps - 1 - j;  // tokens before the current one
                         float4 xv = make_float4(0.f, 0.f, 0.f, 0.f);
                         if (back == 0) xv = load4(a.x + (size_t)b * a.ldx, k4);
                         else if (back <= sd.pos0) xv = load4(hr + (size_t)j * K, k4);
-                        if (blockIdx.x == 0 && j > 0) *(reinterpret_cast<float4*>(hw + (size_t)(j - 1) * K) + k4) = xv;
+                        if (writer && j > 0) *(reinterpret_cast<float4*>(hw + (size_t)(j - 1) * K) + k4) = xv;
                         const float4 wv = __ldg(reinterpret_cast<const float4*>(a.conv_w + (size_t)j * K) + k4);
                         acc.x = fmaf(xv.x, wv.x, acc.x); acc.y = fmaf(xv.y, wv.y, acc.y);
                         acc.z = fmaf(xv.z, wv.z, acc.z); acc.w = fmaf(xv.w, wv.w, acc.w);
                     }
                     v[q] = make_float4(silu(acc.x), silu(acc.y), silu(acc.z), silu(acc.w));
-                    if (blockIdx.x == 0) *(reinterpret_cast<float4*>(a.conv_out + (size_t)b * K) + k4) = v[q];
+                    if (writer) *(reinterpret_cast<float4*>(a.conv_out + (size_t)b * K) + k4) = v[q];
                 }
             }
             uint4 hi, lo;
             split8(v[0], v[1], hi, lo);
-            uint4* p = reinterpret_cast<uint4*>(xs + (size_t)b * stride + (k >> 3) * 32);
+            uint4* p = reinterpret_cast<uint4*>(xs + (size_t)b * stride + ((k - kb) >> 3) * 32);
             p[0] = hi;
             p[1] = lo;
         }
     }
 
     auto stage_plain = [&](int k0, int kend) {
-        const int n8 = (kend - k0) >> 3;
-        for (int i = tid; i < NT * 8 * n8; i += kThreads) {
-            const int b = i / n8, j = i - b * n8;
-            float4 v0 = make_float4(0.f, 0.f, 0.f, 0.f), v1 = v0;
-            if (b < B) {
-                const float* p = a.x + (size_t)b * a.ldx + k0 + j * 8;
-                v0 = load4(p, 0);
-                v1 = load4(p, 1);
+        const int n8 = (kend - k0) >> 3, total = NT * 8 * n8;
+        constexpr int Q = 4;  // groups of eight columns requested before any is used
+        for (int i0 = tid; i0 < total; i0 += Q * kThreads) {
+            float4 v[Q][2];
+            int at[Q];
+#pragma unroll
+            for (int q = 0; q < Q; ++q) {
+                const int i = i0 + q * kThreads, b = i / n8, j = i - b * n8;
+                at[q] = i < total ? b * stride + j * 32 : -1;
+                v[q][0] = v[q][1] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (i < total && b < B) {
+                    const float* p = a.x + (size_t)b * a.ldx + k0 + j * 8;
+                    v[q][0] = load4(p, 0);
+                    v[q][1] = load4(p, 1);
+                }
             }
-            uint4 hi, lo;
-            split8(v0, v1, hi, lo);
-            uint4* p = reinterpret_cast<uint4*>(xs + (size_t)b * stride + j * 32);
-            p[0] = hi;
-            p[1] = lo;
+#pragma unroll
+            for (int q = 0; q < Q; ++q)
+                if (at[q] >= 0) {
+                    uint4 hi, lo;
+                    split8(v[q][0], v[q][1], hi, lo);
+                    uint4* p = reinterpret_cast<uint4*>(xs + at[q]);
+                    p[0] = hi;
+                    p[1] = lo;
+                }
         }
     };
 
     bool staged = PRO != DPRO_PLAIN;  // a plain input of one chunk is staged once for all tiles
     if (staged) __syncthreads();
-    for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x) {
+    for (int tile = tile0; tile < tiles; tile += tile_step) {
         float acc[NT][4];
 #pragma unroll
         for (int t = 0; t < NT; ++t) acc[t][0] = acc[t][1] = acc[t][2] = acc[t][3] = 0.f;
-        for (int k0 = 0; k0 < K; k0 += chunk) {
-            const int kend = min(K, k0 + chunk);
+        for (int k0 = kb; k0 < ke; k0 += chunk) {
+            const int kend = min(ke, k0 + chunk);
             const int pieces = (kend - k0 + 31) >> 5;
             if (!staged) {
-                if (k0 > 0 || tile != (int)blockIdx.x) __syncthreads();  // everyone is done with the previous chunk
+                if (k0 > kb || tile != tile0) __syncthreads();  // everyone is done with the previous chunk
                 stage_plain(k0, kend);
                 __syncthreads();
-                if (K <= chunk) staged = true;
+                if (kslice <= chunk) staged = true;
             }
             if (warp >= pieces) {
                 // nothing of this chunk, but the first pieces of the next one still have to be requested
-                if (kend < K) request(tile, kend, min(K, kend + chunk), warp);
-                else if (tile + (int)gridDim.x < tiles) request(tile + gridDim.x, 0, min(K, chunk), warp);
+                if (kend < ke) request(tile, kend, min(ke, kend + chunk), warp);
+                else if (tile + tile_step < tiles) request(tile + tile_step, kb, min(ke, kb + chunk), warp);
                 continue;
             }
             for (int p0 = warp; p0 < pieces; p0 += kU * kWarps) {
@@ -225,8 +258,8 @@ decode_gemm_kernel(const DecodeGemmArgs a) {
 #pragma unroll
                 for (int u = 0; u < kU; ++u) { cur[u][0] = w[u][0]; cur[u][1] = w[u][1]; }
                 if (p0 + kU * kWarps < pieces) request(tile, k0, kend, p0 + kU * kWarps);
-                else if (kend < K) request(tile, kend, min(K, kend + chunk), warp);
-                else if (tile + (int)gridDim.x < tiles) request(tile + gridDim.x, 0, min(K, chunk), warp);
+                else if (kend < ke) request(tile, kend, min(ke, kend + chunk), warp);
+                else if (tile + tile_step < tiles) request(tile + tile_step, kb, min(ke, kb + chunk), warp);
 #pragma unroll
                 for (int u = 0; u < kU; ++u) {
                     const int p = p0 + u * kWarps;
@@ -259,20 +292,40 @@ decode_gemm_kernel(const DecodeGemmArgs a) {
             red[t][warp][g + 8][2 * c + 1] = acc[t][3];
         }
         __syncthreads();
-        for (int i = tid; i < NT * 128; i += kThreads) {
-            const int n = i & 15, b = i >> 4;
-            const int row = tile * 16 + n;
-            if (b < B && row < N) {
+        if (slices > 1) {
+            for (int i = tid; i < NT * 128; i += kThreads) {
                 float v = 0.f;
 #pragma unroll
-                for (int q = 0; q < kWarps; ++q) v += red[b >> 3][q][n][b & 7];
-                if (a.bias) v += __ldg(a.bias + row);
-                if (a.act == ACT_GELU_ERF) v = gelu_erf(v);
-                else if (a.act == ACT_GELU_TANH) v = gelu_tanh(v);
-                a.out[(size_t)b * a.ldo + row] = v;
+                for (int q = 0; q < kWarps; ++q) v += red[i >> 7][q][i & 15][(i >> 4) & 7];
+                part[i] = v;
+            }
+            cluster_sync_all();
+        }
+        if (rank == 0) {
+            for (int i = tid; i < NT * 128; i += kThreads) {
+                const int n = i & 15, b = i >> 4;
+                const int row = tile * 16 + n;
+                if (b < B && row < N) {
+                    float v = 0.f;
+                    if (slices > 1) {
+                        for (int s = 0; s < slices; ++s) {
+                            float p;
+                            asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(p) : "r"(map_to_cta(smem_u32(part + i), s)) : "memory");
+                            v += p;
+                        }
+                    } else {
+#pragma unroll
+                        for (int q = 0; q < kWarps; ++q) v += red[b >> 3][q][n][b & 7];
+                    }
+                    if (a.bias) v += __ldg(a.bias + row);
+                    if (a.act == ACT_GELU_ERF) v = gelu_erf(v);
+                    else if (a.act == ACT_GELU_TANH) v = gelu_tanh(v);
+                    a.out[(size_t)b * a.ldo + row] = v;
+                }
             }
         }
-        __syncthreads();
+        if (slices > 1) cluster_sync_all();  // the partial sums have been read (and nobody leaves before that)
+        else __syncthreads();
     }
 }
 
@@ -283,13 +336,40 @@ int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
         B200_CUDA(ctx, cudaFuncSetAttribute(decode_gemm_kernel<NT, PRO>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem));
         attr_set[ctx->device & 63] = true;
     }
-    const int chunk = PRO == DPRO_PLAIN ? (a.K < kPlainChunk ? a.K : kPlainChunk) : a.K;
-    const size_t smem = (size_t)NT * 8 * (chunk * 4 + 16);
-    if (smem > (size_t)kMaxSmem) return B200_ERR_LIMIT;
     const int tiles = (a.N + 15) / 16;
+    // K slices while the CTAs of one wave (two per SM) are not used up and a warp keeps at least a piece
+    int slices = 1;
+    if (PRO != DPRO_RESIDUAL)
+        while (slices < 8 && tiles * slices * 2 <= 2 * ctx->num_sms && a.K / (slices * 2) >= 256) slices *= 2;
+    const int kslice = ((a.K + slices - 1) / slices + 31) / 32 * 32;
+    const int chunk = PRO == DPRO_PLAIN ? (kslice < kPlainChunk ? kslice : kPlainChunk) : kslice;
+    const int nr = a.B > 4 ? 8 : (a.B > 2 ? 4 : a.B);
+    const size_t smem = (size_t)NT * 8 * (chunk * 4 + 16) + (PRO == DPRO_RESIDUAL && a.y ? (size_t)nr * a.K * 4 : 0);
+    if (smem > (size_t)kMaxSmem) return B200_ERR_LIMIT;
     const int per_sm = smem > 100 * 1024 ? 1 : 2;
-    const int grid = tiles < per_sm * ctx->num_sms ? tiles : per_sm * ctx->num_sms;
-    cudaError_t le = launch_pdl(ctx, decode_gemm_kernel<NT, PRO>, dim3(grid), dim3(kThreads), smem, a);
+    int grid = tiles * slices;
+    if (grid > per_sm * ctx->num_sms) grid = per_sm * ctx->num_sms / slices * slices;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(grid);
+    cfg.blockDim = dim3(kThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    cudaLaunchAttribute attr[2];
+    int n = 0;
+    if (slices > 1) {
+        attr[n].id = cudaLaunchAttributeClusterDimension;
+        attr[n].val.clusterDim.x = slices;
+        attr[n].val.clusterDim.y = attr[n].val.clusterDim.z = 1;
+        ++n;
+    }
+    if (ctx->pdl) {
+        attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[n].val.programmaticStreamSerializationAllowed = 1;
+        ++n;
+    }
+    cfg.attrs = attr;
+    cfg.numAttrs = n;
+    const cudaError_t le = cudaLaunchKernelEx(&cfg, decode_gemm_kernel<NT, PRO>, a, slices, kslice);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
@@ -297,7 +377,9 @@ int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
 
 }  // namespace
 
-bool decode_gemm_fits(int K, int B) { return (size_t)(B <= 8 ? 8 : 16) * (K * 4 + 16) <= (size_t)kMaxSmem; }
+bool decode_gemm_fits(int K, int B) {
+    return (size_t)(B <= 8 ? 8 : 16) * ((K + 31) / 32 * 128 + 16) + (size_t)(B > 8 ? 8 : B) * K * 4 + (B == 3 || (B > 4 && B < 8) ? (size_t)4 * K * 4 : 0) <= (size_t)kMaxSmem;
+}
 
 int launch_decode_gemm(b200_ctx* ctx, const DecodeGemmArgs& a, int prologue) {
     if (a.B < 1 || a.B > 16 || a.K % 8 || a.N < 1) return B200_ERR_SHAPE;

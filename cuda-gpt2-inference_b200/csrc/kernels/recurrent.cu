@@ -4,6 +4,7 @@
 // All of them treat a step's rows as sequences (SeqDesc): a sequence that starts (pos0 = 0) begins with
 // a zero state whatever its slot holds, any other continues from the slot, so a prompt may be cut anywhere
 // and a slot needs no clearing.  State and everything that enters a recurrence is fp32.
+#include <cstdlib>
 #include <cuda_bf16.h>
 #include "decoder_kernels.h"
 #include "decoder_math.cuh"
@@ -23,7 +24,7 @@ short_conv_kernel(const ShortConvArgs a) {
     griddep_launch_dependents();
     const SeqDesc sd = a.seqs[blockIdx.z];
     const int t0 = blockIdx.y * kConvTok;
-    const int c4 = blockIdx.x * blockDim.x + threadIdx.x;
+    const int c4 = (a.ch0 >> 2) + blockIdx.x * blockDim.x + threadIdx.x;
     if (t0 >= sd.n || c4 * 4 >= a.np) return;
     const int taps = TAPS > 0 ? TAPS : a.taps, hrows = taps - 1;
     const float* hr = a.hist + ((size_t)sd.bank * a.max_slots + sd.slot) * hrows * a.np;
@@ -207,194 +208,293 @@ selective_scan_kernel(const SelectiveScanArgs a) {
 // ------------------------------------------------------------------ gated delta rule
 // The columns of a head's state S [D, Dv] do not touch one another: with S the state before the token,
 //   u = beta (v - g S^T k),   o = g S^T q + (k.q) u,   S <- g S + k u^T
-// - both products read the old state, so one reduction serves them.  L = D / 16 lanes share a group of four
-// columns and keep 16 rows of each in registers (as pairs: one instruction does two multiply-adds); lane l
-// owns rows 4 (l + L i) .. + 3, so the lanes read consecutive 16-byte pieces of k and q.
-constexpr int kDeltaTok = 16, kDeltaRows = 16, kDeltaCols = 4;
-constexpr int kDeltaThreads = 128;
+// - both products read the old state, so one reduction serves them.  The decay is kept out of the state: with
+// S = c R and c the product of the decays since c was last 1,
+//   c <- c g,   u = beta (v - c R^T k),   o = c R^T q + (k.q) u,   R <- R + k (u / c)^T
+// which is three multiply-adds per element instead of four operations; when c has become small R takes it in.
+// L = D / 16 lanes share a group of NC columns and keep 16 rows of each in registers (as pairs: one instruction
+// does two multiply-adds); lane l owns rows 4 (l + L i) .. + 3, so the lanes read consecutive 16-byte pieces of
+// k and q.
+constexpr int kDeltaTok = 16;
+constexpr float kDeltaSmall = 1e-9f;
 
-template <int L>
+template <int L, int NC>
 struct DeltaCore {
-    static constexpr int D = 16 * L;
-    uint64_t S[kDeltaCols][kDeltaRows / 2];
+    static constexpr int D = 16 * L, CNT = 2 * NC;            // totals per token: R^T k of the columns, then R^T q
+    static constexpr int kHeld = L >= CNT ? 1 : CNT / L;      // ... of which a lane holds this many after the reduction
+    static constexpr int kOut = kHeld > NC ? NC : kHeld;      // ... belonging to one of the two products
+    uint64_t S[NC][8];  // R
+    float c;
     __device__ __forceinline__ void zero() {
+        c = 1.f;
 #pragma unroll
-        for (int c = 0; c < kDeltaCols; ++c)
+        for (int j = 0; j < NC; ++j)
 #pragma unroll
-            for (int i = 0; i < kDeltaRows / 2; ++i) S[c][i] = 0ull;
+            for (int i = 0; i < 8; ++i) S[j][i] = 0ull;
     }
     // column j of this group at base + j * D; columns from ncol on are left alone
     __device__ __forceinline__ void load(const float* base, int l, int ncol) {
+        c = 1.f;
 #pragma unroll
-        for (int c = 0; c < kDeltaCols; ++c)
+        for (int j = 0; j < NC; ++j)
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 ulonglong2 v = make_ulonglong2(0ull, 0ull);
-                if (c < ncol) v = *reinterpret_cast<const ulonglong2*>(base + (size_t)c * D + 4 * (l + L * i));
-                S[c][2 * i] = v.x;
-                S[c][2 * i + 1] = v.y;
+                if (j < ncol) v = *reinterpret_cast<const ulonglong2*>(base + (size_t)j * D + 4 * (l + L * i));
+                S[j][2 * i] = v.x;
+                S[j][2 * i + 1] = v.y;
             }
     }
-    __device__ __forceinline__ void store(float* base, int l, int ncol) const {
+    __device__ __forceinline__ void absorb() {
+        const uint64_t cc = pack2(c, c);
 #pragma unroll
-        for (int c = 0; c < kDeltaCols; ++c)
+        for (int j = 0; j < NC; ++j)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) S[j][i] = mul2(cc, S[j][i]);
+        c = 1.f;
+    }
+    __device__ __forceinline__ void store(float* base, int l, int ncol) {
+        absorb();
+#pragma unroll
+        for (int j = 0; j < NC; ++j)
 #pragma unroll
             for (int i = 0; i < 4; ++i)
-                if (c < ncol) *reinterpret_cast<ulonglong2*>(base + (size_t)c * D + 4 * (l + L * i)) = make_ulonglong2(S[c][2 * i], S[c][2 * i + 1]);
+                if (j < ncol) *reinterpret_cast<ulonglong2*>(base + (size_t)j * D + 4 * (l + L * i)) = make_ulonglong2(S[j][2 * i], S[j][2 * i + 1]);
     }
-    // One token.  q, k: D floats in shared memory; v: the group's four values, there too; lane: lane in the warp.
-    // Returns o of column ocol(lane) (valid where owns_o(lane)); with fewer than eight lanes a lane holds
-    // several columns: o[0 .. kHeld).
-    static constexpr int kHeld = L >= 8 ? 1 : 8 / L;         // totals a lane holds after the reduction
-    static constexpr int kOut = kHeld > 4 ? 4 : kHeld;
-    // of the eight totals, 0-3 are S^T k and 4-7 are S^T q of the four columns; lane bit 0 separates the two
-    static __device__ __forceinline__ int ocol(int lane) { return scatter_first<8, L>(lane) & 3; }
-    static __device__ __forceinline__ bool owns_o(int lane) { return (lane & 1) && scatter_owner<8, L>(lane); }
-    __device__ __forceinline__ void token(const float* q, const float* k, const float* v, float g, float beta, float kq, int lane,
+    // o[j] of token() is column ocol + j, on the lanes where owns_o holds (the reduction's first halving, by lane
+    // bit 0, separates R^T k from R^T q)
+    static __device__ __forceinline__ int ocol(int lane) { return scatter_first<CNT, L>(lane) & (NC - 1); }
+    static __device__ __forceinline__ bool owns_o(int lane) { return (lane & 1) && scatter_owner<CNT, L>(lane); }
+    struct Row { uint64_t r[8]; };  // this lane's pairs of a D-vector in shared memory
+    static __device__ __forceinline__ Row row(const float* p, int l) {
+        Row x;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p + 4 * (l + L * i));
+            x.r[2 * i] = v.x;
+            x.r[2 * i + 1] = v.y;
+        }
+        return x;
+    }
+    // One token.  kr: its key; qr: its query on entry, the row at q_next on return (requested as soon as the registers are
+    // free); v: the group's values in shared memory.
+    __device__ __forceinline__ void token(const Row& kr, Row& qr, const float* q_next, const float* v, float g, float beta, float kq, int lane,
                                           float (&o)[kOut]) {
-        const int l = lane & (L - 1);
-        uint64_t kr[8], acc[8];
+        c *= g;
+        if (c < kDeltaSmall) absorb();  // (the same decay in all lanes of a head)
+        const float inv_c = __fdividef(1.0f, c);
+        uint64_t acc[CNT];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const ulonglong2 kv = *reinterpret_cast<const ulonglong2*>(k + 4 * (l + L * i));
-            kr[2 * i] = kv.x;
-            kr[2 * i + 1] = kv.y;
-        }
+        for (int j = 0; j < CNT; ++j) acc[j] = 0ull;
 #pragma unroll
-        for (int c = 0; c < 8; ++c) acc[c] = 0ull;
+        for (int i = 0; i < 8; ++i)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const ulonglong2 qv = *reinterpret_cast<const ulonglong2*>(q + 4 * (l + L * i));
-#pragma unroll
-            for (int c = 0; c < kDeltaCols; ++c) {
-                acc[c] = fma2(kr[2 * i], S[c][2 * i], acc[c]);
-                acc[4 + c] = fma2(qv.x, S[c][2 * i], acc[4 + c]);
-                acc[c] = fma2(kr[2 * i + 1], S[c][2 * i + 1], acc[c]);
-                acc[4 + c] = fma2(qv.y, S[c][2 * i + 1], acc[4 + c]);
+            for (int j = 0; j < NC; ++j) {
+                acc[j] = fma2(kr.r[i], S[j][i], acc[j]);
+                acc[NC + j] = fma2(qr.r[i], S[j][i], acc[NC + j]);
             }
-        }
-        float t[8];
+        qr = row(q_next, lane & (L - 1));
+        float t[CNT];
 #pragma unroll
-        for (int c = 0; c < 8; ++c) {
+        for (int j = 0; j < CNT; ++j) {
             float x, y;
-            unpack2(acc[c], x, y);
-            t[c] = x + y;
+            unpack2(acc[j], x, y);
+            t[j] = x + y;
         }
-        reduce_scatter<8, L>(t, lane);
-        const int first = scatter_first<8, L>(lane);  // t[j] is total number first + j
-        // u on the lanes that hold S^T k (first < 4), handed to the whole group
+        reduce_scatter<CNT, L>(t, lane);
+        const int first = scatter_first<CNT, L>(lane);  // t[j] is total number first + j
         float um[kOut];
 #pragma unroll
-        for (int j = 0; j < kOut; ++j) um[j] = beta * (v[(first + j) & 3] - g * t[j]);
+        for (int j = 0; j < kOut; ++j) um[j] = beta * (v[(first + j) & (NC - 1)] - c * t[j]);
         const int base = lane & ~(L - 1);
-        float u[4];
+        float u[NC];
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-            // the lane whose totals include number c: halving by bits 0, 1, 2 in turn
-            int src = 0;
-            if (L >= 4 && (c & 2)) src |= 2;
-            if (L >= 8 && (c & 1)) src |= 4;
-            u[c] = __shfl_sync(0xffffffffu, um[kHeld >= 4 ? c : (kHeld == 2 ? (c & 1) : 0)], base + src);
-        }
+        for (int j = 0; j < NC; ++j) u[j] = __shfl_sync(0xffffffffu, um[scatter_slot<CNT, L>(j) & (kOut - 1)], base + scatter_lane<CNT, L>(j));
 #pragma unroll
         for (int j = 0; j < kOut; ++j) {
-            const int col = (first + j) & 3;
-            const float uc = (kHeld >= 4) ? u[j & 3] : (col & 2 ? (col & 1 ? u[3] : u[2]) : (col & 1 ? u[1] : u[0]));
-            o[j] = fmaf(g, t[j], kq * uc);
+            const int col = (first + j) & (NC - 1);
+            float uc = u[0];
+#pragma unroll
+            for (int x = 1; x < NC; ++x) uc = col == x ? u[x] : uc;
+            o[j] = fmaf(c, t[j], kq * uc);
         }
-        const uint64_t gg = pack2(g, g);
 #pragma unroll
-        for (int c = 0; c < kDeltaCols; ++c) {
-            const uint64_t uu = pack2(u[c], u[c]);
+        for (int j = 0; j < NC; ++j) {
+            const float us = u[j] * inv_c;
+            const uint64_t uu = pack2(us, us);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) S[c][i] = fma2(kr[i], uu, mul2(gg, S[c][i]));
+            for (int i = 0; i < 8; ++i) S[j][i] = fma2(kr.r[i], uu, S[j][i]);
         }
     }
 };
 
-// Prefill: a CTA walks one (sequence, head) for cols = blockDim.x / L * 4 columns of Dv, in tiles of 16 tokens
-// staged two deep; q and k of a staged tile are made unit vectors in place, one warp per token.
-template <int L>
-__global__ void __launch_bounds__(kDeltaThreads)
+// What the scan wants per token: convolved and activated q and k as unit vectors (q also times D^-1/2) and, per
+// head, {decay, beta, k.q}.  One warp per (sequence, key/value head, run of 16 tokens).
+template <int TAPS>
+__global__ void __launch_bounds__(128)
+delta_prep_kernel(const DeltaArgs a) {
+    constexpr int W = TAPS > 0 ? TAPS : 1;
+    griddep_wait();
+    griddep_launch_dependents();
+    const SeqDesc sd = a.seqs[blockIdx.z];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int t0 = (blockIdx.y * 4 + warp) * kDeltaTok, g = blockIdx.x;
+    if (t0 >= sd.n) return;
+    const int t1 = min(sd.n, t0 + kDeltaTok);
+    const int taps = TAPS > 0 ? TAPS : a.taps, hrows = taps - 1;
+    const float* hr = a.hist + ((size_t)sd.bank * a.max_slots + sd.slot) * hrows * a.np;
+    float* hw = a.hist + ((size_t)(sd.bank ^ 1) * a.max_slots + sd.slot) * hrows * a.np;
+    const float* xin = a.raw + (size_t)sd.row0 * a.ld_raw;
+    float* qkv = const_cast<float*>(a.qkv) + (size_t)sd.row0 * a.ld;
+    const int qc = g * a.Dl, kc = a.k_col + g * a.Dl;
+    auto input = [&](int i, int ch) {
+        if (i >= 0) return xin[(size_t)i * a.ld_raw + ch];
+        if (sd.pos0 + i < 0) return 0.f;
+        return hr[(size_t)(hrows + i) * a.np + ch];
+    };
+    const float qscale = rsqrtf((float)a.D);
+    const int per = a.H / a.G;
+    float sq[kDeltaTok], sk[kDeltaTok], qk[kDeltaTok];  // per token: squares and product of this lane's channels
+#pragma unroll
+    for (int t = 0; t < kDeltaTok; ++t) sq[t] = sk[t] = qk[t] = 0.f;
+    // first pass, 32 channels of q and k at a time: convolution and silu, to memory as they are
+    for (int d = lane; d < a.Dl; d += 32) {
+        float wq[W], wk[W], xq[W], xk[W];
+        if (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j < W; ++j) { wq[j] = __ldg(a.conv_w + (size_t)j * a.np + qc + d); wk[j] = __ldg(a.conv_w + (size_t)j * a.np + kc + d); }
+#pragma unroll
+            for (int j = 0; j + 1 < W; ++j) { xq[j] = input(t0 - (W - 1) + j, qc + d); xk[j] = input(t0 - (W - 1) + j, kc + d); }
+        }
+        float iq[kDeltaTok], ik[kDeltaTok];
+#pragma unroll
+        for (int t = 0; t < kDeltaTok; ++t) {
+            iq[t] = ik[t] = 0.f;
+            if (TAPS > 0 && t0 + t < t1) { iq[t] = input(t0 + t, qc + d); ik[t] = input(t0 + t, kc + d); }
+        }
+#pragma unroll
+        for (int t = 0; t < kDeltaTok; ++t) {
+            float q = 0.f, k = 0.f;
+            if (TAPS > 0) {
+                xq[W - 1] = iq[t];
+                xk[W - 1] = ik[t];
+#pragma unroll
+                for (int j = 0; j < W; ++j) { q = fmaf(xq[j], wq[j], q); k = fmaf(xk[j], wk[j], k); }
+#pragma unroll
+                for (int j = 0; j + 1 < W; ++j) { xq[j] = xq[j + 1]; xk[j] = xk[j + 1]; }
+            } else if (t0 + t < t1) {
+                for (int j = 0; j < taps; ++j) {
+                    q = fmaf(input(t0 + t - hrows + j, qc + d), __ldg(a.conv_w + (size_t)j * a.np + qc + d), q);
+                    k = fmaf(input(t0 + t - hrows + j, kc + d), __ldg(a.conv_w + (size_t)j * a.np + kc + d), k);
+                }
+            }
+            q = silu(q);
+            k = silu(k);
+            if (t0 + t < t1) {
+                qkv[(size_t)(t0 + t) * a.ld + qc + d] = q;
+                qkv[(size_t)(t0 + t) * a.ld + kc + d] = k;
+                sq[t] = fmaf(q, q, sq[t]);
+                sk[t] = fmaf(k, k, sk[t]);
+                qk[t] = fmaf(q, k, qk[t]);
+            }
+        }
+        if (t1 == sd.n)
+            for (int e = 0; e < hrows; ++e) {
+                hw[(size_t)e * a.np + qc + d] = input(sd.n - hrows + e, qc + d);
+                hw[(size_t)e * a.np + kc + d] = input(sd.n - hrows + e, kc + d);
+            }
+    }
+    // sums over the lanes, and the scales applied to what this lane has written
+#pragma unroll
+    for (int t = 0; t < kDeltaTok; ++t) {
+        if (t0 + t >= t1) break;
+        const float rq = qscale / sqrtf(warp_sum(sq[t]) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(sk[t]) + 1e-6f);
+        const float kq = warp_sum(qk[t]) * rq * rk;
+        float* row = qkv + (size_t)(t0 + t) * a.ld;
+        for (int d = lane; d < a.Dl; d += 32) { row[qc + d] *= rq; row[kc + d] *= rk; }
+        const float* gr = a.gates + (size_t)(sd.row0 + t0 + t) * a.ldg;
+        for (int j = lane; j < per; j += 32) {
+            const int h = g * per + j;
+            const float decay = expf(__ldg(a.negA + h) * softplusf_(gr[a.a_col + h] + __ldg(a.dt_bias + h)));
+            a.coef[(size_t)(sd.row0 + t0 + t) * a.H + h] = make_float4(decay, sigmoidf_(gr[a.b_col + h]), kq, 0.f);
+        }
+    }
+}
+
+// Prefill: a CTA walks one (sequence, head) for blockDim.x / L * NC columns of Dv, in tiles of 16 tokens staged two
+// deep by asynchronous copies.
+template <int L, int NC>
+__global__ void __launch_bounds__(128)
 delta_scan_kernel(const DeltaArgs a) {
+    using Core = DeltaCore<L, NC>;
     constexpr int D = 16 * L;
     extern __shared__ __align__(16) float sm[];
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nwarps = blockDim.x >> 5;
-    const int cols = blockDim.x / L * kDeltaCols;
-    const int tile_f = kDeltaTok * (2 * D + cols);
-    float* coef = sm + 2 * tile_f;  // [2][16][4]: g, beta, k.q
+    const int tid = threadIdx.x, lane = tid & 31;
+    const int cols = blockDim.x / L * NC;
+    const int cpad = (cols + 3) & ~3;
+    const int tile_f = kDeltaTok * (2 * D + cpad + 4);  // q, k, v, coefficients
     const int h = blockIdx.x, c0 = blockIdx.y * cols;
     const int kvh = h / (a.H / a.G);
-    const float negA = __ldg(a.negA + h), dtb = __ldg(a.dt_bias + h);
-    const float qscale = rsqrtf((float)a.D);
-    // rows of k and q beyond the head's dimension stay zero in both tiles
-    for (int i = tid; i < 2 * tile_f; i += blockDim.x) sm[i] = 0.f;
+    // rows of k and q beyond the head's dimension and columns beyond Dv stay zero in both tiles
+    for (int i = tid; i < 2 * tile_f + D; i += blockDim.x) sm[i] = 0.f;
     griddep_wait();
     griddep_launch_dependents();
     const SeqDesc sd = a.seqs[blockIdx.z];
     const int grp = tid / L, l = tid & (L - 1);
-    const int gc = c0 + grp * kDeltaCols;         // first column of this group
-    const int ncol = min(kDeltaCols, a.Dv - gc);  // may be <= 0
-    DeltaCore<L> core;
+    const int gc = c0 + grp * NC;           // first column of this group
+    const int ncol = min(NC, a.Dv - gc);    // may be <= 0
+    Core core;
     float* Sg = a.S + (((size_t)sd.slot * a.H + h) * a.Dv + (gc < a.Dv ? gc : 0)) * D;
     if (sd.pos0 > 0) core.load(Sg, l, ncol);
     else core.zero();
     __syncthreads();
 
-    const int d4 = a.Dl >> 2, v4 = min(cols, a.Dvl - c0) >> 2;
+    const int d4 = a.Dl >> 2, v4 = min(cpad, a.Dvl - c0) >> 2;  // (c0 is a multiple of 4)
+    const float* src0 = a.qkv + (size_t)sd.row0 * a.ld;
     auto stage = [&](int t0, int buf) {
         float* q = sm + buf * tile_f;
         const int nt = min(kDeltaTok, sd.n - t0);
         const int per = 2 * d4 + v4;
-        for (int i = tid; i < nt * per; i += blockDim.x) {
-            const int t = i / per, j = i - t * per;
-            const float* row = a.qkv + (size_t)(sd.row0 + t0 + t) * a.ld;
-            if (j < d4) cp_async16(q + t * D + j * 4, row + kvh * a.Dl + j * 4);
-            else if (j < 2 * d4) cp_async16(q + (kDeltaTok + t) * D + (j - d4) * 4, row + a.k_col + kvh * a.Dl + (j - d4) * 4);
-            else cp_async16(q + 2 * kDeltaTok * D + t * cols + (j - 2 * d4) * 4, row + a.v_col + h * a.Dvl + c0 + (j - 2 * d4) * 4);
+        for (int j = tid; j < per; j += blockDim.x) {  // a 16-byte column piece of all tokens
+            const float* src = src0 + (size_t)t0 * a.ld;
+            float* dst;
+            int step;
+            if (j < d4) { src += kvh * a.Dl + j * 4; dst = q + j * 4; step = D; }
+            else if (j < 2 * d4) { src += a.k_col + kvh * a.Dl + (j - d4) * 4; dst = q + kDeltaTok * D + (j - d4) * 4; step = D; }
+            else { src += a.v_col + h * a.Dvl + c0 + (j - 2 * d4) * 4; dst = q + 2 * kDeltaTok * D + (j - 2 * d4) * 4; step = cpad; }
+            for (int t = 0; t < nt; ++t) cp_async16(dst + t * step, src + (size_t)t * a.ld);
         }
+        if (tid < nt) cp_async16(q + kDeltaTok * (2 * D + cpad) + tid * 4, a.coef + (size_t)(sd.row0 + t0 + tid) * a.H + h);
         cp_async_commit();
-        if (tid < nt) {
-            const float* gr = a.gates + (size_t)(sd.row0 + t0 + tid) * a.ldg;
-            coef[(buf * kDeltaTok + tid) * 4] = expf(negA * softplusf_(gr[a.a_col + h] + dtb));
-            coef[(buf * kDeltaTok + tid) * 4 + 1] = sigmoidf_(gr[a.b_col + h]);
-        }
     };
     stage(0, 0);
+    const int oc = Core::ocol(lane);
+    const bool ow = Core::owns_o(lane);
+    float* orow = a.out + (size_t)sd.row0 * a.ldo + h * a.Dvl + gc + oc;
     for (int t0 = 0, it = 0; t0 < sd.n; t0 += kDeltaTok, ++it) {
         const int buf = it & 1, nt = min(kDeltaTok, sd.n - t0);
         if (t0 + kDeltaTok < sd.n) { stage(t0 + kDeltaTok, buf ^ 1); cp_async_wait<1>(); }
         else cp_async_wait<0>();
         __syncthreads();
-        float* q = sm + buf * tile_f;
-        float* k = q + kDeltaTok * D;
-        const float* v = k + kDeltaTok * D;
-        for (int t = warp; t < nt; t += nwarps) {
-            float sq = 0.f, sk = 0.f, dot = 0.f;
-            for (int d = lane; d < D; d += 32) {
-                const float qv = q[t * D + d], kv = k[t * D + d];
-                sq = fmaf(qv, qv, sq);
-                sk = fmaf(kv, kv, sk);
-                dot = fmaf(qv, kv, dot);
-            }
-            sq = warp_sum(sq); sk = warp_sum(sk); dot = warp_sum(dot);
-            const float rq = qscale / sqrtf(sq + 1e-6f), rk = 1.0f / sqrtf(sk + 1e-6f);
-            for (int d = lane; d < D; d += 32) { q[t * D + d] *= rq; k[t * D + d] *= rk; }
-            if (lane == 0) coef[(buf * kDeltaTok + t) * 4 + 2] = dot * rq * rk;
-        }
-        __syncthreads();
-        const int oc = DeltaCore<L>::ocol(lane);
-        const bool ow = DeltaCore<L>::owns_o(lane);
+        const float* q = sm + buf * tile_f;
+        const float* k = q + kDeltaTok * D;
+        const float* v = k + kDeltaTok * D + grp * NC;
+        const float* cf = q + kDeltaTok * (2 * D + cpad);
+        typename Core::Row qr = Core::row(q, l), kr = Core::row(k, l);
+#pragma unroll 2
         for (int t = 0; t < nt; ++t) {
-            const float4 cf = *reinterpret_cast<const float4*>(coef + (buf * kDeltaTok + t) * 4);
-            float o[DeltaCore<L>::kOut];
-            core.token(q + t * D, k + t * D, v + t * cols + grp * kDeltaCols, cf.x, cf.y, cf.z, lane, o);
+            const float4 co = *reinterpret_cast<const float4*>(cf + t * 4);
+            const int tn = min(t + 1, kDeltaTok - 1);
+            const typename Core::Row kn = Core::row(k + tn * D, l);
+            float o[Core::kOut];
+            core.token(kr, qr, q + tn * D, v + t * cpad, co.x, co.y, co.z, lane, o);
+            kr = kn;
             if (ow) {
-                float* orow = a.out + (size_t)(sd.row0 + t0 + t) * a.ldo + h * a.Dvl + gc;
 #pragma unroll
-                for (int j = 0; j < DeltaCore<L>::kOut; ++j)
-                    if (oc + j < ncol) orow[oc + j] = o[j];
+                for (int j = 0; j < Core::kOut; ++j)
+                    if (oc + j < ncol) orow[j] = o[j];
             }
+            orow += a.ldo;
         }
         __syncthreads();
     }
@@ -403,17 +503,18 @@ delta_scan_kernel(const DeltaArgs a) {
 
 // Decode: one CTA per (head, sequence) takes its token through convolution, unit norms, the rule, the
 // output norm and the gate.
-constexpr int kDeltaStepThreads = 256;
+constexpr int kDeltaStepThreads = 256, kDeltaStepCols = 4;
 template <int L>
 __global__ void __launch_bounds__(kDeltaStepThreads)
 delta_step_kernel(const DeltaArgs a) {
-    constexpr int D = 16 * L;
-    extern __shared__ __align__(16) float sm[];  // q [D], k [D], v and o [Dvl + 4 each]
+    constexpr int D = 16 * L, COLS = kDeltaStepThreads / L * kDeltaStepCols;
+    using Core = DeltaCore<L, kDeltaStepCols>;
+    extern __shared__ __align__(16) float sm[];  // q [D], k [D], v and o [vpad each]
     __shared__ float red[8];
     float* q = sm;
     float* k = q + D;
     float* v = k + D;
-    const int vpad = (a.Dvl + kDeltaStepThreads / L * kDeltaCols - 1) & ~3;
+    const int vpad = (a.Dvl + COLS - 1) & ~3;
     float* o = v + vpad;
     const int tid = threadIdx.x, lane = tid & 31;
     const int h = blockIdx.x, per = a.H / a.G, kvh = h / per;
@@ -423,6 +524,15 @@ delta_step_kernel(const DeltaArgs a) {
     griddep_launch_dependents();
     const SeqDesc sd = a.seqs[blockIdx.y];
     const float* row = a.qkv + (size_t)sd.row0 * a.ld;
+    const int grp = tid / L, l = tid & (L - 1);
+    // the state of the first columns is on its way while q, k and v are formed
+    Core core;
+    float* Sh = a.S + ((size_t)sd.slot * a.H + h) * a.Dv * D;
+    auto fetch = [&](int gc) {
+        if (sd.pos0 > 0) core.load(Sh + (size_t)(gc < a.Dv ? gc : 0) * D, l, min(kDeltaStepCols, a.Dv - gc));
+        else core.zero();
+    };
+    fetch(grp * kDeltaStepCols);
     __syncthreads();
     const int hrows = a.taps - 1;
     const float* hr = a.hist + ((size_t)sd.bank * a.max_slots + sd.slot) * hrows * a.np;
@@ -454,23 +564,21 @@ delta_step_kernel(const DeltaArgs a) {
     __syncthreads();
     for (int d = tid; d < D; d += kDeltaStepThreads) { q[d] *= rq; k[d] *= rk; }
     __syncthreads();
-    const int grp = tid / L, l = tid & (L - 1);
-    const int oc = DeltaCore<L>::ocol(lane);
-    const bool ow = DeltaCore<L>::owns_o(lane);
-    for (int c0 = 0; c0 < a.Dv; c0 += kDeltaStepThreads / L * kDeltaCols) {
-        const int gc = c0 + grp * kDeltaCols, ncol = min(kDeltaCols, a.Dv - gc);
-        DeltaCore<L> core;
-        float* Sg = a.S + (((size_t)sd.slot * a.H + h) * a.Dv + (gc < a.Dv ? gc : 0)) * D;
-        if (sd.pos0 > 0) core.load(Sg, l, ncol);
-        else core.zero();
-        float ov[DeltaCore<L>::kOut];
-        core.token(q, k, v + gc, g, beta, dot * rq * rk, lane, ov);
+    const int oc = Core::ocol(lane);
+    const bool ow = Core::owns_o(lane);
+    const typename Core::Row kr = Core::row(k, l);
+    typename Core::Row qr = Core::row(q, l);
+    for (int c0 = 0; c0 < a.Dv; c0 += COLS) {
+        const int gc = c0 + grp * kDeltaStepCols, ncol = min(kDeltaStepCols, a.Dv - gc);
+        if (c0 > 0) fetch(gc);
+        float ov[Core::kOut];
+        core.token(kr, qr, q, v + gc, g, beta, dot * rq * rk, lane, ov);
         if (ow) {
 #pragma unroll
-            for (int j = 0; j < DeltaCore<L>::kOut; ++j)
+            for (int j = 0; j < Core::kOut; ++j)
                 if (oc + j < ncol) o[gc + oc + j] = ov[j];
         }
-        core.store(Sg, l, ncol);
+        core.store(Sh + (size_t)(gc < a.Dv ? gc : 0) * D, l, ncol);
     }
     __syncthreads();
     float s = 0.f;
@@ -567,50 +675,55 @@ int launch_scan_types(b200_ctx* ctx, const SelectiveScanArgs& a, int E, bool x_f
 }
 
 template <int L>
-int launch_delta_one(b200_ctx* ctx, const DeltaArgs& a, int E, bool step) {
-    constexpr int D = 16 * L;
-    cudaError_t le;
-    if (step) {
-        const int vpad = (a.Dvl + kDeltaStepThreads / L * kDeltaCols - 1) & ~3;
-        const size_t smem = (size_t)(2 * D + 2 * vpad) * 4;
-        if (smem > 48 * 1024) return B200_ERR_LIMIT;
-        le = launch_pdl(ctx, delta_step_kernel<L>, dim3(a.H, E), dim3(kDeltaStepThreads), smem, a);
-    } else {
-        int groups = (a.Dv + kDeltaCols - 1) / kDeltaCols;
-        int threads = (groups * L + 31) & ~31;
-        if (threads > kDeltaThreads) threads = kDeltaThreads;
-        // a short grid: narrower column blocks put more SMs to work
-        while (threads > 32 && (long)a.H * E * ((groups * L + threads - 1) / threads) < 2L * ctx->num_sms) threads >>= 1;
-        threads = (threads + 31) & ~31;
-        const int cols = threads / L * kDeltaCols;
-        const size_t smem = (size_t)(2 * kDeltaTok * (2 * D + cols) + 2 * kDeltaTok * 4) * 4;
-        static bool attr_set[64] = {};
-        if (!attr_set[ctx->device & 63]) {
-            B200_CUDA(ctx, cudaFuncSetAttribute(delta_scan_kernel<L>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-            attr_set[ctx->device & 63] = true;
-        }
-        if (smem > 200 * 1024) return B200_ERR_LIMIT;
-        le = launch_pdl(ctx, delta_scan_kernel<L>, dim3(a.H, (a.Dv + cols - 1) / cols, E), dim3(threads), smem, a);
-    }
+int launch_delta_step_one(b200_ctx* ctx, const DeltaArgs& a, int E) {
+    const int vpad = (a.Dvl + kDeltaStepThreads / L * kDeltaStepCols - 1) & ~3;
+    const size_t smem = (size_t)(32 * L + 2 * vpad) * 4;
+    if (smem > 48 * 1024) return B200_ERR_LIMIT;
+    cudaError_t le = launch_pdl(ctx, delta_step_kernel<L>, dim3(a.H, E), dim3(kDeltaStepThreads), smem, a);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
 }
 
-int launch_delta(b200_ctx* ctx, const DeltaArgs& a, int E, bool step) {
-    switch (delta_state_pad(a.D)) {
-        case 32: return launch_delta_one<2>(ctx, a, E, step);
-        case 64: return launch_delta_one<4>(ctx, a, E, step);
-        case 128: return launch_delta_one<8>(ctx, a, E, step);
-        case 256: return launch_delta_one<16>(ctx, a, E, step);
-        default: return B200_ERR_LIMIT;
+template <int L, int NC>
+int launch_delta_scan_one(b200_ctx* ctx, const DeltaArgs& a, int E) {
+    constexpr int D = 16 * L;
+    const int groups = (a.Dv + NC - 1) / NC;
+    // two warps per CTA (a block of columns starts at a multiple of four columns)
+    int threads = (groups * L + 31) & ~31;
+    if (threads > 64) threads = 64;
+    while (threads / L * NC % 4) threads += 32;
+    const int cols = threads / L * NC, cpad = (cols + 3) & ~3;
+    const size_t smem = (size_t)(2 * kDeltaTok * (2 * D + cpad + 4) + D) * 4;
+    if (smem > 200 * 1024) return B200_ERR_LIMIT;
+    static bool attr_set[64] = {};
+    if (!attr_set[ctx->device & 63]) {
+        B200_CUDA(ctx, cudaFuncSetAttribute(delta_scan_kernel<L, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        attr_set[ctx->device & 63] = true;
     }
+    cudaError_t le = launch_pdl(ctx, delta_scan_kernel<L, NC>, dim3(a.H, (a.Dv + cols - 1) / cols, E), dim3(threads), smem, a);
+    ctx->launches++;
+    B200_CUDA(ctx, le);
+    return B200_OK;
+}
+
+// Columns per group: four are the cheapest per column, but with few sequences and heads the warps would be too
+// few to hide the chain from token to token.
+template <int L>
+int launch_delta_scan_l(b200_ctx* ctx, const DeltaArgs& a, int E) {
+    static const int forced = [] { const char* e = getenv("B200_DELTA_COLS"); return e ? atoi(e) : 0; }();  // tuning hook: 1, 2 or 4
+    const long columns = (long)a.H * E * a.Dv;
+    auto warps = [&](int nc) { return columns / nc * L / 32; };
+    const int nc = forced ? forced : (warps(4) >= 6L * ctx->num_sms ? 4 : (warps(2) >= 4L * ctx->num_sms ? 2 : 1));
+    if (nc == 4) return launch_delta_scan_one<L, 4>(ctx, a, E);
+    if (nc == 2) return launch_delta_scan_one<L, 2>(ctx, a, E);
+    return launch_delta_scan_one<L, 1>(ctx, a, E);
 }
 
 }  // namespace
 
 int launch_short_conv(b200_ctx* ctx, const ShortConvArgs& a, int E, int max_n, bool f32) {
-    const dim3 grid((a.np / 4 + 127) / 128, (max_n + kConvTok - 1) / kConvTok, E), block(128);
+    const dim3 grid(((a.np - a.ch0) / 4 + 127) / 128, (max_n + kConvTok - 1) / kConvTok, E), block(128);
     cudaError_t le;
     switch (a.taps) {
         case 2: le = f32 ? launch_pdl(ctx, short_conv_kernel<2, true>, grid, block, 0, a) : launch_pdl(ctx, short_conv_kernel<2, false>, grid, block, 0, a); break;
@@ -649,8 +762,39 @@ int delta_state_pad(int D) {
     return 0;
 }
 
-int launch_delta_scan(b200_ctx* ctx, const DeltaArgs& a, int E) { return launch_delta(ctx, a, E, false); }
-int launch_delta_step(b200_ctx* ctx, const DeltaArgs& a, int E) { return launch_delta(ctx, a, E, true); }
+int launch_delta_prep(b200_ctx* ctx, const DeltaArgs& a, int E, int max_n) {
+    const dim3 grid(a.G, (max_n + 4 * kDeltaTok - 1) / (4 * kDeltaTok), E), block(128);
+    cudaError_t le;
+    switch (a.taps) {
+        case 2: le = launch_pdl(ctx, delta_prep_kernel<2>, grid, block, 0, a); break;
+        case 3: le = launch_pdl(ctx, delta_prep_kernel<3>, grid, block, 0, a); break;
+        case 4: le = launch_pdl(ctx, delta_prep_kernel<4>, grid, block, 0, a); break;
+        default: le = launch_pdl(ctx, delta_prep_kernel<0>, grid, block, 0, a); break;
+    }
+    ctx->launches++;
+    B200_CUDA(ctx, le);
+    return B200_OK;
+}
+
+int launch_delta_scan(b200_ctx* ctx, const DeltaArgs& a, int E) {
+    switch (delta_state_pad(a.D)) {
+        case 32: return launch_delta_scan_l<2>(ctx, a, E);
+        case 64: return launch_delta_scan_l<4>(ctx, a, E);
+        case 128: return launch_delta_scan_l<8>(ctx, a, E);
+        case 256: return launch_delta_scan_l<16>(ctx, a, E);
+        default: return B200_ERR_LIMIT;
+    }
+}
+
+int launch_delta_step(b200_ctx* ctx, const DeltaArgs& a, int E) {
+    switch (delta_state_pad(a.D)) {
+        case 32: return launch_delta_step_one<2>(ctx, a, E);
+        case 64: return launch_delta_step_one<4>(ctx, a, E);
+        case 128: return launch_delta_step_one<8>(ctx, a, E);
+        case 256: return launch_delta_step_one<16>(ctx, a, E);
+        default: return B200_ERR_LIMIT;
+    }
+}
 
 int launch_min_gru(b200_ctx* ctx, const MinGruArgs& a, int E, bool f32) {
     const dim3 grid((a.width + 31) / 32, E);
