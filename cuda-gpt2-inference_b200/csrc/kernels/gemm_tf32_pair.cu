@@ -68,9 +68,14 @@ struct PairCfg {
     static constexpr int B_BYTES = (kMaxW / 2) * 128;            // one plane of this CTA's half of a full-width weight tile
     static constexpr int STAGE_BYTES = PARTS * (A_BYTES + B_BYTES);
     static constexpr int BAR_BYTES = 512;
-    static constexpr int STAGES_RAW = (kGemmMaxSmem - 1024 - BAR_BYTES - kGemmEpiBytes) / STAGE_BYTES;
+    // Staging buffers of an epilogue warp.  A store queues behind the operand loads that are already in the TMA
+    // unit; with one product per K block a tile's loads take no longer than one such wait, so a single buffer
+    // would pace the kernel (bf16: two buffers and a stage less instead).
+    static constexpr int EPI_BUFS = (MODE == PAIR_BF16) ? 2 : 1;
+    static constexpr int EPI_BYTES = kEpiWarps * EPI_BUFS * 4096;
+    static constexpr int STAGES_RAW = (kGemmMaxSmem - 1024 - BAR_BYTES - EPI_BYTES) / STAGE_BYTES;
     static constexpr int STAGES = STAGES_RAW > 8 ? 8 : STAGES_RAW;
-    static constexpr int SMEM = 1024 + STAGES * STAGE_BYTES + kGemmEpiBytes + BAR_BYTES;
+    static constexpr int SMEM = 1024 + STAGES * STAGE_BYTES + EPI_BYTES + BAR_BYTES;
     static constexpr int TMEM_COLS = 512;
     // elements of K per 128-byte block
     static constexpr int BKE = (MODE == PAIR_TF32) ? kGemmBK : (MODE == PAIR_FP8 ? kGemmBKQ : kGemmBKH);
@@ -144,7 +149,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
     uint8_t* smem_a = smem;                                   // [STAGES][PARTS][A_BYTES]
     uint8_t* smem_b = smem_a + STAGES * PARTS * Cfg::A_BYTES;  // [STAGES][PARTS][B_BYTES]
     uint8_t* smem_epi = smem + STAGES * Cfg::STAGE_BYTES;
-    uint64_t* bars = reinterpret_cast<uint64_t*>(smem_epi + kGemmEpiBytes);
+    uint64_t* bars = reinterpret_cast<uint64_t*>(smem_epi + Cfg::EPI_BYTES);
     uint64_t* full_bar = bars;                     // [STAGES] used in the even CTA
     uint64_t* empty_bar = bars + STAGES;           // [STAGES] each CTA
     uint64_t* tmem_full_bar = bars + 2 * STAGES;   // [2] each CTA
@@ -331,11 +336,11 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
             // (measured per launch: 12-14 thousand cycles with one buffer for the accumulating and the
             // two-plane epilogues).
             const bool last_tile = walk.cur >= walk.total;
-            uint8_t* staging = last_tile ? smem + ew * 4 * 4096 : smem_epi + ew * 4096;
+            uint8_t* staging = last_tile ? smem + ew * 4 * 4096 : smem_epi + ew * Cfg::EPI_BUFS * 4096;
             if (c_begin < c_end || args.lse_part != nullptr)  // (an empty share still owes its log-sum-exp slot)
                 gemm_drain_accumulator(args, bias, &tmap_out, tmem_base + acc * kMaxW, q, lane,
                                        m_blk * 2 * BM + (int)rank * BM + q * 32, col0,
-                                       staging, bias_first, c_begin, c_end, last_tile ? 4 : 1, 2 * (col0 / kMaxW) + (ew < 4 ? 0 : 1));
+                                       staging, bias_first, c_begin, c_end, last_tile ? 4 : Cfg::EPI_BUFS, 2 * (col0 / kMaxW) + (ew < 4 ? 0 : 1));
             tc_fence_before_sync();
             __syncwarp();
             if (lane == 0) {

@@ -329,8 +329,9 @@ struct DeltaCore {
 };
 
 // What the scan wants per token: convolved and activated q and k as unit vectors (q also times D^-1/2) and, per
-// head, {decay, beta, k.q}.  One warp per (sequence, key/value head, run of 16 tokens).
-template <int TAPS>
+// head, {decay, beta, k.q}.  One warp per (sequence, key/value head, run of 16 tokens), a lane holding channels
+// lane, lane + 32, ... (V of them) of q and k; two tokens at a time.
+template <int TAPS, int V>
 __global__ void __launch_bounds__(128)
 delta_prep_kernel(const DeltaArgs a) {
     constexpr int W = TAPS > 0 ? TAPS : 1;
@@ -346,7 +347,7 @@ delta_prep_kernel(const DeltaArgs a) {
     float* hw = a.hist + ((size_t)(sd.bank ^ 1) * a.max_slots + sd.slot) * hrows * a.np;
     const float* xin = a.raw + (size_t)sd.row0 * a.ld_raw;
     float* qkv = const_cast<float*>(a.qkv) + (size_t)sd.row0 * a.ld;
-    const int qc = g * a.Dl, kc = a.k_col + g * a.Dl;
+    const int base[2] = {g * a.Dl, a.k_col + g * a.Dl};  // first channel of q and of k
     auto input = [&](int i, int ch) {
         if (i >= 0) return xin[(size_t)i * a.ld_raw + ch];
         if (sd.pos0 + i < 0) return 0.f;
@@ -354,71 +355,93 @@ delta_prep_kernel(const DeltaArgs a) {
     };
     const float qscale = rsqrtf((float)a.D);
     const int per = a.H / a.G;
-    float sq[kDeltaTok], sk[kDeltaTok], qk[kDeltaTok];  // per token: squares and product of this lane's channels
+    float w[2][V][W], win[2][V][W];  // weights and the window of earlier inputs
+    if (TAPS > 0) {
 #pragma unroll
-    for (int t = 0; t < kDeltaTok; ++t) sq[t] = sk[t] = qk[t] = 0.f;
-    // first pass, 32 channels of q and k at a time: convolution and silu, to memory as they are
-    for (int d = lane; d < a.Dl; d += 32) {
-        float wq[W], wk[W], xq[W], xk[W];
-        if (TAPS > 0) {
+        for (int x = 0; x < 2; ++x)
 #pragma unroll
-            for (int j = 0; j < W; ++j) { wq[j] = __ldg(a.conv_w + (size_t)j * a.np + qc + d); wk[j] = __ldg(a.conv_w + (size_t)j * a.np + kc + d); }
+            for (int i = 0; i < V; ++i) {
+                const int d = lane + i * 32;
 #pragma unroll
-            for (int j = 0; j + 1 < W; ++j) { xq[j] = input(t0 - (W - 1) + j, qc + d); xk[j] = input(t0 - (W - 1) + j, kc + d); }
-        }
-        float iq[kDeltaTok], ik[kDeltaTok];
-#pragma unroll
-        for (int t = 0; t < kDeltaTok; ++t) {
-            iq[t] = ik[t] = 0.f;
-            if (TAPS > 0 && t0 + t < t1) { iq[t] = input(t0 + t, qc + d); ik[t] = input(t0 + t, kc + d); }
-        }
-#pragma unroll
-        for (int t = 0; t < kDeltaTok; ++t) {
-            float q = 0.f, k = 0.f;
-            if (TAPS > 0) {
-                xq[W - 1] = iq[t];
-                xk[W - 1] = ik[t];
-#pragma unroll
-                for (int j = 0; j < W; ++j) { q = fmaf(xq[j], wq[j], q); k = fmaf(xk[j], wk[j], k); }
-#pragma unroll
-                for (int j = 0; j + 1 < W; ++j) { xq[j] = xq[j + 1]; xk[j] = xk[j + 1]; }
-            } else if (t0 + t < t1) {
-                for (int j = 0; j < taps; ++j) {
-                    q = fmaf(input(t0 + t - hrows + j, qc + d), __ldg(a.conv_w + (size_t)j * a.np + qc + d), q);
-                    k = fmaf(input(t0 + t - hrows + j, kc + d), __ldg(a.conv_w + (size_t)j * a.np + kc + d), k);
+                for (int j = 0; j < W; ++j) {
+                    w[x][i][j] = d < a.Dl ? __ldg(a.conv_w + (size_t)j * a.np + base[x] + d) : 0.f;
+                    win[x][i][j] = (d < a.Dl && j + 1 < W) ? input(t0 - (W - 1) + j, base[x] + d) : 0.f;
                 }
             }
-            q = silu(q);
-            k = silu(k);
-            if (t0 + t < t1) {
-                qkv[(size_t)(t0 + t) * a.ld + qc + d] = q;
-                qkv[(size_t)(t0 + t) * a.ld + kc + d] = k;
-                sq[t] = fmaf(q, q, sq[t]);
-                sk[t] = fmaf(k, k, sk[t]);
-                qk[t] = fmaf(q, k, qk[t]);
-            }
-        }
-        if (t1 == sd.n)
-            for (int e = 0; e < hrows; ++e) {
-                hw[(size_t)e * a.np + qc + d] = input(sd.n - hrows + e, qc + d);
-                hw[(size_t)e * a.np + kc + d] = input(sd.n - hrows + e, kc + d);
-            }
     }
-    // sums over the lanes, and the scales applied to what this lane has written
+    for (int tb = t0; tb < t1; tb += 2) {
+        float in[2][2][V];  // [token][q, k]
 #pragma unroll
-    for (int t = 0; t < kDeltaTok; ++t) {
-        if (t0 + t >= t1) break;
-        const float rq = qscale / sqrtf(warp_sum(sq[t]) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(sk[t]) + 1e-6f);
-        const float kq = warp_sum(qk[t]) * rq * rk;
-        float* row = qkv + (size_t)(t0 + t) * a.ld;
-        for (int d = lane; d < a.Dl; d += 32) { row[qc + d] *= rq; row[kc + d] *= rk; }
-        const float* gr = a.gates + (size_t)(sd.row0 + t0 + t) * a.ldg;
-        for (int j = lane; j < per; j += 32) {
-            const int h = g * per + j;
-            const float decay = expf(__ldg(a.negA + h) * softplusf_(gr[a.a_col + h] + __ldg(a.dt_bias + h)));
-            a.coef[(size_t)(sd.row0 + t0 + t) * a.H + h] = make_float4(decay, sigmoidf_(gr[a.b_col + h]), kq, 0.f);
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int x = 0; x < 2; ++x)
+#pragma unroll
+                for (int i = 0; i < V; ++i) {
+                    const int d = lane + i * 32;
+                    in[u][x][i] = 0.f;
+                    if (d < a.Dl && tb + u < t1) {
+                        if (TAPS > 0) in[u][x][i] = input(tb + u, base[x] + d);
+                        else
+                            for (int j = 0; j < taps; ++j)
+                                in[u][x][i] = fmaf(input(tb + u - hrows + j, base[x] + d), __ldg(a.conv_w + (size_t)j * a.np + base[x] + d), in[u][x][i]);
+                    }
+                }
+        float sum[2][3];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            sum[u][0] = sum[u][1] = sum[u][2] = 0.f;
+#pragma unroll
+            for (int i = 0; i < V; ++i) {
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    float y = in[u][x][i];
+                    if (TAPS > 0) {
+                        win[x][i][W - 1] = y;
+                        y = 0.f;
+#pragma unroll
+                        for (int j = 0; j < W; ++j) y = fmaf(win[x][i][j], w[x][i][j], y);
+#pragma unroll
+                        for (int j = 0; j + 1 < W; ++j) win[x][i][j] = win[x][i][j + 1];
+                    }
+                    in[u][x][i] = silu(y);
+                }
+                sum[u][0] = fmaf(in[u][0][i], in[u][0][i], sum[u][0]);
+                sum[u][1] = fmaf(in[u][1][i], in[u][1][i], sum[u][1]);
+                sum[u][2] = fmaf(in[u][0][i], in[u][1][i], sum[u][2]);
+            }
+        }
+#pragma unroll
+        for (int s = 16; s >= 1; s >>= 1)
+#pragma unroll
+            for (int u = 0; u < 2; ++u)
+#pragma unroll
+                for (int x = 0; x < 3; ++x) sum[u][x] += __shfl_xor_sync(0xffffffffu, sum[u][x], s);
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int t = tb + u;
+            if (t >= t1) break;
+            const float r[2] = {qscale / sqrtf(sum[u][0] + 1e-6f), 1.0f / sqrtf(sum[u][1] + 1e-6f)};
+            float* row = qkv + (size_t)t * a.ld;
+#pragma unroll
+            for (int x = 0; x < 2; ++x)
+#pragma unroll
+                for (int i = 0; i < V; ++i)
+                    if (lane + i * 32 < a.Dl) row[base[x] + lane + i * 32] = in[u][x][i] * r[x];
+            const float kq = sum[u][2] * r[0] * r[1];
+            const float* gr = a.gates + (size_t)(sd.row0 + t) * a.ldg;
+            for (int j = lane; j < per; j += 32) {
+                const int h = g * per + j;
+                const float decay = expf(__ldg(a.negA + h) * softplusf_(gr[a.a_col + h] + __ldg(a.dt_bias + h)));
+                a.coef[(size_t)(sd.row0 + t) * a.H + h] = make_float4(decay, sigmoidf_(gr[a.b_col + h]), kq, 0.f);
+            }
         }
     }
+    if (t1 == sd.n)  // the last inputs are the history of the next step
+        for (int e = 0; e < hrows; ++e)
+            for (int d = lane; d < a.Dl; d += 32) {
+                hw[(size_t)e * a.np + base[0] + d] = input(sd.n - hrows + e, base[0] + d);
+                hw[(size_t)e * a.np + base[1] + d] = input(sd.n - hrows + e, base[1] + d);
+            }
 }
 
 // Prefill: a CTA walks one (sequence, head) for blockDim.x / L * NC columns of Dv, in tiles of 16 tokens staged two
@@ -589,12 +612,13 @@ delta_step_kernel(const DeltaArgs a) {
 }
 
 // ------------------------------------------------------------------ minGRU
-// A CTA walks one sequence for 32 channels, 128 tokens at a time: each of 16 warps takes 8 consecutive
+// A CTA walks one sequence for 32 channels, 64 tokens at a time: each of 8 warps takes 8 consecutive
 // tokens (lane = channel), first as the affine map S -> A S + b that they amount to, and once the maps
-// of the warps before it are known - through shared memory - as the states themselves.
-constexpr int kGruWarps = 16, kGruTok = 8;
+// of the warps before it are known - through shared memory - as the states themselves.  The inputs of the next
+// 64 tokens are requested before these are worked on.
+constexpr int kGruWarps = 8, kGruTok = 8;
 template <bool F32>
-__global__ void __launch_bounds__(kGruWarps * 32)
+__global__ void __launch_bounds__(kGruWarps * 32, 3)
 min_gru_kernel(const MinGruArgs a) {
     __shared__ float mapA[2][kGruWarps][32], mapB[2][kGruWarps][32];
     griddep_wait();
@@ -606,21 +630,28 @@ min_gru_kernel(const MinGruArgs a) {
     float* Sg = a.S + (size_t)sd.slot * a.width + c;
     float S = (live && sd.pos0 > 0) ? *Sg : 0.f;  // state before the block of tokens (the same in every warp)
     const float* base = a.zx + (size_t)sd.row0 * a.ld + c;
+    float nz[kGruTok], nu[kGruTok], ng[kGruTok];
+    auto request = [&](int tw) {
+#pragma unroll
+        for (int i = 0; i < kGruTok; ++i) {
+            nz[i] = nu[i] = ng[i] = 0.f;
+            if (live && tw + i < sd.n) {
+                const float* r = base + (size_t)(tw + i) * a.ld;
+                nz[i] = r[a.z_col];
+                nu[i] = r[a.x_col];
+                ng[i] = r[a.g_col];
+            }
+        }
+    };
+    request(warp * kGruTok);
     for (int t0 = 0, it = 0; t0 < sd.n; t0 += kGruWarps * kGruTok, ++it) {
         float (&mA)[kGruWarps][32] = mapA[it & 1];
         float (&mB)[kGruWarps][32] = mapB[it & 1];
         const int tw = t0 + warp * kGruTok;
         float zi[kGruTok], ui[kGruTok], gi[kGruTok];
 #pragma unroll
-        for (int i = 0; i < kGruTok; ++i) {
-            zi[i] = ui[i] = gi[i] = 0.f;
-            if (live && tw + i < sd.n) {
-                const float* r = base + (size_t)(tw + i) * a.ld;
-                zi[i] = r[a.z_col];
-                ui[i] = r[a.x_col];
-                gi[i] = r[a.g_col];
-            }
-        }
+        for (int i = 0; i < kGruTok; ++i) { zi[i] = nz[i]; ui[i] = nu[i]; gi[i] = ng[i]; }
+        request(tw + kGruWarps * kGruTok);
         float A = 1.f, b = 0.f;
 #pragma unroll
         for (int i = 0; i < kGruTok; ++i) {
@@ -762,15 +793,25 @@ int delta_state_pad(int D) {
     return 0;
 }
 
-int launch_delta_prep(b200_ctx* ctx, const DeltaArgs& a, int E, int max_n) {
-    const dim3 grid(a.G, (max_n + 4 * kDeltaTok - 1) / (4 * kDeltaTok), E), block(128);
-    cudaError_t le;
+namespace {
+template <int V>
+cudaError_t launch_delta_prep_v(b200_ctx* ctx, const DeltaArgs& a, dim3 grid) {
     switch (a.taps) {
-        case 2: le = launch_pdl(ctx, delta_prep_kernel<2>, grid, block, 0, a); break;
-        case 3: le = launch_pdl(ctx, delta_prep_kernel<3>, grid, block, 0, a); break;
-        case 4: le = launch_pdl(ctx, delta_prep_kernel<4>, grid, block, 0, a); break;
-        default: le = launch_pdl(ctx, delta_prep_kernel<0>, grid, block, 0, a); break;
+        case 2: return launch_pdl(ctx, delta_prep_kernel<2, V>, grid, dim3(128), 0, a);
+        case 3: return launch_pdl(ctx, delta_prep_kernel<3, V>, grid, dim3(128), 0, a);
+        case 4: return launch_pdl(ctx, delta_prep_kernel<4, V>, grid, dim3(128), 0, a);
+        default: return launch_pdl(ctx, delta_prep_kernel<0, V>, grid, dim3(128), 0, a);
     }
+}
+}  // namespace
+
+int launch_delta_prep(b200_ctx* ctx, const DeltaArgs& a, int E, int max_n) {
+    const dim3 grid(a.G, (max_n + 4 * kDeltaTok - 1) / (4 * kDeltaTok), E);
+    cudaError_t le;
+    if (a.Dl <= 32) le = launch_delta_prep_v<1>(ctx, a, grid);
+    else if (a.Dl <= 64) le = launch_delta_prep_v<2>(ctx, a, grid);
+    else if (a.Dl <= 128) le = launch_delta_prep_v<4>(ctx, a, grid);
+    else le = launch_delta_prep_v<8>(ctx, a, grid);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
