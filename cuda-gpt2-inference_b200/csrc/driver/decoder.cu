@@ -198,11 +198,9 @@ struct b200_decoder {
     void *h = nullptr, *conv = nullptr, *mix = nullptr, *q = nullptr, *low = nullptr;
     float* logits = nullptr;
     int logits_rows = 0;
-    // ... and of the decode path (fp32, 16 rows)
-    float *dx[2] = {nullptr, nullptr}, *dproj = nullptr, *dmix = nullptr, *dy = nullptr, *dconv = nullptr, *daux = nullptr, *dlogits = nullptr;
-    void* dh = nullptr;
-    float* partial = nullptr;
-    unsigned int* counters = nullptr;
+    // ... and of the decode path (16 rows: fp32, or split rows of the same size)
+    float *dx = nullptr, *dproj = nullptr, *dy = nullptr, *daux = nullptr, *dlogits = nullptr;
+    void *dh = nullptr, *dmix = nullptr, *dconv = nullptr;
     // step descriptors: a ring of pinned buffers, one device buffer per path
     static constexpr int kRing = 8;
     int* pinned[kRing] = {};
@@ -463,7 +461,7 @@ void load_all(b200_decoder* m) {
 
 // activations, sized from the loaded layers
 void allocate(b200_decoder* m) {
-    size_t proj = 0, mix = 0, conv = 0, aux = 0, wide = 0, q = 0, low = 0, partial = 0, counters = 16;
+    size_t proj = 0, mix = 0, conv = 0, aux = 0, wide = 0, q = 0, low = 0;
     auto up = [](size_t& a, size_t b) { if (b > a) a = b; };
     for (const Layer& L : m->layers) {
         up(proj, L.in.N);
@@ -473,8 +471,6 @@ void allocate(b200_decoder* m) {
         else if (L.spec->kind == MIX_DELTA) { up(conv, 2 * L.np); up(wide, L.spec->heads * L.Dvl); up(aux, 4 * L.spec->heads); }  // (fp32 in either arithmetic)
         else {
             up(q, (size_t)L.att.H * L.att.Dp);
-            up(partial, attention_decode_partial_floats(L.att, 16));
-            up(counters, (size_t)16 * L.att.H);
         }
     }
     const size_t M = m->max_rows, e = elem(m);
@@ -489,16 +485,14 @@ void allocate(b200_decoder* m) {
     m->low = device_zeros(m, M * low * e);
     m->q = device_zeros(m, M * q * e);
     if (!m->f32) {
-        for (float*& p : m->dx) p = static_cast<float*>(device_zeros(m, (size_t)16 * m->Cp * 4));
+        m->dx = static_cast<float*>(device_zeros(m, (size_t)16 * m->Cp * 4));
         m->dy = static_cast<float*>(device_zeros(m, (size_t)16 * m->Cp * 4));
         m->dh = device_zeros(m, (size_t)16 * m->Cp * 4);
         m->dproj = static_cast<float*>(device_zeros(m, (size_t)16 * proj * 4));
-        m->dmix = static_cast<float*>(device_zeros(m, (size_t)16 * mix * 4));
-        m->dconv = static_cast<float*>(device_zeros(m, (size_t)16 * conv * 4));
+        m->dmix = device_zeros(m, (size_t)16 * mix * 4);
+        m->dconv = device_zeros(m, (size_t)16 * conv * 4);
         m->daux = static_cast<float*>(device_zeros(m, (size_t)16 * aux * 4));
         m->dlogits = static_cast<float*>(device_zeros(m, (size_t)16 * m->Vp * 4));
-        m->partial = static_cast<float*>(device_zeros(m, partial * 4));
-        m->counters = static_cast<unsigned int*>(device_zeros(m, counters * 4));
     }
     // descriptors: sequences, tokens, the sequence of every row, wanted rows, query-tile pairs
     m->desc_ints = (size_t)m->max_slots * 8 + 3 * M + 2 * (M / 256 + m->max_slots + 1) + 64;
@@ -622,11 +616,10 @@ int mixer_delta(b200_decoder* m, const Layer& L, const StepView& v) {
     return B200_OK;
 }
 
-MinGruArgs gru_args(const b200_decoder* m, const Layer& L, const SeqDesc* seqs, const float* proj, void* out, size_t out_elem) {
+MinGruArgs gru_args(const Layer& L, const SeqDesc* seqs, const float* proj, void* out) {
     MinGruArgs g{};
     g.zx = proj; g.ld = L.in.N; g.z_col = L.z_col; g.x_col = L.x_col; g.g_col = L.g_col; g.S = L.S;
-    g.out = static_cast<char*>(out) + (size_t)L.att_p * out_elem; g.ldo = L.o.K; g.seqs = seqs; g.width = L.spec->gru_width; g.out_scale = L.spec->right_scale;
-    (void)m;
+    g.out = out; g.ldo = L.o.K; g.seqs = seqs; g.width = L.spec->gru_width; g.out_scale = L.spec->right_scale;
     return g;
 }
 
@@ -638,7 +631,7 @@ int mixer_parallel(b200_decoder* m, const Layer& L, const StepView& v) {
         OP("attention", launch_attention_cached_mma(ctx, L.att, m->q, m->mix, L.o.K, v.seqs, v.pairs, v.num_pairs, v.M, m->max_slots));
     else
         OP("attention", launch_attention_cached_simt(ctx, L.att, m->q, m->mix, L.o.K, v.seqs, v.E, v.max_n, m->f32));
-    OP("min gru", launch_min_gru(ctx, gru_args(m, L, v.seqs, m->proj, m->mix, elem(m)), v.E, m->f32));
+    OP("min gru", launch_min_gru(ctx, gru_args(L, v.seqs, m->proj, static_cast<char*>(m->mix) + L.att_p * elem(m)), v.E, m->f32));
     return B200_OK;
 }
 
@@ -650,7 +643,7 @@ int enqueue_general(b200_decoder* m, const StepView& v) {
     n.x_out = m->x; n.h = m->h; n.M = v.M;
     n.tok = v.tokens; n.embed = m->embed; n.embed_scale = m->spec.embed_scale;
     n.w = m->layers[0].norm1;
-    OP("embed norm", launch_residual_rms(ctx, n, m->f32));
+    OP("embed norm", launch_residual_rms(ctx, n, m->f32 ? H_F32 : H_BF16));
     n.tok = nullptr;
     n.x = m->x;
     n.y = m->y;
@@ -664,14 +657,14 @@ int enqueue_general(b200_decoder* m, const StepView& v) {
         n.wb = L.norm1b;
         if (L.spec->ff > 0) {
             n.w = L.norm2;
-            OP("residual norms", launch_residual_rms(ctx, n, m->f32));
+            OP("residual norms", launch_residual_rms(ctx, n, m->f32 ? H_F32 : H_BF16));
             OP("gemm mlp up", product(m, m->mix, m->h, L.mlp.up, v.M, m->spec.design->mlp_act, true));
             OP("gemm mlp down", product(m, m->y, m->mix, L.mlp.down, v.M));
             n.wb = L.norm2b;
         }
         if (!last) {
             n.w = m->layers[i + 1].norm1;
-            OP("residual norms", launch_residual_rms(ctx, n, m->f32));
+            OP("residual norms", launch_residual_rms(ctx, n, m->f32 ? H_F32 : H_BF16));
         }
     }
     if (v.n_want == 0) return B200_OK;
@@ -679,74 +672,50 @@ int enqueue_general(b200_decoder* m, const StepView& v) {
     n.rows = v.want;
     n.M = v.n_want;
     n.x_out = nullptr;
-    OP("final norm", launch_residual_rms(ctx, n, m->f32));
+    OP("final norm", launch_residual_rms(ctx, n, m->f32 ? H_F32 : H_BF16));
     OP("gemm head", product(m, m->logits, m->h, m->head, v.n_want));
     return B200_OK;
 }
 
 // ------------------------------------------------------------------ decode path
 // One token for each of B <= 16 sequences: descriptors and tokens come from dseqs / dtokens, the logits go to
-// dlogits.  Every norm runs in the prologue of the product that follows it; the residual stream alternates
-// between two buffers because the product's other CTAs still read the old one.
+// dlogits.  The inputs of the products are split rows (decoder_math.cuh), written so by whatever produces them; the
+// short convolutions run in the epilogue of the projection in front of them.
 int enqueue_decode(b200_decoder* m, int B) {
     b200_ctx* ctx = m->ctx;
-    float *xa = m->dx[0], *xb = m->dx[1];
-    const float *pending = nullptr, *pending_w = nullptr;  // branch output and the norm behind it, not yet in the residual
-    bool first = true;
-    const bool fused = decode_gemm_fits(m->Cp, B);
-    auto residual = [&](float* out, int ldo, const Matrix& w, const float* norm, int act) {
-        DecodeGemmArgs a{};
-        a.out = out; a.ldo = ldo; a.W = static_cast<const uint16_t*>(w.w); a.bias = w.bias; a.B = B; a.N = w.N; a.K = w.K; a.act = act;
-        a.status = ctx->d_status;
-        int st;
-        if (fused) {
-            a.x = xa; a.y = pending; a.wb = pending_w; a.w = norm; a.x_out = xb; a.C = m->C; a.eps = m->spec.eps; a.vocab = m->spec.vocab;
-            if (first) { a.tok = m->dtokens; a.embed = static_cast<const uint16_t*>(m->embed); a.embed_scale = m->spec.embed_scale; }
-            st = launch_decode_gemm(ctx, a, DPRO_RESIDUAL);
-        } else {
-            // rows too long for the prologue: a kernel of its own, with fp32 rows between them
-            ResidualNormArgs n{};
-            n.C = m->C; n.Cp = m->Cp; n.eps = m->spec.eps; n.vocab = m->spec.vocab; n.M = B;
-            n.x = xa; n.y = pending; n.wb = pending_w; n.w = norm; n.x_out = xb; n.h = m->dh;
-            st = B200_OK;
-            if (first) {  // the embedding's rows are bf16: into the residual first
-                ResidualNormArgs e = n;
-                e.x = nullptr; e.y = nullptr; e.w = nullptr; e.tok = m->dtokens; e.embed = m->embed; e.embed_scale = m->spec.embed_scale; e.x_out = xa;
-                st = launch_residual_rms(ctx, e, false);
-            }
-            if (st == B200_OK) st = launch_residual_rms(ctx, n, true);
-            a.x = static_cast<const float*>(m->dh); a.ldx = m->Cp;
-            if (st == B200_OK) st = launch_decode_gemm(ctx, a, DPRO_PLAIN);
-        }
-        first = false;
-        std::swap(xa, xb);
+    ResidualNormArgs n{};
+    n.C = m->C; n.Cp = m->Cp; n.eps = m->spec.eps; n.vocab = m->spec.vocab; n.M = B;
+    n.x_out = m->dx; n.h = m->dh;
+    n.tok = m->dtokens; n.embed = m->embed; n.embed_scale = m->spec.embed_scale;
+    auto norm = [&](const float* w) {
+        n.w = w;
+        const int st = launch_residual_rms(ctx, n, H_SPLIT);
+        n.tok = nullptr;
+        n.x = m->dx;
         return st;
     };
-    auto plain = [&](float* out, const float* in, int ldx, const Matrix& w) {
+    auto product_args = [&](const void* x, const Matrix& w) {
         DecodeGemmArgs a{};
-        a.out = out; a.ldo = w.N; a.W = static_cast<const uint16_t*>(w.w); a.bias = w.bias; a.B = B; a.N = w.N; a.K = w.K;
-        a.x = in; a.ldx = ldx; a.status = ctx->d_status;
-        return launch_decode_gemm(ctx, a, DPRO_PLAIN);
+        a.x = static_cast<const uint8_t*>(x); a.W = static_cast<const uint16_t*>(w.w); a.bias = w.bias; a.B = B; a.N = w.N; a.K = w.K;
+        return a;
+    };
+    auto plain = [&](float* out, const void* x, const Matrix& w) {
+        DecodeGemmArgs a = product_args(x, w);
+        a.out = out; a.ldo = w.N;
+        return launch_decode_gemm(ctx, a);
     };
     for (const Layer& L : m->layers) {
         const LayerSpec& s = *L.spec;
-        TRY(residual(m->dproj, L.in.N, L.in, L.norm1, ACT_NONE));
+        TRY(norm(L.norm1));
+        DecodeGemmArgs in = product_args(m->dh, L.in);
+        in.out = m->dproj; in.ldo = L.in.N;
+        if (s.kind != MIX_PARALLEL) {
+            in.seqs = m->dseqs; in.conv_w = L.conv_w; in.conv_b = L.conv_b; in.hist = L.hist; in.conv_n = L.np; in.taps = s.conv; in.max_slots = m->max_slots;
+            if (s.kind == MIX_MAMBA1) in.conv_out = static_cast<uint8_t*>(m->dconv);
+        }
+        TRY(launch_decode_gemm(ctx, in));
         if (s.kind == MIX_MAMBA1) {
-            DecodeGemmArgs a{};
-            a.out = m->daux; a.ldo = L.xp.N; a.W = static_cast<const uint16_t*>(L.xp.w); a.B = B; a.N = L.xp.N; a.K = L.np;
-            a.seqs = m->dseqs; a.conv_w = L.conv_w; a.conv_b = L.conv_b; a.hist = L.hist; a.taps = s.conv; a.max_slots = m->max_slots;
-            a.status = ctx->d_status;
-            if (decode_gemm_fits(L.np, B)) {
-                a.x = m->dproj; a.ldx = L.in.N; a.conv_out = m->dconv;
-                TRY(launch_decode_gemm(ctx, a, DPRO_CONV));
-            } else {
-                ShortConvArgs c{};
-                c.x = m->dproj; c.ldx = L.in.N; c.out = m->dconv; c.ld_out = L.np; c.w = L.conv_w; c.bias = L.conv_b; c.hist = L.hist; c.seqs = m->dseqs;
-                c.np = L.np; c.taps = s.conv; c.max_slots = m->max_slots;
-                TRY(launch_short_conv(ctx, c, B, 1, true));
-                a.x = m->dconv; a.ldx = L.np;
-                TRY(launch_decode_gemm(ctx, a, DPRO_PLAIN));
-            }
+            TRY(plain(m->daux, m->dconv, L.xp));
             SelectiveScanArgs c{};
             c.x = m->dconv; c.ldx = L.np; c.bc = m->daux; c.ldbc = L.xp.N; c.b_col = L.rank_p; c.c_col = L.rank_p + L.sp;
             c.z = m->dproj + L.np; c.ldz = L.in.N; c.A2 = L.A2; c.dt_b = L.dt_b; c.D = L.D; c.S = L.S; c.out = m->dmix; c.ldo = L.o.K; c.seqs = m->dseqs;
@@ -756,22 +725,28 @@ int enqueue_decode(b200_decoder* m, int B) {
         } else if (s.kind == MIX_DELTA) {
             DeltaArgs a = delta_args(m, L, m->dseqs, m->dproj);
             a.qkv = m->dproj; a.ld = L.in.N;
-            a.out = m->dmix; a.ldo = L.o.K;
+            a.out = static_cast<float*>(m->dmix); a.ldo = L.o.K;
             TRY(launch_delta_step(ctx, a, B));
         } else {
-            TRY(launch_attention_cached_decode(ctx, L.att, m->dproj, L.in.N, m->dmix, L.o.K, m->dseqs, B, m->partial, m->counters,
-                                               gru_args(m, L, m->dseqs, m->dproj, m->dmix, 4)));
+            MinGruArgs gru = gru_args(L, m->dseqs, m->dproj, m->dmix);
+            gru.out_col = L.att_p;
+            TRY(launch_attention_cached_decode(ctx, L.att, m->dproj, L.in.N, static_cast<uint8_t*>(m->dmix), L.o.K, m->dseqs, B, gru));
         }
-        TRY(plain(m->dy, m->dmix, L.o.K, L.o));
-        pending = m->dy;
-        pending_w = L.norm1b;
+        TRY(plain(m->dy, m->dmix, L.o));
+        n.y = m->dy;
+        n.wb = L.norm1b;
         if (s.ff > 0) {
-            TRY(residual(m->dmix, L.mlp.up.N, L.mlp.up, L.norm2, m->spec.design->mlp_act));
-            TRY(plain(m->dy, m->dmix, L.mlp.up.N, L.mlp.down));
-            pending_w = L.norm2b;
+            TRY(norm(L.norm2));
+            DecodeGemmArgs up = product_args(m->dh, L.mlp.up);
+            up.act = m->spec.design->mlp_act;
+            up.split_out = static_cast<uint8_t*>(m->dmix);
+            TRY(launch_decode_gemm(ctx, up));
+            TRY(plain(m->dy, m->dmix, L.mlp.down));
+            n.wb = L.norm2b;
         }
     }
-    return residual(m->dlogits, m->Vp, m->head, m->final_norm, ACT_NONE);
+    TRY(norm(m->final_norm));
+    return plain(m->dlogits, m->dh, m->head);
 }
 
 // ------------------------------------------------------------------ steps

@@ -673,24 +673,31 @@ attention_cached_mma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
 }
 
 // ------------------------------------------------------------------ decode
-// Grid (key/value head x head chunk x split, sequence); further CTAs in x run the minGRU step.  GH query heads
-// of a group share every key and value read.  Keys go by in tiles of 128: scores (LK lanes per key, 16 bytes
-// of the key per lane), softmax statistics (a warp per head), probabilities x values (LV lanes per key).
+// A cluster of `splits` CTAs per (sequence, key/value head, chunk of GH query heads), each with its share of the
+// cached positions; further CTAs in x run the minGRU step.  The query heads of a CTA share every key and value
+// read.  Keys go by in tiles of 128: scores (LK lanes per key, 16 bytes of the key per lane), softmax statistics
+// (a warp per head), probabilities x values (LV lanes per key); a tile's keys and first values are requested
+// together, the first tile's before the queries are formed.  The splits' states are merged through the cluster's
+// shared memory.
 constexpr int kDecThreads = 256, kDecTile = 128;
+
+__device__ __forceinline__ float ld_cluster_f32(const float* p, int rank) {
+    float v;
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(map_to_cta(smem_u32(p), rank)) : "memory");
+    return v;
+}
 
 template <int GH, int LK>
 __global__ void __launch_bounds__(kDecThreads)
-attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj, int ld, float* __restrict__ out, int ldo,
-                        const SeqDesc* __restrict__ seqs, int splits, int chunks, float* partial, unsigned int* counters, const MinGruArgs gru) {
+attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj, int ld, uint8_t* __restrict__ out, int ldo,
+                        const SeqDesc* __restrict__ seqs, int splits, int chunks, const MinGruArgs gru) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float ss[GH][kDecTile];
-    __shared__ float stat_m[GH], stat_l[GH], stat_a[GH], s_new[GH];
-    __shared__ int is_last;
+    __shared__ float stat_m[GH], stat_l[GH], stat_a[GH];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     griddep_wait();
     griddep_launch_dependents();
-    const int b = blockIdx.y;
-    const SeqDesc sd = seqs[b];
+    const SeqDesc sd = seqs[blockIdx.y];
     const int att_blocks = c.G * chunks * splits;
     const float* row = proj + (size_t)sd.row0 * ld;
     if ((int)blockIdx.x >= att_blocks) {  // minGRU: one thread per channel
@@ -700,7 +707,7 @@ attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj,
             float* Sp = gru.S + (size_t)sd.slot * gru.width + ch;
             const float S = fmaf(1.f - z, sd.pos0 > 0 ? *Sp : 0.f, z * (u >= 0.f ? u + 0.5f : sigmoidf_(u)));
             *Sp = S;
-            static_cast<float*>(gru.out)[(size_t)sd.row0 * gru.ldo + ch] = S * silu(row[gru.g_col + ch]) * gru.out_scale;
+            store_split(static_cast<uint8_t*>(gru.out) + (size_t)sd.row0 * gru.ldo * 4, gru.out_col + ch, S * silu(row[gru.g_col + ch]) * gru.out_scale);
         }
         return;
     }
@@ -715,6 +722,30 @@ attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj,
     const float2* rot = c.rot + (size_t)pos * (c.rot_dims >> 1);
     __half* Kc = static_cast<__half*>(c.K) + ((size_t)sd.slot * c.G + g) * c.Tp * Dp;
     __half* Vc = static_cast<__half*>(c.V) + ((size_t)sd.slot * c.G + g) * c.Tp * Dvp;
+    const int per = (((pos + splits - 1) / splits + kDecTile - 1) / kDecTile) * kDecTile;  // cached keys per split
+    const int t_begin = min(pos, z * per), t_end = min(pos, t_begin + per);
+    constexpr int KPP = kDecThreads / LK;  // keys per pass
+    constexpr int PASSES = kDecTile / KPP;
+    constexpr int VU = 4;                  // values per thread requested at a time
+    const int sub = lane & (LK - 1);
+    const int LV = Dvp >> 3, vgroups = kDecThreads / LV, vg = tid / LV, vsub = tid - vg * LV;
+    const bool v_live = vg < vgroups;
+    uint4 kv[PASSES], vv[VU];
+    auto request = [&](int t0) {
+#pragma unroll
+        for (int p = 0; p < PASSES; ++p) {
+            const int t = t0 + p * KPP + tid / LK;
+            kv[p] = make_uint4(0u, 0u, 0u, 0u);
+            if (t < t_end && sub * 8 < Dp) kv[p] = *reinterpret_cast<const uint4*>(Kc + (size_t)t * Dp + sub * 8);
+        }
+#pragma unroll
+        for (int u = 0; u < VU; ++u) {
+            const int t = t0 + vg + u * vgroups;
+            vv[u] = make_uint4(0u, 0u, 0u, 0u);
+            if (v_live && t < min(t_end, t0 + kDecTile)) vv[u] = *reinterpret_cast<const uint4*>(Vc + (size_t)t * Dvp + vsub * 8);
+        }
+    };
+    request(t_begin);
     for (int j = warp; j < GH + 2; j += 8) {
         if (j < GH) {
             if (j < nh) head_vector(qs + j * Dp, row + c.q_col + (h0 + j) * c.D, c.D, Dp, c.q_norm != nullptr, c.q_norm, c.eps, c.rot_dims, rot, lane);
@@ -741,37 +772,38 @@ attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj,
         for (int d = lane; d < Dp; d += 32) s = fmaf(qs[warp * Dp + d], kn[d], s);
         s = warp_sum(s);
         if (lane == 0) {
-            s_new[warp] = s;
             stat_m[warp] = z == 0 ? s : -INFINITY;  // the new key belongs to split 0
             stat_l[warp] = z == 0 ? 1.f : 0.f;
         }
     }
     // this lane's piece of the queries
-    const int sub = lane & (LK - 1);
     float q[GH][8];
 #pragma unroll
     for (int j = 0; j < GH; ++j)
 #pragma unroll
         for (int e = 0; e < 8; ++e) q[j][e] = sub * 8 + e < Dp ? qs[j * Dp + sub * 8 + e] : 0.f;
-    const int LV = Dvp >> 3, vgroups = kDecThreads / LV, vg = tid / LV, vsub = tid - vg * LV;
-    const bool v_live = vg < vgroups;
     float acc[GH][8];
 #pragma unroll
     for (int j = 0; j < GH; ++j)
 #pragma unroll
         for (int e = 0; e < 8; ++e) acc[j][e] = (z == 0 && vg == 0) ? vn[vsub * 8 + e] : 0.f;
-    const int per = (((pos + splits - 1) / splits + kDecTile - 1) / kDecTile) * kDecTile;  // cached keys per split
-    const int t_begin = min(pos, z * per), t_end = min(pos, t_begin + per);
-    constexpr int KPP = kDecThreads / LK;  // keys per pass
-    constexpr int PASSES = kDecTile / KPP;
-    for (int t0 = t_begin; t0 < t_end; t0 += kDecTile) {
-        uint4 kv[PASSES];
+    auto add_value = [&](const uint4& x, int t) {
+        const __half2* hp = reinterpret_cast<const __half2*>(&x);
+        float2 f[4];
 #pragma unroll
-        for (int p = 0; p < PASSES; ++p) {
-            const int t = t0 + p * KPP + tid / LK;
-            kv[p] = make_uint4(0u, 0u, 0u, 0u);
-            if (t < t_end && sub * 8 < Dp) kv[p] = *reinterpret_cast<const uint4*>(Kc + (size_t)t * Dp + sub * 8);
+        for (int e = 0; e < 4; ++e) f[e] = __half22float2(hp[e]);
+#pragma unroll
+        for (int j = 0; j < GH; ++j) {
+            const float p = ss[j][t];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                acc[j][2 * e] = fmaf(p, f[e].x, acc[j][2 * e]);
+                acc[j][2 * e + 1] = fmaf(p, f[e].y, acc[j][2 * e + 1]);
+            }
         }
+    };
+    for (int t0 = t_begin; t0 < t_end; t0 += kDecTile) {
+        const int nt = min(kDecTile, t_end - t0);
 #pragma unroll
         for (int p = 0; p < PASSES; ++p) {
             const int kt = p * KPP + tid / LK;
@@ -790,7 +822,7 @@ attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj,
             if (scatter_owner<GH, LK>(lane)) {
                 const int first = scatter_first<GH, LK>(lane);
 #pragma unroll
-                for (int j = 0; j < HELD; ++j) ss[first + j][kt] = t0 + kt < t_end ? s[j] : -INFINITY;
+                for (int j = 0; j < HELD; ++j) ss[first + j][kt] = kt < nt ? s[j] : -INFINITY;
             }
         }
         __syncthreads();
@@ -809,6 +841,7 @@ attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj,
                 s += p;
             }
             s = warp_sum(s);
+            __syncwarp();
             if (lane == 0) {
                 const float al = ex2(m_old - m);
                 stat_a[warp] = al;
@@ -824,40 +857,22 @@ attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj,
 #pragma unroll
                 for (int e = 0; e < 8; ++e) acc[j][e] *= al;
             }
-            const int nt = min(kDecTile, t_end - t0);
-            for (int kt = vg; kt < nt; kt += 4 * vgroups) {
-                uint4 vv[4];
 #pragma unroll
-                for (int u = 0; u < 4; ++u) {
-                    const int t = kt + u * vgroups;
-                    vv[u] = make_uint4(0u, 0u, 0u, 0u);
-                    if (t < nt) vv[u] = *reinterpret_cast<const uint4*>(Vc + (size_t)(t0 + t) * Dvp + vsub * 8);
-                }
+            for (int u = 0; u < VU; ++u)
+                if (vg + u * vgroups < nt) add_value(vv[u], vg + u * vgroups);
+            for (int kt = vg + VU * vgroups; kt < nt; kt += VU * vgroups) {  // value heads of more than 64
 #pragma unroll
-                for (int u = 0; u < 4; ++u) {
-                    const int t = kt + u * vgroups;
-                    if (t < nt) {
-                        const __half2* hp = reinterpret_cast<const __half2*>(&vv[u]);
-                        float2 f[4];
+                for (int u = 0; u < VU; ++u)
+                    if (kt + u * vgroups < nt) vv[u] = *reinterpret_cast<const uint4*>(Vc + (size_t)(t0 + kt + u * vgroups) * Dvp + vsub * 8);
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) f[e] = __half22float2(hp[e]);
-#pragma unroll
-                        for (int j = 0; j < GH; ++j) {
-                            const float p = ss[j][t];
-#pragma unroll
-                            for (int e = 0; e < 4; ++e) {
-                                acc[j][2 * e] = fmaf(p, f[e].x, acc[j][2 * e]);
-                                acc[j][2 * e + 1] = fmaf(p, f[e].y, acc[j][2 * e + 1]);
-                            }
-                        }
-                    }
-                }
+                for (int u = 0; u < VU; ++u)
+                    if (kt + u * vgroups < nt) add_value(vv[u], kt + u * vgroups);
             }
         }
+        if (t0 + kDecTile < t_end) request(t0 + kDecTile);
         __syncthreads();
     }
     // sum of the key groups: each in turn adds its part (a handful of them; fixed order)
-    __syncthreads();
     for (int i = tid; i < GH * Dvp; i += kDecThreads) os[i] = 0.f;
     __syncthreads();
     // groups of one warp first, by shuffles, when they are whole powers of two
@@ -880,42 +895,27 @@ attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj,
         }
         __syncthreads();
     }
+    uint8_t* orow = out + (size_t)sd.row0 * ldo * 4;
     if (splits == 1) {
         for (int i = tid; i < nh * c.Dv; i += kDecThreads) {
             const int j = i / c.Dv, d = i - j * c.Dv;
-            out[(size_t)sd.row0 * ldo + (h0 + j) * c.Dv + d] = os[j * Dvp + d] / stat_l[j] * c.out_scale;
+            store_split(orow, (h0 + j) * c.Dv + d, os[j * Dvp + d] / stat_l[j] * c.out_scale);
         }
         return;
     }
-    const int stride = Dvp + 2;
-    float* mine = partial + (((size_t)b * c.G * chunks + gc) * splits + z) * GH * stride;
-    for (int i = tid; i < GH * Dvp; i += kDecThreads) mine[(i / Dvp) * stride + i % Dvp] = os[i];
-    if (tid < GH) {
-        mine[tid * stride + Dvp] = stat_l[tid];
-        mine[tid * stride + Dvp + 1] = stat_m[tid];
-    }
-    __threadfence();
-    __syncthreads();
-    unsigned int* counter = counters + (size_t)b * c.G * chunks + gc;
-    if (tid == 0) is_last = (atomicAdd(counter, 1u) == (unsigned)splits - 1);
-    __syncthreads();
-    if (!is_last) return;
-    __threadfence();
-    // the last CTA of the group merges the splits, in their order
-    const float* all = partial + ((size_t)b * c.G * chunks + gc) * splits * GH * stride;
-    for (int i = tid; i < nh * c.Dv; i += kDecThreads) {
+    cluster_sync_all();  // every split's state is in its shared memory
+    for (int i = z * kDecThreads + tid; i < nh * c.Dv; i += splits * kDecThreads) {
         const int j = i / c.Dv, d = i - j * c.Dv;
         float m = -INFINITY, L = 0.f, O = 0.f;
-        for (int s = 0; s < splits; ++s) m = fmaxf(m, __ldcg(all + ((size_t)s * GH + j) * stride + Dvp + 1));
+        for (int s = 0; s < splits; ++s) m = fmaxf(m, ld_cluster_f32(stat_m + j, s));
         for (int s = 0; s < splits; ++s) {
-            const float* ps = all + ((size_t)s * GH + j) * stride;
-            const float w = ex2(__ldcg(ps + Dvp + 1) - m);  // 0 for a split without keys
-            L = fmaf(__ldcg(ps + Dvp), w, L);
-            O = fmaf(__ldcg(ps + d), w, O);
+            const float w = ex2(ld_cluster_f32(stat_m + j, s) - m);  // 0 for a split without keys
+            L = fmaf(ld_cluster_f32(stat_l + j, s), w, L);
+            O = fmaf(ld_cluster_f32(os + j * Dvp + d, s), w, O);
         }
-        out[(size_t)sd.row0 * ldo + (h0 + j) * c.Dv + d] = O / L * c.out_scale;
+        store_split(orow, (h0 + j) * c.Dv + d, O / L * c.out_scale);
     }
-    if (tid == 0) *counter = 0u;
+    cluster_sync_all();  // nobody leaves while its state is being read
 }
 
 template <int KD, int VD>
@@ -939,30 +939,47 @@ int decode_heads_per_cta(const CachedAttention& c) {
 }
 
 template <int GH, int LK>
-int launch_decode_one(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, float* out, int ldo, const SeqDesc* seqs, int B,
-                      float* partial, unsigned int* counters, const MinGruArgs& gru) {
+int launch_decode_one(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, uint8_t* out, int ldo, const SeqDesc* seqs, int B,
+                      const MinGruArgs& gru) {
     const int chunks = (c.H / c.G + GH - 1) / GH;
-    int splits = 2 * ctx->num_sms / (B * c.G * chunks);
-    const int most = (c.Tp + kDecTile - 1) / kDecTile;
-    if (splits > kDecodeAttMaxSplits) splits = kDecodeAttMaxSplits;
-    if (splits > most) splits = most;
-    if (splits < 1) splits = 1;
+    int splits = 1;
+    while (splits < 8 && B * c.G * chunks * splits * 2 <= 2 * ctx->num_sms && splits * 2 * kDecTile <= c.Tp) splits *= 2;
     const size_t smem = (size_t)(GH * c.Dp + c.Dp + c.Dvp + GH * c.Dvp) * 4;
     if (smem > 40 * 1024) return B200_ERR_LIMIT;
-    const int gru_blocks = gru.S ? (gru.width + kDecThreads - 1) / kDecThreads : 0;
-    cudaError_t le = launch_pdl(ctx, attention_decode_kernel<GH, LK>, dim3(c.G * chunks * splits + gru_blocks, B), dim3(kDecThreads), smem, c, proj, ld, out,
-                                ldo, seqs, splits, chunks, partial, counters, gru);
+    int gru_blocks = gru.S ? (gru.width + kDecThreads - 1) / kDecThreads : 0;
+    gru_blocks = (gru_blocks + splits - 1) / splits * splits;  // whole clusters
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(c.G * chunks * splits + gru_blocks, B);
+    cfg.blockDim = dim3(kDecThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    cudaLaunchAttribute attr[2];
+    int n = 0;
+    if (splits > 1) {
+        attr[n].id = cudaLaunchAttributeClusterDimension;
+        attr[n].val.clusterDim.x = splits;
+        attr[n].val.clusterDim.y = attr[n].val.clusterDim.z = 1;
+        ++n;
+    }
+    if (ctx->pdl) {
+        attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[n].val.programmaticStreamSerializationAllowed = 1;
+        ++n;
+    }
+    cfg.attrs = attr;
+    cfg.numAttrs = n;
+    const cudaError_t le = cudaLaunchKernelEx(&cfg, attention_decode_kernel<GH, LK>, c, proj, ld, out, ldo, seqs, splits, chunks, gru);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
 }
 
 template <int GH>
-int launch_decode_lk(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, float* out, int ldo, const SeqDesc* seqs, int B,
-                     float* partial, unsigned int* counters, const MinGruArgs& gru) {
-    if (c.Dp <= 64) return launch_decode_one<GH, 8>(ctx, c, proj, ld, out, ldo, seqs, B, partial, counters, gru);
-    if (c.Dp <= 128) return launch_decode_one<GH, 16>(ctx, c, proj, ld, out, ldo, seqs, B, partial, counters, gru);
-    return launch_decode_one<GH, 32>(ctx, c, proj, ld, out, ldo, seqs, B, partial, counters, gru);
+int launch_decode_lk(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, uint8_t* out, int ldo, const SeqDesc* seqs, int B,
+                     const MinGruArgs& gru) {
+    if (c.Dp <= 64) return launch_decode_one<GH, 8>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
+    if (c.Dp <= 128) return launch_decode_one<GH, 16>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
+    return launch_decode_one<GH, 32>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
 }
 
 }  // namespace
@@ -1029,19 +1046,14 @@ int launch_attention_cached_simt(b200_ctx* ctx, const CachedAttention& c, const 
     return B200_OK;
 }
 
-size_t attention_decode_partial_floats(const CachedAttention& c, int B) {
-    const int gh = decode_heads_per_cta(c), chunks = (c.H / c.G + gh - 1) / gh;
-    return (size_t)B * c.G * chunks * kDecodeAttMaxSplits * gh * (c.Dvp + 2);
-}
-
-int launch_attention_cached_decode(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, float* out, int ldo,
-                                   const SeqDesc* seqs, int B, float* partial, unsigned int* counters, const MinGruArgs& gru) {
+int launch_attention_cached_decode(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, uint8_t* out, int ldo,
+                                   const SeqDesc* seqs, int B, const MinGruArgs& gru) {
     if (c.D > kMaxHead || c.Dv > kMaxHead) return B200_ERR_LIMIT;
     switch (decode_heads_per_cta(c)) {
-        case 8: return launch_decode_lk<8>(ctx, c, proj, ld, out, ldo, seqs, B, partial, counters, gru);
-        case 4: return launch_decode_lk<4>(ctx, c, proj, ld, out, ldo, seqs, B, partial, counters, gru);
-        case 2: return launch_decode_lk<2>(ctx, c, proj, ld, out, ldo, seqs, B, partial, counters, gru);
-        default: return launch_decode_lk<1>(ctx, c, proj, ld, out, ldo, seqs, B, partial, counters, gru);
+        case 8: return launch_decode_lk<8>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
+        case 4: return launch_decode_lk<4>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
+        case 2: return launch_decode_lk<2>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
+        default: return launch_decode_lk<1>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
     }
 }
 

@@ -25,7 +25,7 @@ inline int pad_dim(int n) { return n < 64 ? 64 : (n + 7) & ~7; }
 
 // ---- row-wise (rmsnorm.cu)
 // Residual stream of M rows:  r = embed[tok] * scale (tok != null), or x, or x + rms(y) * wb (y != null);
-// x_out = r (if not null);  h = rms(r) * w as f32 / bf16 (if w).  rows != null: row i of the output
+// x_out = r (if not null);  h = rms(r) * w (if w) as bf16, fp32 or split rows (decoder_math.cuh).  rows != null: row i of the output
 // is made from row rows[i] of the inputs.  C columns of Cp.
 struct ResidualNormArgs {
     const float* x; const float* y; const float* wb; const float* w;
@@ -34,7 +34,8 @@ struct ResidualNormArgs {
     const int* rows;
     int M, C, Cp; float eps;
 };
-int launch_residual_rms(b200_ctx* ctx, const ResidualNormArgs& a, bool f32);
+enum : int { H_BF16 = 0, H_F32 = 1, H_SPLIT = 2 };
+int launch_residual_rms(b200_ctx* ctx, const ResidualNormArgs& a, int format);  // H_F32: the embedding table is fp32, else bf16
 // out[r, h*Dv + d] = o / rms(o over the head) * w[d] * silu(gate);  o, gate [M] rows with heads Dvl apart
 int launch_gated_head_norm(b200_ctx* ctx, void* out, int ld_out, const float* o, int ld_o, const float* gate, int ld_gate,
                            const float* w, int M, int H, int Dv, int Dvl, float eps, bool f32);
@@ -46,29 +47,21 @@ enum : int { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_GELU_ERF = 2 };
 // out[M,N] = act(inp[M,K] W[N,K]^T + bias) on the fp32 FMA pipe (no reduced precision anywhere); K, N multiples of 4
 int launch_gemm_fp32(b200_ctx* ctx, float* out, const float* inp, const float* W, const float* bias, int M, int K, int N, int act);
 
-// Decode product (gemm_decode.cu): B <= 16 rows against bf16 weights.  Prologues that form the input:
-//   DPRO_PLAIN     x [B, K] fp32
-//   DPRO_RESIDUAL  r = embed[tok] * scale, or x, or x + rms(y) * wb; input = rms(r) * w; r is stored to
-//                  x_out by one CTA (a buffer other than x)
-//   DPRO_CONV      short causal convolution + bias + silu of column block [0, K) of x (leading dimension ldx)
-//                  with the history bank; the convolved row goes to conv_out, the new history to the other bank
-enum : int { DPRO_PLAIN = 0, DPRO_RESIDUAL = 1, DPRO_CONV = 2 };
+// Decode product (gemm_decode.cu): B <= 16 split rows x [B, K] against bf16 weights [N, K], + bias, then
+//   columns below conv_n: short causal convolution with the history of the row's slot (+ conv_b) and silu; the new
+//     history goes to the other bank
+//   the others: act
+// to out (fp32) and, as split rows, to split_out (all columns) or conv_out (the convolved ones, which then do not go to out).
 struct DecodeGemmArgs {
-    float* out; int ldo;
-    const uint16_t* W;   // [N, K]
-    const float* bias;
+    const uint8_t* x;
+    const uint16_t* W; const float* bias;
     int B, N, K, act;
-    const float* x; int ldx;
-    // DPRO_RESIDUAL
-    const float* y; const float* wb; const float* w; float* x_out;
-    const int* tok; const uint16_t* embed; float embed_scale; int vocab;
-    int C; float eps;
-    // DPRO_CONV
-    const SeqDesc* seqs; const float* conv_w; const float* conv_b; float* hist; int taps; int max_slots; float* conv_out;
-    int* status;
+    float* out; int ldo;
+    uint8_t* split_out;   // [B] rows of N columns
+    const SeqDesc* seqs; const float* conv_w; const float* conv_b; float* hist; int conv_n, taps, max_slots;
+    uint8_t* conv_out;    // [B] rows of conv_n columns
 };
-int launch_decode_gemm(b200_ctx* ctx, const DecodeGemmArgs& a, int prologue);
-bool decode_gemm_fits(int K, int B);  // whether DPRO_RESIDUAL / DPRO_CONV can hold B rows of K on chip
+int launch_decode_gemm(b200_ctx* ctx, const DecodeGemmArgs& a);
 
 // ---- recurrences (recurrent.cu)
 // y = silu(causal depthwise convolution of columns [0, n) of x + bias); weights [taps][np]; history
@@ -86,9 +79,10 @@ int launch_short_conv(b200_ctx* ctx, const ShortConvArgs& a, int E, int max_n, b
 
 // Selective scan with a diagonal state per channel:
 //   dt = softplus(dt_raw + dt_b);  S[c,:] = 2^(dt A2[c,:]) S[c,:] + dt x B;  y = (S C + D x) * silu(z)
-// With Wdt (decode, one token per sequence) dt_raw is formed here: dt_raw[c] = Wdt[c,:] . bc[0..rank).
+// With Wdt (decode, one token per sequence) dt_raw is formed here: dt_raw[c] = Wdt[c,:] . bc[0..rank), and x
+// and out are split rows.
 struct SelectiveScanArgs {
-    const void* x; int ldx;           // convolved input: bf16 (f32: fp32)
+    const void* x; int ldx;           // convolved input: bf16 (f32: fp32; decode: split rows of ldx columns)
     const float* dt; int lddt;        // dt_raw, null with Wdt
     const float* bc; int ldbc;        // per token: [dt: ..| B: at b_col | C: at c_col]
     int b_col, c_col;
@@ -110,7 +104,8 @@ int launch_selective_scan(b200_ctx* ctx, const SelectiveScanArgs& a, int E, int 
 //   prep   convolution + silu of raw's q and k columns -> unit vectors (q also times D^-1/2) in qkv, and coef
 //          (the v columns are a plain short convolution)
 //   scan   qkv, coef -> o in out [M, H*Dvl] fp32
-//   step   one token per sequence, everything from the raw projection (qkv, ld) to the normalised, gated output
+//   step   one token per sequence, from the convolved columns (qkv, ld) to the normalised, gated output as split rows
+//          of ldo columns
 struct DeltaArgs {
     const float* qkv; int ld; int k_col, v_col;
     const float* raw; int ld_raw;
@@ -138,6 +133,7 @@ struct MinGruArgs {
     void* out; int ldo;
     const SeqDesc* seqs;
     int width; float out_scale;
+    int out_col;  // added to the column (the decode kernel, whose split rows cannot be offset by a pointer)
 };
 int launch_min_gru(b200_ctx* ctx, const MinGruArgs& a, int E, bool f32);
 
@@ -154,7 +150,7 @@ struct CachedAttention {
     float scale, eps;
     void* K; void* V;
     float out_scale;
-};
+};  // (scores: (q . k) * scale)
 inline int attention_pad(int d) { return d <= 64 ? 64 : (d + 63) & ~63; }
 // norms and rotation of a step's q (-> q_out [M][H * Dp]) and k, v (-> cache)
 int launch_attention_prep(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, void* q_out, const SeqDesc* seqs,
@@ -166,11 +162,9 @@ int launch_attention_cached_mma(b200_ctx* ctx, const CachedAttention& c, const v
                                 const int2* pairs, int num_pairs, int M, int max_slots);
 int launch_attention_cached_simt(b200_ctx* ctx, const CachedAttention& c, const void* q, void* out, int ldo, const SeqDesc* seqs,
                                  int E, int max_n, bool f32);
-// One token per sequence: norms, rotation, cache append and attention in one kernel (fp16 cache, fp32
-// out [B][ldo]); with gru.S also a minGRU step in further CTAs of the launch.
-constexpr int kDecodeAttMaxSplits = 16;
-int launch_attention_cached_decode(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, float* out, int ldo,
-                                   const SeqDesc* seqs, int B, float* partial, unsigned int* counters, const MinGruArgs& gru);
-size_t attention_decode_partial_floats(const CachedAttention& c, int B);
+// One token per sequence: norms, rotation, cache append and attention in one kernel (fp16 cache; out: split rows of
+// ldo columns); with gru.S also a minGRU step in further CTAs of the launch (gru.out: the same rows, out_col: its first column).
+int launch_attention_cached_decode(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, uint8_t* out, int ldo,
+                                   const SeqDesc* seqs, int B, const MinGruArgs& gru);
 
 }  // namespace b200

@@ -74,6 +74,26 @@ __device__ __forceinline__ void store1(void* base, size_t i, float v) {
     else reinterpret_cast<__nv_bfloat16*>(base)[i] = __float2bfloat16_rn(v);
 }
 
+// Split rows, the operand format of the decode products: eight values as 16 bytes of bf16 and 16 bytes of the
+// bf16 of what that rounding dropped (four bytes per value in all).
+__device__ __forceinline__ void store_split(uint8_t* row, int k, float v) {
+    const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+    __nv_bfloat16* p = reinterpret_cast<__nv_bfloat16*>(row + (k >> 3) * 32 + (k & 7) * 2);
+    p[0] = hi;
+    p[8] = __float2bfloat16_rn(v - __bfloat162float(hi));
+}
+__device__ __forceinline__ void store_split4(uint8_t* row, int k4, float4 v) {  // values 4 k4 .. 4 k4 + 3
+    const uint32_t h0 = pack_bf16(v.x, v.y), h1 = pack_bf16(v.z, v.w);
+    uint2* p = reinterpret_cast<uint2*>(row + (k4 >> 1) * 32 + (k4 & 1) * 8);
+    p[0] = make_uint2(h0, h1);
+    p[2] = make_uint2(pack_bf16(v.x - __uint_as_float(h0 << 16), v.y - __uint_as_float(h0 & 0xffff0000u)),
+                      pack_bf16(v.z - __uint_as_float(h1 << 16), v.w - __uint_as_float(h1 & 0xffff0000u)));
+}
+__device__ __forceinline__ float load_split(const uint8_t* row, int k) {
+    const __nv_bfloat16* p = reinterpret_cast<const __nv_bfloat16*>(row + (k >> 3) * 32 + (k & 7) * 2);
+    return __bfloat162float(p[0]) + __bfloat162float(p[8]);
+}
+
 __device__ __forceinline__ void cp_async16(void* smem_dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst))), "l"(src) : "memory");
 }

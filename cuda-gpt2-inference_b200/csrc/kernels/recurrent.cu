@@ -126,7 +126,8 @@ selective_scan_kernel(const SelectiveScanArgs a) {
             if (c0 + q < a.inner) {
                 if (!STEP) cp_async16(&T.dt[t][q], a.dt + r * a.lddt + c0 + q);
                 cp_async16(&T.z[t][q], a.z + r * a.ldz + c0 + q);
-                if (XF32) cp_async16(T.x + (t * kScanCh + q) * XB, static_cast<const float*>(a.x) + r * a.ldx + c0 + q);
+                if (STEP) {}  // split rows: below
+                else if (XF32) cp_async16(T.x + (t * kScanCh + q) * XB, static_cast<const float*>(a.x) + r * a.ldx + c0 + q);
                 else cp_async8(T.x + (t * kScanCh + q) * XB, static_cast<const uint16_t*>(a.x) + r * a.ldx + c0 + q);
             }
         }
@@ -136,6 +137,8 @@ selective_scan_kernel(const SelectiveScanArgs a) {
             cp_async16(&T.bc[which][t][q], a.bc + (size_t)(sd.row0 + t0 + t) * a.ldbc + (which ? a.c_col : a.b_col) + q);
         }
         cp_async_commit();
+        if (STEP && tid < kScanCh && c0 + tid < a.inner)
+            reinterpret_cast<float*>(T.x)[tid] = load_split(static_cast<const uint8_t*>(a.x) + (size_t)sd.row0 * a.ldx * 4, c0 + tid);
     };
     auto xval = [&](const Tile& T, int t, int k) {
         return XF32 ? reinterpret_cast<const float*>(T.x)[t * kScanCh + k] : bf16_to_f(reinterpret_cast<const uint16_t*>(T.x)[t * kScanCh + k]);
@@ -194,7 +197,8 @@ selective_scan_kernel(const SelectiveScanArgs a) {
             const int t = i / kScanCh, k = i & (kScanCh - 1);
             if (c0 + k < a.inner) {
                 const float v = (T.dt[t][k] + Dc_ch * xval(T, t, k)) * silu(T.z[t][k]);
-                store1<OF32>(a.out, (size_t)(sd.row0 + t0 + t) * a.ldo + c0 + k, v);
+                if (STEP) store_split(static_cast<uint8_t*>(a.out) + (size_t)sd.row0 * a.ldo * 4, c0 + k, v);
+                else store1<OF32>(a.out, (size_t)(sd.row0 + t0 + t) * a.ldo + c0 + k, v);
             }
         }
         __syncthreads();  // the tile may be staged again
@@ -524,8 +528,7 @@ delta_scan_kernel(const DeltaArgs a) {
     core.store(Sg, l, ncol);
 }
 
-// Decode: one CTA per (head, sequence) takes its token through convolution, unit norms, the rule, the
-// output norm and the gate.
+// Decode: one CTA per (head, sequence) takes its token through unit norms, the rule, the output norm and the gate.
 constexpr int kDeltaStepThreads = 256, kDeltaStepCols = 4;
 template <int L>
 __global__ void __launch_bounds__(kDeltaStepThreads)
@@ -548,7 +551,7 @@ delta_step_kernel(const DeltaArgs a) {
     const SeqDesc sd = a.seqs[blockIdx.y];
     const float* row = a.qkv + (size_t)sd.row0 * a.ld;
     const int grp = tid / L, l = tid & (L - 1);
-    // the state of the first columns is on its way while q, k and v are formed
+    // the state of the first columns is on its way while q, k and v are fetched and normalised
     Core core;
     float* Sh = a.S + ((size_t)sd.slot * a.H + h) * a.Dv * D;
     auto fetch = [&](int gc) {
@@ -557,26 +560,10 @@ delta_step_kernel(const DeltaArgs a) {
     };
     fetch(grp * kDeltaStepCols);
     __syncthreads();
-    const int hrows = a.taps - 1;
-    const float* hr = a.hist + ((size_t)sd.bank * a.max_slots + sd.slot) * hrows * a.np;
-    float* hw = a.hist + ((size_t)(sd.bank ^ 1) * a.max_slots + sd.slot) * hrows * a.np;
     for (int i = tid; i < 2 * a.Dl + a.Dvl; i += kDeltaStepThreads) {
-        int ch;
-        float* dst;
-        bool keep;  // this CTA writes the history of the channel (q and k are shared by the heads of a group)
-        if (i < a.Dl) { ch = kvh * a.Dl + i; dst = q + i; keep = h % per == 0; }
-        else if (i < 2 * a.Dl) { ch = a.k_col + kvh * a.Dl + i - a.Dl; dst = k + i - a.Dl; keep = h % per == 0; }
-        else { ch = a.v_col + h * a.Dvl + i - 2 * a.Dl; dst = v + i - 2 * a.Dl; keep = true; }
-        float s = 0.f;
-        for (int j = 0; j < a.taps; ++j) {
-            const int back = hrows - j;
-            float x = 0.f;
-            if (back == 0) x = row[ch];
-            else if (back <= sd.pos0) x = hr[(size_t)j * a.np + ch];
-            if (keep && j > 0) hw[(size_t)(j - 1) * a.np + ch] = x;
-            s = fmaf(x, __ldg(a.conv_w + (size_t)j * a.np + ch), s);
-        }
-        *dst = silu(s);
+        if (i < a.Dl) q[i] = row[kvh * a.Dl + i];
+        else if (i < 2 * a.Dl) k[i - a.Dl] = row[a.k_col + kvh * a.Dl + i - a.Dl];
+        else v[i - 2 * a.Dl] = row[a.v_col + h * a.Dvl + i - 2 * a.Dl];
     }
     __syncthreads();
     float sq = 0.f, sk = 0.f, dot = 0.f;  // every warp for itself
@@ -608,7 +595,8 @@ delta_step_kernel(const DeltaArgs a) {
     for (int d = tid; d < a.Dv; d += kDeltaStepThreads) s += o[d] * o[d];
     const float r = 1.0f / sqrtf(block_sum(s, red) / (float)a.Dv + a.eps);
     for (int d = tid; d < a.Dv; d += kDeltaStepThreads)
-        a.out[(size_t)sd.row0 * a.ldo + h * a.Dv + d] = o[d] * r * __ldg(a.norm_w + d) * silu(row[a.gate_col + h * a.Dvl + d]);
+        store_split(reinterpret_cast<uint8_t*>(a.out) + (size_t)sd.row0 * a.ldo * 4, h * a.Dv + d,
+                    o[d] * r * __ldg(a.norm_w + d) * silu(row[a.gate_col + h * a.Dvl + d]));
 }
 
 // ------------------------------------------------------------------ minGRU

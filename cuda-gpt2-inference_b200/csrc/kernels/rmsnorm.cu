@@ -14,7 +14,7 @@ constexpr int kVpt = 4;  // float4 of a row a thread keeps in registers: rows up
 
 // Pass 1: r (see launch_residual_rms) into registers and x_out, sum of r^2.  Rows longer than the registers
 // hold are read again from x_out.
-template <bool F32>
+template <int OUT>  // H_BF16, H_F32 (with an fp32 embedding table), H_SPLIT
 __global__ void __launch_bounds__(kNormThreads)
 residual_rms_kernel(const ResidualNormArgs a, int* status) {
     __shared__ float red[8];
@@ -48,7 +48,7 @@ residual_rms_kernel(const ResidualNormArgs a, int* status) {
     auto value = [&](int c, float4 yv) {
         float4 r;
         if (a.tok) {
-            r = F32 ? load4(static_cast<const float*>(a.embed) + (size_t)tok * a.Cp, c)
+            r = OUT == H_F32 ? load4(static_cast<const float*>(a.embed) + (size_t)tok * a.Cp, c)
                     : load4(static_cast<const uint16_t*>(a.embed) + (size_t)tok * a.Cp, c);
             r.x *= a.embed_scale; r.y *= a.embed_scale; r.z *= a.embed_scale; r.w *= a.embed_scale;
         } else r = x[c];
@@ -77,7 +77,9 @@ residual_rms_kernel(const ResidualNormArgs a, int* status) {
     const float rstd = 1.0f / sqrtf(block_sum(s, red) * inv_c + a.eps);
     auto emit = [&](int c, float4 r) {
         const float4 w = __ldg(reinterpret_cast<const float4*>(a.w) + c);
-        store4<F32>(a.h, (size_t)row_out * C4 + c, make_float4(r.x * rstd * w.x, r.y * rstd * w.y, r.z * rstd * w.z, r.w * rstd * w.w));
+        const float4 h = make_float4(r.x * rstd * w.x, r.y * rstd * w.y, r.z * rstd * w.z, r.w * rstd * w.w);
+        if (OUT == H_SPLIT) store_split4(static_cast<uint8_t*>(a.h) + (size_t)row_out * a.Cp * 4, c, h);
+        else store4<OUT == H_F32>(a.h, (size_t)row_out * C4 + c, h);
     };
 #pragma unroll
     for (int i = 0; i < kVpt; ++i) {
@@ -139,12 +141,14 @@ __global__ void slice_kernel(void* dst, int ld_dst, const float* __restrict__ sr
 
 }  // namespace
 
-int launch_residual_rms(b200_ctx* ctx, const ResidualNormArgs& a, bool f32) {
+int launch_residual_rms(b200_ctx* ctx, const ResidualNormArgs& a, int format) {
     if (a.M <= 0) return B200_OK;
     int threads = ((a.Cp / 4 + 31) / 32) * 32;
     if (threads > kNormThreads) threads = kNormThreads;
-    cudaError_t le = f32 ? launch_pdl(ctx, residual_rms_kernel<true>, dim3(a.M), dim3(threads), 0, a, ctx->d_status)
-                         : launch_pdl(ctx, residual_rms_kernel<false>, dim3(a.M), dim3(threads), 0, a, ctx->d_status);
+    cudaError_t le;
+    if (format == H_F32) le = launch_pdl(ctx, residual_rms_kernel<H_F32>, dim3(a.M), dim3(threads), 0, a, ctx->d_status);
+    else if (format == H_SPLIT) le = launch_pdl(ctx, residual_rms_kernel<H_SPLIT>, dim3(a.M), dim3(threads), 0, a, ctx->d_status);
+    else le = launch_pdl(ctx, residual_rms_kernel<H_BF16>, dim3(a.M), dim3(threads), 0, a, ctx->d_status);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
