@@ -78,8 +78,9 @@ def operator_costs(cfg, M):
             H, G, D, Dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
             nc = 2 * G * D + H * Dv
             gemm("gemm delta in", C, P(nc + H * Dv + 2 * H))
-            c["conv delta"] = (M * nc * 8.0, 0, M * nc * 2.0 * m["conv"], M * nc * 2.0)
-            c["delta scan"] = (M * (nc + H * Dv + 2 * H) * 4.0, 0, M * H * D * Dv * 7.0, 0)
+            c["conv delta v"] = (M * H * Dv * 8.0, 0, M * H * Dv * 2.0 * m["conv"], M * H * Dv * 2.0)
+            c["delta prep"] = (M * 2 * G * D * 8.0 + M * H * (8 + 16.0), 0, M * 2 * G * D * (2.0 * m["conv"] + 5), M * 2 * G * D * 2.0)
+            c["delta scan"] = (M * (nc + H * Dv + 4 * H) * 4.0, 0, M * H * D * Dv * 6.0, 0)
             c["head norm"] = (M * H * Dv * (4 + 4 + 2.0), 0, 0, M * H * Dv * 2.0)
             gemm("gemm delta o", H * Dv, C)
         else:

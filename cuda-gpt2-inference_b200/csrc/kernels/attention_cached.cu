@@ -24,33 +24,44 @@ template <typename T> __device__ __forceinline__ T to_cache(float v);
 template <> __device__ __forceinline__ float to_cache<float>(float v) { return v; }
 template <> __device__ __forceinline__ __half to_cache<__half>(float v) { return to_half(v); }
 
-// One warp turns the n values at src into the normalised, rotated vector in buf (shared memory, n floats; pad
-// zeros up to n_pad): lane's values i = lane, lane + 32, ...
+// One warp turns the n values at src into the normalised, rotated vector in buf (shared memory; zeros up to n_pad):
+// lane's values i = lane, lane + 32, ...  Everything is requested before anything is used.
 __device__ __forceinline__ void head_vector(float* buf, const float* src, int n, int n_pad, bool norm, const float* w, float eps,
                                             int rot_dims, const float2* rot, int lane) {
-    float v[kMaxHead / 32];
-    float s = 0.f;
+    constexpr int NV = kMaxHead / 32;
+    const int half = rot_dims >> 1;
+    float v[NV], wv[NV];
+    float2 cs[NV / 2];
 #pragma unroll
-    for (int i = 0; i < kMaxHead / 32; ++i) {
+    for (int i = 0; i < NV; ++i) {
         const int d = lane + i * 32;
         v[i] = d < n ? src[d] : 0.f;
-        s = fmaf(v[i], v[i], s);
+        wv[i] = (w && d < n) ? __ldg(w + d) : 1.f;
     }
-    float r = 1.f;
-    if (norm) r = 1.0f / sqrtf(warp_sum(s) / (float)n + eps);
 #pragma unroll
-    for (int i = 0; i < kMaxHead / 32; ++i) {
+    for (int i = 0; i < NV / 2; ++i) cs[i] = lane + i * 32 < half ? __ldg(rot + lane + i * 32) : make_float2(1.f, 0.f);
+    float r = 1.f;
+    if (norm) {
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) s = fmaf(v[i], v[i], s);
+        r = 1.0f / sqrtf(warp_sum(s) / (float)n + eps);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
         const int d = lane + i * 32;
-        if (d < n_pad) buf[d] = d < n ? v[i] * r * (w ? __ldg(w + d) : 1.f) : 0.f;
+        if (d < n_pad) buf[d] = v[i] * r * wv[i];
     }
     __syncwarp();
-    if (rot_dims > 0) {
-        const int half = rot_dims >> 1;
-        for (int i = lane; i < half; i += 32) {
-            const float2 cs = rot[i];
-            const float u = buf[i], x = buf[i + half];
-            buf[i] = u * cs.x - x * cs.y;
-            buf[i + half] = x * cs.x + u * cs.y;
+    if (half > 0) {
+#pragma unroll
+        for (int i = 0; i < NV / 2; ++i) {
+            const int d = lane + i * 32;
+            if (d < half) {
+                const float u = buf[d], x = buf[d + half];
+                buf[d] = u * cs[i].x - x * cs[i].y;
+                buf[d + half] = x * cs[i].x + u * cs[i].y;
+            }
         }
         __syncwarp();
     }
@@ -688,7 +699,7 @@ __device__ __forceinline__ float ld_cluster_f32(const float* p, int rank) {
 }
 
 template <int GH, int LK>
-__global__ void __launch_bounds__(kDecThreads)
+__global__ void __launch_bounds__(kDecThreads, 2)
 attention_decode_kernel(const CachedAttention c, const float* __restrict__ proj, int ld, uint8_t* __restrict__ out, int ldo,
                         const SeqDesc* __restrict__ seqs, int splits, int chunks, const MinGruArgs gru) {
     extern __shared__ __align__(16) float sm[];
@@ -935,7 +946,7 @@ int launch_mma_one(b200_ctx* ctx, const CUtensorMap& tq, const CUtensorMap& tk, 
 
 int decode_heads_per_cta(const CachedAttention& c) {
     const int per = c.H / c.G;
-    return per >= 5 ? 8 : (per >= 3 ? 4 : (per == 2 ? 2 : 1));
+    return per >= 3 ? 4 : per;  // (eight heads' queries and sums would not leave room for two CTAs per SM)
 }
 
 template <int GH, int LK>
@@ -1050,7 +1061,6 @@ int launch_attention_cached_decode(b200_ctx* ctx, const CachedAttention& c, cons
                                    const SeqDesc* seqs, int B, const MinGruArgs& gru) {
     if (c.D > kMaxHead || c.Dv > kMaxHead) return B200_ERR_LIMIT;
     switch (decode_heads_per_cta(c)) {
-        case 8: return launch_decode_lk<8>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
         case 4: return launch_decode_lk<4>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
         case 2: return launch_decode_lk<2>(ctx, c, proj, ld, out, ldo, seqs, B, gru);
         default: return launch_decode_lk<1>(ctx, c, proj, ld, out, ldo, seqs, B, gru);

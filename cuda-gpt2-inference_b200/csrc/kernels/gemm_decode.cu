@@ -25,8 +25,8 @@ namespace {
 
 constexpr int kThreads = 256, kWarps = 8;
 constexpr int kU = 8;             // pieces of a warp on the way
-constexpr int kChunk = 2048;      // input columns staged at a time (kChunk2 with 16 rows)
-constexpr int kChunk2 = 1024;
+constexpr int kTwoCtaSmem = 103 * 1024;  // input rows of a CTA that still leave room for a second one ...
+constexpr int kOneCtaSmem = 200 * 1024;  // ... and the most a CTA can hold
 constexpr int kMaxTaps = 4;       // convolution inputs requested ahead of the product (longer ones behind it)
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t a0, const uint32_t a1, const uint32_t a2, const uint32_t a3,
@@ -204,10 +204,9 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
 
 template <int NT>
 int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
-    constexpr int kMaxSmem = NT * 8 * ((NT == 1 ? kChunk : kChunk2) * 4 + 16);
     static bool attr_set[64] = {};
     if (!attr_set[ctx->device & 63]) {
-        B200_CUDA(ctx, cudaFuncSetAttribute(decode_gemm_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem));
+        B200_CUDA(ctx, cudaFuncSetAttribute(decode_gemm_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kOneCtaSmem));
         attr_set[ctx->device & 63] = true;
     }
     const int tiles = (a.N + 15) / 16;
@@ -215,10 +214,13 @@ int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
     int slices = 1;
     while (slices < 8 && tiles * slices * 2 <= 2 * ctx->num_sms && a.K / (slices * 2) >= 256) slices *= 2;
     const int kslice = ((a.K + slices - 1) / slices + 31) / 32 * 32;
-    const int most = NT == 1 ? kChunk : kChunk2;
-    const int chunk = kslice < most ? kslice : most;
+    // the columns staged at a time: all of the slice, so that they are staged once for all tiles; else as many as
+    // two CTAs per SM can hold
+    auto columns = [](int smem) { return (smem / (NT * 8) - 16) / 4 / 32 * 32; };
+    const int chunk = kslice <= columns(kOneCtaSmem) ? kslice : columns(kTwoCtaSmem);
+    const int per_sm = chunk <= columns(kTwoCtaSmem) ? 2 : 1;
     int grid = tiles * slices;
-    if (grid > 2 * ctx->num_sms) grid = 2 * ctx->num_sms / slices * slices;
+    if (grid > per_sm * ctx->num_sms) grid = per_sm * ctx->num_sms / slices * slices;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(grid);
     cfg.blockDim = dim3(kThreads);
