@@ -268,6 +268,43 @@ def test_slots_are_reused(pkg, ctx, dtype):
     m.close()
 
 
+@pytest.mark.parametrize("layer,width", [
+    (parallel(heads=12, kv_heads=3, dim=64, vdim=64, rot=64), 128),
+    (parallel(heads=14, kv_heads=2, dim=128, vdim=128, rot=64, scale=0.2), 128),
+    (delta(heads=12, kv_heads=6, dim=64, vdim=128), 128),
+    (delta(heads=24, kv_heads=24, dim=64, vdim=128), 128),
+    (delta(heads=16, kv_heads=4, dim=128, vdim=128), 128),
+    (delta(heads=40, kv_heads=20, dim=32, vdim=128), 128),
+    (mamba(inner=1300, state=16, ff=2600), 96)])
+def test_large_steps_equal_small_ones(pkg, ctx, layer, width):
+    """Steps of thousands of rows - persistent kernels with several items per CTA, paired-CTA products with the exact
+    gelu in their epilogue, the delta rule's wider column groups - against each sequence alone."""
+    cfg = config([layer], width=width, vocab=300)
+    n = 12
+    m, _ = model(pkg, ctx, cfg, "bfloat16", seed=16, max_slots=n, max_seq=384, max_rows=4096)
+    toks = [tokens(cfg, 200 + 13 * i, seed=i) for i in range(n)]
+    slots = [m.open() for _ in range(n)]
+    first = [len(t) // 3 + i for i, t in enumerate(toks)]
+    m.step([(s, t[:k]) for s, t, k in zip(slots, toks, first)])
+    rest = [t[k:] for t, k in zip(toks, first)]
+    together = m.step(list(zip(slots, rest)), want=range(sum(map(len, rest))))
+    for s in slots:
+        m.close_slot(s)
+    # all of them once more, in one step from their start
+    slots = [m.open() for _ in range(n)]
+    whole = m.step(list(zip(slots, toks)), want=range(sum(map(len, toks))))
+    for s in slots:
+        m.close_slot(s)
+    r = w = 0
+    for i, t in enumerate(toks):
+        alone = run(m, t, [64])
+        check(together[r:r + len(rest[i])], alone[first[i]:], TOL["bfloat16"], f"sequence {i}, continued")
+        check(whole[w:w + len(t)], alone, TOL["bfloat16"], f"sequence {i}, whole")
+        r += len(rest[i])
+        w += len(t)
+    m.close()
+
+
 def test_long_decoding(pkg, ctx):
     cfg = config([delta(), parallel(), mamba(ff=40)])
     m, w = model(pkg, ctx, cfg, "bfloat16", seed=11, max_seq=600)
