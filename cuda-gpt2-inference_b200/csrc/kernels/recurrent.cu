@@ -359,6 +359,13 @@ delta_prep_kernel(const DeltaArgs a) {
     };
     const float qscale = rsqrtf((float)a.D);
     const int per = a.H / a.G;
+    // the gates of the run's tokens and heads, side by side
+    for (int i = lane; i < (t1 - t0) * per; i += 32) {
+        const int t = t0 + i / per, h = g * per + i % per;
+        const float* gr = a.gates + (size_t)(sd.row0 + t) * a.ldg;
+        const float decay = expf(__ldg(a.negA + h) * softplusf_(gr[a.a_col + h] + __ldg(a.dt_bias + h)));
+        *reinterpret_cast<float2*>(a.coef + (size_t)(sd.row0 + t) * a.H + h) = make_float2(decay, sigmoidf_(gr[a.b_col + h]));
+    }
     float w[2][V][W], win[2][V][W];  // weights and the window of earlier inputs
     if (TAPS > 0) {
 #pragma unroll
@@ -432,12 +439,7 @@ delta_prep_kernel(const DeltaArgs a) {
                 for (int i = 0; i < V; ++i)
                     if (lane + i * 32 < a.Dl) row[base[x] + lane + i * 32] = in[u][x][i] * r[x];
             const float kq = sum[u][2] * r[0] * r[1];
-            const float* gr = a.gates + (size_t)(sd.row0 + t) * a.ldg;
-            for (int j = lane; j < per; j += 32) {
-                const int h = g * per + j;
-                const float decay = expf(__ldg(a.negA + h) * softplusf_(gr[a.a_col + h] + __ldg(a.dt_bias + h)));
-                a.coef[(size_t)(sd.row0 + t) * a.H + h] = make_float4(decay, sigmoidf_(gr[a.b_col + h]), kq, 0.f);
-            }
+            for (int j = lane; j < per; j += 32) a.coef[(size_t)(sd.row0 + t) * a.H + g * per + j].z = kq;
         }
     }
     if (t1 == sd.n)  // the last inputs are the history of the next step
