@@ -1,4 +1,4 @@
-"""Plain numpy restatement of the layered decoders (Vunolorn): one function per mechanism, token by
+"""Plain numpy restatement of the layered decoders (Vunolorn, Pumotar): one function per mechanism, token by
 token, no cache and no batching - a whole sequence in, the logits of every position out.
 
 TEST INFRASTRUCTURE ONLY, like oracle.py: the tests and the smoke check compare the library with
@@ -36,6 +36,17 @@ def gelu_erf(z):
     return 0.5 * z * (1.0 + _erf(z / math.sqrt(2.0)).astype(z.dtype))
 
 
+def gelu_tanh(z):
+    return 0.5 * z * (1.0 + np.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def clamped_swish_gate(g, u, limit):
+    """Gate bounded above, linear part on both sides; the linear part counts from one."""
+    g = np.minimum(g, limit)
+    u = np.clip(u, -limit, limit)
+    return g * sigmoid(1.702 * g) * (u + 1.0)
+
+
 # ---------------------------------------------------------------- norms
 def rms_norm(x, eps, weight=None):
     y = x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps)
@@ -68,6 +79,19 @@ def rotate_half(x, dims, base, positions):
     c, s = np.cos(a).astype(x.dtype)[:, None, :], np.sin(a).astype(x.dtype)[:, None, :]
     u, v = x[..., :half], x[..., half:dims]
     return np.concatenate([u * c - v * s, v * c + u * s, x[..., dims:]], axis=-1)
+
+
+def rotate_pairs(x, base, positions):
+    """x [T, heads, dims]: dimensions 2i and 2i + 1 turn by position * base^(-2i/dims)."""
+    dims = x.shape[-1]
+    y = np.empty_like(x)
+    for i in range(dims // 2):
+        a = positions.astype(np.float64) * float(base) ** (-2.0 * i / dims)
+        c, s = np.cos(a).astype(x.dtype)[:, None], np.sin(a).astype(x.dtype)[:, None]
+        u, v = x[..., 2 * i], x[..., 2 * i + 1]
+        y[..., 2 * i] = u * c - v * s
+        y[..., 2 * i + 1] = v * c + u * s
+    return y
 
 
 def softmax_attention(q, k, v, scale):
@@ -107,6 +131,23 @@ def gated_delta_rule(q, k, v, g, beta):
             u = beta[t, h] * (v[t, h] - kk @ S[h])
             S[h] = S[h] + np.outer(kk, u)
             o[t, h] = qq @ S[h]
+    return o
+
+
+def channel_delta_rule(q, k, v, g, beta):
+    """The delta rule with a decay per key channel: q, k [T, G, D]; v [T, H, Dv]; g [T, H, D]; beta [T, H].
+    Row d of a head's state is multiplied by g[d] before the token is written."""
+    T, H, Dv = v.shape
+    per = H // q.shape[1]
+    S = np.zeros((H, q.shape[2], Dv), v.dtype)
+    o = np.zeros_like(v)
+    for t in range(T):
+        for h in range(H):
+            kk, qq = k[t, h // per], q[t, h // per]
+            S[h] = g[t, h][:, None] * S[h]
+            u = beta[t, h] * (v[t, h] - S[h].T @ kk)
+            S[h] = S[h] + kk[:, None] * u[None, :]
+            o[t, h] = S[h].T @ qq
     return o
 
 
@@ -167,16 +208,67 @@ def mixer_parallel(h, w, p, m, eps):
             + m["right_scale"] * mixer_min_gru(h, w, p + ".right", m["right"], eps))
 
 
-MIXERS = {"mamba1": mixer_mamba1, "delta": mixer_delta, "parallel": mixer_parallel}
+def mixer_latent_attention(h, w, p, m, eps):
+    """Keys and values of all heads come from one low-rank latent per token; the rotated part of the key is
+    shared by the heads."""
+    T, H, D, Dr, Dv, R = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    pos, base = np.arange(T), m["rot"]["base"]
+    q = (h @ w[p + ".q"].T).reshape(T, H, D + Dr)
+    q = np.concatenate([q[..., :D], rotate_pairs(q[..., D:], base, pos)], axis=-1)
+    kv = h @ w[p + ".dkv"].T
+    c = rms_norm(kv[:, :R], eps, w[p + ".dkv.norm"])
+    k_rot = np.broadcast_to(rotate_pairs(kv[:, None, R:], base, pos), (T, H, Dr))
+    k = np.concatenate([(c @ w[p + ".uk"].T).reshape(T, H, D), k_rot], axis=-1)
+    v = (c @ w[p + ".uv"].T).reshape(T, H, Dv)
+    return softmax_attention(q, k, v, m["scale"]).reshape(T, H * Dv) @ w[p + ".o"].T
 
 
+def mixer_channel_delta(h, w, p, m, eps):
+    T, H, G, D, Dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q, k, v = (short_conv_silu(h @ w[f"{p}.{n}"].T, w[f"{p}.{n}.conv"]) for n in "qkv")
+    q = unit_norm(q.reshape(T, G, D)) * D ** -0.5
+    k = unit_norm(k.reshape(T, G, D))
+    beta = sigmoid(h @ w[p + ".b"].T)
+    a = (h @ w[p + ".a1"].T) @ w[p + ".a2"].T
+    g = np.exp(-np.exp(w[p + ".A_log"])[None, :, None] * softplus(a + w[p + ".dt_bias"]).reshape(T, H, D))
+    o = channel_delta_rule(q, k, v.reshape(T, H, Dv), g, beta)
+    gate = sigmoid((h @ w[p + ".g1"].T) @ w[p + ".g2"].T).reshape(T, H, Dv)
+    return (rms_norm(o, eps, w[p + ".norm"]) * gate).reshape(T, H * Dv) @ w[p + ".o"].T
+
+
+MIXERS = {"mamba1": mixer_mamba1, "delta": mixer_delta, "parallel": mixer_parallel,
+          "latent_attention": mixer_latent_attention, "channel_delta": mixer_channel_delta}
+
+
+# ---------------------------------------------------------------- feed-forward
 def dense_mlp(h, w, p):
     return gelu_erf(h @ w[p + ".up"].T) @ w[p + ".down"].T
 
 
-def forward(cfg, w, tokens, layer_outputs=None):
-    """Logits [T, vocab] of a whole sequence; the residual stream after every layer is appended to
-    layer_outputs if a list is given."""
+def gated_mlp(h, w, p):
+    return (gelu_tanh(h @ w[p + ".gate"].T) * (h @ w[p + ".up"].T)) @ w[p + ".down"].T
+
+
+def clamped_mlp(h, w, p, limit):
+    return clamped_swish_gate(h @ w[p + ".gate"].T, h @ w[p + ".up"].T, limit) @ w[p + ".down"].T
+
+
+def table_experts(h, w, p, m, tokens):
+    """Every token id has its experts in a table; they count alike.  The shared expert is weighed by a gate."""
+    top = m["router"]["top"]
+    table = np.asarray(w[p + ".table"]).astype(np.int64)
+    y = np.zeros_like(h)
+    for t, tok in enumerate(tokens):
+        for e in table[tok]:
+            y[t] += clamped_mlp(h[t:t + 1], w, f"{p}.e{e}", m["expert"]["limit"])[0] / top
+    if m.get("shared"):
+        gate = sigmoid(h @ w[p + ".shared.sg"].T)
+        y = y + gate * clamped_mlp(h, w, p + ".shared", m["shared"]["limit"])
+    return y
+
+
+# ---------------------------------------------------------------- models
+def forward_vunolorn(cfg, w, tokens, layer_outputs=None):
     eps = cfg["norm"]["eps"]
     x = w["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]
     for i, layer in enumerate(cfg["layers"]):
@@ -189,6 +281,39 @@ def forward(cfg, w, tokens, layer_outputs=None):
         if layer_outputs is not None:
             layer_outputs.append(x.copy())
     return rms_norm(x, eps, w["final.norm"]) @ w["head"].T
+
+
+def layer_runs(cfg):
+    """The order in which the layers run: those of the loop several times over."""
+    n, loop = len(cfg["layers"]), cfg.get("loop")
+    if not loop:
+        return list(range(n))
+    body = list(range(loop["start"], loop["stop"]))
+    return list(range(loop["start"])) + body * loop["times"] + list(range(loop["stop"], n))
+
+
+def forward_pumotar(cfg, w, tokens, layer_outputs=None):
+    eps, tokens = cfg["norm"]["eps"], np.asarray(tokens)
+    x = w["embed"][tokens] * cfg["embedding"]["scale"]
+    for i in layer_runs(cfg):
+        p, layer = f"l{i}", cfg["layers"][i]
+        x = x + MIXERS[layer["type"]](rms_norm(x, eps, 1 + w[p + ".norm1"]), w, p + ".mix", layer["mixer"], eps)
+        mlp = layer["mlp"]
+        if mlp is not None:
+            h = rms_norm(x, eps, 1 + w[p + ".norm2"])
+            x = x + (gated_mlp(h, w, p + ".mlp") if mlp["kind"] == "dense" else table_experts(h, w, p + ".mlp", mlp, tokens))
+        if layer_outputs is not None:
+            layer_outputs.append(x.copy())
+    return rms_norm(x, eps, 1 + w["final.norm"]) @ w["embed"].T
+
+
+DESIGNS = {"Vunolorn": forward_vunolorn, "Pumotar": forward_pumotar}
+
+
+def forward(cfg, w, tokens, layer_outputs=None):
+    """Logits [T, vocab] of a whole sequence; the residual stream after every layer run is appended to
+    layer_outputs if a list is given."""
+    return DESIGNS[cfg["architecture"]](cfg, w, tokens, layer_outputs)
 
 
 # ---------------------------------------------------------------- random models
