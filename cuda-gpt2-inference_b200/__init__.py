@@ -738,7 +738,8 @@ class Decoder:
     dtype "bfloat16": bf16 weights and matrix products, fp32 residual, norms, scores and recurrences;
     "float32": everything in fp32.  max_rows tokens run at a time (default: max_seq, at most 8192)."""
     ARITHMETIC = {"bfloat16": 0, "float32": 1}
-    ARCHITECTURES = ("Vunolorn",)
+    ARCHITECTURES = ("Vunolorn", "Pumotar")
+    TENSOR_TYPES = {"uint16": 0, "float32": 1, "int32": 2}
 
     def __init__(self, ctx: Context, config, dtype: str = "bfloat16", max_slots: int = 16, max_seq: int = 4096, max_rows: int | None = None):
         import json
@@ -769,14 +770,14 @@ class Decoder:
         self.ctx.check(lib().b200_decoder_load_safetensors(self._h, os.fsencode(path)), "load_safetensors")
 
     def load_tensors(self, tensors):
-        """{name: numpy array}: float32, or uint16 holding bf16 bits."""
+        """{name: numpy array}: float32, uint16 holding bf16 bits, or int32 (tables)."""
         import numpy as np
         for name, a in tensors.items():
             a = np.ascontiguousarray(a)
-            if a.dtype not in (np.float32, np.uint16):
-                raise B200Error(f"{name}: float32 or bf16 bits as uint16, not {a.dtype}")
+            if a.dtype.name not in self.TENSOR_TYPES:
+                raise B200Error(f"{name}: float32, bf16 bits as uint16 or int32, not {a.dtype}")
             shape = (C.c_long * a.ndim)(*a.shape)
-            self.ctx.check(lib().b200_decoder_set_tensor(self._h, name.encode(), _ptr(a), int(a.dtype == np.float32), shape, a.ndim), "set_tensor")
+            self.ctx.check(lib().b200_decoder_set_tensor(self._h, name.encode(), _ptr(a), self.TENSOR_TYPES[a.dtype.name], shape, a.ndim), "set_tensor")
         self.ctx.check(lib().b200_decoder_finish_load(self._h), "finish_load")
 
     def set_graph(self, on: bool):

@@ -29,6 +29,8 @@ DECODER_SOURCES = [
     "kernels/gemm_fp32.cu",
     "kernels/gemm_decode.cu",
     "kernels/recurrent.cu",
+    "kernels/experts.cu",
+    "kernels/attention_latent.cu",
     "kernels/attention_cached.cu",
     "driver/decoder.cu",
 ]

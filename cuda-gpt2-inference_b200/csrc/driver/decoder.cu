@@ -22,6 +22,7 @@
 #include <stdexcept>
 #include <string>
 #include <vector>
+#include <cuda_fp16.h>
 #include "../api/ctx.h"
 #include "../kernels/decoder_kernels.h"
 #include "json.h"
@@ -35,31 +36,42 @@ namespace {
 // What the models of one architecture have in common and config.json does not say.
 struct Design {
     const char* name;
-    int mlp_act;        // of a dense feed-forward
+    int mlp_act;        // of a dense feed-forward: down(act(up)) ...
+    int mlp_gate;       // ... or, not GATE_NONE, down(act(gate) * up)
     bool qk_norm;       // attention: per-head RMS norm of queries and keys, with weights
     bool value_norm;    // attention: values divided by their root mean square
+    bool post_norm;     // an RMS norm behind every sublayer too
+    float norm_offset;  // added to the stored weights of the norms in front of the sublayers and of the last one
+    bool tied_head;     // the logits' matrix is the embedding table
 };
 const Design kDesigns[] = {
-    {"Vunolorn", ACT_GELU_ERF, true, true},
+    {"Vunolorn", ACT_GELU_ERF, GATE_NONE, true, true, true, 0.f, false},
+    {"Pumotar", ACT_NONE, GATE_GELU_TANH, false, false, false, 1.f, true},
 };
 
-enum MixerKind { MIX_MAMBA1, MIX_DELTA, MIX_PARALLEL };
+enum MixerKind { MIX_MAMBA1, MIX_DELTA, MIX_PARALLEL, MIX_LATENT, MIX_CHANNEL_DELTA };
+enum MlpKind { MLP_NONE, MLP_DENSE, MLP_EXPERTS };
 
 struct AttentionSpec { int heads, kv_heads, dim, vdim, rot_dims; double rot_base; float scale; };
 struct LayerSpec {
     MixerKind kind;
     int conv = 0, dt_rank = 0, inner = 0, state = 0;           // mamba1 (and conv of delta)
-    int heads = 0, kv_heads = 0, dim = 0, vdim = 0;            // delta
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0;            // delta, channel_delta; latent_attention (no kv_heads)
+    int kv_rank = 0, rot_dim = 0; double rot_base = 0; float scale = 0.f;  // latent_attention
     AttentionSpec att{};                                       // parallel, left
     int gru_width = 0;                                         // parallel, right
     float left_scale = 1.f, right_scale = 1.f;
-    int ff = 0;                                                // 0: no feed-forward
+    MlpKind mlp = MLP_NONE;
+    int ff = 0;                                                // dense: its width; experts: of one of them
+    int experts = 0, top = 0, shared_ff = 0;                   // (shared_ff 0: no shared expert)
+    float limit = 0.f, shared_limit = 0.f;
 };
 struct ModelSpec {
     const Design* design = nullptr;
     int vocab = 0, width = 0;
     float embed_scale = 1.f, eps = 1e-5f;
     std::vector<LayerSpec> layers;
+    std::vector<int> order;  // the layers in the order in which they run; one that is looped occurs several times
 };
 
 void positive(int v, const char* what) { if (v < 1) throw std::runtime_error(std::string("config: '") + what + "' must be positive"); }
@@ -85,6 +97,14 @@ AttentionSpec parse_attention(const Json& m) {
     return a;
 }
 
+void parse_delta(const Json& m, LayerSpec& l) {
+    l.conv = m.integer("conv"); l.heads = m.integer("heads"); l.kv_heads = m.integer("kv_heads");
+    l.dim = m.integer("dim"); l.vdim = m.integer("vdim");
+    positive(l.conv, "conv"); head_groups(l.heads, l.kv_heads); positive(l.dim, "dim"); positive(l.vdim, "vdim");
+    if (!delta_state_pad(l.dim)) throw std::runtime_error("config: delta 'dim' beyond 256");
+    if (l.vdim > 2048) throw std::runtime_error("config: delta 'vdim' beyond 2048");
+}
+
 // mixer registry: config name -> reader of its sizes
 struct MixerType {
     const char* name;
@@ -97,13 +117,20 @@ const MixerType kMixers[] = {
          positive(l.conv, "conv"); positive(l.dt_rank, "dt_rank"); positive(l.inner, "inner"); positive(l.state, "state");
          if (!selective_state_pad(l.state)) throw std::runtime_error("config: mamba1 'state' beyond 256");
      }},
-    {"delta", [](const Json& m, LayerSpec& l) {
-         l.kind = MIX_DELTA;
-         l.conv = m.integer("conv"); l.heads = m.integer("heads"); l.kv_heads = m.integer("kv_heads");
-         l.dim = m.integer("dim"); l.vdim = m.integer("vdim");
-         positive(l.conv, "conv"); head_groups(l.heads, l.kv_heads); positive(l.dim, "dim"); positive(l.vdim, "vdim");
-         if (!delta_state_pad(l.dim)) throw std::runtime_error("config: delta 'dim' beyond 256");
-         if (l.vdim > 2048) throw std::runtime_error("config: delta 'vdim' beyond 2048");
+    {"delta", [](const Json& m, LayerSpec& l) { l.kind = MIX_DELTA; parse_delta(m, l); }},
+    {"channel_delta", [](const Json& m, LayerSpec& l) { l.kind = MIX_CHANNEL_DELTA; parse_delta(m, l); }},
+    {"latent_attention", [](const Json& m, LayerSpec& l) {
+         l.kind = MIX_LATENT;
+         l.heads = m.integer("heads"); l.dim = m.integer("dim"); l.vdim = m.integer("vdim");
+         l.kv_rank = m.integer("kv_rank"); l.rot_dim = m.integer("rot_dim");
+         positive(l.heads, "heads"); positive(l.dim, "dim"); positive(l.vdim, "vdim"); positive(l.kv_rank, "kv_rank"); positive(l.rot_dim, "rot_dim");
+         l.scale = (float)m.number("scale");
+         if (!(l.scale > 0.f)) throw std::runtime_error("config: attention 'scale' must be positive");
+         const Json& r = m.at("rot");
+         l.rot_base = r.number("base");
+         if (r.integer("dims") != l.rot_dim || l.rot_dim % 2) throw std::runtime_error("config: rot.dims must be rot_dim, and even");
+         if (l.dim + l.rot_dim > 256 || l.vdim > 256) throw std::runtime_error("config: attention heads of more than 256 dimensions");
+         if (l.kv_rank > 512 || !latent_row_pad(l.kv_rank + l.rot_dim)) throw std::runtime_error("config: 'kv_rank' beyond 512, or with rot_dim beyond 640");
      }},
     {"parallel", [](const Json& m, LayerSpec& l) {
          l.kind = MIX_PARALLEL;
@@ -112,6 +139,38 @@ const MixerType kMixers[] = {
          positive(l.gru_width, "width");
          l.left_scale = (float)m.number("left_scale");
          l.right_scale = (float)m.number("right_scale");
+     }},
+};
+
+// feed-forward registry
+struct MlpType {
+    const char* name;
+    void (*parse)(const Json&, LayerSpec&);
+};
+float parse_limit(const Json& m) {
+    const float v = (float)m.number("limit");
+    if (!(v > 0.f)) throw std::runtime_error("config: 'limit' must be positive");
+    return v;
+}
+const MlpType kMlps[] = {
+    {"dense", [](const Json& m, LayerSpec& l) {
+         l.mlp = MLP_DENSE;
+         l.ff = m.integer("ff");
+         positive(l.ff, "ff");
+     }},
+    {"moe", [](const Json& m, LayerSpec& l) {
+         l.mlp = MLP_EXPERTS;
+         const Json &e = m.at("expert"), &r = m.at("router");
+         l.ff = e.integer("ff"); l.limit = parse_limit(e);
+         l.experts = r.integer("experts"); l.top = r.integer("top");
+         positive(l.ff, "ff"); positive(l.experts, "experts"); positive(l.top, "top");
+         if (l.top > l.experts) throw std::runtime_error("config: router.top beyond router.experts");
+         if (l.top > 16 || l.experts > 8192) throw std::runtime_error("config: router.top beyond 16 or router.experts beyond 8192");
+         if (m.has("shared") && !m.at("shared").is_null()) {
+             const Json& s = m.at("shared");
+             l.shared_ff = s.integer("ff"); l.shared_limit = parse_limit(s);
+             positive(l.shared_ff, "ff");
+         }
      }},
 };
 
@@ -138,12 +197,26 @@ ModelSpec parse_config(const char* text) {
         mt->parse(lj.at("mixer"), l);
         const Json& mlp = lj.at("mlp");
         if (!mlp.is_null()) {
-            if (mlp.string("kind") != "dense") throw std::runtime_error("config: unknown feed-forward '" + mlp.string("kind") + "'");
-            l.ff = mlp.integer("ff");
-            positive(l.ff, "ff");
+            const std::string& kind = mlp.string("kind");
+            const MlpType* ft = nullptr;
+            for (const MlpType& t : kMlps)
+                if (kind == t.name) ft = &t;
+            if (!ft) throw std::runtime_error("config: unknown feed-forward '" + kind + "'");
+            ft->parse(mlp, l);
         }
         s.layers.push_back(l);
     }
+    const int n = (int)s.layers.size();
+    int start = 0, stop = 0, times = 1;
+    if (j.has("loop") && !j.at("loop").is_null()) {
+        const Json& lp = j.at("loop");
+        start = lp.integer("start"); stop = lp.integer("stop"); times = lp.integer("times");
+        if (start < 0 || stop < start || stop > n || times < 1) throw std::runtime_error("config: 'loop' must name layers start .. stop - 1 and run them at least once");
+    }
+    for (int i = 0; i < start; ++i) s.order.push_back(i);
+    for (int t = 0; t < times; ++t)
+        for (int i = start; i < stop; ++i) s.order.push_back(i);
+    for (int i = stop; i < n; ++i) s.order.push_back(i);
     return s;
 }
 
@@ -151,7 +224,16 @@ ModelSpec parse_config(const char* text) {
 // A matrix [N, K] in the model's element type; N and K are padded with zeros.
 struct Matrix { void* w = nullptr; int N = 0, K = 0; float* bias = nullptr; };
 
-struct Mlp { Matrix up, down; };
+// Gated feed-forwards: up holds gates and linear parts, blocks of 32 rows of either in turn, [2 F].  Experts: up and down are
+// stacks of one matrix per expert (N, K of one).
+struct Mlp {
+    Matrix up, down, shared_up, shared_down;
+    int gate = GATE_NONE;
+    float* shared_gate = nullptr;
+    int* table = nullptr;
+    MoeRoute route{};  // of a step's pairs
+};
+// a layer run: the passes of a looped layer share the weights, each has its own state
 struct Layer {
     const LayerSpec* spec = nullptr;
     float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
@@ -162,11 +244,18 @@ struct Layer {
     float *conv_w = nullptr, *conv_b = nullptr, *A2 = nullptr, *dt_b = nullptr, *D = nullptr;
     int np = 0, sp = 0, rank_p = 0;
     // delta: in = [q: G*Dl | k: G*Dl | v: H*Dvl | gate: H*Dvl | a: H | b: H]
+    // channel_delta: in = [q | k | v | a1: low_a | g1: low_g | b: H], low = a2 and g2 side by side (each zero on the other's columns)
+    Matrix low;
+    int low_col = 0, low_a = 0, low_g = 0, gate_row = 0;
     float *negA = nullptr, *dt_bias = nullptr, *head_norm = nullptr;
     int Dl = 0, Dvl = 0, k_col = 0, v_col = 0, gate_col = 0, a_col = 0, b_col = 0;
     // parallel: in = [q | k | v | z | x | g], o over [attention: att_p | minGRU]
     CachedAttention att{};
     int z_col = 0, x_col = 0, g_col = 0, att_p = 0;
+    // latent_attention: in = [q | dkv]; kv: a cached row -> its expanded keys and values, which flat addresses
+    LatentAttention lat{};
+    CachedAttention flat{};
+    Matrix kv;
     // what the slots hold
     float *hist = nullptr, *S = nullptr;
 };
@@ -174,6 +263,8 @@ struct Layer {
 struct Slot { bool open = false; int len = 0, bank = 0; };
 
 int round4(int n) { return (n + 3) & ~3; }
+int round8(int n) { return (n + 7) & ~7; }
+int gate_pad(int F) { return F < 64 ? 64 : (F + 31) & ~31; }  // columns of a gated feed-forward of width F
 
 }  // namespace
 
@@ -187,7 +278,7 @@ struct b200_decoder {
     bool use_graph = true;
     TensorStore* store = nullptr;
     std::vector<void*> owned;             // every device allocation
-    std::vector<Layer> layers;
+    std::vector<Layer> layers;            // in the order in which they run
     void* embed = nullptr;
     float* final_norm = nullptr;
     Matrix head;
@@ -196,11 +287,19 @@ struct b200_decoder {
     // activations of the general path
     float *x = nullptr, *proj = nullptr, *y = nullptr, *aux = nullptr, *wide = nullptr;
     void *h = nullptr, *conv = nullptr, *mix = nullptr, *q = nullptr, *low = nullptr;
+    float *gates = nullptr;                          // low-rank decays and output gates
+    void *ql = nullptr, *lat = nullptr, *kv = nullptr;  // latent queries; latents and expanded keys and values of the step (grown on demand)
+    int kv_rows = 0, expand_from = 1;                // expand_from: tokens from which a sequence's step is expanded
+    void *pair_h = nullptr, *pair_mix = nullptr;     // rows of (token, expert) pairs: input, activations, outputs
+    float *pair_y = nullptr, *raw = nullptr, *shared_gate = nullptr;
+    MoeRoute* routes = nullptr;                      // of the layers with experts
+    int num_routes = 0, max_experts = 0;
     float* logits = nullptr;
     int logits_rows = 0;
     // ... and of the decode path (16 rows: fp32, or split rows of the same size)
     float *dx = nullptr, *dproj = nullptr, *dy = nullptr, *daux = nullptr, *dlogits = nullptr;
-    void *dh = nullptr, *dmix = nullptr, *dconv = nullptr;
+    void *dh = nullptr, *dmix = nullptr, *dconv = nullptr, *dql = nullptr, *dpair_mix = nullptr;
+    float *dpair_y = nullptr, *dshared_gate = nullptr;
     // step descriptors: a ring of pinned buffers, one device buffer per path
     static constexpr int kRing = 8;
     int* pinned[kRing] = {};
@@ -245,36 +344,54 @@ void* upload(b200_decoder* m, const void* src, size_t bytes) {
 // Assembles a padded matrix from blocks of tensors, then uploads it in the model's element type.
 class MatrixBuilder {
    public:
-    MatrixBuilder(b200_decoder* m, int N, int K) : m_(m), N_(N), K_(K) {
+    // fp16: of a 16-bit model, elements in fp16 instead of bf16
+    MatrixBuilder(b200_decoder* m, size_t N, int K, bool fp16 = false) : m_(m), N_(N), K_(K), fp16_(fp16) {
         if (m->f32) f_.assign((size_t)N * K, 0.f);
         else h_.assign((size_t)N * K, 0);
     }
     // rows `rows` of t (columns [0, cols)) to (row0, col0), times scale
-    void put(const HostTensor& t, int src_row0, int rows, int cols, int row0, int col0) {
+    void put(const HostTensor& t, int src_row0, int rows, int cols, size_t row0, int col0) {
         for (int r = 0; r < rows; ++r) {
             const size_t s = (size_t)(src_row0 + r) * cols, d = (size_t)(row0 + r) * K_ + col0;
             if (m_->f32) for (int c = 0; c < cols; ++c) f_[d + c] = t.value(s + c);
-            else if (t.f32) for (int c = 0; c < cols; ++c) h_[d + c] = bf16_bits(t.value(s + c));
+            else if (fp16_) for (int c = 0; c < cols; ++c) h_[d + c] = half_bits(t.value(s + c));
+            else if (t.type == TensorType::F32) for (int c = 0; c < cols; ++c) h_[d + c] = bf16_bits(t.value(s + c));
             else memcpy(&h_[d], t.data + 2 * s, (size_t)cols * 2);
         }
     }
-    Matrix build() {
+    void one(size_t row, int col) {
+        if (m_->f32) f_[row * K_ + col] = 1.f;
+        else h_[row * K_ + col] = fp16_ ? half_bits(1.f) : bf16_bits(1.f);
+    }
+    // gates and linear parts [F, cols], in blocks of 32 rows of either, from row0 on
+    void put_gated(const HostTensor& gate, const HostTensor& up, int F, int cols, size_t row0) {
+        for (int f = 0; f < F; f += 32) {
+            const int n = F - f < 32 ? F - f : 32;
+            put(gate, f, n, cols, row0 + 2 * f, 0);
+            put(up, f, n, cols, row0 + 2 * f + 32, 0);
+        }
+    }
+    // parts: how many matrices are stacked
+    Matrix build(int parts = 1) {
         Matrix x;
-        x.N = N_; x.K = K_;
+        x.N = (int)(N_ / parts); x.K = K_;
         x.w = m_->f32 ? upload(m_, f_.data(), f_.size() * 4) : upload(m_, h_.data(), h_.size() * 2);
         return x;
     }
 
    private:
+    static uint16_t half_bits(float v) { const __half h = __float2half_rn(v); uint16_t u; memcpy(&u, &h, 2); return u; }
     b200_decoder* m_;
-    int N_, K_;
+    size_t N_;
+    int K_;
+    bool fp16_;
     std::vector<float> f_;
     std::vector<uint16_t> h_;
 };
 
-float* vector_f32(b200_decoder* m, const HostTensor& t, size_t padded) {
+float* vector_f32(b200_decoder* m, const HostTensor& t, size_t padded, float offset = 0.f) {
     std::vector<float> v(padded, 0.f);
-    for (size_t i = 0; i < t.count(); ++i) v[i] = t.value(i);
+    for (size_t i = 0; i < t.count(); ++i) v[i] = t.value(i) + offset;
     return static_cast<float*>(upload(m, v.data(), padded * 4));
 }
 
@@ -340,8 +457,6 @@ void load_mamba1(b200_decoder* m, Layer& L, const std::string& p) {
     for (int c = 0; c < n; ++c)
         for (int k = 0; k < s.state; ++k) A2[(size_t)c * L.sp + k] = (float)(-exp((double)a.value((size_t)c * s.state + k)) * 1.4426950408889634);
     L.A2 = static_cast<float*>(upload(m, A2.data(), A2.size() * 4));
-    L.hist = static_cast<float*>(device_zeros(m, (size_t)2 * m->max_slots * (s.conv - 1) * L.np * 4));
-    L.S = static_cast<float*>(device_zeros(m, (size_t)m->max_slots * n * L.sp * 4));
 }
 
 void load_delta(b200_decoder* m, Layer& L, const std::string& p) {
@@ -351,7 +466,15 @@ void load_delta(b200_decoder* m, Layer& L, const std::string& p) {
     L.Dl = round4(D); L.Dvl = round4(Dv);
     L.k_col = G * L.Dl; L.v_col = 2 * G * L.Dl;
     L.np = L.v_col + H * L.Dvl;  // the convolved columns
-    L.gate_col = L.np; L.a_col = L.gate_col + H * L.Dvl; L.b_col = L.a_col + H;
+    const bool channel = s.kind == MIX_CHANNEL_DELTA;
+    int ra = 0, rg = 0;
+    if (channel) {
+        ra = w.rows(p + ".a1"); rg = w.rows(p + ".g1");
+        L.low_a = round8(ra); L.low_g = round8(rg);
+        L.low_col = round8(L.np); L.b_col = L.low_col + L.low_a + L.low_g;
+    } else {
+        L.gate_col = L.np; L.a_col = L.gate_col + H * L.Dvl; L.b_col = L.a_col + H;
+    }
     MatrixBuilder b(m, pad_dim(L.b_col + H), m->Cp);
     std::vector<float> taps((size_t)s.conv * L.np, 0.f);
     const struct { const char* n; int heads, dim, dim_l, col; } parts[] = {{".q", G, D, L.Dl, 0}, {".k", G, D, L.Dl, L.k_col}, {".v", H, Dv, L.Dvl, L.v_col}};
@@ -360,9 +483,22 @@ void load_delta(b200_decoder* m, Layer& L, const std::string& p) {
         for (int h = 0; h < a.heads; ++h) b.put(t, h * a.dim, a.dim, C, a.col + h * a.dim_l, 0);
         put_taps(taps, L.np, w.get(p + a.n + ".conv", {(long)a.heads * a.dim, s.conv}), a.heads * a.dim, s.conv, a.dim, a.dim_l, a.col);
     }
-    const HostTensor& g = w.get(p + ".g", {(long)H * Dv, C});
-    for (int h = 0; h < H; ++h) b.put(g, h * Dv, Dv, C, L.gate_col + h * L.Dvl, 0);
-    b.put(w.get(p + ".a", {H, C}), 0, H, C, L.a_col, 0);
+    if (channel) {
+        b.put(w.get(p + ".a1", {ra, C}), 0, ra, C, L.low_col, 0);
+        b.put(w.get(p + ".g1", {rg, C}), 0, rg, C, L.low_col + L.low_a, 0);
+        L.gate_row = round8(H * L.Dl);
+        MatrixBuilder low(m, pad_dim(L.gate_row + H * L.Dvl), pad_dim(L.low_a + L.low_g));
+        const HostTensor &a2 = w.get(p + ".a2", {(long)H * D, ra}), &g2 = w.get(p + ".g2", {(long)H * Dv, rg});
+        for (int h = 0; h < H; ++h) {
+            low.put(a2, h * D, D, ra, h * L.Dl, 0);
+            low.put(g2, h * Dv, Dv, rg, L.gate_row + h * L.Dvl, L.low_a);
+        }
+        L.low = low.build();
+    } else {
+        const HostTensor& g = w.get(p + ".g", {(long)H * Dv, C});
+        for (int h = 0; h < H; ++h) b.put(g, h * Dv, Dv, C, L.gate_col + h * L.Dvl, 0);
+        b.put(w.get(p + ".a", {H, C}), 0, H, C, L.a_col, 0);
+    }
     b.put(w.get(p + ".b", {H, C}), 0, H, C, L.b_col, 0);
     L.in = b.build();
     MatrixBuilder o(m, m->Cp, pad_dim(H * Dv));
@@ -373,10 +509,79 @@ void load_delta(b200_decoder* m, Layer& L, const std::string& p) {
     std::vector<float> negA(H);
     for (int h = 0; h < H; ++h) negA[h] = (float)-exp((double)a.value(h));
     L.negA = static_cast<float*>(upload(m, negA.data(), negA.size() * 4));
-    L.dt_bias = vector_f32(m, w.get(p + ".dt_bias", {H}), H);
+    if (channel) {
+        const HostTensor& t = w.get(p + ".dt_bias", {(long)H * D});
+        std::vector<float> bias((size_t)H * L.Dl, 0.f);
+        for (int h = 0; h < H; ++h)
+            for (int d = 0; d < D; ++d) bias[(size_t)h * L.Dl + d] = t.value((size_t)h * D + d);
+        L.dt_bias = static_cast<float*>(upload(m, bias.data(), bias.size() * 4));
+    } else L.dt_bias = vector_f32(m, w.get(p + ".dt_bias", {H}), H);
     L.head_norm = vector_f32(m, w.get(p + ".norm", {Dv}), Dv);
-    L.hist = static_cast<float*>(device_zeros(m, (size_t)2 * m->max_slots * (s.conv - 1) * L.np * 4));
-    L.S = static_cast<float*>(device_zeros(m, (size_t)m->max_slots * H * Dv * delta_state_pad(D) * 4));
+}
+
+void load_latent(b200_decoder* m, Layer& L, const std::string& p) {
+    const LayerSpec& s = *L.spec;
+    const TensorStore& w = *m->store;
+    const int C = m->C, H = s.heads, D = s.dim, Dr = s.rot_dim, Dv = s.vdim, R = s.kv_rank;
+    LatentAttention& c = L.lat;
+    c.H = H; c.D = D; c.Dr = Dr; c.Dv = Dv; c.R = R;
+    c.Lp = latent_row_pad(R + Dr); c.Tp = m->Tp; c.Dp = attention_pad(D + Dr); c.Dvp = attention_pad(Dv); c.Rp = round8(R);
+    c.q_col = 0; c.c_col = round8(H * (D + Dr));
+    c.rot = rotation_table(m, Dr, s.rot_base);
+    c.scale = s.scale; c.eps = m->spec.eps;
+    MatrixBuilder b(m, pad_dim(c.c_col + R + Dr), m->Cp);
+    b.put(w.get(p + ".q", {(long)H * (D + Dr), C}), 0, H * (D + Dr), C, 0, 0);
+    b.put(w.get(p + ".dkv", {(long)R + Dr, C}), 0, R + Dr, C, c.c_col, 0);
+    L.in = b.build();
+    c.c_norm = vector_f32(m, w.get(p + ".dkv.norm", {R}), R);
+    const HostTensor &uk = w.get(p + ".uk", {(long)H * D, R}), &uv = w.get(p + ".uv", {(long)H * Dv, R});
+    // expanded: per head [W_uk c | rotated part, passed on | zeros], then all heads' [W_uv c | zeros]
+    MatrixBuilder kv(m, (size_t)H * (c.Dp + c.Dvp), c.Lp, true);
+    for (int h = 0; h < H; ++h) {
+        kv.put(uk, h * D, D, R, (size_t)h * c.Dp, 0);
+        for (int j = 0; j < Dr; ++j) kv.one((size_t)h * c.Dp + D + j, R + j);
+        kv.put(uv, h * Dv, Dv, R, (size_t)H * c.Dp + h * c.Dvp, 0);
+    }
+    L.kv = kv.build();
+    CachedAttention& f = L.flat;
+    f.H = f.G = H; f.D = D + Dr; f.Dv = Dv; f.Dp = c.Dp; f.Dvp = c.Dvp; f.Tp = m->Tp;
+    f.scale = s.scale; f.eps = m->spec.eps; f.out_scale = 1.f; f.ld_kv = L.kv.N;
+    if (!m->f32) {
+        MatrixBuilder k(m, (size_t)H * D, c.Rp), v(m, (size_t)H * Dv, c.Rp);
+        k.put(uk, 0, H * D, R, 0, 0);
+        v.put(uv, 0, H * Dv, R, 0, 0);
+        c.Wuk = static_cast<const uint16_t*>(k.build().w);
+        c.Wuv = static_cast<const uint16_t*>(v.build().w);
+    }
+    MatrixBuilder o(m, m->Cp, pad_dim(H * Dv));
+    o.put(w.get(p + ".o", {C, (long)H * Dv}), 0, C, H * Dv, 0, 0);
+    L.o = o.build();
+}
+
+// what every slot holds of a layer run
+void allocate_state(b200_decoder* m, Layer& L) {
+    const LayerSpec& s = *L.spec;
+    const size_t slots = m->max_slots;
+    auto floats = [&](size_t n) { return static_cast<float*>(device_zeros(m, n * 4)); };
+    switch (s.kind) {
+        case MIX_MAMBA1:
+            L.hist = floats(2 * slots * (s.conv - 1) * L.np);
+            L.S = floats(slots * s.inner * L.sp);
+            break;
+        case MIX_DELTA:
+        case MIX_CHANNEL_DELTA:
+            L.hist = floats(2 * slots * (s.conv - 1) * L.np);
+            L.S = floats(slots * s.heads * s.vdim * delta_state_pad(s.dim));
+            break;
+        case MIX_PARALLEL:
+            L.att.K = device_zeros(m, slots * L.att.G * L.att.Tp * L.att.Dp * elem(m));
+            L.att.V = device_zeros(m, slots * L.att.G * L.att.Tp * L.att.Dvp * elem(m));
+            L.S = floats(slots * s.gru_width);
+            break;
+        case MIX_LATENT:
+            L.lat.cache = device_zeros(m, slots * L.lat.Tp * L.lat.Lp * elem(m));
+            break;
+    }
 }
 
 void load_parallel(b200_decoder* m, Layer& L, const std::string& p) {
@@ -419,61 +624,162 @@ void load_parallel(b200_decoder* m, Layer& L, const std::string& p) {
     }
     c.v_norm = m->spec.design->value_norm;
     c.scale = a.scale; c.eps = m->spec.eps; c.out_scale = s.left_scale;
-    c.K = device_zeros(m, (size_t)m->max_slots * c.G * c.Tp * c.Dp * elem(m));
-    c.V = device_zeros(m, (size_t)m->max_slots * c.G * c.Tp * c.Dvp * elem(m));
-    L.S = static_cast<float*>(device_zeros(m, (size_t)m->max_slots * W * 4));
+}
+
+Matrix gated_up(b200_decoder* m, const std::string& p, int F) {
+    const TensorStore& w = *m->store;
+    MatrixBuilder b(m, (size_t)2 * gate_pad(F), m->Cp);
+    b.put_gated(w.get(p + ".gate", {F, m->C}), w.get(p + ".up", {F, m->C}), F, m->C, 0);
+    return b.build();
+}
+Matrix down_matrix(b200_decoder* m, const std::string& p, int F, int Fp) {
+    MatrixBuilder b(m, m->Cp, Fp);
+    b.put(m->store->get(p + ".down", {m->C, F}), 0, m->C, F, 0, 0);
+    return b.build();
+}
+
+void load_mlp(b200_decoder* m, Layer& L, const std::string& p) {
+    const LayerSpec& s = *L.spec;
+    const TensorStore& w = *m->store;
+    const int C = m->C, F = s.ff;
+    Mlp& f = L.mlp;
+    if (s.mlp == MLP_DENSE) {
+        f.gate = m->spec.design->mlp_gate;
+        if (f.gate == GATE_NONE) {
+            MatrixBuilder up(m, pad_dim(F), m->Cp);
+            up.put(w.get(p + ".up", {F, C}), 0, F, C, 0, 0);
+            f.up = up.build();
+            f.down = down_matrix(m, p, F, pad_dim(F));
+        } else {
+            f.up = gated_up(m, p, F);
+            f.down = down_matrix(m, p, F, gate_pad(F));
+        }
+        return;
+    }
+    f.gate = GATE_CLAMP;
+    const int Fp = gate_pad(F), E = s.experts, V = m->spec.vocab;
+    MatrixBuilder up(m, (size_t)E * 2 * Fp, m->Cp), down(m, (size_t)E * m->Cp, Fp);
+    for (int e = 0; e < E; ++e) {
+        const std::string q = p + ".e" + std::to_string(e);
+        up.put_gated(w.get(q + ".gate", {F, C}), w.get(q + ".up", {F, C}), F, C, (size_t)e * 2 * Fp);
+        down.put(w.get(q + ".down", {C, F}), 0, C, F, (size_t)e * m->Cp, 0);
+    }
+    f.up = up.build(E);
+    f.down = down.build(E);
+    const HostTensor& t = w.get(p + ".table", {V, s.top}, true);
+    std::vector<int> table((size_t)V * s.top);
+    for (size_t i = 0; i < table.size(); ++i) {
+        table[i] = t.integer(i);
+        if (table[i] < 0 || table[i] >= E) throw std::runtime_error("weights: '" + p + ".table' names an expert that is not there");
+        for (size_t k = i - i % s.top; k < i; ++k)
+            if (table[k] == table[i]) throw std::runtime_error("weights: '" + p + ".table' names an expert twice for one token");
+    }
+    f.table = static_cast<int*>(upload(m, table.data(), table.size() * 4));
+    if (s.shared_ff > 0) {
+        f.shared_up = gated_up(m, p + ".shared", s.shared_ff);
+        f.shared_down = down_matrix(m, p + ".shared", s.shared_ff, gate_pad(s.shared_ff));
+        f.shared_gate = vector_f32(m, w.get(p + ".shared.sg", {1, C}), m->Cp);
+    }
+}
+
+// the most runs, and rows of padded runs, of the pairs of M tokens
+int most_runs(const b200_decoder* m, const LayerSpec& s, int M, int* rows) {
+    const int P = M * s.top, align = moe_run_rows(P, s.experts, m->f32), runs = (P + (s.experts < P ? s.experts : P) * (align - 1)) / align;
+    if (rows) *rows = runs * align;
+    return runs;
 }
 
 void load_all(b200_decoder* m) {
     const TensorStore& w = *m->store;
     const int C = m->C, V = m->spec.vocab;
+    const Design& design = *m->spec.design;
     {
-        MatrixBuilder b(m, V, m->Cp);
+        MatrixBuilder b(m, m->Vp, m->Cp);
         b.put(w.get("embed", {V, C}), 0, V, C, 0, 0);
-        m->embed = b.build().w;
+        const Matrix e = b.build();
+        m->embed = e.w;
+        if (design.tied_head) m->head = e;
     }
-    m->layers.assign(m->spec.layers.size(), Layer());
-    for (size_t i = 0; i < m->layers.size(); ++i) {
-        Layer& L = m->layers[i];
+    std::vector<Layer> layers(m->spec.layers.size());
+    std::vector<MoeRoute> routes;
+    for (size_t i = 0; i < layers.size(); ++i) {
+        Layer& L = layers[i];
         L.spec = &m->spec.layers[i];
         const std::string p = "l" + std::to_string(i);
-        L.norm1 = vector_f32(m, w.get(p + ".norm1", {C}), m->Cp);
-        L.norm1b = vector_f32(m, w.get(p + ".norm1b", {C}), m->Cp);
-        if (L.spec->kind == MIX_MAMBA1) load_mamba1(m, L, p + ".mix");
-        else if (L.spec->kind == MIX_DELTA) load_delta(m, L, p + ".mix");
-        else load_parallel(m, L, p + ".mix");
-        if (L.spec->ff > 0) {
-            const int F = L.spec->ff, Fp = pad_dim(F);
-            L.norm2 = vector_f32(m, w.get(p + ".norm2", {C}), m->Cp);
-            L.norm2b = vector_f32(m, w.get(p + ".norm2b", {C}), m->Cp);
-            MatrixBuilder up(m, Fp, m->Cp), down(m, m->Cp, Fp);
-            up.put(w.get(p + ".mlp.up", {F, C}), 0, F, C, 0, 0);
-            down.put(w.get(p + ".mlp.down", {C, F}), 0, C, F, 0, 0);
-            L.mlp.up = up.build();
-            L.mlp.down = down.build();
+        L.norm1 = vector_f32(m, w.get(p + ".norm1", {C}), m->Cp, design.norm_offset);
+        if (design.post_norm) L.norm1b = vector_f32(m, w.get(p + ".norm1b", {C}), m->Cp);
+        switch (L.spec->kind) {
+            case MIX_MAMBA1: load_mamba1(m, L, p + ".mix"); break;
+            case MIX_DELTA:
+            case MIX_CHANNEL_DELTA: load_delta(m, L, p + ".mix"); break;
+            case MIX_PARALLEL: load_parallel(m, L, p + ".mix"); break;
+            case MIX_LATENT: load_latent(m, L, p + ".mix"); break;
+        }
+        if (L.spec->mlp != MLP_NONE) {
+            L.norm2 = vector_f32(m, w.get(p + ".norm2", {C}), m->Cp, design.norm_offset);
+            if (design.post_norm) L.norm2b = vector_f32(m, w.get(p + ".norm2b", {C}), m->Cp);
+            load_mlp(m, L, p + ".mlp");
+        }
+        if (L.spec->mlp == MLP_EXPERTS) {
+            MoeRoute& r = L.mlp.route;
+            r.table = L.mlp.table; r.experts = L.spec->experts; r.top = L.spec->top;
+            int runs = 0;
+            for (int M = 1; M <= m->max_rows; ++M) { const int n = most_runs(m, *L.spec, M, nullptr); if (n > runs) runs = n; }
+            r.place = static_cast<int*>(device_zeros(m, (size_t)m->max_rows * r.top * 4));
+            r.blocks = static_cast<int*>(device_zeros(m, (size_t)(1 + runs) * 4));
+            routes.push_back(r);
+            if (r.experts > m->max_experts) m->max_experts = r.experts;
         }
     }
-    m->final_norm = vector_f32(m, w.get("final.norm", {C}), m->Cp);
-    MatrixBuilder b(m, m->Vp, m->Cp);
-    b.put(w.get("head", {V, C}), 0, V, C, 0, 0);
-    m->head = b.build();
+    m->num_routes = (int)routes.size();
+    if (m->num_routes) m->routes = static_cast<MoeRoute*>(upload(m, routes.data(), routes.size() * sizeof(MoeRoute)));
+    for (int i : m->spec.order) {
+        m->layers.push_back(layers[i]);
+        allocate_state(m, m->layers.back());
+    }
+    m->final_norm = vector_f32(m, w.get("final.norm", {C}), m->Cp, design.norm_offset);
+    if (!design.tied_head) {
+        MatrixBuilder b(m, m->Vp, m->Cp);
+        b.put(w.get("head", {V, C}), 0, V, C, 0, 0);
+        m->head = b.build();
+    }
 }
 
 // activations, sized from the loaded layers
 void allocate(b200_decoder* m) {
-    size_t proj = 0, mix = 0, conv = 0, aux = 0, wide = 0, q = 0, low = 0;
+    size_t proj = 0, mix = 0, conv = 0, aux = 0, wide = 0, q = 0, low = 0, gates = 0, ql = 0, raw = 0, decode_pair_mix = 0, top = 0;
+    size_t pair_rows = 0, pair_mix = 0;  // (pair_mix, raw: elements)
+    bool shared = false;
     auto up = [](size_t& a, size_t b) { if (b > a) a = b; };
+    const size_t M = m->max_rows, e = elem(m);
     for (const Layer& L : m->layers) {
+        const LayerSpec& s = *L.spec;
         up(proj, L.in.N);
         up(mix, L.o.K);
-        if (L.spec->ff) up(mix, L.mlp.up.N);
-        if (L.spec->kind == MIX_MAMBA1) { up(conv, L.np); up(aux, L.xp.N); up(wide, L.np); up(low, L.rank_p); }
-        else if (L.spec->kind == MIX_DELTA) { up(conv, 2 * L.np); up(wide, L.spec->heads * L.Dvl); up(aux, 4 * L.spec->heads); }  // (fp32 in either arithmetic)
-        else {
-            up(q, (size_t)L.att.H * L.att.Dp);
+        switch (s.kind) {
+            case MIX_MAMBA1: up(conv, L.np); up(aux, L.xp.N); up(wide, L.np); up(low, L.rank_p); break;
+            case MIX_CHANNEL_DELTA: up(low, L.low.K); up(gates, L.low.N);  // and
+            case MIX_DELTA: up(conv, 2 * L.np); up(wide, s.heads * L.Dvl); up(aux, 4 * s.heads); break;  // (fp32 in either arithmetic)
+            case MIX_PARALLEL: up(q, (size_t)L.att.H * L.att.Dp); break;
+            case MIX_LATENT:
+                up(q, (size_t)L.lat.H * L.lat.Dp);
+                up(ql, (size_t)L.lat.H * L.lat.Lp);
+                break;
+        }
+        if (s.mlp == MLP_DENSE) {
+            up(mix, L.mlp.down.K);
+            if (L.mlp.gate != GATE_NONE) up(raw, M * L.mlp.up.N);
+        } else if (s.mlp == MLP_EXPERTS) {
+            if (s.shared_ff) { shared = true; up(mix, L.mlp.shared_down.K); up(raw, M * L.mlp.shared_up.N); }
+            size_t most = 0;
+            for (int n = 1; n <= m->max_rows; ++n) { int rows; most_runs(m, s, n, &rows); up(most, rows); }
+            up(pair_rows, most);
+            up(pair_mix, most * L.mlp.down.K);
+            up(raw, most * L.mlp.up.N);
+            up(top, s.top);
+            up(decode_pair_mix, (size_t)16 * s.top * L.mlp.down.K);
         }
     }
-    const size_t M = m->max_rows, e = elem(m);
     m->x = static_cast<float*>(device_zeros(m, M * m->Cp * 4));
     m->h = device_zeros(m, M * m->Cp * e);
     m->y = static_cast<float*>(device_zeros(m, M * m->Cp * 4));
@@ -484,6 +790,24 @@ void allocate(b200_decoder* m) {
     m->wide = static_cast<float*>(device_zeros(m, M * wide * 4));
     m->low = device_zeros(m, M * low * e);
     m->q = device_zeros(m, M * q * e);
+    m->gates = static_cast<float*>(device_zeros(m, M * gates * 4));
+    if (pair_rows) {
+        m->pair_h = device_zeros(m, pair_rows * m->Cp * e);
+        m->pair_mix = device_zeros(m, pair_mix * e);
+        m->pair_y = static_cast<float*>(device_zeros(m, pair_rows * m->Cp * 4));
+        if (shared) m->shared_gate = static_cast<float*>(device_zeros(m, M * 4));
+    }
+    if (m->f32) m->raw = static_cast<float*>(device_zeros(m, raw * 4));
+    if (ql && !m->f32) {
+        // a sequence's step is expanded if that takes less: per head and position, n (2 R + Dr) multiply-adds on mma.sync, counted
+        // four times, against n (Dp + Dvp) on tcgen05 and Lp (Dp + Dvp) for the expansion
+        const Layer* first = nullptr;
+        for (const Layer& L : m->layers) if (!first && L.spec->kind == MIX_LATENT) first = &L;
+        const LatentAttention& c = first->lat;
+        const long slow = 4L * (2 * c.R + c.Dr), fast = c.Dp + c.Dvp;
+        m->expand_from = slow > fast ? (int)(c.Lp * fast / (slow - fast)) + 1 : m->max_rows + 1;
+        m->ql = device_zeros(m, M * ql * 2);
+    }
     if (!m->f32) {
         m->dx = static_cast<float*>(device_zeros(m, (size_t)16 * m->Cp * 4));
         m->dy = static_cast<float*>(device_zeros(m, (size_t)16 * m->Cp * 4));
@@ -492,10 +816,17 @@ void allocate(b200_decoder* m) {
         m->dmix = device_zeros(m, (size_t)16 * mix * 4);
         m->dconv = device_zeros(m, (size_t)16 * conv * 4);
         m->daux = static_cast<float*>(device_zeros(m, (size_t)16 * aux * 4));
+        m->dql = device_zeros(m, (size_t)16 * ql * 2);
+        if (pair_rows) {
+            m->dpair_mix = device_zeros(m, decode_pair_mix * 4);
+            m->dpair_y = static_cast<float*>(device_zeros(m, 16 * top * m->Cp * 4));
+            m->dshared_gate = static_cast<float*>(device_zeros(m, 16 * 4));
+        }
         m->dlogits = static_cast<float*>(device_zeros(m, (size_t)16 * m->Vp * 4));
     }
-    // descriptors: sequences, tokens, the sequence of every row, wanted rows, query-tile pairs
-    m->desc_ints = (size_t)m->max_slots * 8 + 3 * M + 2 * (M / 256 + m->max_slots + 1) + 64;
+    // descriptors: sequences, tokens, the sequence of every row, wanted rows, rows and sequences in the latent form, query-tile
+    // pairs of all sequences and of the expanded ones
+    m->desc_ints = (size_t)m->max_slots * 9 + 4 * M + 4 * (M / 256 + m->max_slots + 1) + 64;
     if (m->desc_ints < 16 * 9) m->desc_ints = 16 * 9;
     m->desc = static_cast<int*>(device_zeros(m, m->desc_ints * 4));
     m->dseqs = static_cast<SeqDesc*>(device_zeros(m, 16 * (sizeof(SeqDesc) + 4)));
@@ -559,9 +890,28 @@ int product(b200_decoder* m, void* out, const void* in, const Matrix& w, int M, 
                             static_cast<const uint16_t*>(in), static_cast<const uint16_t*>(w.w), w.bias, M, w.K, w.N, flags);
 }
 
+// down-projection's input: act(gate) * linear part; groups: per run of rows with a matrix of its own
+int gated_product(b200_decoder* m, void* out, const void* in, const Matrix& w, int M, int gate, float limit, const GemmGroups* groups = nullptr) {
+    b200_ctx* ctx = m->ctx;
+    if (m->f32) {
+        TRY(launch_gemm_fp32(ctx, m->raw, static_cast<const float*>(in), static_cast<const float*>(w.w), nullptr, M, w.K, w.N, ACT_NONE, groups));
+        return launch_gated_act(ctx, static_cast<float*>(out), m->raw, M, w.N / 2, gate, limit);
+    }
+    return launch_gemm_bf16(ctx, nullptr, static_cast<uint16_t*>(out), static_cast<const uint16_t*>(in), static_cast<const uint16_t*>(w.w), nullptr, M, w.K, w.N,
+                            gate == GATE_CLAMP ? GEMM_GATED_CLAMP : GEMM_GATED_GELU, nullptr, 0, 0, limit, groups);
+}
+int grouped_product(b200_decoder* m, float* out, const void* in, const Matrix& w, int M, const GemmGroups* groups) {
+    b200_ctx* ctx = m->ctx;
+    if (m->f32) return launch_gemm_fp32(ctx, out, static_cast<const float*>(in), static_cast<const float*>(w.w), nullptr, M, w.K, w.N, ACT_NONE, groups);
+    return launch_gemm_bf16(ctx, out, nullptr, static_cast<const uint16_t*>(in), static_cast<const uint16_t*>(w.w), nullptr, M, w.K, w.N, 0, nullptr, 0, 0, 0.f, groups);
+}
+
 struct StepView {
     const SeqDesc* seqs; const int* tokens; const int* row_seq; const int* want; const int2* pairs;
     int E, M, max_n, n_want, num_pairs;
+    // latent attention: rows and sequences in the latent form, query-tile pairs of the expanded sequences, whose positions are kv_rows rows
+    const int* lat_rows; const int* lat_seqs; const int2* kv_pairs;
+    int num_lat_rows, num_lat_seqs, lat_max_n, lat_max_keys, num_kv_pairs, kv_rows, kv_max_pos0;
 };
 
 int mixer_mamba1(b200_decoder* m, const Layer& L, const StepView& v) {
@@ -592,13 +942,21 @@ DeltaArgs delta_args(const b200_decoder* m, const Layer& L, const SeqDesc* seqs,
     a.H = s.heads; a.G = s.kv_heads; a.D = s.dim; a.Dl = L.Dl; a.Dv = s.vdim; a.Dvl = L.Dvl;
     a.conv_w = L.conv_w; a.hist = L.hist; a.taps = s.conv; a.np = L.np; a.max_slots = m->max_slots;
     a.norm_w = L.head_norm; a.gate_col = L.gate_col; a.eps = m->spec.eps;
+    if (s.kind == MIX_CHANNEL_DELTA) {
+        a.w_low = static_cast<const uint16_t*>(L.low.w); a.ld_low = L.low.K; a.low_col = L.low_col; a.low_a = L.low_a; a.low_g = L.low_g; a.gate_row = L.gate_row;
+    }
     return a;
 }
 
 int mixer_delta(b200_decoder* m, const Layer& L, const StepView& v) {
     b200_ctx* ctx = m->ctx;
     const LayerSpec& s = *L.spec;
+    const bool channel = s.kind == MIX_CHANNEL_DELTA;
     OP("gemm delta in", product(m, m->proj, m->h, L.in, v.M));
+    if (channel) {
+        OP("slice", launch_slice(ctx, m->low, L.low.K, m->proj + L.low_col, L.in.N, L.low_a + L.low_g, v.M, m->f32));
+        OP("gemm delta low rank", product(m, m->gates, m->low, L.low, v.M));
+    }
     ShortConvArgs c{};
     c.x = m->proj; c.ldx = L.in.N; c.out = m->conv; c.ld_out = L.np; c.w = L.conv_w; c.hist = L.hist; c.seqs = v.seqs;
     c.np = L.np; c.taps = s.conv; c.max_slots = m->max_slots;
@@ -608,11 +966,36 @@ int mixer_delta(b200_decoder* m, const Layer& L, const StepView& v) {
     a.qkv = static_cast<const float*>(m->conv);
     a.raw = m->proj; a.ld_raw = L.in.N;
     a.coef = reinterpret_cast<float4*>(m->aux);
+    if (channel) { a.decay = m->gates; a.ld_decay = L.low.N; }
     OP("delta prep", launch_delta_prep(ctx, a, v.E, v.max_n));
     a.out = m->wide; a.ldo = s.heads * L.Dvl;
     OP("delta scan", launch_delta_scan(ctx, a, v.E));
-    OP("head norm", launch_gated_head_norm(ctx, m->mix, L.o.K, m->wide, a.ldo, m->proj + L.gate_col, L.in.N, L.head_norm, v.M, s.heads, s.vdim, L.Dvl,
-                                           m->spec.eps, m->f32));
+    OP("head norm", launch_gated_head_norm(ctx, m->mix, L.o.K, m->wide, a.ldo, channel ? m->gates + L.gate_row : m->proj + L.gate_col, channel ? L.low.N : L.in.N,
+                                           L.head_norm, v.M, s.heads, s.vdim, L.Dvl, m->spec.eps, m->f32, channel));
+    return B200_OK;
+}
+
+int mixer_latent(b200_decoder* m, const Layer& L, const StepView& v) {
+    b200_ctx* ctx = m->ctx;
+    const LatentAttention& c = L.lat;
+    OP("gemm latent in", product(m, m->proj, m->h, L.in, v.M));
+    OP("latent prep", launch_latent_prep(ctx, c, m->proj, L.in.N, m->q, m->lat, v.seqs, v.row_seq, v.M, m->f32));
+    if (v.kv_rows > 0) {
+        if (v.kv_max_pos0 > 0) OP("latent gather", launch_latent_gather(ctx, c, m->lat, v.seqs, v.E, v.kv_max_pos0, m->f32));
+        CachedAttention f = L.flat;
+        f.K = m->kv; f.V = static_cast<char*>(m->kv) + (size_t)c.H * c.Dp * elem(m); f.kv_rows = v.kv_rows;
+        if (m->f32) OP("gemm latent kv", product(m, m->kv, m->lat, L.kv, v.kv_rows));
+        else OP("gemm latent kv", launch_gemm_bf16(ctx, nullptr, static_cast<uint16_t*>(m->kv), static_cast<const uint16_t*>(m->lat), static_cast<const uint16_t*>(L.kv.w),
+                                                   nullptr, v.kv_rows, L.kv.K, L.kv.N, GEMM_FP16));
+        if (!m->f32 && attention_cached_has_mma(f))
+            OP("attention", launch_attention_cached_mma(ctx, f, m->q, m->mix, L.o.K, v.seqs, v.kv_pairs, v.num_kv_pairs, v.M, m->max_slots));
+        else
+            OP("attention", launch_attention_cached_simt(ctx, f, m->q, m->mix, L.o.K, v.seqs, v.E, v.max_n, m->f32));
+    }
+    if (v.num_lat_rows > 0) {
+        OP("latent query", launch_latent_query(ctx, c, m->proj, L.in.N, m->ql, v.seqs, v.row_seq, v.lat_rows, v.num_lat_rows, false));
+        OP("latent attention", launch_latent_attention(ctx, c, m->ql, m->mix, L.o.K, v.seqs, v.lat_seqs, v.num_lat_seqs, v.lat_max_n, v.lat_max_keys, false));
+    }
     return B200_OK;
 }
 
@@ -635,6 +1018,17 @@ int mixer_parallel(b200_decoder* m, const Layer& L, const StepView& v) {
     return B200_OK;
 }
 
+// what the next residual kernel adds: a mixer's (or dense feed-forward's) output ...
+void branch_of_mixer(ResidualNormArgs& n, const Layer& L, const float* y) {
+    n.y = y; n.wb = L.norm1b; n.y_scale = nullptr;
+    n.parts = nullptr; n.part_of = nullptr; n.top = 0;
+}
+// ... or the experts' outputs
+void branch_of_experts(ResidualNormArgs& n, const Layer& L, const float* shared, const float* shared_gate, const float* parts, const int* part_of) {
+    n.y = shared; n.wb = nullptr; n.y_scale = shared ? shared_gate : nullptr;
+    n.parts = parts; n.part_of = part_of; n.top = L.spec->top; n.part_scale = 1.0f / (float)L.spec->top;
+}
+
 // rows of the step -> logits of the wanted rows in m->logits
 int enqueue_general(b200_decoder* m, const StepView& v) {
     b200_ctx* ctx = m->ctx;
@@ -643,24 +1037,49 @@ int enqueue_general(b200_decoder* m, const StepView& v) {
     n.x_out = m->x; n.h = m->h; n.M = v.M;
     n.tok = v.tokens; n.embed = m->embed; n.embed_scale = m->spec.embed_scale;
     n.w = m->layers[0].norm1;
+    if (m->num_routes) OP("expert routes", launch_moe_route(ctx, m->routes, m->num_routes, v.tokens, v.M, m->f32, m->max_experts));
     OP("embed norm", launch_residual_rms(ctx, n, m->f32 ? H_F32 : H_BF16));
     n.tok = nullptr;
     n.x = m->x;
-    n.y = m->y;
     for (size_t i = 0; i < m->layers.size(); ++i) {
         const Layer& L = m->layers[i];
-        if (L.spec->kind == MIX_MAMBA1) TRY(mixer_mamba1(m, L, v));
-        else if (L.spec->kind == MIX_DELTA) TRY(mixer_delta(m, L, v));
-        else TRY(mixer_parallel(m, L, v));
-        OP(L.spec->kind == MIX_MAMBA1 ? "gemm mamba1 o" : (L.spec->kind == MIX_DELTA ? "gemm delta o" : "gemm parallel o"), product(m, m->y, m->mix, L.o, v.M));
+        const Mlp& f = L.mlp;
+        const char* o_name = "";
+        switch (L.spec->kind) {
+            case MIX_MAMBA1: TRY(mixer_mamba1(m, L, v)); o_name = "gemm mamba1 o"; break;
+            case MIX_DELTA:
+            case MIX_CHANNEL_DELTA: TRY(mixer_delta(m, L, v)); o_name = "gemm delta o"; break;
+            case MIX_PARALLEL: TRY(mixer_parallel(m, L, v)); o_name = "gemm parallel o"; break;
+            case MIX_LATENT: TRY(mixer_latent(m, L, v)); o_name = "gemm latent o"; break;
+        }
+        OP(o_name, product(m, m->y, m->mix, L.o, v.M));
         const bool last = i + 1 == m->layers.size();
-        n.wb = L.norm1b;
-        if (L.spec->ff > 0) {
+        branch_of_mixer(n, L, m->y);
+        if (L.spec->mlp == MLP_DENSE) {
             n.w = L.norm2;
             OP("residual norms", launch_residual_rms(ctx, n, m->f32 ? H_F32 : H_BF16));
-            OP("gemm mlp up", product(m, m->mix, m->h, L.mlp.up, v.M, m->spec.design->mlp_act, true));
-            OP("gemm mlp down", product(m, m->y, m->mix, L.mlp.down, v.M));
+            if (f.gate == GATE_NONE) OP("gemm mlp up", product(m, m->mix, m->h, f.up, v.M, m->spec.design->mlp_act, true));
+            else OP("gemm mlp up", gated_product(m, m->mix, m->h, f.up, v.M, f.gate, 0.f));
+            OP("gemm mlp down", product(m, m->y, m->mix, f.down, v.M));
             n.wb = L.norm2b;
+        } else if (L.spec->mlp == MLP_EXPERTS) {
+            const LayerSpec& s = *L.spec;
+            int rows;
+            most_runs(m, s, v.M, &rows);
+            const GemmGroups groups{f.route.blocks, moe_run_rows(v.M * s.top, s.experts, m->f32), s.experts};
+            n.w = L.norm2;
+            n.copy = m->pair_h; n.copy_of = f.route.place; n.copies = s.top;
+            n.gate_w = f.shared_gate; n.gate_out = m->shared_gate;
+            OP("residual norms experts", launch_residual_rms(ctx, n, m->f32 ? H_F32 : H_BF16));
+            n.copies = 0;
+            n.gate_w = nullptr;
+            OP("gemm experts up", gated_product(m, m->pair_mix, m->pair_h, f.up, rows, f.gate, s.limit, &groups));
+            OP("gemm experts down", grouped_product(m, m->pair_y, m->pair_mix, f.down, rows, &groups));
+            if (s.shared_ff) {
+                OP("gemm shared up", gated_product(m, m->mix, m->h, f.shared_up, v.M, f.gate, s.shared_limit));
+                OP("gemm shared down", product(m, m->y, m->mix, f.shared_down, v.M));
+            }
+            branch_of_experts(n, L, s.shared_ff ? m->y : nullptr, m->shared_gate, m->pair_y, f.route.place);
         }
         if (!last) {
             n.w = m->layers[i + 1].norm1;
@@ -709,7 +1128,7 @@ int enqueue_decode(b200_decoder* m, int B) {
         TRY(norm(L.norm1));
         DecodeGemmArgs in = product_args(m->dh, L.in);
         in.out = m->dproj; in.ldo = L.in.N;
-        if (s.kind != MIX_PARALLEL) {
+        if (s.kind != MIX_PARALLEL && s.kind != MIX_LATENT) {
             in.seqs = m->dseqs; in.conv_w = L.conv_w; in.conv_b = L.conv_b; in.hist = L.hist; in.conv_n = L.np; in.taps = s.conv; in.max_slots = m->max_slots;
             if (s.kind == MIX_MAMBA1) in.conv_out = static_cast<uint8_t*>(m->dconv);
         }
@@ -722,7 +1141,10 @@ int enqueue_decode(b200_decoder* m, int B) {
             c.inner = s.inner; c.state_pad = L.sp;
             c.Wdt = static_cast<const uint16_t*>(L.dt.w); c.rank = s.dt_rank; c.ld_wdt = L.rank_p;
             TRY(launch_selective_scan(ctx, c, B, 1, true, true));
-        } else if (s.kind == MIX_DELTA) {
+        } else if (s.kind == MIX_LATENT) {
+            TRY(launch_latent_query(ctx, L.lat, m->dproj, L.in.N, m->dql, m->dseqs, nullptr, nullptr, B, true));
+            TRY(launch_latent_attention(ctx, L.lat, m->dql, m->dmix, L.o.K, m->dseqs, nullptr, B, 1, m->Tp, true));
+        } else if (s.kind == MIX_DELTA || s.kind == MIX_CHANNEL_DELTA) {
             DeltaArgs a = delta_args(m, L, m->dseqs, m->dproj);
             a.qkv = m->dproj; a.ld = L.in.N;
             a.out = static_cast<float*>(m->dmix); a.ldo = L.o.K;
@@ -733,16 +1155,34 @@ int enqueue_decode(b200_decoder* m, int B) {
             TRY(launch_attention_cached_decode(ctx, L.att, m->dproj, L.in.N, static_cast<uint8_t*>(m->dmix), L.o.K, m->dseqs, B, gru));
         }
         TRY(plain(m->dy, m->dmix, L.o));
-        n.y = m->dy;
-        n.wb = L.norm1b;
-        if (s.ff > 0) {
+        branch_of_mixer(n, L, m->dy);
+        const Mlp& f = L.mlp;
+        if (s.mlp == MLP_DENSE) {
             TRY(norm(L.norm2));
-            DecodeGemmArgs up = product_args(m->dh, L.mlp.up);
+            DecodeGemmArgs up = product_args(m->dh, f.up);
             up.act = m->spec.design->mlp_act;
+            up.gate = f.gate;
             up.split_out = static_cast<uint8_t*>(m->dmix);
             TRY(launch_decode_gemm(ctx, up));
-            TRY(plain(m->dy, m->dmix, L.mlp.down));
+            TRY(plain(m->dy, m->dmix, f.down));
             n.wb = L.norm2b;
+        } else if (s.mlp == MLP_EXPERTS) {
+            n.gate_w = f.shared_gate; n.gate_out = m->dshared_gate;
+            TRY(norm(L.norm2));
+            n.gate_w = nullptr;
+            DecodeGemmArgs up = product_args(m->dh, f.up), down = product_args(m->dpair_mix, f.down);
+            up.table = down.table = f.table; up.tok = down.tok = m->dtokens; up.top = down.top = s.top;
+            up.gate = f.gate; up.limit = s.limit; up.split_out = static_cast<uint8_t*>(m->dpair_mix);
+            down.pair_in = 1; down.out = m->dpair_y; down.ldo = f.down.N;
+            if (s.shared_ff) {
+                up.shared = {static_cast<const uint8_t*>(m->dh), static_cast<const uint16_t*>(f.shared_up.w), f.shared_up.N, f.shared_up.K, s.shared_limit, nullptr, 0,
+                             static_cast<uint8_t*>(m->dmix)};
+                down.shared = {static_cast<const uint8_t*>(m->dmix), static_cast<const uint16_t*>(f.shared_down.w), f.shared_down.N, f.shared_down.K, 0.f, m->dy,
+                               f.shared_down.N, nullptr};
+            }
+            TRY(launch_decode_gemm(ctx, up));
+            TRY(launch_decode_gemm(ctx, down));
+            branch_of_experts(n, L, s.shared_ff ? m->dy : nullptr, m->dshared_gate, m->dpair_y, nullptr);
         }
     }
     TRY(norm(m->final_norm));
@@ -763,7 +1203,7 @@ struct Entry { int slot; const int* tokens; int n; };
 SeqDesc describe(b200_decoder* m, int slot, int row0, int n) {
     Slot& s = m->slots[slot];
     SeqDesc d{};
-    d.row0 = row0; d.n = n; d.slot = slot; d.pos0 = s.len; d.bank = s.bank;
+    d.row0 = row0; d.n = n; d.slot = slot; d.pos0 = s.len; d.bank = s.bank; d.kv0 = -1; d.lat0 = row0;
     s.len += n;
     s.bank ^= 1;
     return d;
@@ -812,10 +1252,36 @@ int decode_step(b200_decoder* m, const std::vector<int>& slots, const int* token
     return B200_OK;
 }
 
+// latents and expanded keys and values of `rows` positions
+int reserve_expanded(b200_decoder* m, int rows) {
+    if (rows <= m->kv_rows) return B200_OK;
+    b200_ctx* ctx = m->ctx;
+    size_t lat = 0, kv = 0;
+    for (const Layer& L : m->layers)
+        if (L.spec->kind == MIX_LATENT) { if ((size_t)L.kv.K > lat) lat = L.kv.K; if ((size_t)L.kv.N > kv) kv = L.kv.N; }
+    if (rows < 2 * m->kv_rows) rows = 2 * m->kv_rows;
+    B200_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    if (m->lat) cudaFree(m->lat);
+    if (m->kv) cudaFree(m->kv);
+    m->lat = m->kv = nullptr;
+    m->kv_rows = 0;
+    B200_CUDA(ctx, cudaMalloc(&m->lat, rows * lat * elem(m)));
+    B200_CUDA(ctx, cudaMalloc(&m->kv, rows * kv * elem(m)));
+    m->kv_rows = rows;
+    return B200_OK;
+}
+
 int general_step(b200_decoder* m, const std::vector<Entry>& entries, const std::vector<int>& want) {
     b200_ctx* ctx = m->ctx;
-    int M = 0, max_n = 0;
-    for (const Entry& e : entries) { M += e.n; if (e.n > max_n) max_n = e.n; }
+    int M = 0, max_n = 0, expanded = 0;
+    bool latent = false;
+    for (const Layer& L : m->layers) latent = latent || L.spec->kind == MIX_LATENT;
+    for (const Entry& e : entries) {
+        M += e.n;
+        if (e.n > max_n) max_n = e.n;
+        if (latent && e.n >= m->expand_from) expanded += m->slots[e.slot].len + e.n;
+    }
+    if (expanded) TRY(reserve_expanded(m, expanded));
     const int E = (int)entries.size(), nw = (int)want.size();
     if (nw > m->logits_rows) {
         B200_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
@@ -831,14 +1297,28 @@ int general_step(b200_decoder* m, const std::vector<Entry>& entries, const std::
     int* tok = host + 8 * E;
     int* row_seq = tok + M;
     int* w = row_seq + M;
-    int* pr = w + nw;
+    int* lat_rows = w + nw;
+    int* lat_seqs = lat_rows + M;
+    int* pr = lat_seqs + E;
     if ((pr - host) & 1) ++pr;  // int2
     struct Pair { int seq, pair, keys; };
     std::vector<Pair> pairs;
+    StepView v{};
     int row = 0;
     for (int i = 0; i < E; ++i) {
         const Entry& e = entries[i];
         sd[i] = describe(m, e.slot, row, e.n);
+        if (latent && e.n >= m->expand_from) {
+            sd[i].kv0 = v.kv_rows;
+            v.kv_rows += sd[i].pos0 + e.n;
+            if (sd[i].pos0 > v.kv_max_pos0) v.kv_max_pos0 = sd[i].pos0;
+        } else if (latent) {
+            sd[i].lat0 = v.num_lat_rows;
+            for (int t = 0; t < e.n; ++t) lat_rows[v.num_lat_rows++] = row + t;
+            lat_seqs[v.num_lat_seqs++] = i;
+            if (e.n > v.lat_max_n) v.lat_max_n = e.n;
+            if (sd[i].pos0 + e.n > v.lat_max_keys) v.lat_max_keys = sd[i].pos0 + e.n;
+        }
         for (int t = 0; t < e.n; ++t) { tok[row + t] = e.tokens[t]; row_seq[row + t] = i; }
         for (int p = 0; p * 256 < e.n; ++p) pairs.push_back({i, p, sd[i].pos0 + (e.n < (p + 1) * 256 ? e.n : (p + 1) * 256)});
         row += e.n;
@@ -848,16 +1328,21 @@ int general_step(b200_decoder* m, const std::vector<Entry>& entries, const std::
     for (size_t i = 1; i < pairs.size(); ++i)
         for (size_t j = i; j > 0 && pairs[j - 1].keys < pairs[j].keys; --j) std::swap(pairs[j - 1], pairs[j]);
     for (size_t i = 0; i < pairs.size(); ++i) { pr[2 * i] = pairs[i].seq; pr[2 * i + 1] = pairs[i].pair; }
-    const size_t used = (pr - host) + 2 * pairs.size();
+    int* kpr = pr + 2 * pairs.size();
+    for (const Pair& p : pairs)
+        if (sd[p.seq].kv0 >= 0) { kpr[2 * v.num_kv_pairs] = p.seq; kpr[2 * v.num_kv_pairs + 1] = p.pair; v.num_kv_pairs++; }
+    const size_t used = (kpr - host) + 2 * (size_t)v.num_kv_pairs;
     if (used > m->desc_ints) return B200_ERR_LIMIT;
     B200_CUDA(ctx, cudaMemcpyAsync(m->desc, host, used * 4, cudaMemcpyHostToDevice, ctx->stream));
     B200_CUDA(ctx, cudaEventRecord(m->ring_ev[m->ring], ctx->stream));
-    StepView v;
     v.seqs = reinterpret_cast<const SeqDesc*>(m->desc);
     v.tokens = m->desc + (tok - host);
     v.row_seq = m->desc + (row_seq - host);
     v.want = m->desc + (w - host);
     v.pairs = reinterpret_cast<const int2*>(m->desc + (pr - host));
+    v.kv_pairs = reinterpret_cast<const int2*>(m->desc + (kpr - host));
+    v.lat_rows = m->desc + (lat_rows - host);
+    v.lat_seqs = m->desc + (lat_seqs - host);
     v.E = E; v.M = M; v.max_n = max_n; v.n_want = nw; v.num_pairs = (int)pairs.size();
     return enqueue_general(m, v);
 }
@@ -899,6 +1384,8 @@ int b200_decoder_destroy(b200_decoder* m) {
     for (cudaEvent_t e : m->ev_pool) cudaEventDestroy(e);
     for (void* p : m->owned) cudaFree(p);
     if (m->logits) cudaFree(m->logits);
+    if (m->lat) cudaFree(m->lat);
+    if (m->kv) cudaFree(m->kv);
     if (m->gen_log) cudaFree(m->gen_log);
     for (int i = 0; i < b200_decoder::kRing; ++i) {
         if (m->pinned[i]) cudaFreeHost(m->pinned[i]);
@@ -924,10 +1411,11 @@ int b200_decoder_check_config(const char* config_json, char* message, int messag
 
 int b200_decoder_vocab(const b200_decoder* m) { return m ? m->spec.vocab : 0; }
 
-int b200_decoder_set_tensor(b200_decoder* m, const char* name, const void* data, int is_f32, const long* shape, int ndim) {
+int b200_decoder_set_tensor(b200_decoder* m, const char* name, const void* data, int type, const long* shape, int ndim) {
     if (!m || !name || !data || !shape) return B200_ERR_NULL;
+    if (type < 0 || type > 2) return B200_ERR_SHAPE;
     if (m->ready) return B200_ERR_STATE;
-    m->store->set(name, data, is_f32 != 0, std::vector<long>(shape, shape + ndim));
+    m->store->set(name, data, static_cast<TensorType>(type), std::vector<long>(shape, shape + ndim));
     return B200_OK;
 }
 

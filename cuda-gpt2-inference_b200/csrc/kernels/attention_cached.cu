@@ -199,8 +199,11 @@ attention_simt_kernel(const CachedAttention c, const T* __restrict__ q_in, void*
     if (q0 >= sd.n) return;
     const int kvh = h / (c.H / c.G);
     const int tid = threadIdx.x, nq = min(SQ, sd.n - q0);
-    const T* K = static_cast<const T*>(c.K) + ((size_t)sd.slot * c.G + kvh) * c.Tp * c.Dp;
-    const T* V = static_cast<const T*>(c.V) + ((size_t)sd.slot * c.G + kvh) * c.Tp * c.Dvp;
+    const bool flat = c.ld_kv > 0;
+    if (flat && sd.kv0 < 0) return;
+    const int ldk = flat ? c.ld_kv : c.Dp, ldv = flat ? c.ld_kv : c.Dvp;
+    const T* K = static_cast<const T*>(c.K) + (flat ? (size_t)sd.kv0 * ldk + h * c.Dp : ((size_t)sd.slot * c.G + kvh) * c.Tp * c.Dp);
+    const T* V = static_cast<const T*>(c.V) + (flat ? (size_t)sd.kv0 * ldv + h * c.Dvp : ((size_t)sd.slot * c.G + kvh) * c.Tp * c.Dvp);
     for (int i = tid; i < SQ * c.D; i += 256) {
         const int r = i / c.D, d = i - r * c.D;
         qs[r * Dl + d] = r < nq ? cache_f<T>(q_in + ((size_t)(sd.row0 + q0 + r) * c.H + h) * c.Dp + d) * c.scale : 0.f;
@@ -218,11 +221,11 @@ attention_simt_kernel(const CachedAttention c, const T* __restrict__ q_in, void*
         const int nk = min(SK, keys - k0);
         for (int i = tid; i < SK * c.D; i += 256) {
             const int t = i / c.D, d = i - t * c.D;
-            ks[t * Dl + d] = t < nk ? cache_f<T>(K + (size_t)(k0 + t) * c.Dp + d) : 0.f;
+            ks[t * Dl + d] = t < nk ? cache_f<T>(K + (size_t)(k0 + t) * ldk + d) : 0.f;
         }
         for (int i = tid; i < SK * c.Dv; i += 256) {
             const int t = i / c.Dv, d = i - t * c.Dv;
-            vs[t * Vl + d] = t < nk ? cache_f<T>(V + (size_t)(k0 + t) * c.Dvp + d) : 0.f;
+            vs[t * Vl + d] = t < nk ? cache_f<T>(V + (size_t)(k0 + t) * ldv + d) : 0.f;
         }
         __syncthreads();
         float s[4] = {0.f, 0.f, 0.f, 0.f};
@@ -338,7 +341,7 @@ __device__ __forceinline__ bool pipe_bar_all(int id, bool ok) {
 }
 
 struct Item {
-    int row0, n, q0, pos0, slot, h;
+    int row0, n, q0, pos0, slot, h, kv0;
     // key blocks pipeline x works through (0: the pair has no second tile)
     template <int BKV>
     __device__ __forceinline__ int blocks(int x) const {
@@ -352,7 +355,7 @@ __device__ __forceinline__ Item get_item(const MmaArgs& a, int item) {
     const SeqDesc* s = a.seqs + pr.x;
     Item it;
     it.h = item % a.c.H;
-    it.row0 = __ldg(&s->row0); it.n = __ldg(&s->n); it.pos0 = __ldg(&s->pos0); it.slot = __ldg(&s->slot);
+    it.row0 = __ldg(&s->row0); it.n = __ldg(&s->n); it.pos0 = __ldg(&s->pos0); it.slot = __ldg(&s->slot); it.kv0 = __ldg(&s->kv0);
     it.q0 = pr.y * 2 * BQ;
     return it;
 }
@@ -435,7 +438,9 @@ attention_cached_mma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
                 const Item it = get_item(args, item);
                 const int n0 = it.blocks<BKV>(0), n1 = it.blocks<BKV>(1);
                 const int n_item = n1 > n0 ? n1 : n0;
-                const int kv0 = (it.slot * args.c.G + it.h / (args.c.H / args.c.G)) * args.c.Tp;
+                const bool flat = args.c.ld_kv > 0;
+                const int kv0 = flat ? it.kv0 : (it.slot * args.c.G + it.h / (args.c.H / args.c.G)) * args.c.Tp;
+                const int k_x = flat ? it.h * args.c.Dp : 0, v_x = flat ? it.h * args.c.Dvp : 0;
                 if (!mbar_wait(&q_empty[qs], ((n / QS) & 1) ^ 1, abort_flag)) { ok = false; break; }
                 mbar_arrive_expect_tx(&q_full[qs], (n1 > 0 ? 2 : 1) * KD * QB);
                 for (int x = 0; x < (n1 > 0 ? 2 : 1); ++x)
@@ -447,14 +452,14 @@ attention_cached_mma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
                         const int s = gk & 1;
                         if (!mbar_wait(&k_empty[s], ((gk >> 1) & 1) ^ 1, abort_flag)) { ok = false; break; }
                         mbar_arrive_expect_tx(&k_full[s], KD * KB);
-                        for (int d = 0; d < KD; ++d) tma_load_2d(k_s + (s * KD + d) * KB, &tmap_k, d * 64, kv0 + (j + 1) * BKV, &k_full[s]);
+                        for (int d = 0; d < KD; ++d) tma_load_2d(k_s + (s * KD + d) * KB, &tmap_k, k_x + d * 64, kv0 + (j + 1) * BKV, &k_full[s]);
                     }
                     if (j >= 0) {
                         const uint32_t gv = g + j;
                         const int s = gv & 1;
                         if (!mbar_wait(&v_empty[s], ((gv >> 1) & 1) ^ 1, abort_flag)) { ok = false; break; }
                         mbar_arrive_expect_tx(&v_full[s], VD * KB);
-                        for (int d = 0; d < VD; ++d) tma_load_2d(v_s + (s * VD + d) * KB, &tmap_v, d * 64, kv0 + j * BKV, &v_full[s]);
+                        for (int d = 0; d < VD; ++d) tma_load_2d(v_s + (s * VD + d) * KB, &tmap_v, v_x + d * 64, kv0 + j * BKV, &v_full[s]);
                     }
                 }
                 g += n_item;
@@ -1028,8 +1033,13 @@ int launch_attention_cached_mma(b200_ctx* ctx, const CachedAttention& c, const v
     const uint32_t bkv = c.Dvp > 64 ? 64 : 128;
     // 16-bit elements: the map's number format does not matter, nothing is converted or filled but zeros
     int st = b200_get_tensor_map_bf16(ctx, &tq, q, (uint64_t)M, (uint64_t)c.H * c.Dp, (uint64_t)c.H * c.Dp, BQ, 64);
-    if (st == B200_OK) st = b200_get_tensor_map_bf16(ctx, &tk, c.K, kv_rows, (uint64_t)c.Dp, (uint64_t)c.Dp, bkv, 64);
-    if (st == B200_OK) st = b200_get_tensor_map_bf16(ctx, &tv, c.V, kv_rows, (uint64_t)c.Dvp, (uint64_t)c.Dvp, bkv, 64);
+    if (c.ld_kv > 0) {
+        if (st == B200_OK) st = b200_get_tensor_map_bf16(ctx, &tk, c.K, (uint64_t)c.kv_rows, (uint64_t)c.H * c.Dp, (uint64_t)c.ld_kv, bkv, 64);
+        if (st == B200_OK) st = b200_get_tensor_map_bf16(ctx, &tv, c.V, (uint64_t)c.kv_rows, (uint64_t)c.H * c.Dvp, (uint64_t)c.ld_kv, bkv, 64);
+    } else {
+        if (st == B200_OK) st = b200_get_tensor_map_bf16(ctx, &tk, c.K, kv_rows, (uint64_t)c.Dp, (uint64_t)c.Dp, bkv, 64);
+        if (st == B200_OK) st = b200_get_tensor_map_bf16(ctx, &tv, c.V, kv_rows, (uint64_t)c.Dvp, (uint64_t)c.Dvp, bkv, 64);
+    }
     if (st != B200_OK) return st;
     MmaArgs a;
     a.c = c; a.seqs = seqs; a.pairs = pairs; a.num_items = num_pairs * c.H; a.out = out; a.ldo = ldo;

@@ -17,41 +17,57 @@ struct SeqDesc {
     int slot;  // where the sequence's cache and state live
     int pos0;  // position of its first token in this step
     int bank;  // short-convolution history to read (0 / 1); the other bank is written
-    int pad[3];
+    int kv0;   // latent attention: first row of the sequence's expanded keys and values; -1: the latents are attended to
+    int lat0;  // ... and then the first of its rows among the step's queries that do so
+    int pad;
 };
 
 // leading dimension of a matrix operand with n columns: whole 16-byte pieces, at least one 64-element K block
 inline int pad_dim(int n) { return n < 64 ? 64 : (n + 7) & ~7; }
 
 // ---- row-wise (rmsnorm.cu)
-// Residual stream of M rows:  r = embed[tok] * scale (tok != null), or x, or x + rms(y) * wb (y != null);
+// Residual stream of M rows:  r = embed[tok] * scale (tok != null), or x, or x + branch with branch = rms(y) * wb (wb, y != null),
+// or y * y_scale[row] (y != null; y_scale null: 1) + part_scale * sum of `top` rows of parts (part_of[row * top + j]; null: row * top + j);
 // x_out = r (if not null);  h = rms(r) * w (if w) as bf16, fp32 or split rows (decoder_math.cuh).  rows != null: row i of the output
-// is made from row rows[i] of the inputs.  C columns of Cp.
+// is made from row rows[i] of the inputs.  C columns of Cp.  copies > 0 (bf16, fp32): row i of h also goes to rows copy_of[i * copies + j]
+// of copy.  gate_w: gate_out[i] = sigmoid(h . gate_w).
 struct ResidualNormArgs {
     const float* x; const float* y; const float* wb; const float* w;
     float* x_out; void* h;
     const int* tok; const void* embed; float embed_scale; int vocab;
     const int* rows;
     int M, C, Cp; float eps;
+    const float* y_scale; const float* parts; const int* part_of; int top; float part_scale;
+    void* copy; const int* copy_of; int copies;
+    const float* gate_w; float* gate_out;
 };
 enum : int { H_BF16 = 0, H_F32 = 1, H_SPLIT = 2 };
 int launch_residual_rms(b200_ctx* ctx, const ResidualNormArgs& a, int format);  // H_F32: the embedding table is fp32, else bf16
-// out[r, h*Dv + d] = o / rms(o over the head) * w[d] * silu(gate);  o, gate [M] rows with heads Dvl apart
+// out[r, h*Dv + d] = o / rms(o over the head) * w[d] * silu(gate) (plain_sigmoid: sigmoid(gate));  o, gate [M] rows with heads Dvl apart
 int launch_gated_head_norm(b200_ctx* ctx, void* out, int ld_out, const float* o, int ld_o, const float* gate, int ld_gate,
-                           const float* w, int M, int H, int Dv, int Dvl, float eps, bool f32);
+                           const float* w, int M, int H, int Dv, int Dvl, float eps, bool f32, bool plain_sigmoid = false);
 // dst[r, 0..n) = src[r, col0 ..]  (fp32 -> bf16 or fp32), columns n..ld_dst zero
 int launch_slice(b200_ctx* ctx, void* dst, int ld_dst, const float* src, int ld_src, int n, int M, bool f32);
 
 // ---- matrix products
 enum : int { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_GELU_ERF = 2 };
 // out[M,N] = act(inp[M,K] W[N,K]^T + bias) on the fp32 FMA pipe (no reduced precision anywhere); K, N multiples of 4
-int launch_gemm_fp32(b200_ctx* ctx, float* out, const float* inp, const float* W, const float* bias, int M, int K, int N, int act);
+int launch_gemm_fp32(b200_ctx* ctx, float* out, const float* inp, const float* W, const float* bias, int M, int K, int N, int act,
+                     const GemmGroups* groups = nullptr);
 
 // Decode product (gemm_decode.cu): B <= 16 split rows x [B, K] against bf16 weights [N, K], + bias, then
 //   columns below conv_n: short causal convolution with the history of the row's slot (+ conv_b) and silu; the new
 //     history goes to the other bank
 //   the others: act
 // to out (fp32) and, as split rows, to split_out (all columns) or conv_out (the convolved ones, which then do not go to out).
+// gate != GATE_NONE: W's rows come in blocks of 64, 32 gates and the 32 linear values that belong to them, and the output
+// (split_out) has N / 2 columns.
+// Table-routed experts (top > 0): input row b belongs to the `top` matrices table[tok[b] * top ..] of the stack W [..][N, K],
+// and its products with them are rows b * top + j of the output; pair_in: of the input too (else one row b meets
+// them all).  A matrix is read once however many rows want it.  With shared.W a further matrix of its own
+// height, width, input and output meets every row in the same launch.
+enum : int { GATE_NONE = 0, GATE_GELU_TANH = 1, GATE_CLAMP = 2 };
+struct DecodeGemmShared { const uint8_t* x; const uint16_t* W; int N, K; float limit; float* out; int ldo; uint8_t* split_out; };
 struct DecodeGemmArgs {
     const uint8_t* x;
     const uint16_t* W; const float* bias;
@@ -60,8 +76,20 @@ struct DecodeGemmArgs {
     uint8_t* split_out;   // [B] rows of N columns
     const SeqDesc* seqs; const float* conv_w; const float* conv_b; float* hist; int conv_n, taps, max_slots;
     uint8_t* conv_out;    // [B] rows of conv_n columns
+    int gate; float limit;
+    const int* table; const int* tok; int top, pair_in;
+    DecodeGemmShared shared;
 };
 int launch_decode_gemm(b200_ctx* ctx, const DecodeGemmArgs& a);
+
+// ---- experts (experts.cu)
+struct MoeRoute { const int* table; int experts, top; int* place; int* blocks; };  // table [vocab][top]
+// rows per run (GemmGroups::align) of P pairs
+__host__ __device__ inline int moe_run_rows(int P, int experts, bool f32) { return f32 ? 64 : (P / 1024 >= experts ? 256 : 128); }
+// routes: n of them in device memory
+int launch_moe_route(b200_ctx* ctx, const MoeRoute* routes, int n, const int* tok, int M, bool f32, int max_experts);
+// out[M,F] = act of in[M,2F], whose columns are blocks of 32 gates and their 32 linear values (fp32; F a multiple of 32)
+int launch_gated_act(b200_ctx* ctx, float* out, const float* in, int M, int F, int gate, float limit);
 
 // ---- recurrences (recurrent.cu)
 // y = silu(causal depthwise convolution of columns [0, n) of x + bias); weights [taps][np]; history
@@ -119,6 +147,12 @@ struct DeltaArgs {
     int H, G, D, Dl, Dv, Dvl;
     const float* conv_w; float* hist; int taps, np, max_slots;
     const float* norm_w; int gate_col; float eps;
+    // Decay per key channel: exp(-exp(A_log) softplus(a + dt_bias)) with dt_bias [H][Dl] and a from a low-rank projection.
+    //   decay: rows of ld_decay columns, head h's at h*Dl: a on entry of prep, the decay behind it
+    //   step forms a, and the output gate (through a sigmoid), itself: w_low's row h*Dl + d meets columns low_col .. + low_a of the
+    //   token's row, its row gate_row + h*Dvl + d columns low_a .. low_a + low_g of the same piece
+    float* decay; int ld_decay;
+    const uint16_t* w_low; int ld_low, low_col, low_a, low_g, gate_row;
 };
 int delta_state_pad(int D);  // 0: unsupported
 int launch_delta_prep(b200_ctx* ctx, const DeltaArgs& a, int E, int max_n);
@@ -150,6 +184,9 @@ struct CachedAttention {
     float scale, eps;
     void* K; void* V;
     float out_scale;
+    // > 0: K and V are not the cache but rows of ld_kv columns in which every head has its own Dp / Dvp columns (G = H); a
+    // sequence's positions are the rows from its kv0 on (kv_rows in all)
+    int ld_kv, kv_rows;
 };  // (scores: (q . k) * scale)
 inline int attention_pad(int d) { return d <= 64 ? 64 : (d + 63) & ~63; }
 // norms and rotation of a step's q (-> q_out [M][H * Dp]) and k, v (-> cache)
@@ -166,5 +203,41 @@ int launch_attention_cached_simt(b200_ctx* ctx, const CachedAttention& c, const 
 // ldo columns); with gru.S also a minGRU step in further CTAs of the launch (gru.out: the same rows, out_col: its first column).
 int launch_attention_cached_decode(b200_ctx* ctx, const CachedAttention& c, const float* proj, int ld, uint8_t* out, int ldo,
                                    const SeqDesc* seqs, int B, const MinGruArgs& gru);
+
+// ---- latent attention (attention_latent.cu)
+// Keys and values of all heads are linear in one latent per token, W_uk c and W_uv c, beside a rotated key part that the heads
+// share.  The cache holds the latent and that part: rows [c: R | rotated: Dr | zeros up to Lp], [slots][Tp][Lp], fp16 or fp32.
+// A sequence's step is computed in one of two ways (SeqDesc::kv0):
+//   expanded   many tokens: keys and values of all positions are formed by one product over the cached rows, whose weight
+//              passes the rotated part on, and attended to by the kernels of attention_cached.cu
+//   latent     few tokens (16-bit arithmetic): the queries are taken into the latent's space, q W_uk, scored against the cached rows
+//              themselves, and W_uv is applied to the weighted sum of latents
+struct LatentAttention {
+    int H, D, Dr, Dv, R;           // per head: D unrotated and Dr rotated dimensions, values of Dv
+    int Lp, Tp, Dp, Dvp;           // Dp, Dvp: padded heads of the expanded keys and values
+    int q_col, c_col;              // columns of the projection: heads D + Dr apart; latent, then rotated key part
+    const float2* rot;             // [Tp][Dr / 2] (cos, sin); pairs are neighbouring dimensions
+    const float* c_norm;
+    float scale, eps;
+    void* cache;
+    const uint16_t* Wuk;           // [H * D][Rp] bf16, Rp = R rounded up to 8
+    const uint16_t* Wuv;           // [H * Dv][Rp]
+    int Rp;
+};
+int latent_row_pad(int r);  // Lp of rows of r values; 0: unsupported
+// norm and rotation of the step's rows: -> cache, and for the expanded sequences -> lat (rows kv0 + position, Lp columns) and their
+// queries -> q_out [M][H * Dp]
+int launch_latent_prep(b200_ctx* ctx, const LatentAttention& c, const float* proj, int ld, void* q_out, void* lat, const SeqDesc* seqs, const int* row_seq,
+                       int M, bool f32);
+// cached rows of earlier steps of the expanded sequences -> lat
+int launch_latent_gather(b200_ctx* ctx, const LatentAttention& c, void* lat, const SeqDesc* seqs, int E, int max_pos0, bool f32);
+// queries of rows[0 .. n) (null: 0 .. n - 1) in the latent's space -> ql [n][H][Lp] fp16; append: the rows' latents go to the cache too (one
+// token per sequence: row i is sequence i's)
+int launch_latent_query(b200_ctx* ctx, const LatentAttention& c, const float* proj, int ld, void* ql, const SeqDesc* seqs, const int* row_seq,
+                        const int* rows, int n, bool append);
+// attention of ql's rows over the cached latents, W_uv applied, for sequences list[0 .. n) (null: 0 .. n - 1) of at most max_n
+// tokens that see at most max_keys keys.  out: bf16, or split rows, of ldo columns.
+int launch_latent_attention(b200_ctx* ctx, const LatentAttention& c, const void* ql, void* out, int ldo, const SeqDesc* seqs, const int* list, int n, int max_n,
+                            int max_keys, bool split_rows);
 
 }  // namespace b200

@@ -26,6 +26,12 @@ __device__ __forceinline__ float gelu_erf_h(float z) {
     const float erfc = p * __expf(-x * x);  // of |z| / sqrt(2)
     return z >= 0.f ? z - 0.5f * z * erfc : 0.5f * z * erfc;
 }
+// a gate bounded above and its linear part, bounded on both sides, that counts from one: g sigmoid(1.702 g) (u + 1)
+__device__ __forceinline__ float clamped_gate(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoidf_(1.702f * g) * (u + 1.0f);
+}
 // 2^x on the special-function unit
 __device__ __forceinline__ float ex2(float x) {
     float y;

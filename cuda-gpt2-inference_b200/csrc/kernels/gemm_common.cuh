@@ -61,6 +61,12 @@ struct GemmArgs {
     // the last full round of the resident pairs - are each computed as tail_sub tiles of tile_w / tail_sub
     // columns, so that the partly empty last round costs a fraction of a tile's time (1: off)
     int tail_sub = 1, n_main = 0;
+    float gate_limit = 0.f;              // of GEMM_GATED_CLAMP
+    const int* group_blocks = nullptr;   // grouped product: see GemmGroups
+    int group_align = 0;
+    // tiles along M (of `rows` rows), and the first weight row of a tile's matrix
+    __device__ __forceinline__ int m_blocks(int rows) const { return group_blocks ? __ldg(group_blocks) * (group_align / rows) : num_m_blocks; }
+    __device__ __forceinline__ int weight_row0(int m_blk, int rows) const { return group_blocks ? __ldg(group_blocks + 1 + m_blk / (group_align / rows)) * N : 0; }
 };
 
 // Arg-max keys: the value as an order-preserving 32-bit integer in the high half, the inverted
@@ -166,6 +172,12 @@ __device__ __forceinline__ void gemm_drain_accumulator_bf16(const GemmArgs& args
                             lo[h * 16 + j * 4 + i] = *reinterpret_cast<const uint32_t*>(&ll);
                         }
                     }
+                } else if (args.flags & GEMM_FP16) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const __half2 hh = __floats2half2_rn(fminf(fmaxf(v[2 * i], -65504.f), 65504.f), fminf(fmaxf(v[2 * i + 1], -65504.f), 65504.f));
+                        pk[i] = *reinterpret_cast<const uint32_t*>(&hh);
+                    }
                 } else {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
@@ -208,6 +220,49 @@ __device__ __forceinline__ void gemm_drain_accumulator_bf16(const GemmArgs& args
     }
 }
 
+// Gated outputs: a pair of 32-column chunks - gates, linear values - leaves as 32 16-bit columns, through one of the
+// warp's staging buffers (rows 80 bytes apart) so that four lanes write 64 contiguous bytes of a row.  c_begin, c_end even.
+__device__ __forceinline__ void gemm_drain_accumulator_gated(const GemmArgs& args, uint32_t tmem_acc, int q, int lane, int row0, int col0, uint8_t* stage,
+                                                             int c_begin, int c_end) {
+    const bool clamp = (args.flags & GEMM_GATED_CLAMP) != 0;
+    const int half_n = args.N >> 1;
+#pragma unroll 1
+    for (int c = c_begin; c < c_end; c += 2) {
+        uint32_t r0[32], r1[32];
+        tmem_ld_32x32b_x32(tmem_acc + (uint32_t(q * 32) << 16) + c * 32, r0);
+        tmem_ld_32x32b_x32(tmem_acc + (uint32_t(q * 32) << 16) + c * 32 + 32, r1);
+        tmem_ld_wait();
+        const int cbase = (col0 + c * 32) >> 1;
+        __syncwarp();  // the previous pair has been read back
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            uint32_t pk[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                float v[2];
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const float g = __uint_as_float(r0[8 * j + 2 * i + e]), u = __uint_as_float(r1[8 * j + 2 * i + e]);
+                    v[e] = clamp ? clamped_gate(g, u, args.gate_limit) : gelu_tanh(g) * u;
+                }
+                pk[i] = pack_bf16(v[0], v[1]);
+            }
+            *reinterpret_cast<uint4*>(stage + lane * 80 + j * 16) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+        }
+        __syncwarp();
+        if (cbase < half_n) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int rl = i * 8 + (lane >> 2);
+                if (row0 + rl < args.M)
+                    *reinterpret_cast<uint4*>(args.out_h + (size_t)(row0 + rl) * half_n + cbase + (lane & 3) * 8) =
+                        *reinterpret_cast<const uint4*>(stage + rl * 80 + (lane & 3) * 16);
+            }
+        }
+    }
+    __syncwarp();
+}
+
 //   bias_first : gemm_bias_chunk(bias, args.N, col0, c_begin, lane)
 __device__ __forceinline__ void gemm_drain_accumulator(const GemmArgs& args, const float* bias, const CUtensorMap* tmap_out, uint32_t tmem_acc,
                                                        int q, int lane, int row0, int col0, uint8_t* stage2, float bias_first,
@@ -238,6 +293,10 @@ __device__ __forceinline__ void gemm_drain_accumulator(const GemmArgs& args, con
     if (via_tma) {  // the stores of the previous tile have left the staging buffers
         if (lane == 0) tma_store_wait_read();
         __syncwarp();
+    }
+    if (args.flags & (GEMM_GATED_GELU | GEMM_GATED_CLAMP)) {
+        gemm_drain_accumulator_gated(args, tmem_acc, q, lane, row0, col0, stage2, c_begin, c_end);
+        return;
     }
     if (args.out_h) {
         gemm_drain_accumulator_bf16(args, bias, tmap_out, tmem_acc, q, lane, row0, col0, stage2, bias_first, c_begin, c_end, nbuf);
@@ -377,6 +436,7 @@ int preload_gemm_pair_kernels(b200_ctx* ctx);  // the PAIR_TF32 kernel: loaded n
 int launch_gemm_pair(b200_ctx* ctx, float* out, const void* inp, const void* inp_lo, const void* weight, const void* weight_lo,
                      const float* bias, const float* residual, int M, int K, int N, int flags,
                      unsigned long long* argmax_keys, int argmax_cols, int kind, uint16_t* out_h = nullptr,
-                     int out_planes = 0, int store_period = 0, const GemmRowStats* stats = nullptr, float alpha = 1.0f, int lo_col0 = 0);
+                     int out_planes = 0, int store_period = 0, const GemmRowStats* stats = nullptr, float alpha = 1.0f, int lo_col0 = 0,
+                     float gate_limit = 0.f, const GemmGroups* groups = nullptr);
 
 }  // namespace b200

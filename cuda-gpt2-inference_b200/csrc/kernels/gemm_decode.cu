@@ -16,6 +16,12 @@
 //
 // Narrow outputs: K is cut into slices computed by the CTAs of a cluster, whose partial sums the first of them
 // reads out of the others' shared memory, in rank order.
+//
+// Gated outputs: a tile is eight gate rows and their eight linear rows, so the two meet in the same epilogue.
+//
+// Table-routed experts: blockIdx.y numbers the (input row, choice) pairs.  The first pair of a matrix takes all input rows
+// that chose it, the later ones find that out and leave.  (The ids and the table are read before the previous
+// kernel has finished: they were there before it started.)
 #include "decoder_kernels.h"
 #include "decoder_math.cuh"
 #include "../prim/sm100.cuh"
@@ -27,6 +33,7 @@ constexpr int kThreads = 256, kWarps = 8;
 constexpr int kU = 8;             // pieces of a warp on the way
 constexpr int kTwoCtaSmem = 103 * 1024;  // input rows of a CTA that still leave room for a second one ...
 constexpr int kOneCtaSmem = 200 * 1024;  // ... and the most a CTA can hold
+constexpr int kMaxPairs = 256;    // (input row, expert) pairs
 constexpr int kMaxTaps = 4;       // convolution inputs requested ahead of the product (longer ones behind it)
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t a0, const uint32_t a1, const uint32_t a2, const uint32_t a3,
@@ -44,19 +51,37 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
     extern __shared__ __align__(16) uint8_t xs[];
     __shared__ float red[NT][kWarps][16][9];
     __shared__ float part[NT * 128];
+    __shared__ int expert[kMaxPairs], x_row[NT * 8], o_row[NT * 8];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
-    const int K = a.K, N = a.N, B = a.B;
+    const int B = a.B, pairs = B * a.top, job = blockIdx.y;
+    const bool shared_job = pairs > 0 && job == pairs, routed = pairs > 0 && !shared_job, gated = a.gate != GATE_NONE;
+    const int K = shared_job ? a.shared.K : a.K, N = shared_job ? a.shared.N : a.N;
+    const uint8_t* xin = shared_job ? a.shared.x : a.x;
+    size_t w_off = 0;
+    if (routed) {
+        if (tid < pairs) expert[tid] = __ldg(a.table + (size_t)a.tok[tid / a.top] * a.top + tid % a.top);
+        if (tid < NT * 8) x_row[tid] = o_row[tid] = -1;
+        __syncthreads();
+        const int e = expert[job];
+        if (__syncthreads_or(tid < job && expert[tid] == e)) return;  // an earlier pair's CTAs do this one as well
+        if (tid < pairs && expert[tid] == e) {
+            o_row[tid / a.top] = tid;
+            x_row[tid / a.top] = a.pair_in ? tid : tid / a.top;
+        }
+        __syncthreads();
+        w_off = (size_t)e * N * K;
+    }
     const int tiles = (N + 15) >> 4;
     const int rank = slices > 1 ? (int)cluster_ctarank() : 0;
     const int tile0 = blockIdx.x / slices, tile_step = gridDim.x / slices;
     const int kb = min(K, rank * kslice), ke = min(K, kb + kslice);  // this CTA's columns (may be none)
     const int stride = chunk * 4 + 16;
-    const uint16_t* __restrict__ W = a.W;
+    const uint16_t* __restrict__ W = (shared_job ? a.shared.W : a.W) + w_off;
     // this warp's pieces of a chunk: 32 columns each, number warp, warp + 8, ...
     uint4 w[kU][2];
     auto request = [&](uint4 (&r)[2], int tile, int k0, int kend, int p) {
         const int k = k0 + p * 32 + c * 8;
-        const int r0 = tile * 16 + g, r1 = r0 + 8;
+        const int r0 = gated ? (tile >> 2) * 64 + (tile & 3) * 8 + g : tile * 16 + g, r1 = r0 + (gated ? 32 : 8);
         r[0] = r[1] = make_uint4(0u, 0u, 0u, 0u);
         if (k < kend) {
             if (r0 < N) r[0] = __ldg(reinterpret_cast<const uint4*>(W + (size_t)r0 * K + k));
@@ -99,9 +124,12 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
             if (!staged) {
                 if (k0 > kb || tile != tile0) __syncthreads();  // everyone is done with the previous chunk
                 const int n16 = (kend - k0) >> 2;               // 16-byte pieces of a row
-                for (int b = 0; b < B; ++b)
+                for (int b = 0; b < B; ++b) {
+                    const int xr = routed ? x_row[b] : b;
+                    if (xr < 0) continue;  // (whatever the row holds stays in its own column of the product)
                     for (int i = tid; i < n16; i += kThreads)
-                        cp_async16(xs + (size_t)b * stride + i * 16, a.x + ((size_t)b * K + k0) * 4 + i * 16);
+                        cp_async16(xs + (size_t)b * stride + i * 16, xin + ((size_t)xr * K + k0) * 4 + i * 16);
+                }
                 cp_async_commit();
                 cp_async_wait<0>();
                 __syncthreads();
@@ -158,18 +186,29 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
             }
             cluster_sync_all();
         }
-        if (rank == 0 && eb < B && eb < NT * 8 && er < N) {
+        auto total = [&](int row) {  // of the tile, for input row eb
             float v = 0.f;
             if (slices > 1) {
                 for (int s = 0; s < slices; ++s) {
                     float p;
-                    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(p) : "r"(map_to_cta(smem_u32(part + tid), s)) : "memory");
+                    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(p) : "r"(map_to_cta(smem_u32(part + (tid & ~15) + row), s)) : "memory");
                     v += p;
                 }
             } else {
 #pragma unroll
-                for (int q = 0; q < kWarps; ++q) v += red[eb >> 3][q][tid & 15][eb & 7];
+                for (int q = 0; q < kWarps; ++q) v += red[eb >> 3][q][row][eb & 7];
             }
+            return v;
+        };
+        const int out_row = (eb < B && eb < NT * 8) ? (routed ? o_row[eb] : eb) : -1;
+        if (rank == 0 && out_row >= 0 && gated) {
+            if ((tid & 15) < 8) {
+                const float gv = total(tid & 7), uv = total((tid & 7) + 8);
+                const float v = a.gate == GATE_CLAMP ? clamped_gate(gv, uv, shared_job ? a.shared.limit : a.limit) : gelu_tanh(gv) * uv;
+                store_split((shared_job ? a.shared.split_out : a.split_out) + (size_t)out_row * (N >> 1) * 4, (tile >> 2) * 32 + (tile & 3) * 8 + (tid & 7), v);
+            }
+        } else if (rank == 0 && out_row >= 0 && er < N) {
+            float v = total(tid & 15);
             if (a.bias) v += __ldg(a.bias + er);
             if (conv) {
                 const int hrows = a.taps - 1;
@@ -194,8 +233,9 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
             } else if (a.act == ACT_GELU_ERF) v = gelu_erf(v);
             else if (a.act == ACT_GELU_TANH) v = gelu_tanh(v);
             if (conv && a.conv_out) store_split(a.conv_out + (size_t)eb * a.conv_n * 4, er, v);
-            else if (a.split_out) store_split(a.split_out + (size_t)eb * N * 4, er, v);
-            else a.out[(size_t)eb * a.ldo + er] = v;
+            else if (a.split_out) store_split(a.split_out + (size_t)out_row * N * 4, er, v);
+            else if (shared_job) a.shared.out[(size_t)out_row * a.shared.ldo + er] = v;
+            else a.out[(size_t)out_row * a.ldo + er] = v;
         }
         if (slices > 1) cluster_sync_all();  // the partial sums have been read (and nobody leaves before that)
         else __syncthreads();
@@ -209,20 +249,24 @@ int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
         B200_CUDA(ctx, cudaFuncSetAttribute(decode_gemm_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kOneCtaSmem));
         attr_set[ctx->device & 63] = true;
     }
-    const int tiles = (a.N + 15) / 16;
+    const int jobs = a.top > 0 ? a.B * a.top + (a.shared.W ? 1 : 0) : 1;
+    const int max_n = jobs > 1 && a.shared.N > a.N ? a.shared.N : a.N, max_k = jobs > 1 && a.shared.K > a.K ? a.shared.K : a.K;
+    const int tiles = (max_n + 15) / 16;
     // K slices while the CTAs of one wave (two per SM) are not used up and a warp keeps at least a piece
     int slices = 1;
-    while (slices < 8 && tiles * slices * 2 <= 2 * ctx->num_sms && a.K / (slices * 2) >= 256) slices *= 2;
-    const int kslice = ((a.K + slices - 1) / slices + 31) / 32 * 32;
+    while (slices < 8 && jobs * tiles * slices * 2 <= 2 * ctx->num_sms && max_k / (slices * 2) >= 256) slices *= 2;
+    const int kslice = ((max_k + slices - 1) / slices + 31) / 32 * 32;
     // the columns staged at a time: all of the slice, so that they are staged once for all tiles; else as many as
     // two CTAs per SM can hold
     auto columns = [](int smem) { return (smem / (NT * 8) - 16) / 4 / 32 * 32; };
     const int chunk = kslice <= columns(kOneCtaSmem) ? kslice : columns(kTwoCtaSmem);
     const int per_sm = chunk <= columns(kTwoCtaSmem) ? 2 : 1;
     int grid = tiles * slices;
-    if (grid > per_sm * ctx->num_sms) grid = per_sm * ctx->num_sms / slices * slices;
+    int room = per_sm * ctx->num_sms / jobs;
+    if (room < slices) room = slices;
+    if (grid > room) grid = room / slices * slices;
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(grid);
+    cfg.gridDim = dim3(grid, jobs);
     cfg.blockDim = dim3(kThreads);
     cfg.dynamicSmemBytes = (size_t)NT * 8 * (chunk * 4 + 16);
     cfg.stream = ctx->stream;
@@ -251,6 +295,8 @@ int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
 
 int launch_decode_gemm(b200_ctx* ctx, const DecodeGemmArgs& a) {
     if (a.B < 1 || a.B > 16 || a.K % 8 || a.N < 1) return B200_ERR_SHAPE;
+    if (a.top < 0 || a.B * a.top > kMaxPairs || (a.top > 0 && a.conv_n > 0) || (a.gate != GATE_NONE && (a.N % 64 || !a.split_out))) return B200_ERR_SHAPE;
+    if (a.shared.W && (a.top < 1 || a.shared.K % 8 || (a.gate != GATE_NONE && (a.shared.N % 64 || !a.shared.split_out)))) return B200_ERR_SHAPE;
     return a.B <= 8 ? launch_one<1>(ctx, a) : launch_one<2>(ctx, a);
 }
 

@@ -14,13 +14,18 @@ constexpr int LDT = TM + 4;  // transposed tiles [TK][LDT]
 
 __global__ void __launch_bounds__(kThreads)
 gemm_fp32_kernel(float* __restrict__ out, const float* __restrict__ inp, const float* __restrict__ W,
-                 const float* __restrict__ bias, int M, int K, int N, int act) {
+                 const float* __restrict__ bias, int M, int K, int N, int act, const int* __restrict__ group_blocks, int group_align) {
     __shared__ __align__(16) float as[2][TK][LDT];
     __shared__ __align__(16) float bs[2][TK][LDT];
     griddep_wait();
     griddep_launch_dependents();
     const int tid = threadIdx.x;
     const int m0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
+    if (group_blocks) {  // grouped: runs of group_align rows with a matrix each (GemmGroups)
+        const int run = m0 / group_align;
+        if (run >= group_blocks[0]) return;
+        W += (size_t)group_blocks[1 + run] * N * K;
+    }
     const int lr = tid >> 2, lk = (tid & 3) * 4;  // each thread stages 4 consecutive k of one row of either operand
     const int tx = tid & 15, ty = tid >> 4;
     const bool a_ok = m0 + lr < M, b_ok = n0 + lr < N;
@@ -84,10 +89,11 @@ gemm_fp32_kernel(float* __restrict__ out, const float* __restrict__ inp, const f
 
 }  // namespace
 
-int launch_gemm_fp32(b200_ctx* ctx, float* out, const float* inp, const float* W, const float* bias, int M, int K, int N, int act) {
-    if (K % 4 || N % 4) return B200_ERR_SHAPE;
+int launch_gemm_fp32(b200_ctx* ctx, float* out, const float* inp, const float* W, const float* bias, int M, int K, int N, int act, const GemmGroups* groups) {
+    if (K % 4 || N % 4 || (groups && groups->align % TM)) return B200_ERR_SHAPE;
     if (M <= 0) return B200_OK;
-    cudaError_t le = launch_pdl(ctx, gemm_fp32_kernel, dim3((N + TN - 1) / TN, (M + TM - 1) / TM), dim3(kThreads), 0, out, inp, W, bias, M, K, N, act);
+    cudaError_t le = launch_pdl(ctx, gemm_fp32_kernel, dim3((N + TN - 1) / TN, (M + TM - 1) / TM), dim3(kThreads), 0, out, inp, W, bias, M, K, N, act,
+                                groups ? groups->blocks : nullptr, groups ? groups->align : 0);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;

@@ -89,7 +89,6 @@ gemm_tf32_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
 
     const int warp = threadIdx.x >> 5;
     const int lane = threadIdx.x & 31;
-    const int num_tiles = args.num_m_blocks * args.num_n_blocks;
     constexpr int BKE = BF16 ? kGemmBKH : BK;  // elements per 128-byte K block
     const int num_kb = (args.K + BKE - 1) / BKE;
 
@@ -117,9 +116,10 @@ gemm_tf32_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
     const uint32_t tmem_base = *tmem_holder;
     griddep_wait();  // set-up done; from here on global memory is touched
 
+    const int num_m_blocks = args.m_blocks(BM), num_tiles = num_m_blocks * args.num_n_blocks;
     auto tile_coords = [&](int tile, int& m_blk, int& n_blk) {
         if (args.n_fastest) { n_blk = tile % args.num_n_blocks; m_blk = tile / args.num_n_blocks; }
-        else { m_blk = tile % args.num_m_blocks; n_blk = tile / args.num_m_blocks; }
+        else { m_blk = tile % num_m_blocks; n_blk = tile / num_m_blocks; }
     };
 
     if (warp == 0) {
@@ -130,13 +130,14 @@ gemm_tf32_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
             for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
                 int m_blk, n_blk;
                 tile_coords(tile, m_blk, n_blk);
+                const int row_b = args.weight_row0(m_blk, BM) + n_blk * BN;
                 for (int kb = 0; kb < num_kb; ++kb, ++it) {
                     const int s = it % STAGES;
                     const uint32_t ph = (it / STAGES) & 1;
                     if (!mbar_wait(&empty_bar[s], ph ^ 1, abort_flag)) { ok = false; break; }
                     mbar_arrive_expect_tx(&full_bar[s], Cfg::TX_BYTES);
                     tma_load_2d(smem_a + s * Cfg::A_BYTES, &tmap_a, kb * BKE, m_blk * BM, &full_bar[s]);
-                    tma_load_2d(smem_b + s * Cfg::B_BYTES, &tmap_b, kb * BKE, n_blk * BN, &full_bar[s]);
+                    tma_load_2d(smem_b + s * Cfg::B_BYTES, &tmap_b, kb * BKE, row_b, &full_bar[s]);
                 }
             }
             if (!ok) atomicCAS(args.status, 0, DEV_TIMEOUT_PRODUCER);
@@ -144,7 +145,7 @@ gemm_tf32_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
     } else if (warp == 1) {
         // -------------------------------------------------------------- MMA issuer
         if (lane == 0) {
-            constexpr uint32_t idesc = BF16 ? make_idesc_bf16(BM, BN, 0) : make_idesc_tf32(BM, BN, 0);
+            const uint32_t idesc = !BF16 ? make_idesc_tf32(BM, BN, 0) : ((args.flags & GEMM_FP16) ? make_idesc_f16(BM, BN, 0) : make_idesc_bf16(BM, BN, 0));
             uint32_t it = 0;
             bool ok = true;
             int tile_iter = 0;
@@ -283,7 +284,8 @@ namespace {
 // bf16 != 0: inp / weight hold bf16 elements and out_h (if not null) receives the output as bf16.
 int launch_gemm_any(b200_ctx* ctx, float* out, uint16_t* out_h, const void* inp, const void* weight,
                     const float* bias, const float* residual, int M, int K, int N, int flags,
-                    int mode, unsigned long long* argmax_keys, int argmax_cols, bool bf16, int store_period, const GemmRowStats* stats) {
+                    int mode, unsigned long long* argmax_keys, int argmax_cols, bool bf16, int store_period, const GemmRowStats* stats,
+                    float gate_limit = 0.f, const GemmGroups* groups = nullptr) {
     if ((flags & GEMM_ACCUM_OUT) && (residual || out_h)) { ctx->last_error = "GEMM_ACCUM_OUT: fp32 output without a residual operand"; return B200_ERR_STATE; }
     if (store_period && (store_period % 32 || residual || !argmax_keys)) { ctx->last_error = "store_period: multiple of 32, with the fused arg-max only"; return B200_ERR_STATE; }
     const bool x3 = (mode == B200_TF32X3);
@@ -320,14 +322,18 @@ int launch_gemm_any(b200_ctx* ctx, float* out, uint16_t* out_h, const void* inp,
     bool use_pair = M >= 2048 && (N >= 2048 || K >= 2048);
     if (bf16) use_pair = M >= 2048 && (long)((M + 255) / 256) * ((N + 255) / 256) >= ctx->num_sms / 2;
     if (pair_env >= 0) use_pair = pair_env == 1;
+    if (groups && groups->align < 2 * BM) use_pair = false;
     if (stats) {  // the sampling / log-sum-exp epilogue lives in the CTA-pair kernel
         if (x3) { ctx->last_error = "row statistics are not available with 3xTF32 GEMMs"; return B200_ERR_STATE; }
         use_pair = true;
     }
     if (!x3 && use_pair)
         return launch_gemm_pair(ctx, out, inp, nullptr, weight, nullptr, bias, residual, M, K, N, flags, argmax_keys, argmax_cols,
-                                bf16 ? PAIR_BF16 : PAIR_TF32, out_h, 0, store_period, stats);
+                                bf16 ? PAIR_BF16 : PAIR_TF32, out_h, 0, store_period, stats, 1.0f, 0, gate_limit, groups);
     GemmArgs a;
+    a.gate_limit = gate_limit;
+    if (groups) { a.group_blocks = groups->blocks; a.group_align = groups->align; }
+    const uint64_t w_rows = (uint64_t)N * (groups ? groups->matrices : 1);
     a.out = out; a.out_h = out_h; a.bias = bias; a.residual = residual;
     a.M = M; a.N = N; a.K = K;
     a.num_m_blocks = num_m;
@@ -362,7 +368,7 @@ int launch_gemm_any(b200_ctx* ctx, float* out, uint16_t* out_h, const void* inp,
     if (bf16) {
         st = b200_get_tensor_map_bf16(ctx, &ta, inp, (uint64_t)M, (uint64_t)K, (uint64_t)K, BM, kGemmBKH);
         if (st != B200_OK) return st;
-        st = b200_get_tensor_map_bf16(ctx, &tb, weight, (uint64_t)N, (uint64_t)K, (uint64_t)K, (uint32_t)best_bn, kGemmBKH);
+        st = b200_get_tensor_map_bf16(ctx, &tb, weight, w_rows, (uint64_t)K, (uint64_t)K, (uint32_t)best_bn, kGemmBKH);
         if (st != B200_OK) return st;
     } else {
         st = b200_get_tensor_map(ctx, &ta, static_cast<const float*>(inp), (uint64_t)M, (uint64_t)K, (uint64_t)K, BM, BK);
@@ -371,7 +377,8 @@ int launch_gemm_any(b200_ctx* ctx, float* out, uint16_t* out_h, const void* inp,
         if (st != B200_OK) return st;
     }
     // the output in 32 x 32 boxes of fp32 (32 x 64 of bf16), for the epilogue's TMA stores
-    if (out_h) st = b200_get_tensor_map_bf16(ctx, &to, out_h, (uint64_t)M, (uint64_t)N, (uint64_t)N, 32, 64);
+    if (flags & (GEMM_GATED_GELU | GEMM_GATED_CLAMP)) to = ta;  // (not used: plain stores)
+    else if (out_h) st = b200_get_tensor_map_bf16(ctx, &to, out_h, (uint64_t)M, (uint64_t)N, (uint64_t)N, 32, 64);
     else st = b200_get_tensor_map(ctx, &to, out, (uint64_t)M, (uint64_t)N, (uint64_t)N, 32, 32);
     if (st != B200_OK) return st;
     if (bf16) {
@@ -434,10 +441,14 @@ int launch_gemm_bf16x3(b200_ctx* ctx, float* out, uint16_t* out_planes, const ui
 
 int launch_gemm_bf16(b200_ctx* ctx, float* out, uint16_t* out_h, const uint16_t* inp, const uint16_t* weight,
                      const float* bias, int M, int K, int N, int flags,
-                     unsigned long long* argmax_keys, int argmax_cols, int store_period) {
+                     unsigned long long* argmax_keys, int argmax_cols, int store_period, float gate_limit, const GemmGroups* groups) {
+    const int gated = flags & (GEMM_GATED_GELU | GEMM_GATED_CLAMP);
+    if (gated && (!out_h || N % 64 || bias || (flags & GEMM_FP16))) { ctx->last_error = "bf16 GEMM: a gated output is bf16, N a multiple of 64, no bias"; return B200_ERR_SHAPE; }
+    if (groups && (groups->align != BM && groups->align != 2 * BM)) { ctx->last_error = "grouped GEMM: runs of 128 or 256 rows"; return B200_ERR_SHAPE; }
     if (K % 8 || N % 8) { ctx->last_error = "bf16 GEMM: K and N must be multiples of 8"; return B200_ERR_SHAPE; }
     if ((flags & GEMM_GELU_ERF) && !out_h) { ctx->last_error = "GEMM_GELU_ERF: 16-bit output only"; return B200_ERR_STATE; }
-    return launch_gemm_any(ctx, out, out_h, inp, weight, bias, nullptr, M, K, N, flags & (GEMM_GELU | GEMM_GELU_ERF | GEMM_ROUND_OUT_TF32 | GEMM_ACCUM_OUT), B200_TF32, argmax_keys, argmax_cols, true, store_period, nullptr);
+    return launch_gemm_any(ctx, out, out_h, inp, weight, bias, nullptr, M, K, N, flags & (GEMM_GELU | GEMM_GELU_ERF | GEMM_ROUND_OUT_TF32 | GEMM_ACCUM_OUT | GEMM_GATED_GELU | GEMM_GATED_CLAMP | GEMM_FP16), B200_TF32, argmax_keys, argmax_cols, true, store_period, nullptr,
+                           gate_limit, groups);
 }
 
 // e4m3 operands: always on CTA pairs (the kernel clips ragged edges itself)

@@ -87,9 +87,10 @@ struct PairCfg {
 
 // The tiles of one CTA pair, in order.  Every role of both CTAs walks the same sequence.
 struct TileWalk {
-    int cur, step, total, tiles;
+    int cur, step, total, tiles, m_blocks;
     __device__ TileWalk(const GemmArgs& a, int pair, int num_pairs)
-        : cur(pair), step(num_pairs), tiles(a.num_m_blocks * a.num_n_blocks) {
+        : cur(pair), step(num_pairs), m_blocks(a.m_blocks(2 * BM)) {
+        tiles = m_blocks * a.num_n_blocks;
         total = a.tail_sub > 1 ? a.n_main + (tiles - a.n_main) * a.tail_sub : a.k_splits * tiles;
     }
     // next tile: 256 rows from m_blk * 256, `width` columns from col0, K blocks [kb0, kb1) (slice ks
@@ -112,7 +113,7 @@ struct TileWalk {
         }
         int n_blk;
         if (a.n_fastest) { m_blk = tile / a.num_n_blocks; n_blk = tile - m_blk * a.num_n_blocks; }
-        else { n_blk = tile / a.num_m_blocks; m_blk = tile - n_blk * a.num_m_blocks; }
+        else { n_blk = tile / m_blocks; m_blk = tile - n_blk * m_blocks; }
         col0 = n_blk * a.tile_w;
         const int rest = (a.N - col0 + a.unit_cols - 1) / a.unit_cols * a.unit_cols;
         width = rest < a.tile_w ? rest : a.tile_w;
@@ -211,7 +212,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                 // a ragged last tile is narrower: its halves start closer together, the box keeps its
                 // size (the rows behind the half are loaded but not multiplied)
                 const int row_a = m_blk * 2 * BM + (int)rank * BM;
-                const int row_b = col0 + (int)rank * (width >> 1);
+                const int row_b = args.weight_row0(m_blk, 2 * BM) + col0 + (int)rank * (width >> 1);
                 for (int kb = kb0; kb < kb1; ++kb, ++it) {
                     const int s = it % STAGES;
                     const uint32_t ph = (it / STAGES) & 1;
@@ -247,7 +248,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                 if (!mbar_wait_cluster(&tmem_empty_bar[acc], acc_ph ^ 1, abort_flag)) { ok = false; break; }
                 tc_fence_after_sync();
                 const uint32_t idesc = (MODE == PAIR_TF32) ? make_idesc_tf32(2 * BM, width, 0)
-                                     : (MODE == PAIR_FP8 ? make_idesc_e4m3(2 * BM, width, 0) : make_idesc_bf16(2 * BM, width, 0));
+                                     : (MODE == PAIR_FP8 ? make_idesc_e4m3(2 * BM, width, 0)
+                                     : (MODE == PAIR_BF16 && (args.flags & GEMM_FP16) ? make_idesc_f16(2 * BM, width, 0) : make_idesc_bf16(2 * BM, width, 0)));
                 const uint32_t d_tmem = tmem_base + acc * kMaxW;
                 for (int kb = kb0; kb < kb1; ++kb, ++it) {
                     const int s = it % STAGES;
@@ -421,7 +423,7 @@ int preload_gemm_pair_kernels(b200_ctx* ctx) {
 int launch_gemm_pair(b200_ctx* ctx, float* out, const void* inp, const void* inp_lo, const void* weight, const void* weight_lo,
                      const float* bias, const float* residual, int M, int K, int N, int flags,
                      unsigned long long* argmax_keys, int argmax_cols, int kind, uint16_t* out_h, int out_planes,
-                     int store_period, const GemmRowStats* stats, float alpha, int lo_col0) {
+                     int store_period, const GemmRowStats* stats, float alpha, int lo_col0, float gate_limit, const GemmGroups* groups) {
     const int num_pairs_max = ctx->num_sms / 2;
     const bool half = kind == PAIR_BF16 || kind == PAIR_BF16X3;
     GemmArgs a;
@@ -429,6 +431,9 @@ int launch_gemm_pair(b200_ctx* ctx, float* out, const void* inp, const void* inp
     a.M = M; a.N = N; a.K = K;
     a.alpha = alpha;
     a.lo_col0 = lo_col0;
+    a.gate_limit = gate_limit;
+    if (groups) { a.group_blocks = groups->blocks; a.group_align = groups->align; }
+    const uint64_t w_rows = (uint64_t)N * (groups ? groups->matrices : 1);
     a.tmap_out2 = static_cast<const CUtensorMap*>(ctx->next_gemm_out2);
     ctx->next_gemm_out2 = nullptr;
     a.out2_rows = a.tmap_out2 ? ctx->next_gemm_out2_rows : 0;
@@ -477,7 +482,7 @@ int launch_gemm_pair(b200_ctx* ctx, float* out, const void* inp, const void* inp
             // (8192 x 3072 x 768, split operands): 91 us against 95 without the tail and 97 with 192-wide
             // tiles, which this model would otherwise prefer by a percent - hence the 0.4 of a round.
             const long left = tiles % num_pairs_max;
-            if (ks == 1 && w == kMaxW && N % kMaxW == 0 && !stats && !argmax_keys && tiles > num_pairs_max && left > 0 && left * 4 <= num_pairs_max)
+            if (ks == 1 && w == kMaxW && N % kMaxW == 0 && !stats && !argmax_keys && !groups && tiles > num_pairs_max && left > 0 && left * 4 <= num_pairs_max)
                 waves = (double)(tiles / num_pairs_max) + 0.4;
             const double tensor = 2.0 * w * products, feed = parts * (128.0 + w / 2) * 128.0 / 52.0;
             // a slice also waits for its predecessor's sums to land and for its own before it signals
@@ -504,7 +509,7 @@ int launch_gemm_pair(b200_ctx* ctx, float* out, const void* inp, const void* inp
     const uint32_t box_b = (uint32_t)(best_w / 2);
     if (half) {
         st = b200_get_tensor_map_bf16(ctx, &maps[0], inp, (uint64_t)M, (uint64_t)K, (uint64_t)K, BM, bke);
-        if (st == B200_OK) st = b200_get_tensor_map_bf16(ctx, &maps[2], weight, (uint64_t)N, (uint64_t)K, (uint64_t)K, box_b, bke);
+        if (st == B200_OK) st = b200_get_tensor_map_bf16(ctx, &maps[2], weight, w_rows, (uint64_t)K, (uint64_t)K, box_b, bke);
         if (st != B200_OK) return st;
         if (kind == PAIR_BF16X3) {
             st = b200_get_tensor_map_bf16(ctx, &maps[1], inp_lo, (uint64_t)M, (uint64_t)K, (uint64_t)K, BM, bke);
@@ -525,14 +530,15 @@ int launch_gemm_pair(b200_ctx* ctx, float* out, const void* inp, const void* inp
         maps[1] = maps[0]; maps[3] = maps[2];
     }
     // the output in 32 x 32 boxes of fp32 (32 x 64 of bf16, both planes in one map), for the epilogue's TMA stores
-    if (out_h) st = b200_get_tensor_map_bf16(ctx, &maps[4], out_h, (uint64_t)M * (out_planes ? 2 : 1), (uint64_t)N, (uint64_t)N, 32, 64);
+    if (flags & (GEMM_GATED_GELU | GEMM_GATED_CLAMP)) maps[4] = maps[0];  // (not used: plain stores)
+    else if (out_h) st = b200_get_tensor_map_bf16(ctx, &maps[4], out_h, (uint64_t)M * (out_planes ? 2 : 1), (uint64_t)N, (uint64_t)N, 32, 64);
     else st = b200_get_tensor_map(ctx, &maps[4], out, (uint64_t)M, (uint64_t)N, (uint64_t)N, 32, 32);
     if (st != B200_OK) return st;
     // Tail of the tile sequence in narrow tiles (see GemmArgs::tail_sub): full-width tiles, whole in N, no K
     // slices, no per-tile row statistics; the weight comes in boxes of a quarter of the rows
     maps[5] = maps[2]; maps[6] = maps[3];
     a.tail_sub = 1; a.n_main = 0;
-    if (best_ks == 1 && best_w == kMaxW && N % kMaxW == 0 && !stats && !argmax_keys) {
+    if (best_ks == 1 && best_w == kMaxW && N % kMaxW == 0 && !stats && !argmax_keys && !groups) {
         const uint32_t box_n = (uint32_t)(best_w / 4 / 2);
         if (kind == PAIR_FP8) st = b200_get_tensor_map_u8(ctx, &maps[5], weight, (uint64_t)N, (uint64_t)K, (uint64_t)K, box_n, bke);
         else if (half) st = b200_get_tensor_map_bf16(ctx, &maps[5], weight, (uint64_t)N, (uint64_t)K, (uint64_t)K, box_n, bke);

@@ -56,8 +56,17 @@ int preload_attention_kernel(b200_ctx* ctx);
 // tiles leave as TMA reductions).  With out = the residual stream this is the residual add.
 // GEMM_PLANES_FP16: a split output (launch_gemm_bf16x3 with out_planes) is written as two fp16 planes instead of bf16
 // GEMM_GELU_ERF: the exact gelu instead of the tanh form (16-bit outputs only)
-enum : int { GEMM_GELU = 1, GEMM_ROUND_OUT_TF32 = 2, GEMM_ACCUM_OUT = 4, GEMM_PLANES_FP16 = 8, GEMM_GELU_ERF = 16 };
+// GEMM_GATED_GELU, GEMM_GATED_CLAMP: the columns come in blocks of 64, 32 gates and the 32 linear values that belong to
+// them, and the output has half as many: gelu_tanh(g) u, or clamped_gate(g, u, limit) (decoder_math.cuh) (launch_gemm_bf16
+// with a 16-bit output; N a multiple of 64)
+// GEMM_FP16: both operands, and a 16-bit output, hold fp16 instead of bf16 (launch_gemm_bf16)
+enum : int { GEMM_GELU = 1, GEMM_ROUND_OUT_TF32 = 2, GEMM_ACCUM_OUT = 4, GEMM_PLANES_FP16 = 8, GEMM_GELU_ERF = 16,
+             GEMM_GATED_GELU = 32, GEMM_GATED_CLAMP = 64, GEMM_FP16 = 128 };
 struct GemmRowStats;
+// Grouped product: every run of `align` input rows (128 or 256) meets a weight matrix of its own.  weight holds
+// `matrices` of them, [matrices * N, K]; blocks[0] is the number of runs, blocks[1 + i] the matrix of run i (device memory; M
+// is the most rows there can be).
+struct GemmGroups { const int* blocks; int align, matrices; };
 int launch_gemm_tf32(b200_ctx* ctx, float* out, const float* inp, const float* weight,
                      const float* bias, const float* residual, int M, int K, int N, int flags,
                      int mode, unsigned long long* argmax_keys = nullptr, int argmax_cols = 0, int store_period = 0,
@@ -67,7 +76,8 @@ int launch_gemm_tf32(b200_ctx* ctx, float* out, const float* inp, const float* w
 // flags: GEMM_GELU only.  K and N multiples of 8.
 int launch_gemm_bf16(b200_ctx* ctx, float* out, uint16_t* out_h, const uint16_t* inp, const uint16_t* weight,
                      const float* bias, int M, int K, int N, int flags,
-                     unsigned long long* argmax_keys = nullptr, int argmax_cols = 0, int store_period = 0);
+                     unsigned long long* argmax_keys = nullptr, int argmax_cols = 0, int store_period = 0,
+                     float gate_limit = 0.f, const GemmGroups* groups = nullptr);
 // The same product from split bf16 operands (three kind::f16 products per K step, hi.hi + hi.lo +
 // lo.hi: 16 significant bits per operand).  inp holds two bf16 planes of [M,K]: hi = bf16(x) and,
 // M*K elements further on, lo = bf16(x - hi); weight_hi / weight_lo [N,K] likewise.  The result goes

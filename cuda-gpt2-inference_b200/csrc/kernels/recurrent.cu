@@ -219,10 +219,13 @@ selective_scan_kernel(const SelectiveScanArgs a) {
 // L = D / 16 lanes share a group of NC columns and keep 16 rows of each in registers (as pairs: one instruction
 // does two multiply-adds); lane l owns rows 4 (l + L i) .. + 3, so the lanes read consecutive 16-byte pieces of
 // k and q.
+// With a decay per key channel (CH) g is a vector over the rows of S: every row takes its decay in first, which is
+// a fourth operation per element, and the products read S already decayed:
+//   S <- diag(g) S,   u = beta (v - S^T k),   o = S^T q + (k.q) u,   S <- S + k u^T
 constexpr int kDeltaTok = 16;
 constexpr float kDeltaSmall = 1e-9f;
 
-template <int L, int NC>
+template <int L, int NC, bool CH = false>
 struct DeltaCore {
     static constexpr int D = 16 * L, CNT = 2 * NC;            // totals per token: R^T k of the columns, then R^T q
     static constexpr int kHeld = L >= CNT ? 1 : CNT / L;      // ... of which a lane holds this many after the reduction
@@ -258,7 +261,7 @@ struct DeltaCore {
         c = 1.f;
     }
     __device__ __forceinline__ void store(float* base, int l, int ncol) {
-        absorb();
+        if (!CH) absorb();
 #pragma unroll
         for (int j = 0; j < NC; ++j)
 #pragma unroll
@@ -281,12 +284,22 @@ struct DeltaCore {
         return x;
     }
     // One token.  kr: its key; qr: its query on entry, the row at q_next on return (requested as soon as the registers are
-    // free); v: the group's values in shared memory.
+    // free); v: the group's values in shared memory.  CH: the decays are gr (g is not used), the row at g_next on return.
     __device__ __forceinline__ void token(const Row& kr, Row& qr, const float* q_next, const float* v, float g, float beta, float kq, int lane,
-                                          float (&o)[kOut]) {
-        c *= g;
-        if (c < kDeltaSmall) absorb();  // (the same decay in all lanes of a head)
-        const float inv_c = __fdividef(1.0f, c);
+                                          float (&o)[kOut], Row* gr = nullptr, const float* g_next = nullptr) {
+        float inv_c = 1.f;
+        if constexpr (CH) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+#pragma unroll
+                for (int j = 0; j < NC; ++j) S[j][i] = mul2(gr->r[i], S[j][i]);
+            *gr = row(g_next, lane & (L - 1));
+        } else {
+            c *= g;
+            if (c < kDeltaSmall) absorb();  // (the same decay in all lanes of a head)
+            inv_c = __fdividef(1.0f, c);
+        }
+        const float cs = CH ? 1.f : c;
         uint64_t acc[CNT];
 #pragma unroll
         for (int j = 0; j < CNT; ++j) acc[j] = 0ull;
@@ -309,7 +322,7 @@ struct DeltaCore {
         const int first = scatter_first<CNT, L>(lane);  // t[j] is total number first + j
         float um[kOut];
 #pragma unroll
-        for (int j = 0; j < kOut; ++j) um[j] = beta * (v[(first + j) & (NC - 1)] - c * t[j]);
+        for (int j = 0; j < kOut; ++j) um[j] = beta * (v[(first + j) & (NC - 1)] - cs * t[j]);
         const int base = lane & ~(L - 1);
         float u[NC];
 #pragma unroll
@@ -320,11 +333,11 @@ struct DeltaCore {
             float uc = u[0];
 #pragma unroll
             for (int x = 1; x < NC; ++x) uc = col == x ? u[x] : uc;
-            o[j] = fmaf(c, t[j], kq * uc);
+            o[j] = fmaf(cs, t[j], kq * uc);
         }
 #pragma unroll
         for (int j = 0; j < NC; ++j) {
-            const float us = u[j] * inv_c;
+            const float us = CH ? u[j] : u[j] * inv_c;
             const uint64_t uu = pack2(us, us);
 #pragma unroll
             for (int i = 0; i < 8; ++i) S[j][i] = fma2(kr.r[i], uu, S[j][i]);
@@ -360,10 +373,23 @@ delta_prep_kernel(const DeltaArgs a) {
     const float qscale = rsqrtf((float)a.D);
     const int per = a.H / a.G;
     // the gates of the run's tokens and heads, side by side
+    if (a.decay) {
+        const int d4 = a.Dl >> 2, n4 = per * d4;  // the group's heads are neighbours
+        for (int i = lane; i < (t1 - t0) * n4; i += 32) {
+            const int t = t0 + i / n4, c4 = i % n4;
+            float4* dp = reinterpret_cast<float4*>(a.decay + (size_t)(sd.row0 + t) * a.ld_decay + (size_t)g * per * a.Dl) + c4;
+            const float4 b = __ldg(reinterpret_cast<const float4*>(a.dt_bias + (size_t)g * per * a.Dl) + c4);
+            const float A = __ldg(a.negA + g * per + c4 / d4);
+            float4 x = *dp;
+            x.x = expf(A * softplusf_(x.x + b.x)); x.y = expf(A * softplusf_(x.y + b.y));
+            x.z = expf(A * softplusf_(x.z + b.z)); x.w = expf(A * softplusf_(x.w + b.w));
+            *dp = x;
+        }
+    }
     for (int i = lane; i < (t1 - t0) * per; i += 32) {
         const int t = t0 + i / per, h = g * per + i % per;
         const float* gr = a.gates + (size_t)(sd.row0 + t) * a.ldg;
-        const float decay = expf(__ldg(a.negA + h) * softplusf_(gr[a.a_col + h] + __ldg(a.dt_bias + h)));
+        const float decay = a.decay ? 1.f : expf(__ldg(a.negA + h) * softplusf_(gr[a.a_col + h] + __ldg(a.dt_bias + h)));
         *reinterpret_cast<float2*>(a.coef + (size_t)(sd.row0 + t) * a.H + h) = make_float2(decay, sigmoidf_(gr[a.b_col + h]));
     }
     float w[2][V][W], win[2][V][W];  // weights and the window of earlier inputs
@@ -450,18 +476,21 @@ delta_prep_kernel(const DeltaArgs a) {
             }
 }
 
-// Prefill: a CTA walks one (sequence, head) for blockDim.x / L * NC columns of Dv, in tiles of 16 tokens staged two
-// deep by asynchronous copies.
-template <int L, int NC>
+// Prefill: a CTA walks one (sequence, head) for blockDim.x / L * NC columns of Dv, in tiles of 16 tokens (8 with a decay
+// per channel) staged two deep by asynchronous copies.
+__host__ __device__ constexpr int delta_tile_tokens(bool channel) { return channel ? 8 : kDeltaTok; }
+// floats of a tile: q, k, decays, v, coefficients
+__host__ __device__ constexpr int delta_tile_floats(int D, int cpad, bool channel) { return delta_tile_tokens(channel) * ((channel ? 3 : 2) * D + cpad + 4); }
+template <int L, int NC, bool CH>
 __global__ void __launch_bounds__(128)
 delta_scan_kernel(const DeltaArgs a) {
-    using Core = DeltaCore<L, NC>;
-    constexpr int D = 16 * L;
+    using Core = DeltaCore<L, NC, CH>;
+    constexpr int D = 16 * L, TOK = delta_tile_tokens(CH), VECS = CH ? 3 : 2;
     extern __shared__ __align__(16) float sm[];
     const int tid = threadIdx.x, lane = tid & 31;
     const int cols = blockDim.x / L * NC;
     const int cpad = (cols + 3) & ~3;
-    const int tile_f = kDeltaTok * (2 * D + cpad + 4);  // q, k, v, coefficients
+    const int tile_f = delta_tile_floats(D, cpad, CH);
     const int h = blockIdx.x, c0 = blockIdx.y * cols;
     const int kvh = h / (a.H / a.G);
     // rows of k and q beyond the head's dimension and columns beyond Dv stay zero in both tiles
@@ -482,41 +511,47 @@ delta_scan_kernel(const DeltaArgs a) {
     const float* src0 = a.qkv + (size_t)sd.row0 * a.ld;
     auto stage = [&](int t0, int buf) {
         float* q = sm + buf * tile_f;
-        const int nt = min(kDeltaTok, sd.n - t0);
-        const int per = 2 * d4 + v4;
+        const int nt = min(TOK, sd.n - t0);
+        const int per = VECS * d4 + v4;
         for (int j = tid; j < per; j += blockDim.x) {  // a 16-byte column piece of all tokens
             const float* src = src0 + (size_t)t0 * a.ld;
             float* dst;
-            int step;
-            if (j < d4) { src += kvh * a.Dl + j * 4; dst = q + j * 4; step = D; }
-            else if (j < 2 * d4) { src += a.k_col + kvh * a.Dl + (j - d4) * 4; dst = q + kDeltaTok * D + (j - d4) * 4; step = D; }
-            else { src += a.v_col + h * a.Dvl + c0 + (j - 2 * d4) * 4; dst = q + 2 * kDeltaTok * D + (j - 2 * d4) * 4; step = cpad; }
-            for (int t = 0; t < nt; ++t) cp_async16(dst + t * step, src + (size_t)t * a.ld);
+            int step = D, ld = a.ld;
+            if (j < d4) { src += kvh * a.Dl + j * 4; dst = q + j * 4; }
+            else if (j < 2 * d4) { src += a.k_col + kvh * a.Dl + (j - d4) * 4; dst = q + TOK * D + (j - d4) * 4; }
+            else if (CH && j < 3 * d4) {
+                ld = a.ld_decay;
+                src = a.decay + (size_t)(sd.row0 + t0) * ld + (size_t)h * a.Dl + (j - 2 * d4) * 4;
+                dst = q + 2 * TOK * D + (j - 2 * d4) * 4;
+            } else { src += a.v_col + h * a.Dvl + c0 + (j - VECS * d4) * 4; dst = q + VECS * TOK * D + (j - VECS * d4) * 4; step = cpad; }
+            for (int t = 0; t < nt; ++t) cp_async16(dst + t * step, src + (size_t)t * ld);
         }
-        if (tid < nt) cp_async16(q + kDeltaTok * (2 * D + cpad) + tid * 4, a.coef + (size_t)(sd.row0 + t0 + tid) * a.H + h);
+        if (tid < nt) cp_async16(q + TOK * (VECS * D + cpad) + tid * 4, a.coef + (size_t)(sd.row0 + t0 + tid) * a.H + h);
         cp_async_commit();
     };
     stage(0, 0);
     const int oc = Core::ocol(lane);
     const bool ow = Core::owns_o(lane);
     float* orow = a.out + (size_t)sd.row0 * a.ldo + h * a.Dvl + gc + oc;
-    for (int t0 = 0, it = 0; t0 < sd.n; t0 += kDeltaTok, ++it) {
-        const int buf = it & 1, nt = min(kDeltaTok, sd.n - t0);
-        if (t0 + kDeltaTok < sd.n) { stage(t0 + kDeltaTok, buf ^ 1); cp_async_wait<1>(); }
+    for (int t0 = 0, it = 0; t0 < sd.n; t0 += TOK, ++it) {
+        const int buf = it & 1, nt = min(TOK, sd.n - t0);
+        if (t0 + TOK < sd.n) { stage(t0 + TOK, buf ^ 1); cp_async_wait<1>(); }
         else cp_async_wait<0>();
         __syncthreads();
         const float* q = sm + buf * tile_f;
-        const float* k = q + kDeltaTok * D;
-        const float* v = k + kDeltaTok * D + grp * NC;
-        const float* cf = q + kDeltaTok * (2 * D + cpad);
-        typename Core::Row qr = Core::row(q, l), kr = Core::row(k, l);
+        const float* k = q + TOK * D;
+        const float* gd = k + TOK * D;  // (CH)
+        const float* v = q + VECS * TOK * D + grp * NC;
+        const float* cf = q + TOK * (VECS * D + cpad);
+        typename Core::Row qr = Core::row(q, l), kr = Core::row(k, l), gr;
+        if (CH) gr = Core::row(gd, l);
 #pragma unroll 2
         for (int t = 0; t < nt; ++t) {
             const float4 co = *reinterpret_cast<const float4*>(cf + t * 4);
-            const int tn = min(t + 1, kDeltaTok - 1);
+            const int tn = min(t + 1, TOK - 1);
             const typename Core::Row kn = Core::row(k + tn * D, l);
             float o[Core::kOut];
-            core.token(kr, qr, q + tn * D, v + t * cpad, co.x, co.y, co.z, lane, o);
+            core.token(kr, qr, q + tn * D, v + t * cpad, co.x, co.y, co.z, lane, o, &gr, gd + tn * D);
             kr = kn;
             if (ow) {
 #pragma unroll
@@ -530,14 +565,15 @@ delta_scan_kernel(const DeltaArgs a) {
     core.store(Sg, l, ncol);
 }
 
-// Decode: one CTA per (head, sequence) takes its token through unit norms, the rule, the output norm and the gate.
+// Decode: one CTA per (head, sequence) takes its token through unit norms, the rule, the output norm and the gate.  CH: the
+// decays and the output gate come from low-rank projections, whose second halves are formed here (eight lanes per row).
 constexpr int kDeltaStepThreads = 256, kDeltaStepCols = 4;
-template <int L>
+template <int L, bool CH>
 __global__ void __launch_bounds__(kDeltaStepThreads)
 delta_step_kernel(const DeltaArgs a) {
     constexpr int D = 16 * L, COLS = kDeltaStepThreads / L * kDeltaStepCols;
-    using Core = DeltaCore<L, kDeltaStepCols>;
-    extern __shared__ __align__(16) float sm[];  // q [D], k [D], v and o [vpad each]
+    using Core = DeltaCore<L, kDeltaStepCols, CH>;
+    extern __shared__ __align__(16) float sm[];  // q [D], k [D], v and o [vpad each]; CH: decays [D], gate [vpad], low-rank inputs
     __shared__ float red[8];
     float* q = sm;
     float* k = q + D;
@@ -546,8 +582,11 @@ delta_step_kernel(const DeltaArgs a) {
     float* o = v + vpad;
     const int tid = threadIdx.x, lane = tid & 31;
     const int h = blockIdx.x, per = a.H / a.G, kvh = h / per;
-    const float negA = __ldg(a.negA + h), dtb = __ldg(a.dt_bias + h);
-    for (int i = tid; i < 2 * D + 2 * vpad; i += kDeltaStepThreads) sm[i] = 0.f;
+    const float negA = __ldg(a.negA + h), dtb = CH ? 0.f : __ldg(a.dt_bias + h);
+    float* gd = o + vpad;
+    float* gate = gd + D;
+    float* low = gate + vpad;
+    for (int i = tid; i < (CH ? 3 * D + 3 * vpad : 2 * D + 2 * vpad); i += kDeltaStepThreads) sm[i] = 0.f;
     griddep_wait();
     griddep_launch_dependents();
     const SeqDesc sd = a.seqs[blockIdx.y];
@@ -567,12 +606,40 @@ delta_step_kernel(const DeltaArgs a) {
         else if (i < 2 * a.Dl) k[i - a.Dl] = row[a.k_col + kvh * a.Dl + i - a.Dl];
         else v[i - 2 * a.Dl] = row[a.v_col + h * a.Dvl + i - 2 * a.Dl];
     }
+    if (CH)
+        for (int i = tid; i < a.low_a + a.low_g; i += kDeltaStepThreads) low[i] = row[a.low_col + i];
     __syncthreads();
+    if (CH) {
+        constexpr int LR = 8;
+        const int sub = tid & (LR - 1);
+        for (int r = tid / LR; r < a.D + a.Dv; r += kDeltaStepThreads / LR) {
+            const bool is_g = r >= a.D;
+            const int d = is_g ? r - a.D : r, c0 = is_g ? a.low_a : 0, c1 = is_g ? a.low_a + a.low_g : a.low_a;
+            const uint16_t* wr = a.w_low + (size_t)(is_g ? a.gate_row + h * a.Dvl + d : h * a.Dl + d) * a.ld_low;
+            float s = 0.f;
+#pragma unroll 2
+            for (int c = c0 + sub * 8; c < c1; c += LR * 8) {  // (both halves start at multiples of eight columns)
+                const uint4 u = __ldg(reinterpret_cast<const uint4*>(wr + c));
+                const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    s = fmaf(__uint_as_float(w[e] << 16), low[c + 2 * e], s);
+                    s = fmaf(__uint_as_float(w[e] & 0xffff0000u), low[c + 2 * e + 1], s);
+                }
+            }
+#pragma unroll
+            for (int m = 1; m < LR; m <<= 1) s += __shfl_xor_sync(0xffu << (lane & 24), s, m);
+            if (sub == 0) {
+                if (is_g) gate[d] = sigmoidf_(s);
+                else gd[d] = expf(negA * softplusf_(s + __ldg(a.dt_bias + (size_t)h * a.Dl + d)));
+            }
+        }
+    }
     float sq = 0.f, sk = 0.f, dot = 0.f;  // every warp for itself
     for (int d = lane; d < D; d += 32) { sq = fmaf(q[d], q[d], sq); sk = fmaf(k[d], k[d], sk); dot = fmaf(q[d], k[d], dot); }
     sq = warp_sum(sq); sk = warp_sum(sk); dot = warp_sum(dot);
     const float rq = rsqrtf((float)a.D) / sqrtf(sq + 1e-6f), rk = 1.0f / sqrtf(sk + 1e-6f);
-    const float g = expf(negA * softplusf_(row[a.a_col + h] + dtb)), beta = sigmoidf_(row[a.b_col + h]);
+    const float g = CH ? 1.f : expf(negA * softplusf_(row[a.a_col + h] + dtb)), beta = sigmoidf_(row[a.b_col + h]);
     __syncthreads();
     for (int d = tid; d < D; d += kDeltaStepThreads) { q[d] *= rq; k[d] *= rk; }
     __syncthreads();
@@ -584,7 +651,9 @@ delta_step_kernel(const DeltaArgs a) {
         const int gc = c0 + grp * kDeltaStepCols, ncol = min(kDeltaStepCols, a.Dv - gc);
         if (c0 > 0) fetch(gc);
         float ov[Core::kOut];
-        core.token(kr, qr, q, v + gc, g, beta, dot * rq * rk, lane, ov);
+        typename Core::Row gr;
+        if (CH) gr = Core::row(gd, l);
+        core.token(kr, qr, q, v + gc, g, beta, dot * rq * rk, lane, ov, &gr, gd);
         if (ow) {
 #pragma unroll
             for (int j = 0; j < Core::kOut; ++j)
@@ -598,7 +667,7 @@ delta_step_kernel(const DeltaArgs a) {
     const float r = 1.0f / sqrtf(block_sum(s, red) / (float)a.Dv + a.eps);
     for (int d = tid; d < a.Dv; d += kDeltaStepThreads)
         store_split(reinterpret_cast<uint8_t*>(a.out) + (size_t)sd.row0 * a.ldo * 4, h * a.Dv + d,
-                    o[d] * r * __ldg(a.norm_w + d) * silu(row[a.gate_col + h * a.Dvl + d]));
+                    o[d] * r * __ldg(a.norm_w + d) * (CH ? gate[d] : silu(row[a.gate_col + h * a.Dvl + d])));
 }
 
 // ------------------------------------------------------------------ minGRU
@@ -695,18 +764,18 @@ int launch_scan_types(b200_ctx* ctx, const SelectiveScanArgs& a, int E, bool x_f
     return B200_ERR_SHAPE;
 }
 
-template <int L>
+template <int L, bool CH>
 int launch_delta_step_one(b200_ctx* ctx, const DeltaArgs& a, int E) {
     const int vpad = (a.Dvl + kDeltaStepThreads / L * kDeltaStepCols - 1) & ~3;
-    const size_t smem = (size_t)(32 * L + 2 * vpad) * 4;
-    if (smem > 48 * 1024) return B200_ERR_LIMIT;
-    cudaError_t le = launch_pdl(ctx, delta_step_kernel<L>, dim3(a.H, E), dim3(kDeltaStepThreads), smem, a);
+    const size_t smem = (size_t)(CH ? 48 * L + 3 * vpad + a.low_a + a.low_g : 32 * L + 2 * vpad) * 4;
+    if (smem > 47 * 1024) return B200_ERR_LIMIT;
+    cudaError_t le = launch_pdl(ctx, delta_step_kernel<L, CH>, dim3(a.H, E), dim3(kDeltaStepThreads), smem, a);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
 }
 
-template <int L, int NC>
+template <int L, int NC, bool CH>
 int launch_delta_scan_one(b200_ctx* ctx, const DeltaArgs& a, int E) {
     constexpr int D = 16 * L;
     const int groups = (a.Dv + NC - 1) / NC;
@@ -715,14 +784,14 @@ int launch_delta_scan_one(b200_ctx* ctx, const DeltaArgs& a, int E) {
     if (threads > 64) threads = 64;
     while (threads / L * NC % 4) threads += 32;
     const int cols = threads / L * NC, cpad = (cols + 3) & ~3;
-    const size_t smem = (size_t)(2 * kDeltaTok * (2 * D + cpad + 4) + D) * 4;
+    const size_t smem = (size_t)(2 * delta_tile_floats(D, cpad, CH) + D) * 4;
     if (smem > 200 * 1024) return B200_ERR_LIMIT;
     static bool attr_set[64] = {};
     if (!attr_set[ctx->device & 63]) {
-        B200_CUDA(ctx, cudaFuncSetAttribute(delta_scan_kernel<L, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        B200_CUDA(ctx, cudaFuncSetAttribute(delta_scan_kernel<L, NC, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         attr_set[ctx->device & 63] = true;
     }
-    cudaError_t le = launch_pdl(ctx, delta_scan_kernel<L, NC>, dim3(a.H, (a.Dv + cols - 1) / cols, E), dim3(threads), smem, a);
+    cudaError_t le = launch_pdl(ctx, delta_scan_kernel<L, NC, CH>, dim3(a.H, (a.Dv + cols - 1) / cols, E), dim3(threads), smem, a);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
@@ -730,15 +799,23 @@ int launch_delta_scan_one(b200_ctx* ctx, const DeltaArgs& a, int E) {
 
 // Columns per group: four are the cheapest per column, but with few sequences and heads the warps would be too
 // few to hide the chain from token to token.
-template <int L>
-int launch_delta_scan_l(b200_ctx* ctx, const DeltaArgs& a, int E) {
+template <int L, bool CH>
+int launch_delta_scan_ch(b200_ctx* ctx, const DeltaArgs& a, int E) {
     static const int forced = [] { const char* e = getenv("B200_DELTA_COLS"); return e ? atoi(e) : 0; }();  // tuning hook: 1, 2 or 4
     const long columns = (long)a.H * E * a.Dv;
     auto warps = [&](int nc) { return columns / nc * L / 32; };
     const int nc = forced ? forced : (warps(4) >= 6L * ctx->num_sms ? 4 : (warps(2) >= 4L * ctx->num_sms ? 2 : 1));
-    if (nc == 4) return launch_delta_scan_one<L, 4>(ctx, a, E);
-    if (nc == 2) return launch_delta_scan_one<L, 2>(ctx, a, E);
-    return launch_delta_scan_one<L, 1>(ctx, a, E);
+    if (nc == 4) return launch_delta_scan_one<L, 4, CH>(ctx, a, E);
+    if (nc == 2) return launch_delta_scan_one<L, 2, CH>(ctx, a, E);
+    return launch_delta_scan_one<L, 1, CH>(ctx, a, E);
+}
+template <int L>
+int launch_delta_scan_l(b200_ctx* ctx, const DeltaArgs& a, int E) {
+    return a.decay ? launch_delta_scan_ch<L, true>(ctx, a, E) : launch_delta_scan_ch<L, false>(ctx, a, E);
+}
+template <int L>
+int launch_delta_step_l(b200_ctx* ctx, const DeltaArgs& a, int E) {
+    return a.w_low ? launch_delta_step_one<L, true>(ctx, a, E) : launch_delta_step_one<L, false>(ctx, a, E);
 }
 
 }  // namespace
@@ -819,10 +896,10 @@ int launch_delta_scan(b200_ctx* ctx, const DeltaArgs& a, int E) {
 
 int launch_delta_step(b200_ctx* ctx, const DeltaArgs& a, int E) {
     switch (delta_state_pad(a.D)) {
-        case 32: return launch_delta_step_one<2>(ctx, a, E);
-        case 64: return launch_delta_step_one<4>(ctx, a, E);
-        case 128: return launch_delta_step_one<8>(ctx, a, E);
-        case 256: return launch_delta_step_one<16>(ctx, a, E);
+        case 32: return launch_delta_step_l<2>(ctx, a, E);
+        case 64: return launch_delta_step_l<4>(ctx, a, E);
+        case 128: return launch_delta_step_l<8>(ctx, a, E);
+        case 256: return launch_delta_step_l<16>(ctx, a, E);
         default: return B200_ERR_LIMIT;
     }
 }

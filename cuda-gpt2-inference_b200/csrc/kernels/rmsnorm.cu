@@ -1,5 +1,5 @@
-// Row-wise kernels of the layered decoders: the residual stream with an RMS norm in front of and
-// behind every sublayer, the per-head output norm of the delta rule, and a column slice.  One CTA per
+// Row-wise kernels of the layered decoders: the residual stream with an RMS norm in front of (and, if a design
+// has it, behind) every sublayer, the per-head output norm of the delta rule, and a column slice.  One CTA per
 // row with the row in registers; sums in fp32, eps inside the root.
 #include <cuda_bf16.h>
 #include "decoder_kernels.h"
@@ -34,17 +34,21 @@ residual_rms_kernel(const ResidualNormArgs a, int* status) {
         if (tok < 0 || tok >= a.vocab) { if (threadIdx.x == 0) atomicCAS(status, 0, 201); tok = 0; }
     }
     float rstd_y = 0.f;
+#pragma unroll
+    for (int i = 0; i < kVpt; ++i) v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (y) {
         float s = 0.f;
 #pragma unroll
         for (int i = 0; i < kVpt; ++i) {
             const int c = threadIdx.x + i * blockDim.x;
-            v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
             if (c < C4) { v[i] = y[c]; s += sq4(v[i]); }
         }
-        for (int c = threadIdx.x + kVpt * blockDim.x; c < C4; c += blockDim.x) s += sq4(y[c]);
-        rstd_y = 1.0f / sqrtf(block_sum(s, red) * inv_c + a.eps);
+        if (a.wb) {
+            for (int c = threadIdx.x + kVpt * blockDim.x; c < C4; c += blockDim.x) s += sq4(y[c]);
+            rstd_y = 1.0f / sqrtf(block_sum(s, red) * inv_c + a.eps);
+        }
     }
+    const float y_scale = a.y_scale ? a.y_scale[row] : 1.f;
     auto value = [&](int c, float4 yv) {
         float4 r;
         if (a.tok) {
@@ -52,9 +56,18 @@ residual_rms_kernel(const ResidualNormArgs a, int* status) {
                     : load4(static_cast<const uint16_t*>(a.embed) + (size_t)tok * a.Cp, c);
             r.x *= a.embed_scale; r.y *= a.embed_scale; r.z *= a.embed_scale; r.w *= a.embed_scale;
         } else r = x[c];
-        if (y) {
+        if (a.wb && y) {
             const float4 w = __ldg(reinterpret_cast<const float4*>(a.wb) + c);
             r.x += yv.x * rstd_y * w.x; r.y += yv.y * rstd_y * w.y; r.z += yv.z * rstd_y * w.z; r.w += yv.w * rstd_y * w.w;
+        } else {
+            float4 b = make_float4(yv.x * y_scale, yv.y * y_scale, yv.z * y_scale, yv.w * y_scale);
+            for (int j = 0; j < a.top; ++j) {  // (0: no parts)
+                const int k = row * a.top + j;
+                const float4 e = reinterpret_cast<const float4*>(a.parts + (size_t)(a.part_of ? a.part_of[k] : k) * a.Cp)[c];
+                b.x = fmaf(e.x, a.part_scale, b.x); b.y = fmaf(e.y, a.part_scale, b.y);
+                b.z = fmaf(e.z, a.part_scale, b.z); b.w = fmaf(e.w, a.part_scale, b.w);
+            }
+            r.x += b.x; r.y += b.y; r.z += b.z; r.w += b.w;
         }
         return r;
     };
@@ -75,11 +88,19 @@ residual_rms_kernel(const ResidualNormArgs a, int* status) {
     }
     if (!a.w) return;
     const float rstd = 1.0f / sqrtf(block_sum(s, red) * inv_c + a.eps);
+    float gate = 0.f;
     auto emit = [&](int c, float4 r) {
         const float4 w = __ldg(reinterpret_cast<const float4*>(a.w) + c);
         const float4 h = make_float4(r.x * rstd * w.x, r.y * rstd * w.y, r.z * rstd * w.z, r.w * rstd * w.w);
         if (OUT == H_SPLIT) store_split4(static_cast<uint8_t*>(a.h) + (size_t)row_out * a.Cp * 4, c, h);
-        else store4<OUT == H_F32>(a.h, (size_t)row_out * C4 + c, h);
+        else {
+            store4<OUT == H_F32>(a.h, (size_t)row_out * C4 + c, h);
+            for (int j = 0; j < a.copies; ++j) store4<OUT == H_F32>(a.copy, (size_t)a.copy_of[row_out * a.copies + j] * C4 + c, h);
+        }
+        if (a.gate_w) {
+            const float4 g = __ldg(reinterpret_cast<const float4*>(a.gate_w) + c);
+            gate += (h.x * g.x + h.y * g.y) + (h.z * g.z + h.w * g.w);
+        }
     };
 #pragma unroll
     for (int i = 0; i < kVpt; ++i) {
@@ -89,13 +110,17 @@ residual_rms_kernel(const ResidualNormArgs a, int* status) {
     // (columns beyond the registers are formed again: x_out may alias x, whose row this thread has already replaced)
     for (int c = threadIdx.x + kVpt * blockDim.x; c < C4; c += blockDim.x)
         emit(c, xo ? xo[c] : value(c, y ? y[c] : make_float4(0.f, 0.f, 0.f, 0.f)));
+    if (a.gate_w) {
+        gate = block_sum(gate, red);
+        if (threadIdx.x == 0) a.gate_out[row_out] = sigmoidf_(gate);
+    }
 }
 
 // one warp per (row, head)
 template <bool F32>
 __global__ void __launch_bounds__(256)
 gated_head_norm_kernel(void* out, int ld_out, const float* __restrict__ o, int ld_o, const float* __restrict__ gate, int ld_gate,
-                       const float* __restrict__ w, int M, int H, int Dv, int Dvl, float eps) {
+                       const float* __restrict__ w, int M, int H, int Dv, int Dvl, float eps, bool plain_sigmoid) {
     griddep_wait();
     griddep_launch_dependents();
     const int lane = threadIdx.x & 31;
@@ -118,13 +143,13 @@ gated_head_norm_kernel(void* out, int ld_out, const float* __restrict__ o, int l
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
             const int d = lane + i * 32;
-            if (d < Dv) store1<F32>(out, ob + d, v[i] * r * __ldg(w + d) * silu(g[i]));
+            if (d < Dv) store1<F32>(out, ob + d, v[i] * r * __ldg(w + d) * (plain_sigmoid ? sigmoidf_(g[i]) : silu(g[i])));
         }
         return;
     }
     for (int d = lane; d < Dv; d += 32) s += oh[d] * oh[d];
     const float r = 1.0f / sqrtf(warp_sum(s) / (float)Dv + eps);
-    for (int d = lane; d < Dv; d += 32) store1<F32>(out, ob + d, oh[d] * r * __ldg(w + d) * silu(gh[d]));
+    for (int d = lane; d < Dv; d += 32) store1<F32>(out, ob + d, oh[d] * r * __ldg(w + d) * (plain_sigmoid ? sigmoidf_(gh[d]) : silu(gh[d])));
 }
 
 template <bool F32>
@@ -155,10 +180,10 @@ int launch_residual_rms(b200_ctx* ctx, const ResidualNormArgs& a, int format) {
 }
 
 int launch_gated_head_norm(b200_ctx* ctx, void* out, int ld_out, const float* o, int ld_o, const float* gate, int ld_gate,
-                           const float* w, int M, int H, int Dv, int Dvl, float eps, bool f32) {
+                           const float* w, int M, int H, int Dv, int Dvl, float eps, bool f32, bool plain_sigmoid) {
     const unsigned grid = (unsigned)(((size_t)M * H + 7) / 8);
-    cudaError_t le = f32 ? launch_pdl(ctx, gated_head_norm_kernel<true>, dim3(grid), dim3(256), 0, out, ld_out, o, ld_o, gate, ld_gate, w, M, H, Dv, Dvl, eps)
-                         : launch_pdl(ctx, gated_head_norm_kernel<false>, dim3(grid), dim3(256), 0, out, ld_out, o, ld_o, gate, ld_gate, w, M, H, Dv, Dvl, eps);
+    cudaError_t le = f32 ? launch_pdl(ctx, gated_head_norm_kernel<true>, dim3(grid), dim3(256), 0, out, ld_out, o, ld_o, gate, ld_gate, w, M, H, Dv, Dvl, eps, plain_sigmoid)
+                         : launch_pdl(ctx, gated_head_norm_kernel<false>, dim3(grid), dim3(256), 0, out, ld_out, o, ld_o, gate, ld_gate, w, M, H, Dv, Dvl, eps, plain_sigmoid);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;

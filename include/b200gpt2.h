@@ -444,8 +444,9 @@ void* b200_gpt2_activation(b200_gpt2* model, const char* name);
 
 /* ---------------------------------------------------------------- layered decoders */
 /* Decoder-only models whose configuration lists their layers (config.json; "architecture" selects the
- * design, e.g. "Vunolorn"), each with a mixer - selective scan, gated delta rule, or softmax attention
- * beside a minGRU - and a feed-forward.  Sequences live in slots, which hold a sequence's key/value cache,
+ * design: "Vunolorn", "Pumotar"), each with a mixer - selective scan, gated delta rule with a decay per head or
+ * per key channel, softmax attention beside a minGRU, latent attention - and a feed-forward, dense or of
+ * table-routed experts.  Sequences live in slots, which hold a sequence's key/value or latent cache,
  * recurrent state and convolution history; a step runs any number of new tokens of any open slots.
  *
  * arithmetic: B200_DECODER_BF16 - bf16 weights and matrix-product operands, fp16 key/value cache, fp32
@@ -462,10 +463,10 @@ int b200_decoder_destroy(b200_decoder* model);
 /* Reads a configuration without a device: B200_OK, or B200_ERR_SHAPE with the reason in message (may be NULL). */
 int b200_decoder_check_config(const char* config_json, char* message, int message_bytes);
 int b200_decoder_vocab(const b200_decoder* model);
-/* Weights: a safetensors file, or tensors one by one (host memory, bf16 or fp32; copied) and finish_load.
- * Names and shapes are checked against the configuration. */
+/* Weights: a safetensors file, or tensors one by one (host memory; copied) and finish_load.  type: 0 bf16, 1 fp32,
+ * 2 int32 (tables).  Names and shapes are checked against the configuration. */
 int b200_decoder_load_safetensors(b200_decoder* model, const char* path);
-int b200_decoder_set_tensor(b200_decoder* model, const char* name, const void* data, int is_f32, const long* shape, int ndim);
+int b200_decoder_set_tensor(b200_decoder* model, const char* name, const void* data, int type, const long* shape, int ndim);
 int b200_decoder_finish_load(b200_decoder* model);
 /* decode steps replayed as CUDA graphs (default 1; needs a stream other than the default one) */
 int b200_decoder_set_graph(b200_decoder* model, int use_graph);
