@@ -1123,8 +1123,8 @@ def main():
                              "fused_residual_layernorm", "rowwise"],
                     help="per-kernel sweep at 8192 rows instead of the forward benchmark")
     ap.add_argument("--layered", nargs="?", const="all", default=None,
-                    help="instead of the forward benchmark: prefill and decode of the layered decoders beside GPT-2 of equal width "
-                         "and depth (sizes 768, 1600, with commas between them; default all)")
+                    help="instead of the forward benchmark: prefill and decode of the layered decoders beside the closest model of "
+                         "equal width and depth (768, 1600, pumotar-768, pumotar-1600, with commas between them; default all)")
     ap.add_argument("--case", type=int, default=None, help="with --op: run only this case of the family")
     ap.add_argument("--modes", default="tf32", choices=["tf32", "both"], help="with --op matmul: also time 3xTF32")
     ap.add_argument("--flush-l2", action="store_true", help="with --op: cold L2 before every launch")

@@ -1083,7 +1083,7 @@ int enqueue_general(b200_decoder* m, const StepView& v) {
         }
         if (!last) {
             n.w = m->layers[i + 1].norm1;
-            OP("residual norms", launch_residual_rms(ctx, n, m->f32 ? H_F32 : H_BF16));
+            OP(n.top ? "residual norms parts" : "residual norms", launch_residual_rms(ctx, n, m->f32 ? H_F32 : H_BF16));
         }
     }
     if (v.n_want == 0) return B200_OK;

@@ -320,10 +320,13 @@ def forward(cfg, w, tokens, layer_outputs=None):
 def tensor_shapes(cfg):
     """name -> shape of every tensor of the model."""
     C, V = cfg["width"], cfg["vocab"]
+    post_norm = own_head = cfg["architecture"] == "Vunolorn"
     s = {"embed": (V, C)}
     for i, layer in enumerate(cfg["layers"]):
         p, m = f"l{i}", layer["mixer"]
-        s[p + ".norm1"] = s[p + ".norm1b"] = (C,)
+        s[p + ".norm1"] = (C,)
+        if post_norm:
+            s[p + ".norm1b"] = (C,)
         if layer["type"] == "mamba1":
             n, r, st = m["inner"], m["dt_rank"], m["state"]
             s.update({p + ".mix.in": (2 * n, C), p + ".mix.conv": (n, m["conv"]), p + ".mix.conv.b": (n,),
@@ -336,6 +339,18 @@ def tensor_shapes(cfg):
                 s[f"{p}.mix.{n}.conv"] = (rows, m["conv"])
             s.update({p + ".mix.b": (H, C), p + ".mix.A_log": (H,), p + ".mix.norm": (Dv,), p + ".mix.a": (H, C),
                       p + ".mix.dt_bias": (H,), p + ".mix.g": (H * Dv, C), p + ".mix.o": (C, H * Dv)})
+        elif layer["type"] == "channel_delta":
+            H, G, D, Dv, x = m["heads"], m["kv_heads"], m["dim"], m["vdim"], p + ".mix"
+            ra, rg = low_ranks(layer)
+            for n, rows in (("q", G * D), ("k", G * D), ("v", H * Dv)):
+                s[f"{x}.{n}"] = (rows, C)
+                s[f"{x}.{n}.conv"] = (rows, m["conv"])
+            s.update({x + ".b": (H, C), x + ".A_log": (H,), x + ".norm": (Dv,), x + ".a1": (ra, C), x + ".a2": (H * D, ra),
+                      x + ".dt_bias": (H * D,), x + ".g1": (rg, C), x + ".g2": (H * Dv, rg), x + ".o": (C, H * Dv)})
+        elif layer["type"] == "latent_attention":
+            H, D, Dr, Dv, R, x = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], p + ".mix"
+            s.update({x + ".q": (H * (D + Dr), C), x + ".dkv": (R + Dr, C), x + ".dkv.norm": (R,), x + ".uk": (H * D, R),
+                      x + ".uv": (H * Dv, R), x + ".o": (C, H * Dv)})
         else:
             l, r = m["left"], m["right"]
             a, b = p + ".mix.left", p + ".mix.right"
@@ -344,12 +359,33 @@ def tensor_shapes(cfg):
                       a + ".o": (C, l["heads"] * l["vdim"])})
             W = r["width"]
             s.update({b + ".z": (W, C), b + ".z.b": (W,), b + ".x": (W, C), b + ".x.b": (W,), b + ".g": (W, C), b + ".o": (C, W)})
-        if layer["mlp"] is not None:
-            F = layer["mlp"]["ff"]
-            s.update({p + ".norm2": (C,), p + ".norm2b": (C,), p + ".mlp.up": (F, C), p + ".mlp.down": (C, F)})
+        mlp = layer["mlp"]
+        if mlp is None:
+            continue
+        s[p + ".norm2"] = (C,)
+        gated = lambda q, F: {q + ".gate": (F, C), q + ".up": (F, C), q + ".down": (C, F)}
+        if post_norm:
+            F = mlp["ff"]
+            s.update({p + ".norm2b": (C,), p + ".mlp.up": (F, C), p + ".mlp.down": (C, F)})
+        elif mlp["kind"] == "dense":
+            s.update(gated(p + ".mlp", mlp["ff"]))
+        else:
+            for e in range(mlp["router"]["experts"]):
+                s.update(gated(f"{p}.mlp.e{e}", mlp["expert"]["ff"]))
+            s[p + ".mlp.table"] = (V, mlp["router"]["top"])
+            if mlp.get("shared"):
+                s.update(gated(p + ".mlp.shared", mlp["shared"]["ff"]))
+                s[p + ".mlp.shared.sg"] = (1, C)
     s["final.norm"] = (C,)
-    s["head"] = (V, C)
+    if own_head:
+        s["head"] = (V, C)
     return s
+
+
+def low_ranks(layer):
+    """Ranks of the low-rank decay and output gate, which only the tensors' shapes give: picked here from the sizes."""
+    m = layer["mixer"]
+    return m.get("ranks", (m["dim"] // 3 + 1, m["vdim"] // 2 + 3))
 
 
 def to_bf16(a):
@@ -365,7 +401,14 @@ def random_weights(cfg, seed):
     w = {}
     for name, shape in tensor_shapes(cfg).items():
         leaf = name.rsplit(".", 1)[-1]
-        if "norm" in leaf:
+        if leaf == "table":  # the entries of a row differ
+            i = int(name[1:].split(".")[0])
+            experts = cfg["layers"][i]["mlp"]["router"]["experts"]
+            w[name] = np.stack([rng.permutation(experts)[:shape[1]] for _ in range(shape[0])]).astype(np.int32)
+            continue
+        if name == "final.norm" or leaf in ("norm1", "norm2"):
+            a = (0.0 if cfg["architecture"] == "Pumotar" else 1.0) + 0.3 * rng.standard_normal(shape)
+        elif "norm" in leaf:
             a = 1.0 + 0.3 * rng.standard_normal(shape)
         elif leaf == "A_log":
             a = rng.uniform(-2.0, 1.5, shape)
@@ -379,6 +422,8 @@ def random_weights(cfg, seed):
             a = rng.standard_normal(shape) / math.sqrt(shape[1])
         elif name == "embed":
             a = rng.standard_normal(shape) / cfg["embedding"]["scale"]
+            if cfg["architecture"] == "Pumotar":  # (the layers' part of the residual stream is to outweigh the token's own embedding)
+                a *= 0.2
         else:
             a = rng.standard_normal(shape) / math.sqrt(shape[1])
         w[name] = to_bf16(a)
@@ -386,17 +431,23 @@ def random_weights(cfg, seed):
 
 
 def as_float64(w):
-    return {k: v.astype(np.float64) for k, v in w.items()}
+    return {k: v if v.dtype == np.int32 else v.astype(np.float64) for k, v in w.items()}
+
+
+def as_bits(w):
+    """The weights as the library takes them: bf16 bits, int32 tables."""
+    return {k: v if v.dtype == np.int32 else (v.view(np.uint32) >> 16).astype(np.uint16) for k, v in w.items()}
 
 
 def save_safetensors(path, w):
-    """Writes the weights as bf16 (their values must be exact in bf16)."""
+    """Writes the weights as bf16 (their values must be exact in bf16), tables as int32."""
     import json
     import struct
     head, off, blobs = {}, 0, []
     for name, a in w.items():
-        b = (np.ascontiguousarray(a, np.float32).view(np.uint32) >> 16).astype(np.uint16).tobytes()
-        head[name] = {"dtype": "BF16", "shape": list(a.shape), "data_offsets": [off, off + len(b)]}
+        table = a.dtype == np.int32
+        b = a.astype("<i4").tobytes() if table else (np.ascontiguousarray(a, np.float32).view(np.uint32) >> 16).astype(np.uint16).tobytes()
+        head[name] = {"dtype": "I32" if table else "BF16", "shape": list(a.shape), "data_offsets": [off, off + len(b)]}
         off += len(b)
         blobs.append(b)
     h = json.dumps(head).encode()
