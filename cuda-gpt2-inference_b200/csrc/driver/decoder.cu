@@ -1171,7 +1171,7 @@ int enqueue_decode(b200_decoder* m, int B) {
             TRY(norm(L.norm2));
             n.gate_w = nullptr;
             DecodeGemmArgs up = product_args(m->dh, f.up), down = product_args(m->dpair_mix, f.down);
-            up.table = down.table = f.table; up.tok = down.tok = m->dtokens; up.top = down.top = s.top;
+            up.table = down.table = f.table; up.tok = down.tok = m->dtokens; up.top = down.top = s.top; up.experts = down.experts = s.experts;
             up.gate = f.gate; up.limit = s.limit; up.split_out = static_cast<uint8_t*>(m->dpair_mix);
             down.pair_in = 1; down.out = m->dpair_y; down.ldo = f.down.N;
             if (s.shared_ff) {

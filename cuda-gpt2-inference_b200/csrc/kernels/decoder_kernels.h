@@ -77,7 +77,7 @@ struct DecodeGemmArgs {
     const SeqDesc* seqs; const float* conv_w; const float* conv_b; float* hist; int conv_n, taps, max_slots;
     uint8_t* conv_out;    // [B] rows of conv_n columns
     int gate; float limit;
-    const int* table; const int* tok; int top, pair_in;
+    const int* table; const int* tok; int top, experts, pair_in;
     DecodeGemmShared shared;
 };
 int launch_decode_gemm(b200_ctx* ctx, const DecodeGemmArgs& a);

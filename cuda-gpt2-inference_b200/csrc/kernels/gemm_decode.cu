@@ -19,9 +19,10 @@
 //
 // Gated outputs: a tile is eight gate rows and their eight linear rows, so the two meet in the same epilogue.
 //
-// Table-routed experts: blockIdx.y numbers the (input row, choice) pairs.  The first pair of a matrix takes all input rows
-// that chose it, the later ones find that out and leave.  (The ids and the table are read before the previous
-// kernel has finished: they were there before it started.)
+// Table-routed experts (ROUTED): every CTA looks the rows' experts up and lists the matrices that occur; the tiles of all of
+// them, and of the shared expert, are one sequence, cut into equal shares of weight bytes, and a matrix is multiplied with
+// all rows at once, of which those that did not choose it are dropped.  (The ids and the table are read before the
+// previous kernel has finished: they were there before it started.)
 #include "decoder_kernels.h"
 #include "decoder_math.cuh"
 #include "../prim/sm100.cuh"
@@ -45,58 +46,100 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t a0, const
 
 // Input rows in shared memory: row b at b * stride, as in memory.  stride = 4 * columns + 16, so that the lanes of
 // a quarter warp (two rows, four groups of eight columns) touch all banks once.
-template <int NT>  // blocks of eight input rows
+template <int NT, bool ROUTED>  // blocks of eight input rows
 __global__ void __launch_bounds__(kThreads, 2)
 decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, const int chunk) {
     extern __shared__ __align__(16) uint8_t xs[];
     __shared__ float red[NT][kWarps][16][9];
     __shared__ float part[NT * 128];
-    __shared__ int expert[kMaxPairs], x_row[NT * 8], o_row[NT * 8];
+    __shared__ uint16_t expert[ROUTED ? kMaxPairs : 1], listed[ROUTED ? kMaxPairs : 1];
+    __shared__ uint8_t first[ROUTED ? kMaxPairs : 1];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
-    const int B = a.B, pairs = B * a.top, job = blockIdx.y;
-    const bool shared_job = pairs > 0 && job == pairs, routed = pairs > 0 && !shared_job, gated = a.gate != GATE_NONE;
-    const int K = shared_job ? a.shared.K : a.K, N = shared_job ? a.shared.N : a.N;
-    const uint8_t* xin = shared_job ? a.shared.x : a.x;
-    size_t w_off = 0;
-    if (routed) {
-        if (tid < pairs) expert[tid] = __ldg(a.table + (size_t)a.tok[tid / a.top] * a.top + tid % a.top);
-        if (tid < NT * 8) x_row[tid] = o_row[tid] = -1;
+    const int B = a.B;
+    const bool gated = a.gate != GATE_NONE;
+    const int rank = slices > 1 ? (int)cluster_ctarank() : 0;
+    const int stride = chunk * 4 + 16;
+    // the cluster's tiles: item, item + step, ...
+    const int tiles = (a.N + 15) >> 4;
+    int item = blockIdx.x / slices, items = tiles, step = gridDim.x / slices, matrices = 1;
+    if (ROUTED) {
+        const int pairs = B * a.top;
+        if (tid < pairs) expert[tid] = (uint16_t)__ldg(a.table + (size_t)a.tok[tid / a.top] * a.top + tid % a.top);
         __syncthreads();
-        const int e = expert[job];
-        if (__syncthreads_or(tid < job && expert[tid] == e)) return;  // an earlier pair's CTAs do this one as well
-        if (tid < pairs && expert[tid] == e) {
-            o_row[tid / a.top] = tid;
-            x_row[tid / a.top] = a.pair_in ? tid : tid / a.top;
+        if (tid < pairs) {
+            bool seen = false;
+            for (int p = 0; p < tid; ++p) seen = seen || expert[p] == expert[tid];
+            first[tid] = !seen;
+        }
+        matrices = __syncthreads_count(tid < pairs && first[tid]);
+        if (tid < pairs && first[tid]) {
+            int n = 0;
+            for (int p = 0; p < tid; ++p) n += first[p];
+            listed[n] = expert[tid];
         }
         __syncthreads();
-        w_off = (size_t)e * N * K;
+        // shares of equal K elements, cut where a tile ends
+        const int shared_tiles = a.shared.W ? (a.shared.N + 15) >> 4 : 0;
+        const long routed_cost = (long)matrices * tiles * a.K, cost = routed_cost + (long)shared_tiles * a.shared.K;
+        auto cut = [&](int i) {
+            const long at = cost * i / step;
+            return at <= routed_cost ? (int)((at + a.K - 1) / a.K) : matrices * tiles + (int)((at - routed_cost + a.shared.K - 1) / a.shared.K);
+        };
+        const int share = item;
+        item = cut(share);
+        items = cut(share + 1);
+        step = 1;
     }
-    const int tiles = (N + 15) >> 4;
-    const int rank = slices > 1 ? (int)cluster_ctarank() : 0;
-    const int tile0 = blockIdx.x / slices, tile_step = gridDim.x / slices;
-    const int kb = min(K, rank * kslice), ke = min(K, kb + kslice);  // this CTA's columns (may be none)
-    const int stride = chunk * 4 + 16;
-    const uint16_t* __restrict__ W = (shared_job ? a.shared.W : a.W) + w_off;
+    struct Tile { const uint16_t* W; int N, K, kb, ke, tile, matrix; };  // kb .. ke: this CTA's columns (may be none)
+    auto tile_of = [&](int i) {
+        Tile t;
+        t.N = a.N; t.K = a.K; t.W = a.W; t.tile = i; t.matrix = 0;
+        if (ROUTED) {
+            t.matrix = min(i / tiles, matrices);
+            t.tile = i - t.matrix * tiles;
+            if (t.matrix == matrices) { t.N = a.shared.N; t.K = a.shared.K; t.W = a.shared.W; }
+            else t.W += (size_t)listed[t.matrix] * a.N * a.K;
+        }
+        const int ks = ROUTED ? ((t.K + slices - 1) / slices + 31) / 32 * 32 : kslice;
+        t.kb = min(t.K, rank * ks);
+        t.ke = min(t.K, t.kb + ks);
+        return t;
+    };
+    // row of input row b's products with the matrix (-1: it did not choose it)
+    auto pair_row = [&](int b, const Tile& t) {
+        if (!ROUTED || t.matrix == matrices) return b;
+        const int e = listed[t.matrix];
+        int r = -1;
+        for (int j = 0; j < a.top; ++j) if (expert[b * a.top + j] == e) r = b * a.top + j;
+        return r;
+    };
     // this warp's pieces of a chunk: 32 columns each, number warp, warp + 8, ...
     uint4 w[kU][2];
-    auto request = [&](uint4 (&r)[2], int tile, int k0, int kend, int p) {
+    auto request = [&](uint4 (&r)[2], const Tile& t, int k0, int kend, int p) {
         const int k = k0 + p * 32 + c * 8;
-        const int r0 = gated ? (tile >> 2) * 64 + (tile & 3) * 8 + g : tile * 16 + g, r1 = r0 + (gated ? 32 : 8);
+        const int r0 = gated ? (t.tile >> 2) * 64 + (t.tile & 3) * 8 + g : t.tile * 16 + g, r1 = r0 + (gated ? 32 : 8);
         r[0] = r[1] = make_uint4(0u, 0u, 0u, 0u);
         if (k < kend) {
-            if (r0 < N) r[0] = __ldg(reinterpret_cast<const uint4*>(W + (size_t)r0 * K + k));
-            if (r1 < N) r[1] = __ldg(reinterpret_cast<const uint4*>(W + (size_t)r1 * K + k));
+            if (r0 < t.N) r[0] = __ldg(reinterpret_cast<const uint4*>(t.W + (size_t)r0 * t.K + k));
+            if (r1 < t.N) r[1] = __ldg(reinterpret_cast<const uint4*>(t.W + (size_t)r1 * t.K + k));
         }
     };
+    Tile now = tile_of(item);
+    const int item0 = item;
+    if (item < items) {
 #pragma unroll
-    for (int u = 0; u < kU; ++u) request(w[u], tile0, kb, min(ke, kb + chunk), warp + u * kWarps);
+        for (int u = 0; u < kU; ++u) request(w[u], now, now.kb, min(now.ke, now.kb + chunk), warp + u * kWarps);
+    }
     for (int i = tid; i < (NT * 8 - B) * (stride >> 4); i += kThreads)
         reinterpret_cast<uint4*>(xs + (size_t)B * stride)[i] = make_uint4(0u, 0u, 0u, 0u);
     griddep_wait();
     griddep_launch_dependents();
 
-    bool staged = false;  // an input of one chunk is staged once for all tiles
-    for (int tile = tile0; tile < tiles; tile += tile_step) {
+    bool staged = false;  // an input of one chunk is staged once for all tiles that share it
+    for (; item < items; item += step) {
+        const Tile next = tile_of(item + step < items ? item + step : item);
+        const int tile = now.tile, N = now.N, kb = now.kb, ke = now.ke;
+        const bool shared_tile = ROUTED && now.matrix == matrices;
         // what the epilogue's convolution wants, on its way during the product (thread tid: column tid & 15, row tid >> 4)
         float cx[kMaxTaps], cw[kMaxTaps];
         const int er = tile * 16 + (tid & 15), eb = tid >> 4;
@@ -122,13 +165,14 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
             const int kend = min(ke, k0 + chunk);
             const int pieces = (kend - k0 + 31) >> 5;
             if (!staged) {
-                if (k0 > kb || tile != tile0) __syncthreads();  // everyone is done with the previous chunk
+                if (k0 > kb || item != item0) __syncthreads();  // everyone is done with the previous chunk
                 const int n16 = (kend - k0) >> 2;               // 16-byte pieces of a row
+                const uint8_t* xin = shared_tile ? a.shared.x : a.x;
                 for (int b = 0; b < B; ++b) {
-                    const int xr = routed ? x_row[b] : b;
+                    const int xr = ROUTED && a.pair_in ? pair_row(b, now) : b;
                     if (xr < 0) continue;  // (whatever the row holds stays in its own column of the product)
                     for (int i = tid; i < n16; i += kThreads)
-                        cp_async16(xs + (size_t)b * stride + i * 16, xin + ((size_t)xr * K + k0) * 4 + i * 16);
+                        cp_async16(xs + (size_t)b * stride + i * 16, xin + ((size_t)xr * now.K + k0) * 4 + i * 16);
                 }
                 cp_async_commit();
                 cp_async_wait<0>();
@@ -137,7 +181,8 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
             }
             // where the pieces behind this chunk's lie
             const bool more = kend < ke;
-            const int tn = more ? tile : tile + tile_step, kn = more ? kend : kb, en = more ? min(ke, kend + chunk) : (tn < tiles ? min(ke, kb + chunk) : kb);
+            const Tile behind = more ? now : next;
+            const int kn = more ? kend : next.kb, en = more ? min(ke, kend + chunk) : (item + step < items ? min(next.ke, next.kb + chunk) : next.kb);
             int p0 = warp;
             do {
                 const bool last = p0 + kU * kWarps >= pieces;
@@ -161,8 +206,8 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
                             mma_bf16(acc[t], w[u][0].z, w[u][1].z, w[u][0].w, w[u][1].w, lo.z, lo.w);
                         }
                     }
-                    if (last) request(w[u], tn, kn, en, warp + u * kWarps);
-                    else request(w[u], tile, k0, kend, p + kU * kWarps);
+                    if (last) request(w[u], behind, kn, en, warp + u * kWarps);
+                    else request(w[u], now, k0, kend, p + kU * kWarps);
                 }
                 p0 += kU * kWarps;
             } while (p0 < pieces);
@@ -200,12 +245,12 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
             }
             return v;
         };
-        const int out_row = (eb < B && eb < NT * 8) ? (routed ? o_row[eb] : eb) : -1;
+        const int out_row = (eb < B && eb < NT * 8) ? pair_row(eb, now) : -1;
         if (rank == 0 && out_row >= 0 && gated) {
             if ((tid & 15) < 8) {
                 const float gv = total(tid & 7), uv = total((tid & 7) + 8);
-                const float v = a.gate == GATE_CLAMP ? clamped_gate(gv, uv, shared_job ? a.shared.limit : a.limit) : gelu_tanh(gv) * uv;
-                store_split((shared_job ? a.shared.split_out : a.split_out) + (size_t)out_row * (N >> 1) * 4, (tile >> 2) * 32 + (tile & 3) * 8 + (tid & 7), v);
+                const float v = a.gate == GATE_CLAMP ? clamped_gate(gv, uv, shared_tile ? a.shared.limit : a.limit) : gelu_tanh(gv) * uv;
+                store_split((shared_tile ? a.shared.split_out : a.split_out) + (size_t)out_row * (N >> 1) * 4, (tile >> 2) * 32 + (tile & 3) * 8 + (tid & 7), v);
             }
         } else if (rank == 0 && out_row >= 0 && er < N) {
             float v = total(tid & 15);
@@ -234,27 +279,30 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
             else if (a.act == ACT_GELU_TANH) v = gelu_tanh(v);
             if (conv && a.conv_out) store_split(a.conv_out + (size_t)eb * a.conv_n * 4, er, v);
             else if (a.split_out) store_split(a.split_out + (size_t)out_row * N * 4, er, v);
-            else if (shared_job) a.shared.out[(size_t)out_row * a.shared.ldo + er] = v;
+            else if (shared_tile) a.shared.out[(size_t)out_row * a.shared.ldo + er] = v;
             else a.out[(size_t)out_row * a.ldo + er] = v;
         }
         if (slices > 1) cluster_sync_all();  // the partial sums have been read (and nobody leaves before that)
         else __syncthreads();
+        if (ROUTED && (a.pair_in || a.shared.x != a.x) && next.matrix != now.matrix) staged = false;
+        now = next;
     }
 }
 
-template <int NT>
+template <int NT, bool ROUTED>
 int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
     static bool attr_set[64] = {};
     if (!attr_set[ctx->device & 63]) {
-        B200_CUDA(ctx, cudaFuncSetAttribute(decode_gemm_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kOneCtaSmem));
+        B200_CUDA(ctx, cudaFuncSetAttribute(decode_gemm_kernel<NT, ROUTED>, cudaFuncAttributeMaxDynamicSharedMemorySize, kOneCtaSmem));
         attr_set[ctx->device & 63] = true;
     }
-    const int jobs = a.top > 0 ? a.B * a.top + (a.shared.W ? 1 : 0) : 1;
-    const int max_n = jobs > 1 && a.shared.N > a.N ? a.shared.N : a.N, max_k = jobs > 1 && a.shared.K > a.K ? a.shared.K : a.K;
-    const int tiles = (max_n + 15) / 16;
+    // (routed: at most as many matrices as pairs or experts; they are not known here)
+    const int max_k = ROUTED && a.shared.W && a.shared.K > a.K ? a.shared.K : a.K;
+    int tiles = (a.N + 15) / 16;
+    if (ROUTED) tiles = tiles * (a.B * a.top < a.experts ? a.B * a.top : a.experts) + (a.shared.W ? (a.shared.N + 15) / 16 : 0);
     // K slices while the CTAs of one wave (two per SM) are not used up and a warp keeps at least a piece
     int slices = 1;
-    while (slices < 8 && jobs * tiles * slices * 2 <= 2 * ctx->num_sms && max_k / (slices * 2) >= 256) slices *= 2;
+    while (slices < 8 && tiles * slices * 2 <= 2 * ctx->num_sms && max_k / (slices * 2) >= 256) slices *= 2;
     const int kslice = ((max_k + slices - 1) / slices + 31) / 32 * 32;
     // the columns staged at a time: all of the slice, so that they are staged once for all tiles; else as many as
     // two CTAs per SM can hold
@@ -262,11 +310,9 @@ int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
     const int chunk = kslice <= columns(kOneCtaSmem) ? kslice : columns(kTwoCtaSmem);
     const int per_sm = chunk <= columns(kTwoCtaSmem) ? 2 : 1;
     int grid = tiles * slices;
-    int room = per_sm * ctx->num_sms / jobs;
-    if (room < slices) room = slices;
-    if (grid > room) grid = room / slices * slices;
+    if (grid > per_sm * ctx->num_sms) grid = per_sm * ctx->num_sms / slices * slices;
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(grid, jobs);
+    cfg.gridDim = dim3(grid);
     cfg.blockDim = dim3(kThreads);
     cfg.dynamicSmemBytes = (size_t)NT * 8 * (chunk * 4 + 16);
     cfg.stream = ctx->stream;
@@ -285,7 +331,7 @@ int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
     }
     cfg.attrs = attr;
     cfg.numAttrs = n;
-    const cudaError_t le = cudaLaunchKernelEx(&cfg, decode_gemm_kernel<NT>, a, slices, kslice, chunk);
+    const cudaError_t le = cudaLaunchKernelEx(&cfg, decode_gemm_kernel<NT, ROUTED>, a, slices, kslice, chunk);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
@@ -297,7 +343,8 @@ int launch_decode_gemm(b200_ctx* ctx, const DecodeGemmArgs& a) {
     if (a.B < 1 || a.B > 16 || a.K % 8 || a.N < 1) return B200_ERR_SHAPE;
     if (a.top < 0 || a.B * a.top > kMaxPairs || (a.top > 0 && a.conv_n > 0) || (a.gate != GATE_NONE && (a.N % 64 || !a.split_out))) return B200_ERR_SHAPE;
     if (a.shared.W && (a.top < 1 || a.shared.K % 8 || (a.gate != GATE_NONE && (a.shared.N % 64 || !a.shared.split_out)))) return B200_ERR_SHAPE;
-    return a.B <= 8 ? launch_one<1>(ctx, a) : launch_one<2>(ctx, a);
+    if (a.top > 0) return a.B <= 8 ? launch_one<1, true>(ctx, a) : launch_one<2, true>(ctx, a);
+    return a.B <= 8 ? launch_one<1, false>(ctx, a) : launch_one<2, false>(ctx, a);
 }
 
 }  // namespace b200
