@@ -244,7 +244,7 @@ __global__ void __launch_bounds__(kLatThreads)
 latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, void* out, int ldo, const SeqDesc* __restrict__ seqs,
                         const int* __restrict__ list, int splits, bool split_rows) {
     extern __shared__ __align__(16) uint8_t raw[];
-    __shared__ float stat_m[16 * MT], stat_l[16 * MT], stat_a[16 * MT];
+    __shared__ float stat_m[16 * MT], stat_l[16 * MT], stat_a[16 * MT], weight[16 * MT][8];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c2 = (lane & 3) * 2;
     const int ld = c.Lp + 8;  // halves
     __half* ks = reinterpret_cast<__half*>(raw);           // [2][64][ld]
@@ -391,48 +391,78 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
                 const int r = m * 16 + g + (e >> 1) * 8, d = oc0 + j * 8 + c2 + (e & 1);
                 if (d < c.Rp) os[r * ldf + d] = o[m][j][e];
             }
+    const int mine = z < np ? (np - z + splits - 1) / splits : 0;  // pairs z, z + splits, ...
+    // the values: W_uv, a warp working on U outputs at a time, 256 latent columns in a step; a step's weights are on their way during
+    // the step before, the first ones' during the merge
+    constexpr int U = 8;
+    const int outputs = mine * c.Dv, chunks = (c.Rp + 255) >> 8;
+    uint4 w[U];
+    auto fetch = [&](int i0, int d0) {
+        const bool live = i0 < outputs && d0 < c.Rp;
+        int k = min(i0, max(outputs - 1, 0)) / c.Dv, v = i0 - k * c.Dv, h = (pair0 + z + k * splits) % c.H;
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            w[u] = make_uint4(0u, 0u, 0u, 0u);
+            if (live && i0 + u < outputs) w[u] = __ldg(reinterpret_cast<const uint4*>(c.Wuv + (size_t)(h * c.Dv + v) * c.Rp + d0));
+            if (++v == c.Dv) { v = 0; ++k; h = (pair0 + z + k * splits) % c.H; }
+        }
+    };
+    fetch(warp * U, lane * 8);
     if (splits > 1) cluster_sync_all();
     else __syncthreads();
-    const int mine = z < np ? (np - z + splits - 1) / splits : 0;  // pairs z, z + splits, ...
-    for (int i = tid; i < mine * ldf; i += kLatThreads) {
-        const int k = i / ldf, d = i - k * ldf, r = z + k * splits;
-        float m = -INFINITY, l = 0.f, v = 0.f;
-        if (splits == 1) { v = os[r * ldf + d]; l = stat_l[r]; }
-        else {
-            for (int s = 0; s < splits; ++s) m = fmaxf(m, ld_cluster_f32(stat_m + r, s));
-            for (int s = 0; s < splits; ++s) {
-                const float w = ex2(ld_cluster_f32(stat_m + r, s) - m);  // 0 for a split that saw no key of the pair's
-                l = fmaf(ld_cluster_f32(stat_l + r, s), w, l);
-                v = fmaf(ld_cluster_f32(os + r * ldf + d, s), w, v);
-            }
-        }
-        om[i] = d < c.R ? v / l : 0.f;
+    if (tid < mine * 8) {  // a split's share in a pair's sum
+        const int k = tid >> 3, s = tid & 7, r = z + k * splits;
+        float m = s < splits ? (splits > 1 ? ld_cluster_f32(stat_m + r, s) : stat_m[r]) : -INFINITY, top = m;
+        const float l = s < splits ? (splits > 1 ? ld_cluster_f32(stat_l + r, s) : stat_l[r]) : 0.f;
+        const uint32_t group = 0xffu << (lane & 24);
+#pragma unroll
+        for (int d = 1; d < 8; d <<= 1) top = fmaxf(top, __shfl_xor_sync(group, top, d));
+        const float e = ex2(m - top);  // 0 for a split that saw no key of the pair's
+        float sum = l * e;
+#pragma unroll
+        for (int d = 1; d < 8; d <<= 1) sum += __shfl_xor_sync(group, sum, d);
+        weight[k][s] = e / sum;
     }
     __syncthreads();
-    constexpr int U = 8;  // outputs a warp works on at a time
-    const int outputs = mine * c.Dv;
+    for (int i = tid; i < mine * ldf; i += kLatThreads) {
+        const int k = i / ldf, d = i - k * ldf;
+        const float* src = os + (z + k * splits) * ldf + d;
+        float v = 0.f;
+        if (splits == 1) v = *src * weight[k][0];
+        else {
+            float x[8];
+#pragma unroll
+            for (int s = 0; s < 8; ++s) x[s] = s < splits ? ld_cluster_f32(src, s) : 0.f;
+#pragma unroll
+            for (int s = 0; s < 8; ++s) v = fmaf(x[s], weight[k][s], v);
+        }
+        om[i] = d < c.R ? v : 0.f;
+    }
+    __syncthreads();
     for (int i0 = warp * U; i0 < outputs; i0 += 8 * U) {
         float acc[U];
 #pragma unroll
         for (int u = 0; u < U; ++u) acc[u] = 0.f;
-        for (int d0 = lane * 8; d0 < c.Rp; d0 += 256) {
-            uint4 w[U];
+        for (int ch = 0; ch < chunks; ++ch) {
+            const int d0 = ch * 256 + lane * 8;
+            uint4 x[U];
+#pragma unroll
+            for (int u = 0; u < U; ++u) x[u] = w[u];
+            if (ch + 1 < chunks) fetch(i0, d0 + 256);
+            else fetch(i0 + 8 * U, lane * 8);
+            if (d0 >= c.Rp) continue;
+            int k = i0 / c.Dv, v = i0 - k * c.Dv;
 #pragma unroll
             for (int u = 0; u < U; ++u) {
-                const int i = min(i0 + u, outputs - 1), k = i / c.Dv, h = (pair0 + z + k * splits) % c.H;
-                w[u] = __ldg(reinterpret_cast<const uint4*>(c.Wuv + (size_t)(h * c.Dv + i - k * c.Dv) * c.Rp + d0));
-            }
-#pragma unroll
-            for (int u = 0; u < U; ++u) {
-                const int k = min(i0 + u, outputs - 1) / c.Dv;
                 const float4 x0 = *reinterpret_cast<const float4*>(om + k * ldf + d0), x1 = *reinterpret_cast<const float4*>(om + k * ldf + d0 + 4);
-                const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
-                const uint32_t y[4] = {w[u].x, w[u].y, w[u].z, w[u].w};
+                const float z8[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+                const uint32_t y[4] = {x[u].x, x[u].y, x[u].z, x[u].w};
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    acc[u] = fmaf(__uint_as_float(y[e] << 16), x[2 * e], acc[u]);
-                    acc[u] = fmaf(__uint_as_float(y[e] & 0xffff0000u), x[2 * e + 1], acc[u]);
+                    acc[u] = fmaf(__uint_as_float(y[e] << 16), z8[2 * e], acc[u]);
+                    acc[u] = fmaf(__uint_as_float(y[e] & 0xffff0000u), z8[2 * e + 1], acc[u]);
                 }
+                if (++v == c.Dv) { v = 0; k = min(k + 1, mine - 1); }  // (outputs beyond the end: weights of zero)
             }
         }
         reduce_scatter<U, 32>(acc, lane);
@@ -533,7 +563,9 @@ int launch_latent_query(b200_ctx* ctx, const LatentAttention& c, const float* pr
 
 int launch_latent_attention(b200_ctx* ctx, const LatentAttention& c, const void* ql, void* out, int ldo, const SeqDesc* seqs, const int* list, int n, int max_n,
                             int max_keys, bool split_rows) {
-    if ((long)max_n * c.H > 16) return launch_latent_mt<2>(ctx, c, ql, out, ldo, seqs, list, n, max_n, max_keys, split_rows);
+    // tiles of 32 pairs read the rows once for twice as many, tiles of 16 take half as long
+    const long pairs = (long)max_n * c.H;
+    if (pairs > 16 && (pairs + 15) / 16 * n * 8 > ctx->num_sms) return launch_latent_mt<2>(ctx, c, ql, out, ldo, seqs, list, n, max_n, max_keys, split_rows);
     return launch_latent_mt<1>(ctx, c, ql, out, ldo, seqs, list, n, max_n, max_keys, split_rows);
 }
 

@@ -78,12 +78,12 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
             listed[n] = expert[tid];
         }
         __syncthreads();
-        // shares of equal K elements, cut where a tile ends
-        const int shared_tiles = a.shared.W ? (a.shared.N + 15) >> 4 : 0;
-        const long routed_cost = (long)matrices * tiles * a.K, cost = routed_cost + (long)shared_tiles * a.shared.K;
-        auto cut = [&](int i) {
-            const long at = cost * i / step;
-            return at <= routed_cost ? (int)((at + a.K - 1) / a.K) : matrices * tiles + (int)((at - routed_cost + a.shared.K - 1) / a.shared.K);
+        // shares of equal cost, in units of 64 columns of a tile, cut where a tile ends
+        const unsigned shared_tiles = a.shared.W ? (a.shared.N + 15) >> 4 : 0, ku = (a.K + 63) >> 6, kus = (a.shared.K + 63) >> 6;
+        const unsigned routed_cost = matrices * tiles * ku, cost = routed_cost + shared_tiles * kus, whole = cost / step, rest = cost % step;
+        auto cut = [&](unsigned i) {
+            const unsigned at = whole * i + rest * i / step;
+            return (int)(at <= routed_cost ? (at + ku - 1) / ku : matrices * tiles + (at - routed_cost + kus - 1) / kus);
         };
         const int share = item;
         item = cut(share);
@@ -91,16 +91,16 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
         step = 1;
     }
     struct Tile { const uint16_t* W; int N, K, kb, ke, tile, matrix; };  // kb .. ke: this CTA's columns (may be none)
-    auto tile_of = [&](int i) {
+    // (slices: a power of two)
+    const int log_slices = __ffs(slices) - 1;
+    auto tile_at = [&](int matrix, int tile) {
         Tile t;
-        t.N = a.N; t.K = a.K; t.W = a.W; t.tile = i; t.matrix = 0;
+        t.N = a.N; t.K = a.K; t.W = a.W; t.tile = tile; t.matrix = matrix;
         if (ROUTED) {
-            t.matrix = min(i / tiles, matrices);
-            t.tile = i - t.matrix * tiles;
-            if (t.matrix == matrices) { t.N = a.shared.N; t.K = a.shared.K; t.W = a.shared.W; }
-            else t.W += (size_t)listed[t.matrix] * a.N * a.K;
+            if (matrix == matrices) { t.N = a.shared.N; t.K = a.shared.K; t.W = a.shared.W; }
+            else t.W += (size_t)listed[matrix] * a.N * a.K;
         }
-        const int ks = ROUTED ? ((t.K + slices - 1) / slices + 31) / 32 * 32 : kslice;
+        const int ks = ROUTED ? (((t.K + slices - 1) >> log_slices) + 31) & ~31 : kslice;
         t.kb = min(t.K, rank * ks);
         t.ke = min(t.K, t.kb + ks);
         return t;
@@ -124,7 +124,8 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
             if (r1 < t.N) r[1] = __ldg(reinterpret_cast<const uint4*>(t.W + (size_t)r1 * t.K + k));
         }
     };
-    Tile now = tile_of(item);
+    const int matrix0 = ROUTED ? min(item / tiles, matrices) : 0;
+    Tile now = tile_at(matrix0, item - matrix0 * tiles);
     const int item0 = item;
     if (item < items) {
 #pragma unroll
@@ -137,7 +138,12 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
 
     bool staged = false;  // an input of one chunk is staged once for all tiles that share it
     for (; item < items; item += step) {
-        const Tile next = tile_of(item + step < items ? item + step : item);
+        Tile next = now;
+        if (!ROUTED) next.tile += step;
+        else if (item + step < items) {
+            if (now.matrix < matrices && now.tile + 1 == tiles) next = tile_at(now.matrix + 1, 0);
+            else next.tile++;
+        }
         const int tile = now.tile, N = now.N, kb = now.kb, ke = now.ke;
         const bool shared_tile = ROUTED && now.matrix == matrices;
         // what the epilogue's convolution wants, on its way during the product (thread tid: column tid & 15, row tid >> 4)

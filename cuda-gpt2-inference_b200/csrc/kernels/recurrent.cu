@@ -586,6 +586,32 @@ delta_step_kernel(const DeltaArgs a) {
     float* gd = o + vpad;
     float* gate = gd + D;
     float* low = gate + vpad;
+    // CH: rows r, r + 32, ... of the low-rank matrices are this group of eight lanes'; RU of them on their way at a time, the
+    // first ones before the previous kernel has finished
+    constexpr int LR = 8, RU = 4;
+    const int sub = tid & (LR - 1), low_rows = a.D + a.Dv;
+    uint4 wl[RU][2];
+    auto low_row = [&](int r, int& c0, int& c1) {
+        const bool is_g = r >= a.D;
+        c0 = is_g ? a.low_a : 0;  // (both halves start at multiples of eight columns)
+        c1 = is_g ? a.low_a + a.low_g : a.low_a;
+        return a.w_low + (size_t)(is_g ? a.gate_row + h * a.Dvl + r - a.D : h * a.Dl + r) * a.ld_low;
+    };
+    auto low_fetch = [&](int r0) {
+#pragma unroll
+        for (int u = 0; u < RU; ++u) {
+            const int r = r0 + u * (kDeltaStepThreads / LR);
+            int c0, c1;
+            const uint16_t* wr = low_row(r < low_rows ? r : 0, c0, c1);
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                const int col = c0 + (sub + x * LR) * 8;
+                wl[u][x] = make_uint4(0u, 0u, 0u, 0u);
+                if (r < low_rows && col < c1) wl[u][x] = __ldg(reinterpret_cast<const uint4*>(wr + col));
+            }
+        }
+    };
+    if (CH) low_fetch(tid / LR);
     for (int i = tid; i < (CH ? 3 * D + 3 * vpad : 2 * D + 2 * vpad); i += kDeltaStepThreads) sm[i] = 0.f;
     griddep_wait();
     griddep_launch_dependents();
@@ -610,28 +636,39 @@ delta_step_kernel(const DeltaArgs a) {
         for (int i = tid; i < a.low_a + a.low_g; i += kDeltaStepThreads) low[i] = row[a.low_col + i];
     __syncthreads();
     if (CH) {
-        constexpr int LR = 8;
-        const int sub = tid & (LR - 1);
-        for (int r = tid / LR; r < a.D + a.Dv; r += kDeltaStepThreads / LR) {
-            const bool is_g = r >= a.D;
-            const int d = is_g ? r - a.D : r, c0 = is_g ? a.low_a : 0, c1 = is_g ? a.low_a + a.low_g : a.low_a;
-            const uint16_t* wr = a.w_low + (size_t)(is_g ? a.gate_row + h * a.Dvl + d : h * a.Dl + d) * a.ld_low;
-            float s = 0.f;
-#pragma unroll 2
-            for (int c = c0 + sub * 8; c < c1; c += LR * 8) {  // (both halves start at multiples of eight columns)
-                const uint4 u = __ldg(reinterpret_cast<const uint4*>(wr + c));
-                const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+        for (int r0 = tid / LR; r0 < low_rows; r0 += RU * (kDeltaStepThreads / LR)) {
+            float s[RU];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    s = fmaf(__uint_as_float(w[e] << 16), low[c + 2 * e], s);
-                    s = fmaf(__uint_as_float(w[e] & 0xffff0000u), low[c + 2 * e + 1], s);
-                }
+            for (int u = 0; u < RU; ++u) {
+                s[u] = 0.f;
+                const int r = r0 + u * (kDeltaStepThreads / LR);
+                if (r >= low_rows) continue;
+                int c0, c1;
+                const uint16_t* wr = low_row(r, c0, c1);
+                auto add = [&](const uint4& v, int col) {
+                    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        s[u] = fmaf(__uint_as_float(w[e] << 16), low[col + 2 * e], s[u]);
+                        s[u] = fmaf(__uint_as_float(w[e] & 0xffff0000u), low[col + 2 * e + 1], s[u]);
+                    }
+                };
+#pragma unroll
+                for (int x = 0; x < 2; ++x)
+                    if (c0 + (sub + x * LR) * 8 < c1) add(wl[u][x], c0 + (sub + x * LR) * 8);
+                for (int col = c0 + (sub + 2 * LR) * 8; col < c1; col += LR * 8)  // ranks beyond 128
+                    add(__ldg(reinterpret_cast<const uint4*>(wr + col)), col);
             }
+            low_fetch(r0 + RU * (kDeltaStepThreads / LR));
 #pragma unroll
-            for (int m = 1; m < LR; m <<= 1) s += __shfl_xor_sync(0xffu << (lane & 24), s, m);
-            if (sub == 0) {
-                if (is_g) gate[d] = sigmoidf_(s);
-                else gd[d] = expf(negA * softplusf_(s + __ldg(a.dt_bias + (size_t)h * a.Dl + d)));
+            for (int u = 0; u < RU; ++u) {
+                const int r = r0 + u * (kDeltaStepThreads / LR);
+#pragma unroll
+                for (int m = 1; m < LR; m <<= 1) s[u] += __shfl_xor_sync(0xffu << (lane & 24), s[u], m);
+                if (sub == 0 && r < low_rows) {
+                    if (r >= a.D) gate[r - a.D] = sigmoidf_(s[u]);
+                    else gd[r] = expf(negA * softplusf_(s[u] + __ldg(a.dt_bias + (size_t)h * a.Dl + r)));
+                }
             }
         }
     }
