@@ -727,6 +727,7 @@ void load_all(b200_decoder* m) {
             for (int M = 1; M <= m->max_rows; ++M) { const int n = most_runs(m, *L.spec, M, nullptr); if (n > runs) runs = n; }
             r.place = static_cast<int*>(device_zeros(m, (size_t)m->max_rows * r.top * 4));
             r.blocks = static_cast<int*>(device_zeros(m, (size_t)(1 + runs) * 4));
+            r.decode = static_cast<DecodeRoute*>(device_zeros(m, sizeof(DecodeRoute)));
             routes.push_back(r);
             if (r.experts > m->max_experts) m->max_experts = r.experts;
         }
@@ -1123,6 +1124,7 @@ int enqueue_decode(b200_decoder* m, int B) {
         a.out = out; a.ldo = w.N;
         return launch_decode_gemm(ctx, a);
     };
+    if (m->num_routes) TRY(launch_decode_routes(ctx, m->routes, m->num_routes, m->dtokens, B));
     for (const Layer& L : m->layers) {
         const LayerSpec& s = *L.spec;
         TRY(norm(L.norm1));
@@ -1171,7 +1173,7 @@ int enqueue_decode(b200_decoder* m, int B) {
             TRY(norm(L.norm2));
             n.gate_w = nullptr;
             DecodeGemmArgs up = product_args(m->dh, f.up), down = product_args(m->dpair_mix, f.down);
-            up.table = down.table = f.table; up.tok = down.tok = m->dtokens; up.top = down.top = s.top; up.experts = down.experts = s.experts;
+            up.route = down.route = f.route.decode; up.top = down.top = s.top; up.experts = down.experts = s.experts;
             up.gate = f.gate; up.limit = s.limit; up.split_out = static_cast<uint8_t*>(m->dpair_mix);
             down.pair_in = 1; down.out = m->dpair_y; down.ldo = f.down.N;
             if (s.shared_ff) {

@@ -219,6 +219,11 @@ __device__ __forceinline__ float ld_cluster_f32(const float* p, int rank) {
     asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(map_to_cta(smem_u32(p), rank)) : "memory");
     return v;
 }
+__device__ __forceinline__ float4 ld_cluster_f32x4(const float* p, int rank) {
+    float4 v;
+    asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(map_to_cta(smem_u32(p), rank)) : "memory");
+    return v;
+}
 __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
 }
@@ -251,12 +256,14 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
     __half* qs = ks + 2 * kLatKeys * ld;                   // [16 MT][ld]
     float* ss = reinterpret_cast<float*>(qs + 16 * MT * ld);  // [16 MT][kLatS]
     __half* ps = reinterpret_cast<__half*>(ss + 16 * MT * kLatS);  // [16 MT][kLatP]
-    griddep_wait();
-    griddep_launch_dependents();
+    // Descriptors, lists and the rows that earlier steps cached were there before the previous kernel started (every kernel of a
+    // step waits for the one before it), and weights always: they are asked for before that kernel has finished.
     const int z = blockIdx.x % splits;
     const SeqDesc sd = seqs[list ? list[blockIdx.y] : blockIdx.y];
     const int pair0 = blockIdx.x / splits * 16 * MT, np = min(16 * MT, sd.n * c.H - pair0);  // (token, head) pairs
     if (np <= 0) return;  // (the whole cluster)
+    const int mine = z < np ? (np - z + splits - 1) / splits : 0;  // pairs z, z + splits, ... are this CTA's to finish
+    if (tid < min(mine, c.H)) l2_prefetch_bulk(c.Wuv + (size_t)((pair0 + z + tid * splits) % c.H) * c.Dv * c.Rp, (uint32_t)c.Dv * c.Rp * 2);
     const int keys = sd.pos0 + (pair0 + np - 1) / c.H + 1;
     const int per = ((keys + splits - 1) / splits + kLatKeys - 1) / kLatKeys * kLatKeys;
     const int t_begin = min(keys, z * per), t_end = min(keys, t_begin + per);
@@ -265,22 +272,32 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
     auto stage = [&](int t0, int buf) {
         __half* dst = ks + buf * kLatKeys * ld;
         const int nk = min(kLatKeys, t_end - t0);
-        for (int i = tid; i < kLatKeys * p16; i += kLatThreads) {
-            const int r = i / p16, p = i - r * p16;
-            if (r < nk) cp_async16(dst + r * ld + p * 8, rows + (size_t)(t0 + r) * c.Lp + p * 8);
-            else *reinterpret_cast<uint4*>(dst + r * ld + p * 8) = make_uint4(0u, 0u, 0u, 0u);
+        for (int p = lane; p < p16; p += 32) {  // a warp per row
+#pragma unroll
+            for (int i = 0; i < kLatKeys / 8; ++i) {
+                const int r = warp + i * 8;
+                if (r < nk) cp_async16(dst + r * ld + p * 8, rows + (size_t)(t0 + r) * c.Lp + p * 8);
+                else *reinterpret_cast<uint4*>(dst + r * ld + p * 8) = make_uint4(0u, 0u, 0u, 0u);
+            }
         }
         cp_async_commit();
     };
+    const bool early = t_begin < t_end && min(t_end, t_begin + kLatKeys) <= sd.pos0;  // rows of earlier steps only
+    if (early) stage(t_begin, 0);
+    griddep_wait();
+    griddep_launch_dependents();
     {
         const __half* q = ql + ((size_t)sd.lat0 * c.H + pair0) * c.Lp;
-        for (int i = tid; i < 16 * MT * p16; i += kLatThreads) {
-            const int r = i / p16, p = i - r * p16;
-            if (r < np) cp_async16(qs + r * ld + p * 8, q + (size_t)r * c.Lp + p * 8);
-            else *reinterpret_cast<uint4*>(qs + r * ld + p * 8) = make_uint4(0u, 0u, 0u, 0u);
+        for (int p = lane; p < p16; p += 32) {
+#pragma unroll
+            for (int i = 0; i < 2 * MT; ++i) {
+                const int r = warp + i * 8;
+                if (r < np) cp_async16(qs + r * ld + p * 8, q + (size_t)r * c.Lp + p * 8);
+                else *reinterpret_cast<uint4*>(qs + r * ld + p * 8) = make_uint4(0u, 0u, 0u, 0u);
+            }
         }
     }
-    if (t_begin < t_end) stage(t_begin, 0);
+    if (!early && t_begin < t_end) stage(t_begin, 0);
     else cp_async_commit();
     if (tid < 16 * MT) { stat_m[tid] = -INFINITY; stat_l[tid] = 0.f; }
     const float scale = c.scale * 1.4426950408889634f;
@@ -379,7 +396,7 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
     cp_async_wait<0>();
     __syncthreads();
     // this split's sums, where the staged rows were; then the merged ones of this CTA's pairs behind them
-    const int ldf = c.Rp;
+    const int ldf = c.Rp + (c.Rp % 32 == 0 ? 8 : 0);  // (at most Lp + 8)
     float* os = reinterpret_cast<float*>(ks);
     float* om = reinterpret_cast<float*>(ks + kLatKeys * ld);
 #pragma unroll
@@ -391,7 +408,6 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
                 const int r = m * 16 + g + (e >> 1) * 8, d = oc0 + j * 8 + c2 + (e & 1);
                 if (d < c.Rp) os[r * ldf + d] = o[m][j][e];
             }
-    const int mine = z < np ? (np - z + splits - 1) / splits : 0;  // pairs z, z + splits, ...
     // the values: W_uv, a warp working on U outputs at a time, 256 latent columns in a step; a step's weights are on their way during
     // the step before, the first ones' during the merge
     constexpr int U = 8;
@@ -424,19 +440,22 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
         weight[k][s] = e / sum;
     }
     __syncthreads();
-    for (int i = tid; i < mine * ldf; i += kLatThreads) {
-        const int k = i / ldf, d = i - k * ldf;
+    const int r4 = c.Rp >> 2;  // (columns R .. Rp of the sums belong to the rotated part: their weights in W_uv are zeros)
+    for (int i = tid; i < mine * r4; i += kLatThreads) {
+        const int k = i / r4, d = (i - k * r4) * 4;
         const float* src = os + (z + k * splits) * ldf + d;
-        float v = 0.f;
-        if (splits == 1) v = *src * weight[k][0];
-        else {
-            float x[8];
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f), x[8];
 #pragma unroll
-            for (int s = 0; s < 8; ++s) x[s] = s < splits ? ld_cluster_f32(src, s) : 0.f;
-#pragma unroll
-            for (int s = 0; s < 8; ++s) v = fmaf(x[s], weight[k][s], v);
+        for (int s = 0; s < 8; ++s) {
+            x[s] = v;
+            if (s < splits) x[s] = splits > 1 ? ld_cluster_f32x4(src, s) : *reinterpret_cast<const float4*>(src);
         }
-        om[i] = d < c.R ? v : 0.f;
+#pragma unroll
+        for (int s = 0; s < 8; ++s) {
+            const float w8 = weight[k][s];
+            v.x = fmaf(x[s].x, w8, v.x); v.y = fmaf(x[s].y, w8, v.y); v.z = fmaf(x[s].z, w8, v.z); v.w = fmaf(x[s].w, w8, v.w);
+        }
+        *reinterpret_cast<float4*>(om + k * ldf + d) = v;
     }
     __syncthreads();
     for (int i0 = warp * U; i0 < outputs; i0 += 8 * U) {

@@ -62,11 +62,13 @@ int launch_gemm_fp32(b200_ctx* ctx, float* out, const float* inp, const float* W
 // to out (fp32) and, as split rows, to split_out (all columns) or conv_out (the convolved ones, which then do not go to out).
 // gate != GATE_NONE: W's rows come in blocks of 64, 32 gates and the 32 linear values that belong to them, and the output
 // (split_out) has N / 2 columns.
-// Table-routed experts (top > 0): input row b belongs to the `top` matrices table[tok[b] * top ..] of the stack W [..][N, K],
+// Table-routed experts (top > 0): input row b belongs to the `top` matrices that `route` gives it of the stack W [..][N, K],
 // and its products with them are rows b * top + j of the output; pair_in: of the input too (else one row b meets
 // them all).  A matrix is read once however many rows want it.  With shared.W a further matrix of its own
 // height, width, input and output meets every row in the same launch.
 enum : int { GATE_NONE = 0, GATE_GELU_TANH = 1, GATE_CLAMP = 2 };
+constexpr int kMaxPairs = 256;  // (input row, expert) pairs
+struct DecodeRoute { int matrices; uint16_t listed[kMaxPairs], expert[kMaxPairs]; };  // matrices that occur; the one of every pair
 struct DecodeGemmShared { const uint8_t* x; const uint16_t* W; int N, K; float limit; float* out; int ldo; uint8_t* split_out; };
 struct DecodeGemmArgs {
     const uint8_t* x;
@@ -77,13 +79,15 @@ struct DecodeGemmArgs {
     const SeqDesc* seqs; const float* conv_w; const float* conv_b; float* hist; int conv_n, taps, max_slots;
     uint8_t* conv_out;    // [B] rows of conv_n columns
     int gate; float limit;
-    const int* table; const int* tok; int top, experts, pair_in;
+    const DecodeRoute* route; int top, experts, pair_in;  // (route: read before the previous kernel has finished)
     DecodeGemmShared shared;
 };
 int launch_decode_gemm(b200_ctx* ctx, const DecodeGemmArgs& a);
 
 // ---- experts (experts.cu)
-struct MoeRoute { const int* table; int experts, top; int* place; int* blocks; };  // table [vocab][top]
+struct MoeRoute { const int* table; int experts, top; int* place; int* blocks; DecodeRoute* decode; };  // table [vocab][top]
+// decode: the routes of B tokens' pairs -> MoeRoute::decode
+int launch_decode_routes(b200_ctx* ctx, const MoeRoute* routes, int n, const int* tok, int B);
 // rows per run (GemmGroups::align) of P pairs
 __host__ __device__ inline int moe_run_rows(int P, int experts, bool f32) { return f32 ? 64 : (P / 1024 >= experts ? 256 : 128); }
 // routes: n of them in device memory

@@ -57,6 +57,34 @@ moe_route_kernel(const MoeRoute* __restrict__ routes, const int* __restrict__ to
     for (int p = tid; p < P; p += kRouteThreads) r.place[p] = atomicAdd(cursor + __ldg(r.table + (size_t)tok[p / r.top] * r.top + p % r.top), 1);
 }
 
+// One CTA per feed-forward layer: the experts of B <= 16 tokens and, each once, the ones that occur (in the order of the pairs)
+__global__ void __launch_bounds__(kMaxPairs)
+decode_routes_kernel(const MoeRoute* __restrict__ routes, const int* __restrict__ tok, int B) {
+    __shared__ int expert[kMaxPairs];
+    __shared__ int first[kMaxPairs];
+    griddep_wait();
+    griddep_launch_dependents();
+    const MoeRoute r = routes[blockIdx.x];
+    const int tid = threadIdx.x, pairs = B * r.top;
+    if (tid < pairs) expert[tid] = __ldg(r.table + (size_t)tok[tid / r.top] * r.top + tid % r.top);
+    __syncthreads();
+    bool seen = false;
+    if (tid < pairs) {
+        for (int p = 0; p < tid; ++p) seen = seen || expert[p] == expert[tid];
+        first[tid] = !seen;
+    }
+    const int n = __syncthreads_count(tid < pairs && !seen);
+    if (tid < pairs) {
+        r.decode->expert[tid] = (uint16_t)expert[tid];
+        if (!seen) {
+            int at = 0;
+            for (int p = 0; p < tid; ++p) at += first[p];
+            r.decode->listed[at] = (uint16_t)expert[tid];
+        }
+    }
+    if (tid == 0) r.decode->matrices = n;
+}
+
 // fp32 rows of n pairs of 32 gates and 32 linear values -> n * 32 columns
 __global__ void __launch_bounds__(256)
 gated_act_kernel(float* __restrict__ out, const float* __restrict__ in, int F, size_t total4, int gate, float limit) {
@@ -82,6 +110,13 @@ gated_act_kernel(float* __restrict__ out, const float* __restrict__ in, int F, s
 int launch_moe_route(b200_ctx* ctx, const MoeRoute* routes, int n, const int* tok, int M, bool f32, int max_experts) {
     if ((size_t)max_experts * 4 > 40 * 1024) return B200_ERR_LIMIT;
     cudaError_t le = launch_pdl(ctx, moe_route_kernel, dim3(n), dim3(kRouteThreads), (size_t)max_experts * 4, routes, tok, M, f32);
+    ctx->launches++;
+    B200_CUDA(ctx, le);
+    return B200_OK;
+}
+
+int launch_decode_routes(b200_ctx* ctx, const MoeRoute* routes, int n, const int* tok, int B) {
+    cudaError_t le = launch_pdl(ctx, decode_routes_kernel, dim3(n), dim3(kMaxPairs), 0, routes, tok, B);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;

@@ -19,10 +19,9 @@
 //
 // Gated outputs: a tile is eight gate rows and their eight linear rows, so the two meet in the same epilogue.
 //
-// Table-routed experts (ROUTED): every CTA looks the rows' experts up and lists the matrices that occur; the tiles of all of
-// them, and of the shared expert, are one sequence, cut into equal shares of weight bytes, and a matrix is multiplied with
-// all rows at once, of which those that did not choose it are dropped.  (The ids and the table are read before the
-// previous kernel has finished: they were there before it started.)
+// Table-routed experts (ROUTED): the tiles of all matrices that occur, and of the shared expert, are one sequence, cut into equal
+// shares of weight bytes, and a matrix is multiplied with all rows at once, of which those that did not choose it are
+// dropped.  (Which ones occur is read before the previous kernel has finished: it was there before that one started.)
 #include "decoder_kernels.h"
 #include "decoder_math.cuh"
 #include "../prim/sm100.cuh"
@@ -34,7 +33,6 @@ constexpr int kThreads = 256, kWarps = 8;
 constexpr int kU = 8;             // pieces of a warp on the way
 constexpr int kTwoCtaSmem = 103 * 1024;  // input rows of a CTA that still leave room for a second one ...
 constexpr int kOneCtaSmem = 200 * 1024;  // ... and the most a CTA can hold
-constexpr int kMaxPairs = 256;    // (input row, expert) pairs
 constexpr int kMaxTaps = 4;       // convolution inputs requested ahead of the product (longer ones behind it)
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t a0, const uint32_t a1, const uint32_t a2, const uint32_t a3,
@@ -53,7 +51,6 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
     __shared__ float red[NT][kWarps][16][9];
     __shared__ float part[NT * 128];
     __shared__ uint16_t expert[ROUTED ? kMaxPairs : 1], listed[ROUTED ? kMaxPairs : 1];
-    __shared__ uint8_t first[ROUTED ? kMaxPairs : 1];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
     const int B = a.B;
     const bool gated = a.gate != GATE_NONE;
@@ -64,18 +61,10 @@ decode_gemm_kernel(const DecodeGemmArgs a, const int slices, const int kslice, c
     int item = blockIdx.x / slices, items = tiles, step = gridDim.x / slices, matrices = 1;
     if (ROUTED) {
         const int pairs = B * a.top;
-        if (tid < pairs) expert[tid] = (uint16_t)__ldg(a.table + (size_t)a.tok[tid / a.top] * a.top + tid % a.top);
-        __syncthreads();
+        matrices = a.route->matrices;
         if (tid < pairs) {
-            bool seen = false;
-            for (int p = 0; p < tid; ++p) seen = seen || expert[p] == expert[tid];
-            first[tid] = !seen;
-        }
-        matrices = __syncthreads_count(tid < pairs && first[tid]);
-        if (tid < pairs && first[tid]) {
-            int n = 0;
-            for (int p = 0; p < tid; ++p) n += first[p];
-            listed[n] = expert[tid];
+            expert[tid] = a.route->expert[tid];
+            listed[tid] = a.route->listed[tid];
         }
         __syncthreads();
         // shares of equal cost, in units of 64 columns of a tile, cut where a tile ends

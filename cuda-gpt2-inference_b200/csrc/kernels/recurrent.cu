@@ -586,46 +586,43 @@ delta_step_kernel(const DeltaArgs a) {
     float* gd = o + vpad;
     float* gate = gd + D;
     float* low = gate + vpad;
-    // CH: rows r, r + 32, ... of the low-rank matrices are this group of eight lanes'; RU of them on their way at a time, the
-    // first ones before the previous kernel has finished
-    constexpr int LR = 8, RU = 4;
-    const int sub = tid & (LR - 1), low_rows = a.D + a.Dv;
-    uint4 wl[RU][2];
-    auto low_row = [&](int r, int& c0, int& c1) {
-        const bool is_g = r >= a.D;
-        c0 = is_g ? a.low_a : 0;  // (both halves start at multiples of eight columns)
-        c1 = is_g ? a.low_a + a.low_g : a.low_a;
-        return a.w_low + (size_t)(is_g ? a.gate_row + h * a.Dvl + r - a.D : h * a.Dl + r) * a.ld_low;
-    };
-    auto low_fetch = [&](int r0) {
-#pragma unroll
-        for (int u = 0; u < RU; ++u) {
-            const int r = r0 + u * (kDeltaStepThreads / LR);
-            int c0, c1;
-            const uint16_t* wr = low_row(r < low_rows ? r : 0, c0, c1);
-#pragma unroll
-            for (int x = 0; x < 2; ++x) {
-                const int col = c0 + (sub + x * LR) * 8;
-                wl[u][x] = make_uint4(0u, 0u, 0u, 0u);
-                if (r < low_rows && col < c1) wl[u][x] = __ldg(reinterpret_cast<const uint4*>(wr + col));
-            }
-        }
-    };
-    if (CH) low_fetch(tid / LR);
-    for (int i = tid; i < (CH ? 3 * D + 3 * vpad : 2 * D + 2 * vpad); i += kDeltaStepThreads) sm[i] = 0.f;
-    griddep_wait();
-    griddep_launch_dependents();
+    // The descriptor and the state were there before the previous kernel started (every kernel of a step waits for the one before
+    // it): they are asked for before that kernel has finished, and so are weights.
     const SeqDesc sd = a.seqs[blockIdx.y];
-    const float* row = a.qkv + (size_t)sd.row0 * a.ld;
     const int grp = tid / L, l = tid & (L - 1);
-    // the state of the first columns is on its way while q, k and v are fetched and normalised
     Core core;
     float* Sh = a.S + ((size_t)sd.slot * a.H + h) * a.Dv * D;
     auto fetch = [&](int gc) {
         if (sd.pos0 > 0) core.load(Sh + (size_t)(gc < a.Dv ? gc : 0) * D, l, min(kDeltaStepCols, a.Dv - gc));
         else core.zero();
     };
-    fetch(grp * kDeltaStepCols);
+    if (!CH) fetch(grp * kDeltaStepCols);
+    // CH: rows r, r + 32, ... of a low-rank matrix are this group of eight lanes', columns sub * 8 .. and 64 + sub * 8 .. of each
+    // this lane's (more than 128 columns: one at a time); RU rows on their way at a time
+    constexpr int LR = 8, RU = 4, LROWS = kDeltaStepThreads / LR;
+    const int sub = tid & (LR - 1);
+    uint4 wl[RU][2];
+    const uint16_t* low_w[2] = {a.w_low + (size_t)h * a.Dl * a.ld_low, a.w_low + (size_t)(a.gate_row + h * a.Dvl) * a.ld_low + a.low_a};
+    auto low_fetch = [&](int half, int r0) {
+        const int rows = half ? a.Dv : a.D, cols = half ? a.low_g : a.low_a;
+#pragma unroll
+        for (int u = 0; u < RU; ++u)
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                const int r = r0 + u * LROWS, col = (sub + x * LR) * 8;
+                wl[u][x] = make_uint4(0u, 0u, 0u, 0u);
+                if (r < rows && col < cols) wl[u][x] = __ldg(reinterpret_cast<const uint4*>(low_w[half] + (size_t)r * a.ld_low + col));
+            }
+    };
+    if (CH) {
+        if (tid == 0 && sd.pos0 > 0) l2_prefetch_bulk(Sh, (uint32_t)a.Dv * D * 4);
+        low_fetch(0, tid / LR);
+    }
+    const float norm_w = tid < a.Dv ? __ldg(a.norm_w + tid) : 0.f;
+    for (int i = tid; i < (CH ? 3 * D + 3 * vpad : 2 * D + 2 * vpad); i += kDeltaStepThreads) sm[i] = 0.f;
+    griddep_wait();
+    griddep_launch_dependents();
+    const float* row = a.qkv + (size_t)sd.row0 * a.ld;
     __syncthreads();
     for (int i = tid; i < 2 * a.Dl + a.Dvl; i += kDeltaStepThreads) {
         if (i < a.Dl) q[i] = row[kvh * a.Dl + i];
@@ -636,41 +633,50 @@ delta_step_kernel(const DeltaArgs a) {
         for (int i = tid; i < a.low_a + a.low_g; i += kDeltaStepThreads) low[i] = row[a.low_col + i];
     __syncthreads();
     if (CH) {
-        for (int r0 = tid / LR; r0 < low_rows; r0 += RU * (kDeltaStepThreads / LR)) {
-            float s[RU];
+        for (int half = 0; half < 2; ++half) {
+            const int rows = half ? a.Dv : a.D, cols = half ? a.low_g : a.low_a;
+            const float* lo = low + (half ? a.low_a : 0);
+            float4 x[2][2];
 #pragma unroll
-            for (int u = 0; u < RU; ++u) {
-                s[u] = 0.f;
-                const int r = r0 + u * (kDeltaStepThreads / LR);
-                if (r >= low_rows) continue;
-                int c0, c1;
-                const uint16_t* wr = low_row(r, c0, c1);
-                auto add = [&](const uint4& v, int col) {
-                    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        s[u] = fmaf(__uint_as_float(w[e] << 16), low[col + 2 * e], s[u]);
-                        s[u] = fmaf(__uint_as_float(w[e] & 0xffff0000u), low[col + 2 * e + 1], s[u]);
-                    }
-                };
-#pragma unroll
-                for (int x = 0; x < 2; ++x)
-                    if (c0 + (sub + x * LR) * 8 < c1) add(wl[u][x], c0 + (sub + x * LR) * 8);
-                for (int col = c0 + (sub + 2 * LR) * 8; col < c1; col += LR * 8)  // ranks beyond 128
-                    add(__ldg(reinterpret_cast<const uint4*>(wr + col)), col);
+            for (int i = 0; i < 2; ++i) {
+                const int col = (sub + i * LR) * 8;
+                x[i][0] = x[i][1] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (col < cols) { x[i][0] = *reinterpret_cast<const float4*>(lo + col); x[i][1] = *reinterpret_cast<const float4*>(lo + col + 4); }
             }
-            low_fetch(r0 + RU * (kDeltaStepThreads / LR));
+            auto add = [&](float s, const uint4& w, const float4& p, const float4& q4) {
+                s = fmaf(__uint_as_float(w.x << 16), p.x, s); s = fmaf(__uint_as_float(w.x & 0xffff0000u), p.y, s);
+                s = fmaf(__uint_as_float(w.y << 16), p.z, s); s = fmaf(__uint_as_float(w.y & 0xffff0000u), p.w, s);
+                s = fmaf(__uint_as_float(w.z << 16), q4.x, s); s = fmaf(__uint_as_float(w.z & 0xffff0000u), q4.y, s);
+                s = fmaf(__uint_as_float(w.w << 16), q4.z, s); s = fmaf(__uint_as_float(w.w & 0xffff0000u), q4.w, s);
+                return s;
+            };
+            for (int r0 = tid / LR; r0 < rows; r0 += RU * LROWS) {
+                float s[RU];
 #pragma unroll
-            for (int u = 0; u < RU; ++u) {
-                const int r = r0 + u * (kDeltaStepThreads / LR);
+                for (int u = 0; u < RU; ++u) {
+                    s[u] = add(add(0.f, wl[u][0], x[0][0], x[0][1]), wl[u][1], x[1][0], x[1][1]);
+                    const int r = r0 + u * LROWS;
+                    if (r < rows)
+                        for (int col = (sub + 2 * LR) * 8; col < cols; col += LR * 8)
+                            s[u] = add(s[u], __ldg(reinterpret_cast<const uint4*>(low_w[half] + (size_t)r * a.ld_low + col)),
+                                       *reinterpret_cast<const float4*>(lo + col), *reinterpret_cast<const float4*>(lo + col + 4));
+                }
+                if (r0 + RU * LROWS < rows) low_fetch(half, r0 + RU * LROWS);
+                else if (half == 0) low_fetch(1, tid / LR);
 #pragma unroll
-                for (int m = 1; m < LR; m <<= 1) s[u] += __shfl_xor_sync(0xffu << (lane & 24), s[u], m);
-                if (sub == 0 && r < low_rows) {
-                    if (r >= a.D) gate[r - a.D] = sigmoidf_(s[u]);
-                    else gd[r] = expf(negA * softplusf_(s[u] + __ldg(a.dt_bias + (size_t)h * a.Dl + r)));
+                for (int u = 0; u < RU; ++u) {
+                    const int r = r0 + u * LROWS;
+#pragma unroll
+                    for (int m = 1; m < LR; m <<= 1) s[u] += __shfl_xor_sync(0xffu << (lane & 24), s[u], m);
+                    if (sub == 0 && r < rows) {
+                        if (half) gate[r] = sigmoidf_(s[u]);
+                        else gd[r] = expf(negA * softplusf_(s[u] + __ldg(a.dt_bias + (size_t)h * a.Dl + r)));
+                    }
                 }
             }
+            if (half == 0 && tid / LR >= rows) low_fetch(1, tid / LR);  // (a group without a row in the first half)
         }
+        fetch(grp * kDeltaStepCols);
     }
     float sq = 0.f, sk = 0.f, dot = 0.f;  // every warp for itself
     for (int d = lane; d < D; d += 32) { sq = fmaf(q[d], q[d], sq); sk = fmaf(k[d], k[d], sk); dot = fmaf(q[d], k[d], dot); }
@@ -704,7 +710,7 @@ delta_step_kernel(const DeltaArgs a) {
     const float r = 1.0f / sqrtf(block_sum(s, red) / (float)a.Dv + a.eps);
     for (int d = tid; d < a.Dv; d += kDeltaStepThreads)
         store_split(reinterpret_cast<uint8_t*>(a.out) + (size_t)sd.row0 * a.ldo * 4, h * a.Dv + d,
-                    o[d] * r * __ldg(a.norm_w + d) * (CH ? gate[d] : silu(row[a.gate_col + h * a.Dvl + d])));
+                    o[d] * r * (d < kDeltaStepThreads ? norm_w : __ldg(a.norm_w + d)) * (CH ? gate[d] : silu(row[a.gate_col + h * a.Dvl + d])));
 }
 
 // ------------------------------------------------------------------ minGRU
