@@ -289,6 +289,8 @@ struct b200_decoder {
     void *h = nullptr, *conv = nullptr, *mix = nullptr, *q = nullptr, *low = nullptr;
     float *gates = nullptr;                          // low-rank decays and output gates
     void *ql = nullptr, *lat = nullptr, *kv = nullptr;  // latent queries; latents and expanded keys and values of the step (grown on demand)
+    LatentParts lat_parts{};  // (pairs: set per layer)
+    long lat_rows_room = 0;
     int kv_rows = 0, expand_from = 1;                // expand_from: tokens from which a sequence's step is expanded
     void *pair_h = nullptr, *pair_mix = nullptr;     // rows of (token, expert) pairs: input, activations, outputs
     float *pair_y = nullptr, *raw = nullptr, *shared_gate = nullptr;
@@ -807,7 +809,20 @@ void allocate(b200_decoder* m) {
         const LatentAttention& c = first->lat;
         const long slow = 4L * (2 * c.R + c.Dr), fast = c.Dp + c.Dvp;
         m->expand_from = slow > fast ? (int)(c.Lp * fast / (slow - fast)) + 1 : m->max_rows + 1;
-        m->ql = device_zeros(m, M * ql * 2);
+        // rows in the latent form: sequences below that many tokens, and decoding ones
+        long rows = (long)m->max_slots * (m->expand_from - 1), pairs = 0, values = 0;
+        if (rows > (long)M) rows = (long)M;
+        if (rows < 16) rows = 16;
+        m->ql = device_zeros(m, rows * ql * 2);
+        for (const Layer& L : m->layers) {
+            if (L.spec->kind != MIX_LATENT) continue;
+            const long most = (rows > 256 ? rows : 256) * L.lat.H;  // 16 decoding rows in up to 16 shares
+            if (most > pairs) pairs = most;
+            if (most * L.lat.Rp > values) values = most * L.lat.Rp;
+        }
+        m->lat_parts.o = static_cast<float*>(device_zeros(m, values * 4));
+        m->lat_parts.ml = static_cast<float2*>(device_zeros(m, pairs * sizeof(float2)));
+        m->lat_rows_room = rows > 256 ? rows : 256;
     }
     if (!m->f32) {
         m->dx = static_cast<float*>(device_zeros(m, (size_t)16 * m->Cp * 4));
@@ -976,6 +991,12 @@ int mixer_delta(b200_decoder* m, const Layer& L, const StepView& v) {
     return B200_OK;
 }
 
+LatentParts latent_parts(const b200_decoder* m, const Layer& L) {
+    LatentParts p = m->lat_parts;
+    p.pairs = m->lat_rows_room * L.lat.H;
+    return p;
+}
+
 int mixer_latent(b200_decoder* m, const Layer& L, const StepView& v) {
     b200_ctx* ctx = m->ctx;
     const LatentAttention& c = L.lat;
@@ -995,7 +1016,8 @@ int mixer_latent(b200_decoder* m, const Layer& L, const StepView& v) {
     }
     if (v.num_lat_rows > 0) {
         OP("latent query", launch_latent_query(ctx, c, m->proj, L.in.N, m->ql, v.seqs, v.row_seq, v.lat_rows, v.num_lat_rows, false));
-        OP("latent attention", launch_latent_attention(ctx, c, m->ql, m->mix, L.o.K, v.seqs, v.lat_seqs, v.num_lat_seqs, v.lat_max_n, v.lat_max_keys, false));
+        OP("latent attention", launch_latent_attention(ctx, c, m->ql, latent_parts(m, L), m->mix, L.o.K, v.seqs, v.lat_seqs, v.num_lat_seqs, v.lat_rows, v.num_lat_rows, v.lat_max_n,
+                                                       v.lat_max_keys, false));
     }
     return B200_OK;
 }
@@ -1145,7 +1167,7 @@ int enqueue_decode(b200_decoder* m, int B) {
             TRY(launch_selective_scan(ctx, c, B, 1, true, true));
         } else if (s.kind == MIX_LATENT) {
             TRY(launch_latent_query(ctx, L.lat, m->dproj, L.in.N, m->dql, m->dseqs, nullptr, nullptr, B, true));
-            TRY(launch_latent_attention(ctx, L.lat, m->dql, m->dmix, L.o.K, m->dseqs, nullptr, B, 1, m->Tp, true));
+            TRY(launch_latent_attention(ctx, L.lat, m->dql, latent_parts(m, L), m->dmix, L.o.K, m->dseqs, nullptr, B, nullptr, B, 1, m->Tp, true));
         } else if (s.kind == MIX_DELTA || s.kind == MIX_CHANNEL_DELTA) {
             DeltaArgs a = delta_args(m, L, m->dseqs, m->dproj);
             a.qkv = m->dproj; a.ld = L.in.N;

@@ -4,6 +4,8 @@
 //   latent_query                 the latent form's queries, q W_uk beside the rotated part (and, decoding, the cache append)
 //   latent_attention             the latent form: all heads of a token read the same cached rows, which therefore serve as the
 //                                keys and, their first R columns, as the values of a whole tile of (token, head) pairs
+//   latent_value                 the weighted sums of latents through W_uv
+#include <cstdlib>
 #include <cuda_fp16.h>
 #include "decoder_kernels.h"
 #include "decoder_math.cuh"
@@ -206,24 +208,13 @@ latent_query_kernel(const LatentAttention c, const float* __restrict__ proj, int
 }
 
 // ------------------------------------------------------------------ attention over latents
-// A cluster of `splits` CTAs per tile of 16 MT (token, head) pairs of one sequence, each with its share of the cached
-// positions.  Positions go by in tiles of 64, staged two deep (cp.async): scores on m16n8k16 fp16 tensor-core instructions, a
-// warp taking eight positions over the whole row; softmax by rows; then the same staged rows are the values, a warp taking
-// 8 NTW columns.  (tcgen05 would want 64 rows or more of pairs and the probabilities in tensor memory or shared memory;
-// a decoding token brings as many pairs as the model has heads.)  The splits' states are merged through the cluster's shared memory, each
-// CTA for its share of the pairs, and goes on to the values: W_uv, a warp per output.
+// A CTA per tile of 16 MT (token, head) pairs of one sequence and share of its cached positions.  Positions go by in tiles of
+// 64, staged two deep by bulk copies (one per row, so that rows can lie 16 bytes apart from whole bank rows): scores on
+// m16n8k16 fp16 tensor-core instructions, a warp taking eight positions over the whole row; softmax by rows; then the
+// same staged rows are the values, a warp taking 8 NTW columns.  (tcgen05 would want 64 rows or more of pairs; a decoding token
+// brings as many as the model has heads.)  latent_value merges the shares and goes on to the values.
 constexpr int kLatThreads = 256, kLatKeys = 64, kLatP = kLatKeys + 8, kLatS = kLatKeys + 4;
 
-__device__ __forceinline__ float ld_cluster_f32(const float* p, int rank) {
-    float v;
-    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(map_to_cta(smem_u32(p), rank)) : "memory");
-    return v;
-}
-__device__ __forceinline__ float4 ld_cluster_f32x4(const float* p, int rank) {
-    float4 v;
-    asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(map_to_cta(smem_u32(p), rank)) : "memory");
-    return v;
-}
 __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
 }
@@ -246,10 +237,12 @@ inline size_t latent_smem(int Lp, int MT) {
 
 template <int MT, int NTW>
 __global__ void __launch_bounds__(kLatThreads)
-latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, void* out, int ldo, const SeqDesc* __restrict__ seqs,
-                        const int* __restrict__ list, int splits, bool split_rows) {
-    extern __shared__ __align__(16) uint8_t raw[];
-    __shared__ float stat_m[16 * MT], stat_l[16 * MT], stat_a[16 * MT], weight[16 * MT][8];
+latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, const LatentParts parts, const SeqDesc* __restrict__ seqs,
+                        const int* __restrict__ list, int splits, int* status) {
+    extern __shared__ __align__(128) uint8_t raw[];
+    __shared__ float stat_m[16 * MT], stat_l[16 * MT], stat_a[16 * MT];
+    __shared__ uint64_t full[2];
+    __shared__ volatile int abort_flag;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c2 = (lane & 3) * 2;
     const int ld = c.Lp + 8;  // halves
     __half* ks = reinterpret_cast<__half*>(raw);           // [2][64][ld]
@@ -257,38 +250,43 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
     float* ss = reinterpret_cast<float*>(qs + 16 * MT * ld);  // [16 MT][kLatS]
     __half* ps = reinterpret_cast<__half*>(ss + 16 * MT * kLatS);  // [16 MT][kLatP]
     // Descriptors, lists and the rows that earlier steps cached were there before the previous kernel started (every kernel of a
-    // step waits for the one before it), and weights always: they are asked for before that kernel has finished.
+    // step waits for the one before it): they are asked for before that kernel has finished.
     const int z = blockIdx.x % splits;
     const SeqDesc sd = seqs[list ? list[blockIdx.y] : blockIdx.y];
     const int pair0 = blockIdx.x / splits * 16 * MT, np = min(16 * MT, sd.n * c.H - pair0);  // (token, head) pairs
-    if (np <= 0) return;  // (the whole cluster)
-    const int mine = z < np ? (np - z + splits - 1) / splits : 0;  // pairs z, z + splits, ... are this CTA's to finish
-    if (tid < min(mine, c.H)) l2_prefetch_bulk(c.Wuv + (size_t)((pair0 + z + tid * splits) % c.H) * c.Dv * c.Rp, (uint32_t)c.Dv * c.Rp * 2);
+    if (np <= 0) return;
+    if (tid == 0) {
+        mbar_init(&full[0], 1);
+        mbar_init(&full[1], 1);
+        abort_flag = 0;
+        fence_barrier_init();
+    }
+    if (tid < 16 * MT) { stat_m[tid] = -INFINITY; stat_l[tid] = 0.f; }
+    __syncthreads();
     const int keys = sd.pos0 + (pair0 + np - 1) / c.H + 1;
-    const int per = ((keys + splits - 1) / splits + kLatKeys - 1) / kLatKeys * kLatKeys;
+    const int per = ((keys + splits - 1) / splits + 15) & ~15;
     const int t_begin = min(keys, z * per), t_end = min(keys, t_begin + per);
     const __half* rows = static_cast<const __half*>(c.cache) + (size_t)sd.slot * c.Tp * c.Lp;
     const int p16 = c.Lp >> 3;  // 16-byte pieces of a row
     auto stage = [&](int t0, int buf) {
         __half* dst = ks + buf * kLatKeys * ld;
         const int nk = min(kLatKeys, t_end - t0);
-        for (int p = lane; p < p16; p += 32) {  // a warp per row
-#pragma unroll
-            for (int i = 0; i < kLatKeys / 8; ++i) {
-                const int r = warp + i * 8;
-                if (r < nk) cp_async16(dst + r * ld + p * 8, rows + (size_t)(t0 + r) * c.Lp + p * 8);
-                else *reinterpret_cast<uint4*>(dst + r * ld + p * 8) = make_uint4(0u, 0u, 0u, 0u);
-            }
+        if (warp == 0) {
+            if (lane == 0) mbar_arrive_expect_tx(&full[buf], (uint32_t)nk * c.Lp * 2);
+            __syncwarp();
+            for (int r = lane; r < nk; r += 32) bulk_load(dst + r * ld, rows + (size_t)(t0 + r) * c.Lp, (uint32_t)c.Lp * 2, &full[buf]);
         }
-        cp_async_commit();
+        for (int r = nk + warp; r < kLatKeys; r += 8)  // (the last tile: rows behind the end are zeros)
+            for (int p = lane; p < p16; p += 32) *reinterpret_cast<uint4*>(dst + r * ld + p * 8) = make_uint4(0u, 0u, 0u, 0u);
     };
     const bool early = t_begin < t_end && min(t_end, t_begin + kLatKeys) <= sd.pos0;  // rows of earlier steps only
     if (early) stage(t_begin, 0);
     griddep_wait();
     griddep_launch_dependents();
+    if (!early && t_begin < t_end) stage(t_begin, 0);
     {
         const __half* q = ql + ((size_t)sd.lat0 * c.H + pair0) * c.Lp;
-        for (int p = lane; p < p16; p += 32) {
+        for (int p = lane; p < p16; p += 32) {  // a warp per row
 #pragma unroll
             for (int i = 0; i < 2 * MT; ++i) {
                 const int r = warp + i * 8;
@@ -296,10 +294,9 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
                 else *reinterpret_cast<uint4*>(qs + r * ld + p * 8) = make_uint4(0u, 0u, 0u, 0u);
             }
         }
+        cp_async_commit();
+        cp_async_wait<0>();
     }
-    if (!early && t_begin < t_end) stage(t_begin, 0);
-    else cp_async_commit();
-    if (tid < 16 * MT) { stat_m[tid] = -INFINITY; stat_l[tid] = 0.f; }
     const float scale = c.scale * 1.4426950408889634f;
     float o[MT][NTW][4];
 #pragma unroll
@@ -308,9 +305,16 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
         for (int j = 0; j < NTW; ++j) o[m][j][0] = o[m][j][1] = o[m][j][2] = o[m][j][3] = 0.f;
     const int oc0 = warp * 8 * NTW;
     for (int t0 = t_begin, n = 0; t0 < t_end; t0 += kLatKeys, ++n) {
-        if (t0 + kLatKeys < t_end) { stage(t0 + kLatKeys, (n + 1) & 1); cp_async_wait<1>(); }
-        else cp_async_wait<0>();
-        __syncthreads();
+        const bool more = t0 + kLatKeys < t_end;
+        if (more) stage(t0 + kLatKeys, (n + 1) & 1);
+        if (!__syncthreads_and(mbar_wait(&full[n & 1], (n >> 1) & 1, &abort_flag))) {
+            if (tid == 0) {
+                atomicCAS(status, 0, DEV_TIMEOUT_PRODUCER);
+                volatile int none = 0;
+                if (more) mbar_wait(&full[(n + 1) & 1], ((n + 1) >> 1) & 1, &none);  // its own copies in flight
+            }
+            return;
+        }
         const __half* kt = ks + (n & 1) * kLatKeys * ld;
         {
             float s[MT][2][4];  // two chains per tile of pairs
@@ -393,111 +397,116 @@ latent_attention_kernel(const LatentAttention c, const __half* __restrict__ ql, 
         }
         __syncthreads();  // the tile and the probabilities may be written again
     }
-    cp_async_wait<0>();
-    __syncthreads();
-    // this split's sums, where the staged rows were; then the merged ones of this CTA's pairs behind them
-    const int ldf = c.Rp + (c.Rp % 32 == 0 ? 8 : 0);  // (at most Lp + 8)
-    float* os = reinterpret_cast<float*>(ks);
-    float* om = reinterpret_cast<float*>(ks + kLatKeys * ld);
+    // this share's sums (a share without keys has none)
+    const size_t pair_index = (size_t)sd.lat0 * c.H + pair0;
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int j = 0; j < NTW; ++j)
+        for (int e = 0; e < 2; ++e) {
+            const int r = m * 16 + g + e * 8;
+            if (r >= np || t_begin >= t_end) continue;
+            float* dst = parts.o + ((pair_index + r) * splits + z) * c.Rp;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int r = m * 16 + g + (e >> 1) * 8, d = oc0 + j * 8 + c2 + (e & 1);
-                if (d < c.Rp) os[r * ldf + d] = o[m][j][e];
+            for (int j = 0; j < NTW; ++j) {
+                const int d = oc0 + j * 8 + c2;
+                if (d < c.Rp) *reinterpret_cast<float2*>(dst + d) = make_float2(o[m][j][2 * e], o[m][j][2 * e + 1]);
             }
-    // the values: W_uv, a warp working on U outputs at a time, 256 latent columns in a step; a step's weights are on their way during
-    // the step before, the first ones' during the merge
-    constexpr int U = 8;
-    const int outputs = mine * c.Dv, chunks = (c.Rp + 255) >> 8;
-    uint4 w[U];
-    auto fetch = [&](int i0, int d0) {
-        const bool live = i0 < outputs && d0 < c.Rp;
-        int k = min(i0, max(outputs - 1, 0)) / c.Dv, v = i0 - k * c.Dv, h = (pair0 + z + k * splits) % c.H;
-#pragma unroll
-        for (int u = 0; u < U; ++u) {
-            w[u] = make_uint4(0u, 0u, 0u, 0u);
-            if (live && i0 + u < outputs) w[u] = __ldg(reinterpret_cast<const uint4*>(c.Wuv + (size_t)(h * c.Dv + v) * c.Rp + d0));
-            if (++v == c.Dv) { v = 0; ++k; h = (pair0 + z + k * splits) % c.H; }
         }
+    if (tid < np) parts.ml[(pair_index + tid) * splits + z] = make_float2(stat_m[tid], stat_l[tid]);
+}
+
+// The shares' sums of four rows' head, merged, through W_uv: a warp works on four outputs at a time, lane l on latent columns 8l .. of
+// each 256.
+constexpr int kValueRows = 4, kMaxSplits = 16;
+__global__ void __launch_bounds__(256)
+latent_value_kernel(const LatentAttention c, const LatentParts parts, int splits, const int* __restrict__ rows, int n, void* out, int ldo, bool split_rows) {
+    __shared__ __align__(16) float om[kValueRows][kMaxLatent];
+    __shared__ float weight[kValueRows][kMaxSplits];
+    constexpr int U = 4, CH = kMaxLatent / 256;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, i0 = blockIdx.y * kValueRows, nr = min(kValueRows, n - i0);
+    uint4 w[U][CH];
+    auto fetch = [&](int v0) {
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+#pragma unroll
+            for (int x = 0; x < CH; ++x) {
+                const int v = v0 + u, d = x * 256 + lane * 8;
+                w[u][x] = make_uint4(0u, 0u, 0u, 0u);
+                if (v < c.Dv && d < c.Rp) w[u][x] = __ldg(reinterpret_cast<const uint4*>(c.Wuv + (size_t)(h * c.Dv + v) * c.Rp + d));
+            }
     };
-    fetch(warp * U, lane * 8);
-    if (splits > 1) cluster_sync_all();
-    else __syncthreads();
-    if (tid < mine * 8) {  // a split's share in a pair's sum
-        const int k = tid >> 3, s = tid & 7, r = z + k * splits;
-        float m = s < splits ? (splits > 1 ? ld_cluster_f32(stat_m + r, s) : stat_m[r]) : -INFINITY, top = m;
-        const float l = s < splits ? (splits > 1 ? ld_cluster_f32(stat_l + r, s) : stat_l[r]) : 0.f;
-        const uint32_t group = 0xffu << (lane & 24);
+    fetch(warp * U);
+    griddep_wait();
+    griddep_launch_dependents();
+    if (warp < nr) {  // a share's weight in its pair's sum
+        const float2 ml = lane < splits ? parts.ml[((size_t)(i0 + warp) * c.H + h) * splits + lane] : make_float2(-INFINITY, 0.f);
+        float top = ml.x;
 #pragma unroll
-        for (int d = 1; d < 8; d <<= 1) top = fmaxf(top, __shfl_xor_sync(group, top, d));
-        const float e = ex2(m - top);  // 0 for a split that saw no key of the pair's
-        float sum = l * e;
-#pragma unroll
-        for (int d = 1; d < 8; d <<= 1) sum += __shfl_xor_sync(group, sum, d);
-        weight[k][s] = e / sum;
+        for (int d = 16; d >= 1; d >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, d));  // finite: every pair sees key 0
+        const float e = ex2(ml.x - top);
+        const float sum = warp_sum(ml.y * e);
+        if (lane < splits) weight[warp][lane] = e / sum;
     }
     __syncthreads();
     const int r4 = c.Rp >> 2;  // (columns R .. Rp of the sums belong to the rotated part: their weights in W_uv are zeros)
-    for (int i = tid; i < mine * r4; i += kLatThreads) {
-        const int k = i / r4, d = (i - k * r4) * 4;
-        const float* src = os + (z + k * splits) * ldf + d;
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f), x[8];
+    for (int i = tid; i < kValueRows * r4; i += 256) {
+        const int r = i / r4, d = (i - r * r4) * 4;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (r < nr) {
+            const float* src = parts.o + ((size_t)(i0 + r) * c.H + h) * splits * c.Rp + d;
+            for (int s0 = 0; s0 < splits; s0 += 8) {
+                float4 x[8];
 #pragma unroll
-        for (int s = 0; s < 8; ++s) {
-            x[s] = v;
-            if (s < splits) x[s] = splits > 1 ? ld_cluster_f32x4(src, s) : *reinterpret_cast<const float4*>(src);
-        }
-#pragma unroll
-        for (int s = 0; s < 8; ++s) {
-            const float w8 = weight[k][s];
-            v.x = fmaf(x[s].x, w8, v.x); v.y = fmaf(x[s].y, w8, v.y); v.z = fmaf(x[s].z, w8, v.z); v.w = fmaf(x[s].w, w8, v.w);
-        }
-        *reinterpret_cast<float4*>(om + k * ldf + d) = v;
-    }
-    __syncthreads();
-    for (int i0 = warp * U; i0 < outputs; i0 += 8 * U) {
-        float acc[U];
-#pragma unroll
-        for (int u = 0; u < U; ++u) acc[u] = 0.f;
-        for (int ch = 0; ch < chunks; ++ch) {
-            const int d0 = ch * 256 + lane * 8;
-            uint4 x[U];
-#pragma unroll
-            for (int u = 0; u < U; ++u) x[u] = w[u];
-            if (ch + 1 < chunks) fetch(i0, d0 + 256);
-            else fetch(i0 + 8 * U, lane * 8);
-            if (d0 >= c.Rp) continue;
-            int k = i0 / c.Dv, v = i0 - k * c.Dv;
-#pragma unroll
-            for (int u = 0; u < U; ++u) {
-                const float4 x0 = *reinterpret_cast<const float4*>(om + k * ldf + d0), x1 = *reinterpret_cast<const float4*>(om + k * ldf + d0 + 4);
-                const float z8[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
-                const uint32_t y[4] = {x[u].x, x[u].y, x[u].z, x[u].w};
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    acc[u] = fmaf(__uint_as_float(y[e] << 16), z8[2 * e], acc[u]);
-                    acc[u] = fmaf(__uint_as_float(y[e] & 0xffff0000u), z8[2 * e + 1], acc[u]);
+                for (int s = 0; s < 8; ++s) {
+                    x[s] = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (s0 + s < splits && weight[r][s0 + s] > 0.f) x[s] = *reinterpret_cast<const float4*>(src + (size_t)(s0 + s) * c.Rp);
                 }
-                if (++v == c.Dv) { v = 0; k = min(k + 1, mine - 1); }  // (outputs beyond the end: weights of zero)
+#pragma unroll
+                for (int s = 0; s < 8; ++s) {
+                    const float f = s0 + s < splits ? weight[r][s0 + s] : 0.f;
+                    v.x = fmaf(x[s].x, f, v.x); v.y = fmaf(x[s].y, f, v.y); v.z = fmaf(x[s].z, f, v.z); v.w = fmaf(x[s].w, f, v.w);
+                }
             }
         }
-        reduce_scatter<U, 32>(acc, lane);
-        const int i = i0 + scatter_first<U, 32>(lane);
-        if (i < outputs && scatter_owner<U, 32>(lane)) {
-            const int k = i / c.Dv, pair = pair0 + z + k * splits, h = pair % c.H, row = sd.row0 + pair / c.H, col = h * c.Dv + i - k * c.Dv;
+        *reinterpret_cast<float4*>(&om[r][d]) = v;
+    }
+    __syncthreads();
+    for (int v0 = warp * U; v0 < c.Dv; v0 += 8 * U) {
+        float acc[U * kValueRows];
+#pragma unroll
+        for (int i = 0; i < U * kValueRows; ++i) acc[i] = 0.f;
+#pragma unroll
+        for (int x = 0; x < CH; ++x) {
+            const int d = x * 256 + lane * 8;
+            if (d >= c.Rp) continue;
+#pragma unroll
+            for (int r = 0; r < kValueRows; ++r) {
+                const float4 a = *reinterpret_cast<const float4*>(&om[r][d]), b = *reinterpret_cast<const float4*>(&om[r][d + 4]);
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+                    float s = acc[u * kValueRows + r];
+                    s = fmaf(__uint_as_float(w[u][x].x << 16), a.x, s); s = fmaf(__uint_as_float(w[u][x].x & 0xffff0000u), a.y, s);
+                    s = fmaf(__uint_as_float(w[u][x].y << 16), a.z, s); s = fmaf(__uint_as_float(w[u][x].y & 0xffff0000u), a.w, s);
+                    s = fmaf(__uint_as_float(w[u][x].z << 16), b.x, s); s = fmaf(__uint_as_float(w[u][x].z & 0xffff0000u), b.y, s);
+                    s = fmaf(__uint_as_float(w[u][x].w << 16), b.z, s); s = fmaf(__uint_as_float(w[u][x].w & 0xffff0000u), b.w, s);
+                    acc[u * kValueRows + r] = s;
+                }
+            }
+        }
+        fetch(v0 + 8 * U);
+        reduce_scatter<U * kValueRows, 32>(acc, lane);
+        const int t = scatter_first<U * kValueRows, 32>(lane), v = v0 + t / kValueRows, r = t % kValueRows;
+        if (v < c.Dv && r < nr && scatter_owner<U * kValueRows, 32>(lane)) {
+            const int row = rows ? rows[i0 + r] : i0 + r, col = h * c.Dv + v;
             if (split_rows) store_split(static_cast<uint8_t*>(out) + (size_t)row * ldo * 4, col, acc[0]);
             else store1<false>(out, (size_t)row * ldo + col, acc[0]);
         }
     }
-    if (splits > 1) cluster_sync_all();  // nobody leaves while its sums are being read
 }
 
 template <int MT, int NTW>
-int launch_latent_one(b200_ctx* ctx, const LatentAttention& c, const void* ql, void* out, int ldo, const SeqDesc* seqs, const int* list, int n, int max_n,
-                      int max_keys, bool split_rows) {
+int launch_latent_one(b200_ctx* ctx, const LatentAttention& c, const void* ql, const LatentParts& parts, const SeqDesc* seqs, const int* list, int n, int max_n,
+                      int splits) {
     const size_t smem = latent_smem(c.Lp, MT);
     static size_t attr_set[64] = {};
     if (attr_set[ctx->device & 63] < smem) {
@@ -505,40 +514,19 @@ int launch_latent_one(b200_ctx* ctx, const LatentAttention& c, const void* ql, v
         attr_set[ctx->device & 63] = smem;
     }
     const int per_seq = (int)(((long)max_n * c.H + 16 * MT - 1) / (16 * MT));
-    int splits = 1;
-    while (splits < 8 && (long)n * per_seq * splits * 2 <= ctx->num_sms && splits * 2 * kLatKeys <= max_keys) splits *= 2;
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(per_seq * splits, n);
-    cfg.blockDim = dim3(kLatThreads);
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = ctx->stream;
-    cudaLaunchAttribute attr[2];
-    int na = 0;
-    if (splits > 1) {
-        attr[na].id = cudaLaunchAttributeClusterDimension;
-        attr[na].val.clusterDim.x = splits;
-        attr[na].val.clusterDim.y = attr[na].val.clusterDim.z = 1;
-        ++na;
-    }
-    if (ctx->pdl) {
-        attr[na].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-        attr[na].val.programmaticStreamSerializationAllowed = 1;
-        ++na;
-    }
-    cfg.attrs = attr;
-    cfg.numAttrs = na;
-    const cudaError_t le = cudaLaunchKernelEx(&cfg, latent_attention_kernel<MT, NTW>, c, static_cast<const __half*>(ql), out, ldo, seqs, list, splits, split_rows);
+    cudaError_t le = launch_pdl(ctx, latent_attention_kernel<MT, NTW>, dim3(per_seq * splits, n), dim3(kLatThreads), smem, c, static_cast<const __half*>(ql), parts, seqs,
+                                list, splits, ctx->d_status);
     ctx->launches++;
     B200_CUDA(ctx, le);
     return B200_OK;
 }
 
 template <int MT>
-int launch_latent_mt(b200_ctx* ctx, const LatentAttention& c, const void* ql, void* out, int ldo, const SeqDesc* seqs, const int* list, int n, int max_n,
-                     int max_keys, bool split_rows) {
-    if (c.R <= 128) return launch_latent_one<MT, 2>(ctx, c, ql, out, ldo, seqs, list, n, max_n, max_keys, split_rows);
-    if (c.R <= 256) return launch_latent_one<MT, 4>(ctx, c, ql, out, ldo, seqs, list, n, max_n, max_keys, split_rows);
-    return launch_latent_one<MT, 8>(ctx, c, ql, out, ldo, seqs, list, n, max_n, max_keys, split_rows);
+int launch_latent_mt(b200_ctx* ctx, const LatentAttention& c, const void* ql, const LatentParts& parts, const SeqDesc* seqs, const int* list, int n, int max_n,
+                     int splits) {
+    if (c.R <= 128) return launch_latent_one<MT, 2>(ctx, c, ql, parts, seqs, list, n, max_n, splits);
+    if (c.R <= 256) return launch_latent_one<MT, 4>(ctx, c, ql, parts, seqs, list, n, max_n, splits);
+    return launch_latent_one<MT, 8>(ctx, c, ql, parts, seqs, list, n, max_n, splits);
 }
 
 }  // namespace
@@ -580,12 +568,29 @@ int launch_latent_query(b200_ctx* ctx, const LatentAttention& c, const float* pr
     return B200_OK;
 }
 
-int launch_latent_attention(b200_ctx* ctx, const LatentAttention& c, const void* ql, void* out, int ldo, const SeqDesc* seqs, const int* list, int n, int max_n,
-                            int max_keys, bool split_rows) {
-    // tiles of 32 pairs read the rows once for twice as many, tiles of 16 take half as long
+int launch_latent_attention(b200_ctx* ctx, const LatentAttention& c, const void* ql, const LatentParts& parts, void* out, int ldo, const SeqDesc* seqs,
+                            const int* list, int n, const int* rows, int n_rows, int max_n, int max_keys, bool split_rows) {
+    // shares of the positions, while there is room on the SMs and a share keeps a tile
     const long pairs = (long)max_n * c.H;
-    if (pairs > 16 && (pairs + 15) / 16 * n * 8 > ctx->num_sms) return launch_latent_mt<2>(ctx, c, ql, out, ldo, seqs, list, n, max_n, max_keys, split_rows);
-    return launch_latent_mt<1>(ctx, c, ql, out, ldo, seqs, list, n, max_n, max_keys, split_rows);
+    const int resident = ctx->num_sms * (latent_smem(c.Lp, 1) > 112 * 1024 ? 1 : 2);
+    // tiles of 32 pairs read the rows once for twice as many, tiles of 16 take half as long
+    const int mt = pairs > 16 && (pairs + 15) / 16 * n * 4 > resident ? 2 : 1;
+    const long tiles = (pairs + 16 * mt - 1) / (16 * mt) * n;
+    long splits = resident / tiles;
+    if (splits > (max_keys + kLatKeys - 1) / kLatKeys) splits = (max_keys + kLatKeys - 1) / kLatKeys;
+    if (splits > kMaxSplits) splits = kMaxSplits;
+    if (splits > parts.pairs / ((long)n_rows * c.H)) splits = parts.pairs / ((long)n_rows * c.H);
+    static const int forced = [] { const char* e = getenv("B200_LATENT_SPLITS"); return e ? atoi(e) : 0; }();  // tuning hook: 1 .. 16
+    if (forced >= 1 && forced <= kMaxSplits && forced <= parts.pairs / ((long)n_rows * c.H)) splits = forced;
+    if (splits < 1) splits = 1;
+    if ((long)n_rows * c.H > parts.pairs) return B200_ERR_LIMIT;
+    const int st = mt == 2 ? launch_latent_mt<2>(ctx, c, ql, parts, seqs, list, n, max_n, (int)splits) : launch_latent_mt<1>(ctx, c, ql, parts, seqs, list, n, max_n, (int)splits);
+    if (st != B200_OK) return st;
+    cudaError_t le = launch_pdl(ctx, latent_value_kernel, dim3(c.H, (n_rows + kValueRows - 1) / kValueRows), dim3(256), 0, c, parts, (int)splits, rows, n_rows, out, ldo,
+                                split_rows);
+    ctx->launches++;
+    B200_CUDA(ctx, le);
+    return B200_OK;
 }
 
 }  // namespace b200

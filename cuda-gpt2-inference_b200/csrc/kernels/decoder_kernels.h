@@ -239,9 +239,11 @@ int launch_latent_gather(b200_ctx* ctx, const LatentAttention& c, void* lat, con
 // token per sequence: row i is sequence i's)
 int launch_latent_query(b200_ctx* ctx, const LatentAttention& c, const float* proj, int ld, void* ql, const SeqDesc* seqs, const int* row_seq,
                         const int* rows, int n, bool append);
-// attention of ql's rows over the cached latents, W_uv applied, for sequences list[0 .. n) (null: 0 .. n - 1) of at most max_n
-// tokens that see at most max_keys keys.  out: bf16, or split rows, of ldo columns.
-int launch_latent_attention(b200_ctx* ctx, const LatentAttention& c, const void* ql, void* out, int ldo, const SeqDesc* seqs, const int* list, int n, int max_n,
-                            int max_keys, bool split_rows);
+// weighted sums of latents of (token, head) pairs over shares of the positions, their maxima and sums of weights; pairs: how many there is room for
+struct LatentParts { float* o; float2* ml; long pairs; };
+// attention of ql's n_rows rows (rows[i] of the step; null: i) over the cached latents, W_uv applied, for sequences list[0 .. n) (null:
+// 0 .. n - 1) of at most max_n tokens that see at most max_keys keys.  out: bf16, or split rows, of ldo columns.  Two launches.
+int launch_latent_attention(b200_ctx* ctx, const LatentAttention& c, const void* ql, const LatentParts& parts, void* out, int ldo, const SeqDesc* seqs,
+                            const int* list, int n, const int* rows, int n_rows, int max_n, int max_keys, bool split_rows);
 
 }  // namespace b200

@@ -142,6 +142,12 @@ __device__ __forceinline__ void tma_reduce_add_2d(const CUtensorMap* map, int x,
                  ::"l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(smem_u32(smem_src))
                  : "memory");
 }
+// Untiled copy of `bytes` (a multiple of 16; both addresses 16-byte aligned) to shared memory, completion on an mbarrier.
+__device__ __forceinline__ void bulk_load(void* smem_dst, const void* src, uint32_t bytes, uint64_t* bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                 ::"r"(smem_u32(smem_dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar))
+                 : "memory");
+}
 // Brings `bytes` (a multiple of 16) at a 16-byte aligned address into L2, without waiting.
 __device__ __forceinline__ void l2_prefetch_bulk(const void* p, uint32_t bytes) {
     asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(p), "r"(bytes) : "memory");
