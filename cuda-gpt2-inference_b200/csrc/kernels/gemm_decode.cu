@@ -298,6 +298,9 @@ int launch_one(b200_ctx* ctx, const DecodeGemmArgs& a) {
     // K slices while the CTAs of one wave (two per SM) are not used up and a warp keeps at least a piece
     int slices = 1;
     while (slices < 8 && tiles * slices * 2 <= 2 * ctx->num_sms && max_k / (slices * 2) >= 256) slices *= 2;
+    // (routed: and as many as it takes for a slice to be staged once for all of its tiles)
+    const int two_ctas = (kTwoCtaSmem / (NT * 8) - 16) / 4 / 32 * 32;
+    while (ROUTED && slices < 8 && (max_k + slices - 1) / slices > two_ctas) slices *= 2;
     const int kslice = ((max_k + slices - 1) / slices + 31) / 32 * 32;
     // the columns staged at a time: all of the slice, so that they are staged once for all tiles; else as many as
     // two CTAs per SM can hold
