@@ -1,6 +1,6 @@
 // Layered decoders: models whose configuration lists their layers, each with a mixer of some kind and a
-// feed-forward, served from per-sequence slots that hold whatever the mixers remember (key/value cache, recurrent
-// state, convolution history).
+// feed-forward, served from per-sequence slots that hold whatever the mixers remember (key/value or latent cache,
+// recurrent state, convolution history).
 //
 //   configuration  ModelSpec, read from config.json; a Design (registry below) fixes what all models of an
 //                  architecture share
